@@ -6,4 +6,7 @@ from .scaling import (estimate_flops, num_matmul_params, num_scaling_params, tra
                       PEAK_FLOPS_B200, PEAK_BANDWIDTH_B200)
 from .data import PackedBatches, DevicePackedBatches, Feeder, bos_token_id
 from .checkpoints import optimizer_state, restore_optimizer_, save_checkpoint, load_checkpoint
-from .generation import KVCache, prefill, decode_step, generate, sample_token
+from .generation import KVCache, prefill, decode_step, extend, generate, sample_token
+from .decoder import Decoder, DecoderConfig, DecoderState, LayerConfig, decoder_layout
+from .models import MODELS, load_model, register
+from .weights import SafeTensors, save_safetensors

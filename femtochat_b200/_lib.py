@@ -43,6 +43,22 @@ class OptimizerConfig(C.Structure):
     ]
 
 
+class LayerConfigC(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "weights_of", "heads", "kv_heads", "dim", "vdim", "conv", "decay_rank", "gate_rank",
+                                         "q_rank", "kv_rank", "rot_dim", "rot_dims", "ff")] + [
+        ("scale", C.c_float), ("rot_base", C.c_double), ("h_decay", C.POINTER(C.c_float))]
+
+
+class DecoderConfigC(C.Structure):
+    _fields_ = [("vocab", C.c_int32), ("width", C.c_int32), ("n_layer", C.c_int32), ("compute_dtype", C.c_int32), ("index_base", C.c_int32),
+                ("max_batch", C.c_int32), ("max_rows", C.c_int32), ("norm_eps", C.c_float), ("residual_mult", C.c_float),
+                ("h_layers", C.POINTER(LayerConfigC))]
+
+
+class DecoderTensorC(C.Structure):
+    _fields_ = [("name", C.c_char * 48), ("offset", C.c_int64), ("rows", C.c_int64), ("cols", C.c_int64)]
+
+
 class FemtoError(RuntimeError):
     def __init__(self, code, msg):
         super().__init__(f"libfemto error {code}: {msg}")
@@ -74,6 +90,11 @@ SIGNATURES = {
     "femto_kv_cache_length": (I32, [P]),
     "femto_prefill": (I32, [P, P, P, P, P, I32, I32, P, P]),
     "femto_decode_step": (I32, [P, P, P, P, P, I32, P, P]),
+    "femto_kv_cache_reset": (I32, [P, P]),
+    "femto_decoder_layout": (I32, [C.POINTER(DecoderConfigC), C.POINTER(DecoderTensorC), I32]),
+    "femto_decoder_nparams": (I64, [C.POINTER(DecoderConfigC)]),
+    "femto_decoder_create": (I32, [C.POINTER(DecoderConfigC), C.POINTER(P)]),
+    "femto_decoder_step": (I32, [P, P, P, P, I32, I32, C.POINTER(I32), I32, P, P, P]),
     "femto_pack_batch": (I32, [P, I64, P, I32, I32, I32, I32, I32, P, P, P, P, P]),
     "femto_feeder_create": (I32, [I32, I32, I32, C.POINTER(P)]),
     "femto_feeder_destroy": (I32, [P]),

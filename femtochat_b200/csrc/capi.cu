@@ -3,6 +3,7 @@
 
 #include <vector>
 
+#include "decoder.cuh"
 #include "model.cuh"
 #include "streaming.cuh"
 
@@ -170,9 +171,34 @@ int32_t femto_create(const femto_config* cfg, int32_t rank, int32_t world, const
   return 0;
 }
 
+int32_t femto_decoder_layout(const femto_decoder_config* cfg, femto_decoder_tensor* out, int32_t capacity) {
+  DecoderStack d;
+  FEMTO_TRY(decoder_fill(&d, cfg));
+  for (int i = 0; i < (int)d.tensors.size() && i < capacity; i++) out[i] = d.tensors[i];
+  return (int32_t)d.tensors.size();
+}
+int64_t femto_decoder_nparams(const femto_decoder_config* cfg) {
+  DecoderStack d;
+  const int r = decoder_fill(&d, cfg);
+  return r ? (int64_t)r : (int64_t)d.nparams;
+}
+int32_t femto_decoder_create(const femto_decoder_config* cfg, femto_handle** out) {
+  if (!out) return femto_fail(FEMTO_ERR_ARG, "h_out is NULL");
+  *out = nullptr;
+  DecoderStack d;
+  FEMTO_TRY(decoder_fill(&d, cfg));
+  FEMTO_TRY(require_device());
+  return decoder_create(cfg, out);
+}
+
 int32_t femto_destroy(femto_handle* h) {
   if (!h) return 0;
   cudaDeviceSynchronize();
+  if (h->dec) {
+    decoder_free(h->dec);
+    delete h;
+    return 0;
+  }
   dp_destroy(h->dp);
   model_free(h);
   delete h;
@@ -181,7 +207,7 @@ int32_t femto_destroy(femto_handle* h) {
 
 int32_t femto_refresh_weights(femto_handle* h, const float* theta, void* stream) {
   if (!h || !theta) return femto_fail(FEMTO_ERR_ARG, "NULL argument");
-  return model_refresh(h, theta, (cudaStream_t)stream);
+  return h->dec ? decoder_refresh(h, theta, (cudaStream_t)stream) : model_refresh(h, theta, (cudaStream_t)stream);
 }
 
 int32_t femto_loss_and_gradient(femto_handle* h, const float* theta, float* delta, const int32_t* tokens,
@@ -221,6 +247,7 @@ int32_t femto_loss_and_gradient_host(femto_handle* h, const float* theta, float*
                                      int32_t reduction, int32_t accumulate, float* h_loss, int32_t* h_n_valid,
                                      void* stream) {
   if (!h || !h_tokens || !h_targets || !h_loss) return femto_fail(FEMTO_ERR_ARG, "NULL argument");
+  if (h->dec) return femto_fail(FEMTO_ERR_UNSUPPORTED, "a decoder that lists its layers does not train");
   if (B <= 0 || B > h->maxB) return femto_fail(FEMTO_ERR_SHAPE, "B=%d outside 1..max_batch=%d", B, h->maxB);
   cudaStream_t s = (cudaStream_t)stream;
   const size_t bytes = sizeof(int) * (size_t)B * h->T;
@@ -269,6 +296,7 @@ int32_t femto_set_overlap(femto_handle* h, int32_t enable) {
 
 int32_t femto_optimizer_state_sizes(femto_handle* h, int64_t* out4) {
   if (!h || !out4) return femto_fail(FEMTO_ERR_ARG, "NULL argument");
+  if (h->dec) return femto_fail(FEMTO_ERR_UNSUPPORTED, "a decoder that lists its layers does not train");
   long long v[4];
   optimizer_state_sizes(h, v);
   for (int i = 0; i < 4; i++) out4[i] = v[i];

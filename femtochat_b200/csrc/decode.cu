@@ -7,20 +7,10 @@
 #include <algorithm>
 #include <vector>
 
+#include "decoder.cuh"
+#include "kv_cache.cuh"
 #include "model.cuh"
 #include "streaming.cuh"
-
-struct femto_kv_cache {
-  femto_handle* h = nullptr;
-  int maxB = 0, maxT = 0, B = 0, len = 0;     // len: tokens cached per column (all columns alike)
-  char* mem = nullptr;
-  std::vector<void*> K, V;                    // per block: [maxB][maxT][kv] of the compute type
-  void* xe_prev = nullptr;                    // [maxB][d] normalised embedding of the last token (smear)
-  void* xe_new = nullptr;                     // [maxB][d]
-  int *tok0 = nullptr, *pos = nullptr, *doc_start = nullptr, *lastpos = nullptr;   // [maxB]
-  float* part = nullptr;                      // split-key partials of the decode attention / split-K of the products
-  size_t part_floats = 0;
-};
 
 namespace {
 
@@ -408,6 +398,7 @@ extern "C" int32_t femto_kv_cache_create(femto_handle* h, int32_t max_batch, int
   if (!h || !out || max_batch <= 0 || max_len <= 0) return femto_fail(FEMTO_ERR_ARG, "bad argument");
   *out = nullptr;
   if (max_batch > h->maxB) return femto_fail(FEMTO_ERR_SHAPE, "max_batch %d exceeds the handle's %d", max_batch, h->maxB);
+  if (h->dec) return decoder_cache_create(h, max_batch, max_len, out);
   femto_kv_cache* c = new femto_kv_cache();
   c->h = h; c->maxB = max_batch; c->maxT = max_len;
   const size_t es = h->bf ? 2 : 4;
@@ -445,6 +436,13 @@ extern "C" int32_t femto_kv_cache_destroy(femto_kv_cache* c) {
   return 0;
 }
 
+extern "C" int32_t femto_kv_cache_reset(femto_kv_cache* c, void* stream) {
+  if (!c) return femto_fail(FEMTO_ERR_ARG, "NULL cache");
+  if (c->h->dec) return decoder_cache_reset(c, (cudaStream_t)stream);
+  c->B = 0; c->len = 0;   // a GPT cache is written from its start by the next femto_prefill
+  return 0;
+}
+
 extern "C" int32_t femto_kv_cache_length(femto_kv_cache* c) { return c ? c->len : FEMTO_ERR_ARG; }
 
 extern "C" int32_t femto_prefill(femto_handle* h, femto_kv_cache* c, const float* theta, const int32_t* tokens,
@@ -452,6 +450,11 @@ extern "C" int32_t femto_prefill(femto_handle* h, femto_kv_cache* c, const float
   if (!h || !c || !theta || !tokens || !logits_out) return femto_fail(FEMTO_ERR_ARG, "NULL argument");
   if (c->h != h) return femto_fail(FEMTO_ERR_ARG, "the cache belongs to another handle");
   if (B <= 0 || B > c->maxB || Tp <= 0 || Tp > c->maxT) return femto_fail(FEMTO_ERR_SHAPE, "prompt [%d][%d] exceeds the cache [%d][%d]", B, Tp, c->maxB, c->maxT);
+  if (h->dec) {
+    if (positions) return femto_fail(FEMTO_ERR_UNSUPPORTED, "this model counts positions from the start of the sequence");
+    FEMTO_TRY(decoder_cache_reset(c, (cudaStream_t)stream));
+    return decoder_step(h, c, theta, tokens, B, Tp, nullptr, 0, logits_out, nullptr, (cudaStream_t)stream);
+  }
   if ((long long)B * Tp > h->maxN) return femto_fail(FEMTO_ERR_SHAPE, "prompt of %d x %d tokens exceeds the workspace (%d tokens)", B, Tp, h->maxN);
   StepExtra ex;
   ex.T = Tp; ex.cache = c; ex.last_logits = logits_out;
@@ -466,7 +469,17 @@ extern "C" int32_t femto_decode_step(femto_handle* h, femto_kv_cache* c, const f
   if (c->len <= 0) return femto_fail(FEMTO_ERR_STATE, "femto_prefill must run before the first femto_decode_step");
   if (B != c->B) return femto_fail(FEMTO_ERR_SHAPE, "B=%d differs from the prompt's %d columns", B, c->B);
   if (c->len >= c->maxT) return femto_fail(FEMTO_ERR_SHAPE, "the cache is full (%d tokens per column)", c->maxT);
+  if (h->dec) {
+    if (positions) return femto_fail(FEMTO_ERR_UNSUPPORTED, "this model counts positions from the start of the sequence");
+    return decoder_step(h, c, theta, tokens, B, 1, nullptr, 0, logits_out, nullptr, (cudaStream_t)stream);
+  }
   if (!h->weights_valid) return femto_fail(FEMTO_ERR_STATE, "call femto_refresh_weights before the first step");
   return h->bf ? decode_t<bf16>(c, theta, tokens, positions, B, logits_out, (cudaStream_t)stream)
                : decode_t<float>(c, theta, tokens, positions, B, logits_out, (cudaStream_t)stream);
+}
+
+extern "C" int32_t femto_decoder_step(femto_handle* h, femto_kv_cache* c, const float* theta, const int32_t* tokens, int32_t B, int32_t T,
+                                      const int32_t* h_want, int32_t n_want, float* logits_out, float* residuals_out, void* stream) {
+  if (!h) return femto_fail(FEMTO_ERR_ARG, "NULL handle");
+  return decoder_step(h, c, theta, tokens, B, T, h_want, n_want, logits_out, residuals_out, (cudaStream_t)stream);
 }

@@ -1,0 +1,446 @@
+// Decoders given as a list of layers: configuration, flat layout, packed weights, cache and the forward schedule.  One
+// schedule serves prompts, portions of prompts and single tokens: it runs the tokens it is given from the states that
+// earlier calls left.
+#include "decoder.cuh"
+
+#include <math.h>
+#include <string.h>
+
+#include <algorithm>
+
+#include "streaming.cuh"
+
+// ---- configuration and layout -------------------------------------------------------------------------------------
+static int check_layer(const femto_decoder_config& cfg, int i) {
+  const femto_layer_config& c = cfg.h_layers[i];
+#define NEED(cond, what) if (!(cond)) return femto_fail(FEMTO_ERR_SHAPE, "layer %d: %s", i, what)
+  NEED(c.heads > 0 && c.dim > 0 && c.vdim > 0, "heads, dim and vdim must be positive");
+  NEED(c.ff >= 0, "ff is negative");
+  NEED(c.weights_of < cfg.n_layer && c.weights_of != i, "weights_of names no other layer");
+  switch (c.mixer) {
+    case FEMTO_MIXER_LIGHTNING:
+      NEED(c.h_decay != nullptr, "lightning attention needs one decay per head");
+      NEED(c.dim <= 256, "dim above 256 is not supported");
+      break;
+    case FEMTO_MIXER_CHANNEL_DELTA:
+      NEED(c.kv_heads > 0 && c.heads % c.kv_heads == 0, "heads must be a multiple of kv_heads");
+      NEED(c.conv >= 1, "conv must be positive");
+      NEED(c.decay_rank > 0 && c.gate_rank > 0, "the low-rank projections need a rank");
+      NEED(c.dim <= 256 && c.vdim <= 256, "dim or vdim above 256 is not supported");
+      break;
+    case FEMTO_MIXER_LATENT_ATTENTION:
+      NEED(c.q_rank > 0 && c.kv_rank > 0 && c.rot_dim >= 0, "q_rank and kv_rank must be positive");
+      NEED(c.rot_dims >= 0 && c.rot_dims <= c.rot_dim && c.rot_dims % 2 == 0, "rot_dims must be even and at most rot_dim");
+      NEED(c.kv_rank <= 1024 && c.vdim <= 256 && c.dim + c.rot_dim <= 512, "kv_rank above 1024, vdim above 256 or dim + rot_dim above 512 is not supported");
+      break;
+    default: return femto_fail(FEMTO_ERR_ARG, "layer %d: unknown mixer %d", i, c.mixer);
+  }
+#undef NEED
+  return 0;
+}
+
+int decoder_fill(DecoderStack* d, const femto_decoder_config* cfg) {
+  if (!cfg || !cfg->h_layers) return femto_fail(FEMTO_ERR_ARG, "config is NULL");
+  if (cfg->vocab <= 0 || cfg->width <= 0 || cfg->n_layer <= 0) return femto_fail(FEMTO_ERR_ARG, "vocab, width and n_layer must be positive");
+  if (cfg->compute_dtype != FEMTO_F32 && cfg->compute_dtype != FEMTO_BF16) return femto_fail(FEMTO_ERR_ARG, "compute_dtype must be FEMTO_F32 or FEMTO_BF16");
+  if (cfg->index_base != 0 && cfg->index_base != 1) return femto_fail(FEMTO_ERR_ARG, "index_base must be 0 or 1");
+  d->cfg = *cfg;
+  d->layer_cfg.assign(cfg->h_layers, cfg->h_layers + cfg->n_layer);
+  d->cfg.h_layers = d->layer_cfg.data();
+  d->bf = cfg->compute_dtype == FEMTO_BF16;
+  d->layers.assign(cfg->n_layer, DecLayer());
+  for (int i = 0; i < cfg->n_layer; i++) {
+    FEMTO_TRY(check_layer(*cfg, i));
+    DecLayer& l = d->layers[i];
+    l.c = cfg->h_layers[i];
+    l.own = i;
+    for (int hops = 0; d->layer_cfg[l.own].weights_of >= 0; hops++) {
+      if (hops > cfg->n_layer) return femto_fail(FEMTO_ERR_SHAPE, "layer %d: weights_of goes round in a circle", i);
+      l.own = d->layer_cfg[l.own].weights_of;
+    }
+    const femto_layer_config &a = l.c, &o = d->layer_cfg[l.own];
+    if (a.mixer != o.mixer || a.heads != o.heads || a.kv_heads != o.kv_heads || a.dim != o.dim || a.vdim != o.vdim || a.conv != o.conv ||
+        a.q_rank != o.q_rank || a.kv_rank != o.kv_rank || a.rot_dim != o.rot_dim || a.ff != o.ff)
+      return femto_fail(FEMTO_ERR_SHAPE, "layer %d differs in its sizes from layer %d, whose weights it uses", i, l.own);
+    l.c.decay_rank = o.decay_rank; l.c.gate_rank = o.gate_rank;
+    if (a.mixer == FEMTO_MIXER_LIGHTNING) l.decay.assign(a.h_decay, a.h_decay + a.heads);
+    l.c.h_decay = nullptr;
+  }
+  // flat layout, and the derived sizes of every layer
+  long long pos = 0;
+  d->tensors.clear();
+  auto take = [&](const std::string& name, long long rows, long long cols) {
+    femto_decoder_tensor t;
+    memset(&t, 0, sizeof(t));
+    strncpy(t.name, name.c_str(), sizeof(t.name) - 1);
+    t.offset = pos; t.rows = rows; t.cols = cols;
+    pos += (rows * std::max(1LL, cols) + 3) / 4 * 4;   // every tensor on a 16-byte boundary
+    d->tensors.push_back(t);
+    return t.offset;
+  };
+  const long long w = cfg->width;
+  d->off_embed = take("embed", cfg->vocab, w);
+  for (int i = 0; i < cfg->n_layer; i++) {
+    DecLayer& l = d->layers[i];
+    const femto_layer_config& c = l.c;
+    const long long H = c.heads, D = c.dim, E = c.vdim, G = c.kv_heads;
+    auto seg = [&](long long n) { const int at = l.n_in; l.n_in += round_up((int)n, 8); return at; };
+    l.ffp = round_up(c.ff, 32);
+    const std::string p = "l" + std::to_string(i) + ".", x = p + "mix.";
+    const bool mine = l.own == i;
+    auto put = [&](const std::string& name, long long rows, long long cols) { return mine ? take(name, rows, cols) : -1LL; };
+    l.norm1 = put(p + "norm1", w, 0); l.norm1b = put(p + "norm1b", w, 0);
+    if (c.mixer == FEMTO_MIXER_LIGHTNING) {
+      l.s_q = seg(H * D); l.s_k = seg(H * D); l.s_v = seg(H * E); l.s_g = seg(H * E);
+      put(x + "q", H * D, w); put(x + "k", H * D, w); put(x + "v", H * E, w); put(x + "g", H * E, w);
+      l.mix_norm = put(x + "norm", H * E, 0);
+    } else if (c.mixer == FEMTO_MIXER_CHANNEL_DELTA) {
+      l.ra = round_up(c.decay_rank, 8); l.rg = round_up(c.gate_rank, 8);
+      l.s_q = seg(G * D); l.s_k = seg(G * D); l.s_v = seg(H * E); l.s_b = seg(H); l.s_a1 = seg(c.decay_rank); l.s_g1 = seg(c.gate_rank);
+      put(x + "q", G * D, w); put(x + "k", G * D, w); put(x + "v", H * E, w); put(x + "b", H, w);
+      put(x + "a1", c.decay_rank, w); put(x + "g1", c.gate_rank, w);
+      put(x + "a2", H * D, c.decay_rank); put(x + "g2", H * E, c.gate_rank);
+      l.conv_q = put(x + "q.conv", G * D, c.conv); l.conv_k = put(x + "k.conv", G * D, c.conv); l.conv_v = put(x + "v.conv", H * E, c.conv);
+      l.a_log = put(x + "A_log", H, 0); l.dt_bias = put(x + "dt_bias", H * D, 0); l.mix_norm = put(x + "norm", E, 0);
+    } else {
+      l.qp = round_up(c.q_rank, 8); l.lp = round_up(c.kv_rank, 8); l.ld = round_up(l.lp + c.rot_dim, 8);
+      l.s_q = seg(c.q_rank); l.s_dkv = seg(c.kv_rank + c.rot_dim); l.s_g = seg(H);
+      put(x + "dq", c.q_rank, w); put(x + "dkv", c.kv_rank + c.rot_dim, w); put(x + "g", H, w);
+      put(x + "uq", H * (D + c.rot_dim), c.q_rank); put(x + "uk", H * D, c.kv_rank); put(x + "uv", H * E, c.kv_rank);
+      l.dq_norm = put(x + "dq.norm", c.q_rank, 0); l.dkv_norm = put(x + "dkv.norm", c.kv_rank, 0);
+    }
+    put(x + "o", w, H * E);
+    if (c.ff > 0) {
+      l.norm2 = put(p + "norm2", w, 0); l.norm2b = put(p + "norm2b", w, 0);
+      put(p + "mlp.gate", c.ff, w); put(p + "mlp.up", c.ff, w); put(p + "mlp.down", w, c.ff);
+    }
+  }
+  for (auto& l : d->layers) {
+    const DecLayer& o = d->layers[l.own];
+    l.norm1 = o.norm1; l.norm1b = o.norm1b; l.norm2 = o.norm2; l.norm2b = o.norm2b; l.mix_norm = o.mix_norm; l.conv_q = o.conv_q;
+    l.conv_k = o.conv_k; l.conv_v = o.conv_v; l.a_log = o.a_log; l.dt_bias = o.dt_bias; l.dq_norm = o.dq_norm; l.dkv_norm = o.dkv_norm;
+  }
+  d->off_final = take("final.norm", w, 0);
+  d->nparams = pos;
+  return 0;
+}
+
+// ---- weights and workspace ------------------------------------------------------------------------------------------
+namespace {
+struct Carver {
+  char* base = nullptr;
+  size_t off = 0;
+  template <typename P> void take(P*& p, size_t bytes) {
+    off = (off + 255) & ~(size_t)255;
+    p = base ? reinterpret_cast<P*>(base + off) : nullptr;
+    off += bytes;
+  }
+};
+
+void carve(DecoderStack* d, Carver& b) {
+  const size_t es = d->bf ? 2 : 4, R = d->cfg.max_rows, w = d->cfg.width;
+  b.take(d->status, 256);
+  b.take(d->embed, es * d->cfg.vocab * w);
+  size_t n_in = 0, mix = 0, ff = 0, qk = 0, hd = 0, heads = 0, g2 = 0, cq = 0, q = 0, qa = 0, vv = 0;
+  for (size_t i = 0; i < d->layers.size(); i++) {
+    DecLayer& l = d->layers[i];
+    const femto_layer_config& c = l.c;
+    const size_t H = c.heads, D = c.dim, E = c.vdim;
+    n_in = std::max(n_in, (size_t)l.n_in); mix = std::max(mix, H * E); ff = std::max(ff, (size_t)l.ffp);
+    if (c.mixer == FEMTO_MIXER_CHANNEL_DELTA) {
+      qk = std::max(qk, c.kv_heads * D); hd = std::max(hd, H * D); heads = std::max(heads, H); g2 = std::max(g2, H * E); vv = std::max(vv, H * E);
+    }
+    if (c.mixer == FEMTO_MIXER_LATENT_ATTENTION) {
+      cq = std::max(cq, (size_t)l.qp); q = std::max(q, H * (D + c.rot_dim)); qa = std::max(qa, H * l.ld);
+    }
+    b.take(l.decay_dev, 4 * H);
+    if (l.own != (int)i) continue;
+    b.take(l.w_in, es * l.n_in * w); b.take(l.w_o, es * w * H * E);
+    if (c.mixer == FEMTO_MIXER_CHANNEL_DELTA) { b.take(l.w_a2, es * H * D * l.ra); b.take(l.w_g2, es * H * E * l.rg); }
+    if (c.mixer == FEMTO_MIXER_LATENT_ATTENTION) { b.take(l.w_uq, es * H * (D + c.rot_dim) * l.qp); b.take(l.w_kv, es * H * (D + E) * l.lp); }
+    if (c.ff > 0) { b.take(l.w_gu, es * 2 * l.ffp * w); b.take(l.w_down, es * w * l.ffp); }
+  }
+  for (auto& l : d->layers) {
+    const DecLayer& o = d->layers[l.own];
+    l.w_in = o.w_in; l.w_o = o.w_o; l.w_a2 = o.w_a2; l.w_g2 = o.w_g2; l.w_uq = o.w_uq; l.w_kv = o.w_kv; l.w_gu = o.w_gu; l.w_down = o.w_down;
+  }
+  b.take(d->tok0, 4 * R); b.take(d->want, 4 * R);
+  b.take(d->x, 4 * R * w); b.take(d->hn, es * R * w); b.take(d->y, es * R * w);
+  b.take(d->proj, es * R * n_in); b.take(d->mixo, es * R * mix); b.take(d->mixg, es * R * mix);
+  b.take(d->gu, es * R * 2 * ff); b.take(d->act, es * R * ff);
+  b.take(d->qn, 4 * R * qk); b.take(d->kn, 4 * R * qk); b.take(d->gd, 4 * R * hd); b.take(d->beta, 4 * R * heads);
+  b.take(d->vv, es * R * vv); b.take(d->g2, es * R * g2);
+  b.take(d->cq, es * R * cq); b.take(d->q, es * R * q);
+  b.take(d->qabs, 4 * std::min(R, (size_t)d->cfg.max_batch * LATENT_FEW) * qa);
+  d->gemm_ws_bytes = (size_t)64 << 20;
+  b.take(d->gemm_ws, d->gemm_ws_bytes);
+}
+}  // namespace
+
+int decoder_create(const femto_decoder_config* cfg, femto_handle** out) {
+  DecoderStack* d = new DecoderStack();
+  int r = decoder_fill(d, cfg);
+  if (!r && (cfg->max_batch <= 0 || cfg->max_rows < cfg->max_batch)) r = femto_fail(FEMTO_ERR_ARG, "max_batch must be positive and max_rows at least max_batch");
+  if (r) { delete d; return r; }
+  Carver dry;
+  carve(d, dry);
+  const size_t bytes = dry.off + 256;
+  cudaError_t e = cudaMalloc(&d->arena, bytes);
+  if (e == cudaSuccess) e = cudaMemset(d->arena, 0, bytes);   // padding columns of packed weights stay zero
+  if (e != cudaSuccess) {
+    r = femto_fail(FEMTO_ERR_NOMEM, "%.2f GiB of weights and workspace: %s", bytes / 1073741824.0, cudaGetErrorString(e));
+    if (d->arena) cudaFree(d->arena);
+    delete d;
+    return r;
+  }
+  Carver real;
+  real.base = d->arena;
+  carve(d, real);
+  for (auto& l : d->layers)
+    if (!l.decay.empty()) cudaMemcpy(l.decay_dev, l.decay.data(), 4 * l.decay.size(), cudaMemcpyHostToDevice);
+  femto_handle* h = new femto_handle();
+  h->dec = d;
+  h->bf = d->bf;
+  h->nparams = d->nparams;
+  h->maxB = cfg->max_batch;
+  h->status = d->status;
+  e = cudaDeviceSynchronize();
+  if (e != cudaSuccess) { r = femto_fail((int)e, "device error while creating the decoder: %s", cudaGetErrorString(e)); decoder_free(d); delete h; return r; }
+  *out = h;
+  return 0;
+}
+
+void decoder_free(DecoderStack* d) {
+  if (!d) return;
+  if (d->arena) cudaFree(d->arena);
+  delete d;
+}
+
+template <typename T> static int refresh_t(DecoderStack* d, const float* theta, cudaStream_t s) {
+  auto find = [&](const std::string& name) -> const femto_decoder_tensor* {
+    for (const auto& t : d->tensors) if (name == t.name) return &t;
+    return nullptr;
+  };
+  const int w = d->cfg.width;
+  auto pack = [&](const std::string& name, void* dst, int ldd, int row, int group, int step) {
+    const femto_decoder_tensor* t = find(name);
+    if (!t) return femto_fail(FEMTO_ERR_STATE, "no tensor %s", name.c_str());
+    return pack_rows<T>(theta + t->offset, (int)t->rows, (int)t->cols, (T*)dst, ldd, row, group, step, s);
+  };
+  const int all = 1 << 30;
+  FEMTO_TRY(pack("embed", d->embed, w, 0, all, 0));
+  for (size_t i = 0; i < d->layers.size(); i++) {
+    DecLayer& l = d->layers[i];
+    if (l.own != (int)i) continue;
+    const femto_layer_config& c = l.c;
+    const std::string p = "l" + std::to_string(i) + ".", x = p + "mix.";
+    if (c.mixer == FEMTO_MIXER_LATENT_ATTENTION) {
+      FEMTO_TRY(pack(x + "dq", l.w_in, w, l.s_q, all, 0)); FEMTO_TRY(pack(x + "dkv", l.w_in, w, l.s_dkv, all, 0));
+      FEMTO_TRY(pack(x + "g", l.w_in, w, l.s_g, all, 0));
+      FEMTO_TRY(pack(x + "uq", l.w_uq, l.qp, 0, all, 0));
+      FEMTO_TRY(pack(x + "uk", l.w_kv, l.lp, 0, all, 0)); FEMTO_TRY(pack(x + "uv", l.w_kv, l.lp, c.heads * c.dim, all, 0));
+    } else {
+      FEMTO_TRY(pack(x + "q", l.w_in, w, l.s_q, all, 0)); FEMTO_TRY(pack(x + "k", l.w_in, w, l.s_k, all, 0));
+      FEMTO_TRY(pack(x + "v", l.w_in, w, l.s_v, all, 0));
+      if (c.mixer == FEMTO_MIXER_LIGHTNING) {
+        FEMTO_TRY(pack(x + "g", l.w_in, w, l.s_g, all, 0));
+      } else {
+        FEMTO_TRY(pack(x + "b", l.w_in, w, l.s_b, all, 0)); FEMTO_TRY(pack(x + "a1", l.w_in, w, l.s_a1, all, 0));
+        FEMTO_TRY(pack(x + "g1", l.w_in, w, l.s_g1, all, 0));
+        FEMTO_TRY(pack(x + "a2", l.w_a2, l.ra, 0, all, 0)); FEMTO_TRY(pack(x + "g2", l.w_g2, l.rg, 0, all, 0));
+      }
+    }
+    FEMTO_TRY(pack(x + "o", l.w_o, c.heads * c.vdim, 0, all, 0));
+    if (c.ff > 0) {   // groups of 32 gate rows and 32 up rows alternate, so that one epilogue sees both of a column
+      FEMTO_TRY(pack(p + "mlp.gate", l.w_gu, w, 0, 32, 64)); FEMTO_TRY(pack(p + "mlp.up", l.w_gu, w, 32, 32, 64));
+      FEMTO_TRY(pack(p + "mlp.down", l.w_down, l.ffp, 0, all, 0));
+    }
+  }
+  d->weights_valid = true;
+  return 0;
+}
+
+int decoder_refresh(femto_handle* h, const float* theta, cudaStream_t s) {
+  return h->dec->bf ? refresh_t<bf16>(h->dec, theta, s) : refresh_t<float>(h->dec, theta, s);
+}
+
+// ---- cache ----------------------------------------------------------------------------------------------------------
+int decoder_cache_create(femto_handle* h, int max_batch, int max_len, femto_kv_cache** out) {
+  DecoderStack* d = h->dec;
+  femto_kv_cache* c = new femto_kv_cache();
+  c->h = h; c->maxB = max_batch; c->maxT = max_len;
+  c->state.resize(d->layers.size());
+  const size_t es = d->bf ? 2 : 4, B = max_batch;
+  size_t exp_bytes = 0;
+  for (auto& l : d->layers) {
+    const femto_layer_config& q = l.c;
+    if (q.mixer != FEMTO_MIXER_LATENT_ATTENTION) continue;
+    exp_bytes = std::max(exp_bytes, es * B * max_len * (size_t)q.heads * (q.dim + q.vdim));
+    c->part_floats = std::max(c->part_floats, (size_t)std::max(64, max_batch * LATENT_FEW) * q.heads * (size_t)(l.lp + 2) * 2);
+  }
+  auto lay = [&](Carver& b) {
+    for (size_t i = 0; i < d->layers.size(); i++) {
+      const DecLayer& l = d->layers[i];
+      const femto_layer_config& q = l.c;
+      LayerState& s = c->state[i];
+      if (q.mixer != FEMTO_MIXER_LATENT_ATTENTION) { s.S_bytes = 4 * B * q.heads * q.dim * q.vdim; b.take(s.S, s.S_bytes); }
+      if (q.mixer == FEMTO_MIXER_CHANNEL_DELTA) {
+        s.tail_bytes = es * B * (q.conv - 1) * (2 * (size_t)q.kv_heads * q.dim + (size_t)q.heads * q.vdim);
+        b.take(s.tail[0], s.tail_bytes); b.take(s.tail[1], s.tail_bytes);
+      }
+      if (q.mixer == FEMTO_MIXER_LATENT_ATTENTION) { s.ld = l.ld; b.take(s.latent, es * B * max_len * l.ld); }
+    }
+    b.take(c->part, 4 * c->part_floats);
+    b.take(c->kv_exp, exp_bytes);
+  };
+  Carver dry;
+  lay(dry);
+  const size_t bytes = dry.off + 256;
+  cudaError_t e = cudaMalloc(&c->mem, bytes);
+  if (e == cudaSuccess) e = cudaMemset(c->mem, 0, bytes);
+  if (e == cudaSuccess) e = cudaDeviceSynchronize();
+  if (e != cudaSuccess) {
+    if (c->mem) cudaFree(c->mem);
+    delete c;
+    return femto_fail(FEMTO_ERR_NOMEM, "%.2f GiB of cache: %s", bytes / 1073741824.0, cudaGetErrorString(e));
+  }
+  Carver real;
+  real.base = c->mem;
+  lay(real);
+  *out = c;
+  return 0;
+}
+
+int decoder_cache_reset(femto_kv_cache* c, cudaStream_t s) {
+  for (auto& l : c->state) {
+    if (l.S_bytes) FEMTO_TRY(fill_zero(l.S, l.S_bytes, s));
+    if (l.tail_bytes) FEMTO_TRY(fill_zero(l.tail[l.tail_now], l.tail_bytes, s));
+  }
+  c->B = 0; c->len = 0;
+  return 0;
+}
+
+// ---- forward ---------------------------------------------------------------------------------------------------------
+template <typename T>
+static int mixer_t(DecoderStack* d, femto_kv_cache* c, int i, const float* theta, int B, int Tn, int first, cudaStream_t s) {
+  typedef DecStream<T> S;
+  const DecLayer& l = d->layers[i];
+  const femto_layer_config& q = l.c;
+  LayerState& st = c->state[i];
+  const int R = B * Tn, w = d->cfg.width, H = q.heads, D = q.dim, E = q.vdim;
+  const float eps = d->cfg.norm_eps;
+  T* proj = (T*)d->proj;
+  FEMTO_TRY(rows_linear<T>(d, d->hn, w, l.w_in, w, proj, l.n_in, R, l.n_in, w, EPI_STORE, s));
+  T* out = (T*)d->mixg;
+  if (q.mixer == FEMTO_MIXER_LIGHTNING) {
+    RecurrenceArgs a;
+    a.q = proj + l.s_q; a.k = proj + l.s_k; a.v = proj + l.s_v; a.ldq = a.ldk = a.ldv = l.n_in;
+    a.decay = l.decay_dev; a.S = st.S; a.o = d->mixo; a.B = B; a.T = Tn; a.heads = a.qk_heads = H; a.dim = D; a.vdim = E;
+    FEMTO_TRY(recurrence<T>(a, s));
+    FEMTO_TRY(S::gated_norm((const T*)d->mixo, theta + l.mix_norm, true, proj + l.s_g, l.n_in, out, R, 1, H * E, eps, s));
+  } else if (q.mixer == FEMTO_MIXER_CHANNEL_DELTA) {
+    FEMTO_TRY(rows_linear<T>(d, proj + l.s_a1, l.n_in, l.w_a2, l.ra, d->gd, H * D, R, H * D, l.ra, EPI_F32, s));
+    FEMTO_TRY(rows_linear<T>(d, proj + l.s_g1, l.n_in, l.w_g2, l.rg, d->g2, H * E, R, H * E, l.rg, EPI_STORE, s));
+    DeltaPrepArgs p;
+    p.proj = proj; p.ldp = l.n_in; p.s_q = l.s_q; p.s_k = l.s_k; p.s_v = l.s_v; p.s_b = l.s_b;
+    p.conv_q = theta + l.conv_q; p.conv_k = theta + l.conv_k; p.conv_v = theta + l.conv_v; p.a_log = theta + l.a_log; p.dt_bias = theta + l.dt_bias;
+    p.tail_in = st.tail[st.tail_now]; p.tail_out = st.tail[st.tail_now ^ 1];
+    p.qn = d->qn; p.kn = d->kn; p.gd = d->gd; p.beta = d->beta; p.vv = d->vv;
+    p.B = B; p.T = Tn; p.heads = H; p.kv_heads = q.kv_heads; p.dim = D; p.vdim = E; p.taps = q.conv;
+    FEMTO_TRY(delta_prep<T>(p, s));
+    st.tail_now ^= 1;
+    RecurrenceArgs a;
+    a.q = d->qn; a.k = d->kn; a.v = d->vv; a.ldq = a.ldk = (long long)q.kv_heads * D; a.ldv = (long long)H * E;
+    a.g = d->gd; a.beta = d->beta; a.S = st.S; a.o = d->mixo; a.B = B; a.T = Tn; a.heads = H; a.qk_heads = q.kv_heads; a.dim = D; a.vdim = E;
+    FEMTO_TRY(recurrence<T>(a, s));
+    FEMTO_TRY(S::gated_norm((const T*)d->mixo, theta + l.mix_norm, false, (const T*)d->g2, (long long)H * E, out, R, H, E, eps, s));
+  } else {
+    FEMTO_TRY(S::norm_cols(proj + l.s_q, l.n_in, theta + l.dq_norm, (T*)d->cq, l.qp, R, q.q_rank, eps, s));
+    FEMTO_TRY(rows_linear<T>(d, d->cq, l.qp, l.w_uq, l.qp, d->q, H * (D + q.rot_dim), R, H * (D + q.rot_dim), l.qp, EPI_STORE, s));
+    LatentArgs a;
+    a.q = d->q; a.dkv = proj + l.s_dkv; a.ld_dkv = l.n_in; a.dkv_norm = theta + l.dkv_norm; a.gate = proj + l.s_g; a.ld_gate = l.n_in;
+    a.latent = st.latent; a.ld = l.ld; a.lp = l.lp; a.maxT = c->maxT; a.w_kv = l.w_kv; a.kv = c->kv_exp;
+    a.qabs = d->qabs; a.part = c->part; a.part_floats = c->part_floats; a.o = out;
+    a.B = B; a.T = Tn; a.first = first; a.heads = H; a.dim = D; a.rot_dim = q.rot_dim; a.rot_dims = q.rot_dims; a.vdim = E; a.kv_rank = q.kv_rank;
+    a.scale = q.scale; a.eps = eps; a.rot_base = q.rot_base; a.d = d;
+    FEMTO_TRY(latent_prep<T>(a, s));
+    FEMTO_TRY(latent_attention<T>(a, s));
+  }
+  return rows_linear<T>(d, out, H * E, l.w_o, H * E, d->y, w, R, w, H * E, EPI_STORE, s);
+}
+
+// Tokens [t0, t0 + Tn) of every column.
+template <typename T>
+static int pass_t(DecoderStack* d, femto_kv_cache* c, const float* theta, const int* tokens, int ld_tok, int B, int Tn, float* residuals,
+                  cudaStream_t s) {
+  typedef DecStream<T> S;
+  const int R = B * Tn, w = d->cfg.width, L = d->cfg.n_layer;
+  const float eps = d->cfg.norm_eps, m = d->cfg.residual_mult;
+  FEMTO_TRY(S::embed((const T*)d->embed, tokens, ld_tok, B, Tn, d->cfg.index_base, d->cfg.vocab, theta + d->layers[0].norm1, d->x, (T*)d->hn,
+                     w, eps, d->status, s));
+  for (int i = 0; i < L; i++) {
+    const DecLayer& l = d->layers[i];
+    FEMTO_TRY(mixer_t<T>(d, c, i, theta, B, Tn, c->len, s));
+    const float* next = i + 1 < L ? theta + d->layers[i + 1].norm1 : nullptr;
+    const bool mlp = l.c.ff > 0;
+    FEMTO_TRY(S::resid_norm(d->x, (const T*)d->y, theta + l.norm1b, m, mlp ? theta + l.norm2 : next, mlp || next ? (T*)d->hn : nullptr, R, w, eps, s));
+    if (mlp) {
+      FEMTO_TRY(rows_linear<T>(d, d->hn, w, l.w_gu, w, d->gu, 2 * l.ffp, R, 2 * l.ffp, w, EPI_STORE, s));
+      FEMTO_TRY(S::gated_mlp((const T*)d->gu, (T*)d->act, R, l.ffp, s));
+      FEMTO_TRY(rows_linear<T>(d, d->act, l.ffp, l.w_down, l.ffp, d->y, w, R, w, l.ffp, EPI_STORE, s));
+      FEMTO_TRY(S::resid_norm(d->x, (const T*)d->y, theta + l.norm2b, m, next, next ? (T*)d->hn : nullptr, R, w, eps, s));
+    }
+    if (residuals) CUDA_TRY(cudaMemcpyAsync(residuals + (size_t)i * R * w, d->x, 4 * (size_t)R * w, cudaMemcpyDeviceToDevice, s));
+  }
+  return 0;
+}
+
+// Logits of n rows of the residual stream (rows want[0..n), or each column's last) as fp32 [n][vocab].
+template <typename T>
+static int logits_t(DecoderStack* d, const float* theta, const int* want, int stride, int n, float* out, cudaStream_t s) {
+  const int w = d->cfg.width;
+  FEMTO_TRY(DecStream<T>::gather_norm(d->x, want, stride, theta + d->off_final, (T*)d->hn, n, w, d->cfg.norm_eps, s));
+  return rows_linear<T>(d, d->hn, w, d->embed, w, out, d->cfg.vocab, n, d->cfg.vocab, w, EPI_F32, s);
+}
+
+int decoder_step(femto_handle* h, femto_kv_cache* c, const float* theta, const int* tokens, int B, int T, const int* h_want, int n_want,
+                 float* logits_out, float* residuals_out, cudaStream_t s) {
+  DecoderStack* d = h->dec;
+  if (!d) return femto_fail(FEMTO_ERR_UNSUPPORTED, "the handle's model does not list its layers");
+  if (!c || !theta || !tokens || (h_want && (!logits_out || n_want <= 0))) return femto_fail(FEMTO_ERR_ARG, "NULL argument");
+  if (c->h != h) return femto_fail(FEMTO_ERR_ARG, "the cache belongs to another handle");
+  if (!d->weights_valid) return femto_fail(FEMTO_ERR_STATE, "call femto_refresh_weights before the first step");
+  if (B <= 0 || B > c->maxB || T <= 0) return femto_fail(FEMTO_ERR_SHAPE, "step [%d][%d] exceeds the cache's %d columns", B, T, c->maxB);
+  if (c->len > 0 && B != c->B) return femto_fail(FEMTO_ERR_SHAPE, "B=%d differs from the %d columns in the cache", B, c->B);
+  if ((long long)c->len + T > c->maxT) return femto_fail(FEMTO_ERR_SHAPE, "%d + %d tokens exceed the cache (%d per column)", c->len, T, c->maxT);
+  for (int i = 0; i < (h_want ? n_want : 0); i++)
+    if (h_want[i] < 0 || h_want[i] >= B * T || (i > 0 && h_want[i] <= h_want[i - 1]))
+      return femto_fail(FEMTO_ERR_ARG, "wanted positions must ascend within 0..%d", B * T - 1);
+  const int portion = d->cfg.max_rows / B;
+  if (residuals_out && T > portion) return femto_fail(FEMTO_ERR_SHAPE, "residuals of %d x %d tokens exceed max_rows", B, T);
+  c->B = B;
+  for (int t0 = 0; t0 < T; t0 += portion) {
+    const int n = std::min(portion, T - t0);
+    FEMTO_TRY(d->bf ? pass_t<bf16>(d, c, theta, tokens + t0, T, B, n, residuals_out, s)
+                    : pass_t<float>(d, c, theta, tokens + t0, T, B, n, residuals_out, s));
+    c->len += n;
+    if (!h_want) {
+      if (logits_out && t0 + n == T)
+        FEMTO_TRY(d->bf ? logits_t<bf16>(d, theta, nullptr, n, B, logits_out, s) : logits_t<float>(d, theta, nullptr, n, B, logits_out, s));
+      continue;
+    }
+    // runs of wanted positions whose logits lie together in the output
+    for (int i = 0; i < n_want;) {
+      const auto here = [&](int k) { const int t = h_want[k] % T; return t >= t0 && t < t0 + n; };
+      if (!here(i)) { i++; continue; }
+      std::vector<int> rows;
+      int k = i;
+      for (; k < n_want && here(k); k++) rows.push_back(h_want[k] / T * n + h_want[k] % T - t0);
+      CUDA_TRY(cudaMemcpyAsync(d->want, rows.data(), 4 * rows.size(), cudaMemcpyHostToDevice, s));   // pageable: staged before it returns
+      float* out = logits_out + (size_t)i * d->cfg.vocab;
+      FEMTO_TRY(d->bf ? logits_t<bf16>(d, theta, d->want, 0, (int)rows.size(), out, s) : logits_t<float>(d, theta, d->want, 0, (int)rows.size(), out, s));
+      i = k;
+    }
+  }
+  return 0;
+}

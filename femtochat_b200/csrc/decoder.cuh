@@ -1,0 +1,136 @@
+// Decoders given as a list of layers (include/femto.h: femto_decoder_*): derived sizes, packed weights and workspace,
+// and the mixers' entry points.  Inference only; the state that outlives a call is in the cache (kv_cache.cuh).
+#pragma once
+#include <string>
+#include <vector>
+
+#include "kv_cache.cuh"
+
+static inline int round_up(int n, int k) { return (n + k - 1) / k * k; }
+
+// The packed input projection of a mixer is ONE product: its segments follow each other in the columns of a row of
+// `proj`, every segment starting at a multiple of 8 (16-byte loads, TMA operands); the gaps come from zero weights.
+struct DecLayer {
+  femto_layer_config c;
+  int own = 0;                        // layer that holds the tensors
+  std::vector<float> decay;
+  float* decay_dev = nullptr;
+  // element offsets into Theta of what is read there in fp32
+  long long norm1 = -1, norm1b = -1, norm2 = -1, norm2b = -1, mix_norm = -1, conv_q = -1, conv_k = -1, conv_v = -1,
+            a_log = -1, dt_bias = -1, dq_norm = -1, dkv_norm = -1;
+  // packed compute-type weights, row-major [out][in]
+  void *w_in = nullptr, *w_o = nullptr, *w_a2 = nullptr, *w_g2 = nullptr, *w_uq = nullptr, *w_kv = nullptr, *w_gu = nullptr,
+       *w_down = nullptr;
+  int n_in = 0;                       // columns of proj
+  int s_q = 0, s_k = 0, s_v = 0, s_g = 0, s_b = 0, s_a1 = 0, s_g1 = 0, s_dkv = 0;   // segment starts
+  int ra = 0, rg = 0;                 // decay_rank / gate_rank rounded up to 8
+  int qp = 0, lp = 0, ld = 0;         // q_rank, kv_rank rounded up to 8; pitch of a cached latent row
+  int ffp = 0;                        // ff rounded up to 32: the feed-forward's products are this wide
+  int qk_heads() const { return c.mixer == FEMTO_MIXER_CHANNEL_DELTA ? c.kv_heads : c.heads; }
+};
+
+struct DecoderStack {
+  femto_decoder_config cfg;
+  std::vector<DecLayer> layers;
+  std::vector<femto_decoder_tensor> tensors;
+  std::vector<femto_layer_config> layer_cfg;
+  long long nparams = 0, off_embed = 0, off_final = 0;
+  bool bf = false, weights_valid = false;
+  char* arena = nullptr;
+  unsigned int* status = nullptr;
+  void* embed = nullptr;              // [vocab][width] compute type: input table and output head
+  // workspace of one internal pass of up to max_rows tokens
+  int* tok0 = nullptr;
+  int* want = nullptr;                // [max_rows]
+  float* x = nullptr;                 // residual stream, fp32
+  void *hn = nullptr, *y = nullptr, *proj = nullptr, *mixo = nullptr, *mixg = nullptr, *gu = nullptr, *act = nullptr;
+  float *qn = nullptr, *kn = nullptr, *gd = nullptr, *beta = nullptr;
+  void *vv = nullptr, *g2 = nullptr, *cq = nullptr, *q = nullptr;
+  float* qabs = nullptr;              // latent attention, few rows: queries in the latent space
+  void* gemm_ws = nullptr;
+  size_t gemm_ws_bytes = 0;
+};
+
+int decoder_fill(DecoderStack* d, const femto_decoder_config* cfg);
+int decoder_create(const femto_decoder_config* cfg, femto_handle** out);
+void decoder_free(DecoderStack* d);
+int decoder_refresh(femto_handle* h, const float* theta, cudaStream_t s);
+int decoder_step(femto_handle* h, femto_kv_cache* c, const float* theta, const int* tokens, int B, int T, const int* h_want,
+                 int n_want, float* logits_out, float* residuals_out, cudaStream_t s);
+int decoder_cache_create(femto_handle* h, int max_batch, int max_len, femto_kv_cache** out);
+int decoder_cache_reset(femto_kv_cache* c, cudaStream_t s);
+
+// ---- streaming kernels (decoder_stream.cu) ------------------------------------------------------------------------
+template <typename T> struct DecStream {
+  // x = table[token] (fp32), h = rms_norm(x) w
+  static int embed(const T* table, const int* tokens, int ld_tok, int B, int T_, int base, int vocab, const float* w, float* x,
+                   T* h, int d, float eps, unsigned int* status, cudaStream_t s);
+  // x += m rms_norm(y) w_post;  h = rms_norm(x) w_pre (skipped when h is NULL)
+  static int resid_norm(float* x, const T* y, const float* w_post, float m, const float* w_pre, T* h, int rows, int d, float eps,
+                        cudaStream_t s);
+  // h[i] = rms_norm(x[row i]) w, row i = want ? want[i] : (i + 1) stride - 1
+  static int gather_norm(const float* x, const int* want, int stride, const float* w, T* h, int n, int d, float eps,
+                         cudaStream_t s);
+  // out[r][g] = rms_norm over each of `groups` runs of `size` of in[r], times w (size, or groups*size when w_all), times sigmoid(gate)
+  static int gated_norm(const T* in, const float* w, bool w_all, const T* gate, long long ldg, T* out, int rows, int groups, int size,
+                        float eps, cudaStream_t s);
+  // out[r][0..size) = rms_norm(in[r]) w, out[r][size..ldo) = 0
+  static int norm_cols(const T* in, long long ldi, const float* w, T* out, long long ldo, int rows, int size, float eps, cudaStream_t s);
+  // act[r][j] = silu(gate) * up from rows of interleaved groups of 32 gate and 32 up columns
+  static int gated_mlp(const T* gu, T* act, int rows, int ffp, cudaStream_t s);
+};
+// weight packing: dst[(r / group) * step + r % group + dst_row][c] = src[r][c], c < cols (dst pitch ldd)
+template <typename T>
+int pack_rows(const float* src, int rows, int cols, T* dst, long long ldd, int dst_row, int group, int step, cudaStream_t s);
+
+// ---- products -------------------------------------------------------------------------------------------------------
+// C[M][N] = X[M][K] W[N][K]^T; epi EPI_STORE (compute type) or EPI_F32.  Up to 8 rows stream the weights once through
+// a row-dot kernel, more rows take the tensor-core GEMM.
+template <typename T>
+int rows_linear(DecoderStack* d, const void* X, long long ldx, const void* W, long long ldw, void* C, long long ldc, int M, int N, int K,
+                int epi, cudaStream_t s);
+
+// ---- recurrences (recurrence.cu) ------------------------------------------------------------------------------------
+struct RecurrenceArgs {
+  const void *q = nullptr, *k = nullptr, *v = nullptr;   // q, k: fp32 rows when qk_f32, else the compute type with silu applied here
+  long long ldq = 0, ldk = 0, ldv = 0;
+  const float* g = nullptr;      // [rows][heads * dim] decays per channel, or NULL: decay[heads]
+  const float* beta = nullptr;   // [rows][heads], or NULL: plain sum of outer products
+  const float* decay = nullptr;
+  float* S = nullptr;            // [B][heads][vdim][dim]
+  void* o = nullptr;             // [rows][heads * vdim]
+  int B = 0, T = 0, heads = 0, qk_heads = 0, dim = 0, vdim = 0;
+};
+template <typename T> int recurrence(const RecurrenceArgs& a, cudaStream_t s);
+
+// Short causal convolutions + silu, unit vectors, decays and step sizes of the gated delta rule.
+struct DeltaPrepArgs {
+  const void* proj = nullptr; long long ldp = 0;
+  int s_q = 0, s_k = 0, s_v = 0, s_b = 0;
+  const float *conv_q = nullptr, *conv_k = nullptr, *conv_v = nullptr, *a_log = nullptr, *dt_bias = nullptr;
+  const void* tail_in = nullptr; void* tail_out = nullptr;
+  float *qn = nullptr, *kn = nullptr, *gd = nullptr, *beta = nullptr; void* vv = nullptr;   // gd holds W_a2 W_a1 h on entry
+  int B = 0, T = 0, heads = 0, kv_heads = 0, dim = 0, vdim = 0, taps = 0;
+};
+template <typename T> int delta_prep(const DeltaPrepArgs& a, cudaStream_t s);
+
+// ---- latent attention (latent_attention.cu) -------------------------------------------------------------------------
+struct LatentArgs {
+  void* q = nullptr;             // [rows][heads (dim + rot_dim)], rotated in place by latent_prep
+  const void* dkv = nullptr; long long ld_dkv = 0;     // new rows of W_dkv h (kv_rank, rot_dim)
+  const float* dkv_norm = nullptr;
+  const void* gate = nullptr; long long ld_gate = 0;   // one logit per head
+  void* latent = nullptr;        // cache [maxB][maxT][ld]
+  int ld = 0, lp = 0, maxT = 0;
+  const void* w_kv = nullptr;    // [heads dim + heads vdim][lp]
+  void* kv = nullptr;            // expanded keys and values, [B][maxT][heads (dim + vdim)]
+  float* qabs = nullptr; float* part = nullptr; size_t part_floats = 0;
+  void* o = nullptr;             // [rows][heads vdim]
+  int B = 0, T = 0, first = 0, heads = 0, dim = 0, rot_dim = 0, rot_dims = 0, vdim = 0, kv_rank = 0;
+  float scale = 1.f, eps = 0.f; double rot_base = 1.0;
+  DecoderStack* d = nullptr;
+};
+template <typename T> int latent_prep(const LatentArgs& a, cudaStream_t s);
+template <typename T> int latent_attention(const LatentArgs& a, cudaStream_t s);
+constexpr int LATENT_FEW = 8;          // columns with at most this many new tokens attend in the latent space
+constexpr int LATENT_MAX_SPLITS = 64;

@@ -1,0 +1,338 @@
+// HBM-streaming kernels of the layer-listing decoders: embedding, norms around each sublayer with the fp32 residual
+// sum, gated norms, the feed-forward's gate, weight packing, and the product of a few rows with a [out][in] weight.
+#include "decoder.cuh"
+
+namespace {
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+
+// Sum over the 256 threads of a block; every thread gets it.
+__device__ __forceinline__ float block_sum(float v) {
+  __shared__ float red[8];
+  v = warp_sum(v);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; i++) t += red[i];
+  return t;
+}
+
+constexpr int RT = 256;   // threads of a row kernel: one row per block
+
+template <typename T>
+__global__ void __launch_bounds__(RT) k_dec_embed(const T* __restrict__ table, const int* __restrict__ tokens, int ld_tok, int T_,
+                                                  int base, int vocab, const float* __restrict__ w, float* __restrict__ x,
+                                                  T* __restrict__ h, int d, float eps, unsigned int* status) {
+  pdl_trigger();
+  const int row = blockIdx.x;
+  int tk = tokens[(long long)(row / T_) * ld_tok + row % T_] - base;
+  if (tk < 0 || tk >= vocab) { if (threadIdx.x == 0) atomicOr(status, ST_BAD_TOKEN); tk = min(max(tk, 0), vocab - 1); }
+  const T* src = table + (long long)tk * d;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < d; c += RT) { const float f = to_f<T>(src[c]); ss += f * f; }
+  const float inv = 1.f / sqrtf(block_sum(ss) / d + eps);
+  for (int c = threadIdx.x; c < d; c += RT) {
+    const float f = to_f<T>(src[c]);
+    x[(long long)row * d + c] = f;
+    h[(long long)row * d + c] = from_f<T>(f * inv * w[c]);
+  }
+}
+
+// NV 4-element vectors per thread stay in registers between the two norms (NV = 0: any width, through memory).
+template <typename T, int NV>
+__global__ void __launch_bounds__(RT) k_resid_norm(float* __restrict__ x, const T* __restrict__ y, const float* __restrict__ w_post,
+                                                   float m, const float* __restrict__ w_pre, T* __restrict__ h, int d, float eps) {
+  pdl_trigger();
+  const long long base = (long long)blockIdx.x * d;
+  if constexpr (NV > 0) {
+    float f[NV][4], r[NV][4];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+      const int c = (i * RT + threadIdx.x) * 4;
+      if (c < d) {
+        if constexpr (sizeof(T) == 4) {
+          const float4 q = *reinterpret_cast<const float4*>(y + base + c);
+          f[i][0] = q.x; f[i][1] = q.y; f[i][2] = q.z; f[i][3] = q.w;
+        } else {
+          const uint2 q = *reinterpret_cast<const uint2*>(y + base + c);
+          const bf16* hq = reinterpret_cast<const bf16*>(&q);
+#pragma unroll
+          for (int e = 0; e < 4; e++) f[i][e] = __bfloat162float(hq[e]);
+        }
+        const float4 q = *reinterpret_cast<const float4*>(x + base + c);
+        r[i][0] = q.x; r[i][1] = q.y; r[i][2] = q.z; r[i][3] = q.w;
+#pragma unroll
+        for (int e = 0; e < 4; e++) ss += f[i][e] * f[i][e];
+      }
+    }
+    float inv = 1.f / sqrtf(block_sum(ss) / d + eps);
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+      const int c = (i * RT + threadIdx.x) * 4;
+      if (c < d) {
+        const float4 w = *reinterpret_cast<const float4*>(w_post + c);
+        r[i][0] += m * (f[i][0] * inv * w.x); r[i][1] += m * (f[i][1] * inv * w.y);
+        r[i][2] += m * (f[i][2] * inv * w.z); r[i][3] += m * (f[i][3] * inv * w.w);
+        *reinterpret_cast<float4*>(x + base + c) = make_float4(r[i][0], r[i][1], r[i][2], r[i][3]);
+#pragma unroll
+        for (int e = 0; e < 4; e++) ss += r[i][e] * r[i][e];
+      }
+    }
+    if (!h) return;
+    inv = 1.f / sqrtf(block_sum(ss) / d + eps);
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+      const int c = (i * RT + threadIdx.x) * 4;
+      if (c < d) {
+        const float4 w = *reinterpret_cast<const float4*>(w_pre + c);
+        const float o[4] = {r[i][0] * inv * w.x, r[i][1] * inv * w.y, r[i][2] * inv * w.z, r[i][3] * inv * w.w};
+        if constexpr (sizeof(T) == 4) {
+          *reinterpret_cast<float4*>(h + base + c) = make_float4(o[0], o[1], o[2], o[3]);
+        } else {
+          uint2 q;
+          __nv_bfloat162* hq = reinterpret_cast<__nv_bfloat162*>(&q);
+          hq[0] = __floats2bfloat162_rn(o[0], o[1]); hq[1] = __floats2bfloat162_rn(o[2], o[3]);
+          *reinterpret_cast<uint2*>(h + base + c) = q;
+        }
+      }
+    }
+  } else {
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < d; c += RT) { const float f = to_f<T>(y[base + c]); ss += f * f; }
+    float inv = 1.f / sqrtf(block_sum(ss) / d + eps);
+    ss = 0.f;
+    for (int c = threadIdx.x; c < d; c += RT) {
+      const float r = x[base + c] + m * (to_f<T>(y[base + c]) * inv * w_post[c]);
+      x[base + c] = r;
+      ss += r * r;
+    }
+    if (!h) return;
+    inv = 1.f / sqrtf(block_sum(ss) / d + eps);
+    for (int c = threadIdx.x; c < d; c += RT) h[base + c] = from_f<T>(x[base + c] * inv * w_pre[c]);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(RT) k_gather_norm(const float* __restrict__ x, const int* __restrict__ want, int stride,
+                                                    const float* __restrict__ w, T* __restrict__ h, int d, float eps) {
+  pdl_trigger();
+  const int i = blockIdx.x;
+  const float* src = x + (long long)(want ? want[i] : (i + 1) * stride - 1) * d;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < d; c += RT) ss += src[c] * src[c];
+  const float inv = 1.f / sqrtf(block_sum(ss) / d + eps);
+  for (int c = threadIdx.x; c < d; c += RT) h[(long long)i * d + c] = from_f<T>(src[c] * inv * w[c]);
+}
+
+// One warp per (row, group).
+template <typename T, int V>
+__global__ void __launch_bounds__(256) k_gated_norm(const T* __restrict__ in, const float* __restrict__ w, int w_all,
+                                                    const T* __restrict__ gate, long long ldg, T* __restrict__ out, long long n,
+                                                    int groups, int size, float eps) {
+  pdl_trigger();
+  const long long it = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (it >= n) return;
+  const int lane = threadIdx.x & 31, g = (int)(it % groups);
+  const long long row = it / groups;
+  const T* a = in + it * size;
+  const T* gt = gate + row * ldg + (long long)g * size;
+  const float* wg = w + (w_all ? (long long)g * size : 0);
+  float ss = 0.f;
+  for (int c = lane * V; c < size; c += 32 * V) {
+    float f[V];
+    load_vec<T, V>(a + c, f);
+#pragma unroll
+    for (int e = 0; e < V; e++) ss += f[e] * f[e];
+  }
+  const float inv = 1.f / sqrtf(warp_sum(ss) / size + eps);
+  for (int c = lane * V; c < size; c += 32 * V) {
+    float f[V], z[V];
+    load_vec<T, V>(a + c, f);
+    load_vec<T, V>(gt + c, z);
+#pragma unroll
+    for (int e = 0; e < V; e++) f[e] = f[e] * inv * wg[c + e] * sigmoid_f(z[e]);
+    store_vec<T, V>(out + it * size + c, f);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) k_norm_cols(const T* __restrict__ in, long long ldi, const float* __restrict__ w, T* __restrict__ out,
+                                                   long long ldo, int rows, int size, float eps) {
+  pdl_trigger();
+  const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= rows) return;
+  const T* a = in + (long long)row * ldi;
+  float ss = 0.f;
+  for (int c = lane; c < size; c += 32) { const float f = to_f<T>(a[c]); ss += f * f; }
+  const float inv = 1.f / sqrtf(warp_sum(ss) / size + eps);
+  for (int c = lane; c < ldo; c += 32) out[(long long)row * ldo + c] = from_f<T>(c < size ? to_f<T>(a[c]) * inv * w[c] : 0.f);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) k_gated_mlp(const T* __restrict__ gu, T* __restrict__ act, long long n, int ffp) {
+  pdl_trigger();
+  constexpr int V = VecN<T>::n;
+  const long long i = ((long long)blockIdx.x * 256 + threadIdx.x) * V;
+  if (i >= n) return;
+  const long long row = i / ffp;
+  const int j = (int)(i % ffp);
+  const T* src = gu + row * 2 * ffp + (j >> 5) * 64 + (j & 31);
+  float a[V], b[V];
+  load_vec<T, V>(src, a);
+  load_vec<T, V>(src + 32, b);
+#pragma unroll
+  for (int e = 0; e < V; e++) a[e] = a[e] * sigmoid_f(a[e]) * b[e];
+  store_vec<T, V>(act + i, a);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) k_pack_rows(const float* __restrict__ src, long long n, int cols, T* __restrict__ dst, long long ldd,
+                                                   int dst_row, int group, int step) {
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= n) return;
+  const int r = (int)(i / cols), c = (int)(i % cols);
+  dst[(long long)(dst_row + (r / group) * step + r % group) * ldd + c] = from_f<T>(src[i]);
+}
+
+// C[m][n] = sum_k X[m][k] W[n][k] for M <= 8 rows: one warp per output column, 16-byte loads of W, X in shared memory.
+// Every weight is read exactly once.
+constexpr int RL_ROWS = 8;
+template <typename T, int MR, bool VEC>
+__global__ void __launch_bounds__(256) k_rows_linear(const T* __restrict__ X, long long ldx, const T* __restrict__ W, long long ldw,
+                                                     void* __restrict__ C, long long ldc, int M, int N, int K, int f32_out) {
+  pdl_trigger();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int n = blockIdx.x * 8 + warp;
+  if (n >= N) return;
+  const T* wr = W + (long long)n * ldw;
+  float acc[MR];
+#pragma unroll
+  for (int m = 0; m < MR; m++) acc[m] = 0.f;
+  if constexpr (VEC) {
+    constexpr int V = VecN<T>::n;
+#pragma unroll 4
+    for (int k = lane * V; k < K; k += 32 * V) {
+      float w[V];
+      load_vec<T, V>(wr + k, w);
+#pragma unroll
+      for (int m = 0; m < MR; m++) {
+        if (m < M) {
+          float x[V];
+          load_vec<T, V>(X + m * ldx + k, x);
+#pragma unroll
+          for (int e = 0; e < V; e++) acc[m] = fmaf(x[e], w[e], acc[m]);
+        }
+      }
+    }
+  } else {
+    for (int k = lane; k < K; k += 32) {
+      const float w = to_f<T>(wr[k]);
+#pragma unroll
+      for (int m = 0; m < MR; m++)
+        if (m < M) acc[m] = fmaf(to_f<T>(X[m * ldx + k]), w, acc[m]);
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < MR; m++) {
+    if (m >= M) break;
+    const float v = warp_sum(acc[m]);
+    if (lane == 0) {
+      if (f32_out) reinterpret_cast<float*>(C)[m * ldc + n] = v;
+      else reinterpret_cast<T*>(C)[m * ldc + n] = from_f<T>(v);
+    }
+  }
+}
+
+}  // namespace
+
+template <typename T>
+int DecStream<T>::embed(const T* table, const int* tokens, int ld_tok, int B, int T_, int base, int vocab, const float* w, float* x, T* h,
+                        int d, float eps, unsigned int* status, cudaStream_t s) {
+  k_dec_embed<T><<<B * T_, RT, 0, s>>>(table, tokens, ld_tok, T_, base, vocab, w, x, h, d, eps, status);
+  KERNEL_CHECK();
+  return 0;
+}
+template <typename T>
+int DecStream<T>::resid_norm(float* x, const T* y, const float* w_post, float m, const float* w_pre, T* h, int rows, int d, float eps,
+                             cudaStream_t s) {
+  const bool vec = (d & 3) == 0 && aligned16(x) && aligned16(y) && aligned16(w_post) && (!h || (aligned16(w_pre) && aligned16(h)));
+  const int nv = vec ? cdiv(d, RT * 4) : 0;
+  if (nv == 1) k_resid_norm<T, 1><<<rows, RT, 0, s>>>(x, y, w_post, m, w_pre, h, d, eps);
+  else if (nv == 2) k_resid_norm<T, 2><<<rows, RT, 0, s>>>(x, y, w_post, m, w_pre, h, d, eps);
+  else if (nv == 3 || nv == 4) k_resid_norm<T, 4><<<rows, RT, 0, s>>>(x, y, w_post, m, w_pre, h, d, eps);
+  else k_resid_norm<T, 0><<<rows, RT, 0, s>>>(x, y, w_post, m, w_pre, h, d, eps);
+  KERNEL_CHECK();
+  return 0;
+}
+template <typename T>
+int DecStream<T>::gather_norm(const float* x, const int* want, int stride, const float* w, T* h, int n, int d, float eps, cudaStream_t s) {
+  k_gather_norm<T><<<n, RT, 0, s>>>(x, want, stride, w, h, d, eps);
+  KERNEL_CHECK();
+  return 0;
+}
+template <typename T>
+int DecStream<T>::gated_norm(const T* in, const float* w, bool w_all, const T* gate, long long ldg, T* out, int rows, int groups, int size,
+                             float eps, cudaStream_t s) {
+  const long long n = (long long)rows * groups;
+  constexpr int V = VecN<T>::n;
+  if (size % V == 0 && ldg % V == 0 && aligned16(in) && aligned16(gate) && aligned16(out))
+    k_gated_norm<T, V><<<cdiv(n, 8), 256, 0, s>>>(in, w, w_all, gate, ldg, out, n, groups, size, eps);
+  else
+    k_gated_norm<T, 1><<<cdiv(n, 8), 256, 0, s>>>(in, w, w_all, gate, ldg, out, n, groups, size, eps);
+  KERNEL_CHECK();
+  return 0;
+}
+template <typename T>
+int DecStream<T>::norm_cols(const T* in, long long ldi, const float* w, T* out, long long ldo, int rows, int size, float eps, cudaStream_t s) {
+  k_norm_cols<T><<<cdiv(rows, 8), 256, 0, s>>>(in, ldi, w, out, ldo, rows, size, eps);
+  KERNEL_CHECK();
+  return 0;
+}
+template <typename T> int DecStream<T>::gated_mlp(const T* gu, T* act, int rows, int ffp, cudaStream_t s) {
+  const long long n = (long long)rows * ffp;
+  k_gated_mlp<T><<<cdiv(n, 256 * VecN<T>::n), 256, 0, s>>>(gu, act, n, ffp);
+  KERNEL_CHECK();
+  return 0;
+}
+template struct DecStream<float>;
+template struct DecStream<bf16>;
+
+template <typename T>
+int pack_rows(const float* src, int rows, int cols, T* dst, long long ldd, int dst_row, int group, int step, cudaStream_t s) {
+  const long long n = (long long)rows * cols;
+  k_pack_rows<T><<<cdiv(n, 256), 256, 0, s>>>(src, n, cols, dst, ldd, dst_row, group, step);
+  KERNEL_CHECK();
+  return 0;
+}
+template int pack_rows<float>(const float*, int, int, float*, long long, int, int, int, cudaStream_t);
+template int pack_rows<bf16>(const float*, int, int, bf16*, long long, int, int, int, cudaStream_t);
+
+template <typename T>
+int rows_linear(DecoderStack* d, const void* X, long long ldx, const void* W, long long ldw, void* C, long long ldc, int M, int N, int K,
+                int epi, cudaStream_t s) {
+  if (M <= RL_ROWS) {
+    constexpr int V = VecN<T>::n;
+    const bool vec = K % V == 0 && ldx % V == 0 && ldw % V == 0 && aligned16(X) && aligned16(W);
+    const int grid = cdiv(N, 8), f32 = epi == EPI_F32;
+#define LAUNCH(MR, VEC) k_rows_linear<T, MR, VEC><<<grid, 256, 0, s>>>((const T*)X, ldx, (const T*)W, ldw, C, ldc, M, N, K, f32)
+    if (!vec) LAUNCH(8, false);
+    else if (M == 1) LAUNCH(1, true);
+    else if (M == 2) LAUNCH(2, true);
+    else if (M <= 4) LAUNCH(4, true);
+    else LAUNCH(8, true);
+#undef LAUNCH
+    KERNEL_CHECK();
+    return 0;
+  }
+  GemmArgs g;
+  g.ws = d->gemm_ws; g.ws_bytes = d->gemm_ws_bytes; g.status = d->status;
+  g.A = X; g.lda = ldx; g.a_kmajor = true; g.B = W; g.ldb = ldw; g.b_kmajor = true;
+  g.C = C; g.ldc = ldc; g.M = M; g.N = N; g.K = K; g.epi = epi; g.beta = 0.f;
+  return gemm<T>(g, s);
+}
+template int rows_linear<float>(DecoderStack*, const void*, long long, const void*, long long, void*, long long, int, int, int, int, cudaStream_t);
+template int rows_linear<bf16>(DecoderStack*, const void*, long long, const void*, long long, void*, long long, int, int, int, int, cudaStream_t);

@@ -586,6 +586,7 @@ static int step_t(femto_handle* h, const float* theta, float* delta, const int* 
 int model_step(femto_handle* h, const float* theta, float* delta, const int* tokens, const int* targets,
                const int* positions, int B, int reduction, bool backward, bool accumulate, float* loss_out,
                int* nvalid_out, cudaStream_t s, float* logits_out, float* token_losses_out, const StepExtra* ex) {
+  if (h && h->dec) return femto_fail(FEMTO_ERR_UNSUPPORTED, "a decoder that lists its layers runs through femto_prefill, femto_decode_step and femto_decoder_step");
   const bool prompt = ex && ex->cache && ex->last_logits;
   if (!h || !theta || !tokens || (!logits_out && !prompt && (!targets || (!loss_out && !token_losses_out))))
     return femto_fail(FEMTO_ERR_ARG, "NULL argument");

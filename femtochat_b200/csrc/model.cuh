@@ -19,6 +19,7 @@ struct LayerBuf {
 };
 
 struct DpState;  // NCCL communicator (dp.cu)
+struct DecoderStack;   // a model that lists its layers (decoder.cuh)
 
 struct femto_handle {
   femto_config cfg;
@@ -73,6 +74,7 @@ struct femto_handle {
   DpState* dp = nullptr;
   bool overlap_sync = false;     // sum delta over ranks in buckets while the reverse pass runs
   bool delta_synced = false;     // the last step already reduced delta (femto_grad_sync only joins)
+  DecoderStack* dec = nullptr;   // set: this handle is a layer-listing decoder and none of the GPT fields above is used
   std::string err;
 };
 

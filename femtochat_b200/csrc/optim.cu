@@ -611,6 +611,7 @@ int optimizer_state_sizes(femto_handle* h, long long* out4) {
 int optimizer_create(femto_handle* h, const femto_optimizer_config* cfg, float* adam_m, float* adam_v, float* muon_m,
                      float* muon_v, femto_optimizer** out) {
   if (!h || !cfg || !adam_m || !adam_v || !muon_m || !muon_v || !out) return femto_fail(FEMTO_ERR_ARG, "NULL argument");
+  if (h->dec) return femto_fail(FEMTO_ERR_UNSUPPORTED, "a decoder that lists its layers does not train");
   if (cfg->ns_steps < 0 || cfg->ns_steps > 5) return femto_fail(FEMTO_ERR_ARG, "ns_steps must be 0..5");
   femto_optimizer* o = new femto_optimizer();
   o->h = h; o->cfg = *cfg; o->adam_m = adam_m; o->adam_v = adam_v; o->muon_m = muon_m; o->muon_v = muon_v;

@@ -7,6 +7,7 @@ import math
 from typing import Optional
 
 from . import _lib
+from .handle import Handle
 from .parameters import GPTConfig, Layout, Params, parameter_layout, paramview
 
 
@@ -56,13 +57,14 @@ def initialize_(params, layout: Layout, seed: int = 123, all_nonzero: bool = Fal
     uniform(layout.smear_gate, 0.0, 0.02)
 
 
-class GradientState:
+class GradientState(Handle):
     """What `gradient_state` returns (ext/FemtoChatEnzymeExt.jl:27-36): built once per
     (config, batch shape), reused for every batch.  Owns the library handle."""
 
     def __init__(self, config: GPTConfig, max_batch: int, compute_type="float32", short_window: int = 0,
                  doc_mask: bool = False, index_base: int = 1, rank: int = 0, world: int = 1, nccl_id: bytes = None):
         import torch
+        super().__init__()
         self.config = config
         self.max_batch = max_batch
         self.compute_type = compute_type
@@ -76,28 +78,6 @@ class GradientState:
         self._loss = torch.zeros(1, dtype=torch.float32, device="cuda")
         self._nvalid = torch.zeros(1, dtype=torch.int32, device="cuda")
         self._weights_of = None
-
-    def refresh_weights(self, theta) -> None:
-        _lib.check(_lib.lib().femto_refresh_weights(self.h, _lib.ptr(theta), _lib.stream_ptr()))
-
-    def status_word(self) -> int:
-        out = C.c_int32(0)
-        _lib.check(_lib.lib().femto_status_word(self.h, C.byref(out)))
-        return out.value
-
-    def launch_count(self) -> int:
-        return int(_lib.lib().femto_launch_count(self.h))
-
-    def close(self) -> None:
-        if self.h:
-            _lib.lib().femto_destroy(self.h)
-            self.h = None
-
-    def __del__(self):
-        try:
-            self.close()
-        except Exception:
-            pass
 
 
 def gradient_state(params: Params, config: GPTConfig, layout: Layout, tokens, targets, positions=None, **options):
@@ -163,6 +143,24 @@ class GPT:
         self.compute_type = compute_type
         self.options = options
         self._state: Optional[GradientState] = None
+
+    @property
+    def index_base(self) -> int:
+        return self.options.get("index_base", 1)
+
+    @classmethod
+    def from_weights(cls, config_json: dict, tensors, compute_type="float32", **options) -> "GPT":
+        """`config_json`: GPTConfig's fields beside "architecture"; `tensors`: one row-major [in][out] tensor per entry of
+        the layout, named "wte", "lm_head", "smear_gate", "lam_s", "lam_y" and "l<block>.<name>"."""
+        import torch
+        config = GPTConfig(**{k: v for k, v in config_json.items() if k in GPTConfig.__dataclass_fields__})
+        layout = parameter_layout(config)
+        theta = torch.zeros(layout.nparams, dtype=torch.float32, device="cuda")
+        for name, spec in layout.named():
+            if name not in tensors:
+                raise ValueError(f"no tensor {name}")
+            theta[spec.offset:spec.offset + spec.size].copy_(tensors[name].reshape(-1))
+        return cls(Params(theta), config, layout, compute_type=compute_type, **options)
 
     def state(self, B: int) -> GradientState:
         if self._state is None or self._state.max_batch < B:

@@ -77,6 +77,16 @@ class Layout:
     padded_vocab_size: int
     nparams: int
 
+    def named(self):
+        """(name, spec) of every tensor; a block's tensors are called l<block>.<name>."""
+        for name, spec in (("wte", self.embedding), ("lm_head", self.lm_head), ("smear_gate", self.smear_gate), ("lam_s", self.lam_s),
+                           ("lam_y", self.lam_y)):
+            yield name, spec
+        for i, blk in enumerate(self.blocks):
+            for name, spec in blk.items():
+                if spec is not None:
+                    yield f"l{i}.{name}", spec
+
 
 def parameter_layout(config: GPTConfig, pad_vocab_size_to: int = 64) -> Layout:
     """src/parameters.jl:219-337."""
@@ -119,12 +129,16 @@ def window_sizes(config: GPTConfig, short_window: int = 0) -> List[Tuple[int, in
 
 
 class Params:
-    """src/parameters.jl:31-62: flat parameter vector Θ and its fp32 gradient vector δ."""
+    """src/parameters.jl:31-62: flat parameter vector Θ and its fp32 gradient vector δ (delta=False: none, for models
+    that only run forward)."""
 
     def __init__(self, theta, delta=None):
         import torch
         if theta.dim() != 1:
             raise ValueError("Θ must be a vector")
+        if delta is False:
+            self.theta, self.delta = theta, None
+            return
         if delta is None:
             delta = torch.zeros_like(theta, dtype=torch.float32)
         if delta.dtype != torch.float32:

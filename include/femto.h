@@ -141,6 +141,60 @@ int32_t femto_prefill(femto_handle* h, femto_kv_cache* c, const float* theta, co
 int32_t femto_decode_step(femto_handle* h, femto_kv_cache* c, const float* theta, const int32_t* tokens,
                           const int32_t* positions, int32_t B, float* logits_out, void* stream);
 
+/* ---- decoders that list their layers ------------------------------------------------------------------------------ */
+/* A decoder-only model given as a list of layers, each a token mixer and an optional gated feed-forward, with an RMS norm
+ * before and after both:  x += m norm1b(mixer(norm1(x))),  x += m norm2b(mlp(norm2(x)));  the residual stream x is fp32 in
+ * every build.  No counterpart in the reference: the handle is a femto_handle like any other, and
+ * femto_refresh_weights, femto_kv_cache_*, femto_prefill, femto_decode_step, femto_status_word, femto_launch_count and
+ * femto_destroy take it; calls that train do not (FEMTO_ERR_UNSUPPORTED).  The model "Virolorn" is built of these. */
+#define FEMTO_MIXER_LIGHTNING 1        /* S <- decay_h S + k v^T, o = S^T q, one constant decay per head */
+#define FEMTO_MIXER_CHANNEL_DELTA 2    /* gated delta rule with a data-dependent decay per head and key channel */
+#define FEMTO_MIXER_LATENT_ATTENTION 3 /* softmax attention over a cached low-rank latent plus one rotated key part */
+
+typedef struct femto_layer_config {
+  int32_t mixer;       /* FEMTO_MIXER_* */
+  int32_t weights_of;  /* -1, or the layer whose tensors this one uses (it keeps a state of its own) */
+  int32_t heads, kv_heads, dim, vdim; /* dim: query/key size per head (unrotated part for latent attention) */
+  int32_t conv;        /* CHANNEL_DELTA: taps of the causal convolutions on q, k and v */
+  int32_t decay_rank, gate_rank;      /* CHANNEL_DELTA: inner sizes of the two low-rank projections */
+  int32_t q_rank, kv_rank, rot_dim, rot_dims; /* LATENT_ATTENTION; the first rot_dims of the rot_dim part are rotated */
+  int32_t ff;          /* inner size of the gated feed-forward, 0 = the layer has none */
+  float scale;         /* LATENT_ATTENTION: factor on the scores */
+  double rot_base;     /* LATENT_ATTENTION: pair i turns by position * rot_base^(-2i/rot_dims) */
+  const float* h_decay; /* LIGHTNING: [heads], host memory, read during the call */
+} femto_layer_config;
+
+typedef struct femto_decoder_config {
+  int32_t vocab, width, n_layer;
+  int32_t compute_dtype; /* FEMTO_F32: everything in fp32; FEMTO_BF16: products and activations in bf16 */
+  int32_t index_base;    /* token ids start at 0 or 1 */
+  int32_t max_batch;     /* most columns of a call */
+  int32_t max_rows;      /* tokens (over all columns) that one internal pass takes; longer prompts are fed in portions */
+  float norm_eps, residual_mult;
+  const femto_layer_config* h_layers; /* [n_layer], host memory */
+} femto_decoder_config;
+
+/* One tensor of the flat fp32 parameter vector: a weight is row-major [rows][cols] = [out][in]. */
+typedef struct femto_decoder_tensor {
+  char name[48]; /* "embed", "final.norm", "l<i>.norm1", "l<i>.mix.q", "l<i>.mlp.gate", ... */
+  int64_t offset, rows, cols; /* cols == 0: a vector */
+} femto_decoder_tensor;
+
+/* Writes up to `capacity` descriptors in flat order; returns the number of tensors (or < 0). */
+int32_t femto_decoder_layout(const femto_decoder_config* h_cfg, femto_decoder_tensor* h_out, int32_t capacity);
+int64_t femto_decoder_nparams(const femto_decoder_config* h_cfg);
+int32_t femto_decoder_create(const femto_decoder_config* h_cfg, femto_handle** h_out);
+/* The next T tokens of every column (int32 [B][T]) from the cache and states that earlier calls left; any T >= 1.
+ * Logits fp32 [n_want][vocab] of the positions h_want (host array, ascending indices b*T + t), or, with h_want NULL, of
+ * each column's last position ([B][vocab]; logits_out may then be NULL: none are computed).  An empty cache starts B
+ * columns.  residuals_out (NULL, or fp32 [n_layer][B*T][width]) receives the residual stream after every layer; with it
+ * B*T may not exceed max_rows.  femto_prefill is femto_kv_cache_reset + this call, femto_decode_step this call with T = 1. */
+int32_t femto_decoder_step(femto_handle* h, femto_kv_cache* c, const float* theta, const int32_t* tokens, int32_t B,
+                           int32_t T, const int32_t* h_want, int32_t n_want, float* logits_out, float* residuals_out,
+                           void* stream);
+/* Forgets what the cache holds (recurrent states back to zero), so that another request can use it. */
+int32_t femto_kv_cache_reset(femto_kv_cache* c, void* stream);
+
 /* ---- batch producer (src/dataloader.jl:241-274; scripts/train.jl:144-145) ---------------------- */
 /* One run of a document inside a batch column: rows row..row+n-1 of column col take the tokens
  * stream[src..src+n-1]; positions count up from pos0; the target of the last row is `next` (0-based id of the
