@@ -172,6 +172,14 @@ void carve(DecoderStack* d, Carver& b) {
   b.take(d->vv, es * R * vv); b.take(d->g2, es * R * g2);
   b.take(d->cq, es * R * cq); b.take(d->q, es * R * q);
   b.take(d->qabs, 4 * std::min(R, (size_t)d->cfg.max_batch * LATENT_FEW) * qa);
+  size_t items = 0;
+  for (const auto& l : d->layers)
+    if (d->bf && l.c.mixer != FEMTO_MIXER_LATENT_ATTENTION && l.c.dim <= 128 && l.c.vdim <= 128)
+      items = std::max(items, chunked_recurrence_item_bytes(l.c.dim, l.c.vdim) * l.c.heads * d->cfg.max_batch);
+  // the chunks of a segment go through memory once between the two kernels: a segment that stays in L2, at least one chunk
+  const size_t chunks = items ? std::max<size_t>(1, std::min<size_t>(((size_t)80 << 20) / items, R / d->cfg.max_batch / 64 + 1)) : 0;
+  d->chunk_ws_bytes = items * chunks;
+  b.take(d->chunk_ws, d->chunk_ws_bytes);
   d->gemm_ws_bytes = (size_t)64 << 20;
   b.take(d->gemm_ws, d->gemm_ws_bytes);
 }
@@ -333,10 +341,14 @@ static int mixer_t(DecoderStack* d, femto_kv_cache* c, int i, const float* theta
   FEMTO_TRY(rows_linear<T>(d, d->hn, w, l.w_in, w, proj, l.n_in, R, l.n_in, w, EPI_STORE, s));
   T* out = (T*)d->mixg;
   if (q.mixer == FEMTO_MIXER_LIGHTNING) {
+    ChunkArgs ca;
+    ca.proj = proj; ca.ldp = l.n_in; ca.s_q = l.s_q; ca.s_k = l.s_k; ca.s_v = l.s_v; ca.decay = l.decay_dev; ca.S = st.S; ca.o = d->mixo;
+    ca.B = B; ca.T = Tn; ca.heads = ca.qk_heads = H; ca.dim = D; ca.vdim = E; ca.ws = d->chunk_ws; ca.ws_bytes = d->chunk_ws_bytes; ca.status = d->status;
     RecurrenceArgs a;
     a.q = proj + l.s_q; a.k = proj + l.s_k; a.v = proj + l.s_v; a.ldq = a.ldk = a.ldv = l.n_in;
     a.decay = l.decay_dev; a.S = st.S; a.o = d->mixo; a.B = B; a.T = Tn; a.heads = a.qk_heads = H; a.dim = D; a.vdim = E;
-    FEMTO_TRY(recurrence<T>(a, s));
+    if (sizeof(T) == 2 && chunked_recurrence_supported(ca)) FEMTO_TRY(chunked_recurrence(ca, s));
+    else FEMTO_TRY(recurrence<T>(a, s));
     FEMTO_TRY(S::gated_norm((const T*)d->mixo, theta + l.mix_norm, true, proj + l.s_g, l.n_in, out, R, 1, H * E, eps, s));
   } else if (q.mixer == FEMTO_MIXER_CHANNEL_DELTA) {
     FEMTO_TRY(rows_linear<T>(d, proj + l.s_a1, l.n_in, l.w_a2, l.ra, d->gd, H * D, R, H * D, l.ra, EPI_F32, s));
@@ -347,12 +359,19 @@ static int mixer_t(DecoderStack* d, femto_kv_cache* c, int i, const float* theta
     p.tail_in = st.tail[st.tail_now]; p.tail_out = st.tail[st.tail_now ^ 1];
     p.qn = d->qn; p.kn = d->kn; p.gd = d->gd; p.beta = d->beta; p.vv = d->vv;
     p.B = B; p.T = Tn; p.heads = H; p.kv_heads = q.kv_heads; p.dim = D; p.vdim = E; p.taps = q.conv;
-    FEMTO_TRY(delta_prep<T>(p, s));
+    ChunkArgs ca;
+    ca.proj = proj; ca.ldp = l.n_in; ca.s_q = l.s_q; ca.s_k = l.s_k; ca.s_v = l.s_v; ca.s_b = l.s_b; ca.conv_q = p.conv_q; ca.conv_k = p.conv_k;
+    ca.conv_v = p.conv_v; ca.a_log = p.a_log; ca.dt_bias = p.dt_bias; ca.graw = d->gd; ca.tail_in = p.tail_in; ca.S = st.S; ca.o = d->mixo;
+    ca.B = B; ca.T = Tn; ca.heads = H; ca.qk_heads = q.kv_heads; ca.dim = D; ca.vdim = E; ca.taps = q.conv; ca.ws = d->chunk_ws;
+    ca.ws_bytes = d->chunk_ws_bytes; ca.status = d->status;
+    const bool chunked = sizeof(T) == 2 && chunked_recurrence_supported(ca);
+    if (chunked) { FEMTO_TRY(chunked_recurrence(ca, s)); FEMTO_TRY(conv_tail<T>(p, s)); }
+    else FEMTO_TRY(delta_prep<T>(p, s));
     st.tail_now ^= 1;
     RecurrenceArgs a;
     a.q = d->qn; a.k = d->kn; a.v = d->vv; a.ldq = a.ldk = (long long)q.kv_heads * D; a.ldv = (long long)H * E;
     a.g = d->gd; a.beta = d->beta; a.S = st.S; a.o = d->mixo; a.B = B; a.T = Tn; a.heads = H; a.qk_heads = q.kv_heads; a.dim = D; a.vdim = E;
-    FEMTO_TRY(recurrence<T>(a, s));
+    if (!chunked) FEMTO_TRY(recurrence<T>(a, s));
     FEMTO_TRY(S::gated_norm((const T*)d->mixo, theta + l.mix_norm, false, (const T*)d->g2, (long long)H * E, out, R, H, E, eps, s));
   } else {
     FEMTO_TRY(S::norm_cols(proj + l.s_q, l.n_in, theta + l.dq_norm, (T*)d->cq, l.qp, R, q.q_rank, eps, s));

@@ -47,6 +47,8 @@ struct DecoderStack {
   float *qn = nullptr, *kn = nullptr, *gd = nullptr, *beta = nullptr;
   void *vv = nullptr, *g2 = nullptr, *cq = nullptr, *q = nullptr;
   float* qabs = nullptr;              // latent attention, few rows: queries in the latent space
+  char* chunk_ws = nullptr;           // chunked recurrences: operands of the chunks of one segment
+  size_t chunk_ws_bytes = 0;
   void* gemm_ws = nullptr;
   size_t gemm_ws_bytes = 0;
 };
@@ -113,6 +115,26 @@ struct DeltaPrepArgs {
   int B = 0, T = 0, heads = 0, kv_heads = 0, dim = 0, vdim = 0, taps = 0;
 };
 template <typename T> int delta_prep(const DeltaPrepArgs& a, cudaStream_t s);
+template <typename T> int conv_tail(const DeltaPrepArgs& a, cudaStream_t s);   // only the kept inputs
+
+// The same recurrences for many tokens in bf16 models, chunk by chunk on the tensor cores (chunked_recurrence.cu);
+// convolutions, unit vectors and decays included.
+struct ChunkArgs {
+  const void* proj = nullptr; long long ldp = 0;        // packed projections; q, k (and v, without convolutions) get silu here
+  int s_q = 0, s_k = 0, s_v = 0, s_b = 0;
+  const float *conv_q = nullptr, *conv_k = nullptr, *conv_v = nullptr, *a_log = nullptr, *dt_bias = nullptr;
+  const float* graw = nullptr;   // [rows][heads * dim] W_a2 W_a1 h, or NULL: decayed sum with decay[heads]
+  const float* decay = nullptr;
+  const void* tail_in = nullptr;
+  float* S = nullptr; void* o = nullptr;
+  int B = 0, T = 0, heads = 0, qk_heads = 0, dim = 0, vdim = 0, taps = 1;
+  char* ws = nullptr; size_t ws_bytes = 0;
+  unsigned int* status = nullptr;
+  int t0 = 0, chunks = 0; size_t item_bytes = 0;        // set per segment
+};
+size_t chunked_recurrence_item_bytes(int dim, int vdim);
+bool chunked_recurrence_supported(const ChunkArgs& a);
+int chunked_recurrence(const ChunkArgs& a, cudaStream_t s);
 
 // ---- latent attention (latent_attention.cu) -------------------------------------------------------------------------
 struct LatentArgs {
@@ -132,5 +154,7 @@ struct LatentArgs {
 };
 template <typename T> int latent_prep(const LatentArgs& a, cudaStream_t s);
 template <typename T> int latent_attention(const LatentArgs& a, cudaStream_t s);
+bool latent_attention_tc_supported(const LatentArgs& a);       // latent_attention_sm100.cu: the prompt's attention on the tensor cores
+int latent_attention_tc(const LatentArgs& a, cudaStream_t s);
 constexpr int LATENT_FEW = 8;          // columns with at most this many new tokens attend in the latent space
 constexpr int LATENT_MAX_SPLITS = 64;

@@ -610,6 +610,20 @@ int make_tmap_4d_slabs_bf16(CUtensorMap* out, const void* base, uint64_t extent,
   return r == CUDA_SUCCESS ? 0 : 1;
 }
 
+int make_tmap_nd_bf16(CUtensorMap* out, const void* base, int rank, const uint64_t* dims, const uint64_t* strides_elems, const uint32_t* box_in) {
+  PFN_encodeTiled enc = get_encode();
+  if (!enc) return femto_fail(FEMTO_ERR_UNSUPPORTED, "cuTensorMapEncodeTiled is not available from the driver");
+  cuuint64_t d[5], st[4];
+  cuuint32_t box[5], estr[5] = {1, 1, 1, 1, 1};
+  for (int i = 0; i < rank; i++) { d[i] = dims[i] ? dims[i] : 1; box[i] = box_in[i]; }
+  for (int i = 0; i + 1 < rank; i++) st[i] = strides_elems[i] * 2;
+  CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, rank, const_cast<void*>(base), d, st, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS)
+    return femto_fail(FEMTO_ERR_ALIGN, "cuTensorMapEncodeTiled (%dd) failed (%d): inner extent %llu", rank, (int)r, (unsigned long long)d[0]);
+  return 0;
+}
+
 int make_tmap_2d_bf16(CUtensorMap* out, const void* base, uint64_t dim0, uint64_t dim1, uint64_t stride1_elems,
                       uint32_t box0, uint32_t box1) {
   PFN_encodeTiled enc = get_encode();

@@ -290,6 +290,7 @@ template <typename T> int latent_attention(const LatentArgs& a, cudaStream_t s) 
     g.A = reinterpret_cast<const T*>(g.A) + g.strideA;
     g.C = reinterpret_cast<T*>(g.C) + g.strideC;
   }
+  if (sizeof(T) == 2 && latent_attention_tc_supported(a)) return latent_attention_tc(a, s);
   const size_t smem = 4 * (size_t)((SQ + SK) * (a.dim + a.rot_dim + 1) + SK * a.vdim + SQ * (SK + 1) + 2 * SQ);
   FEMTO_TRY(allow_smem(k_latent_attn_simt<T>, smem));
   k_latent_attn_simt<T><<<dim3(cdiv(a.T, SQ), a.heads, a.B), 128, smem, s>>>(a, N);

@@ -198,17 +198,22 @@ template <typename T> int recurrence(const RecurrenceArgs& a, cudaStream_t s) {
 template int recurrence<float>(const RecurrenceArgs&, cudaStream_t);
 template int recurrence<bf16>(const RecurrenceArgs&, cudaStream_t);
 
+template <typename T> int conv_tail(const DeltaPrepArgs& a, cudaStream_t s) {
+  if (a.taps <= 1) return 0;
+  const long long m = (long long)a.B * (a.taps - 1) * (2 * a.kv_heads * a.dim + a.heads * a.vdim);
+  k_conv_tail<T><<<cdiv(m, 256), 256, 0, s>>>(a);
+  KERNEL_CHECK();
+  return 0;
+}
+template int conv_tail<float>(const DeltaPrepArgs&, cudaStream_t);
+template int conv_tail<bf16>(const DeltaPrepArgs&, cudaStream_t);
+
 template <typename T> int delta_prep(const DeltaPrepArgs& a, cudaStream_t s) {
   if (a.dim > 256 || a.vdim > 256) return femto_fail(FEMTO_ERR_UNSUPPORTED, "delta rule: dim %d / vdim %d > 256", a.dim, a.vdim);
   const long long n = (long long)a.B * a.T * (2 * a.kv_heads + 2 * a.heads);
   k_delta_prep<T><<<cdiv(n, 8), 256, 0, s>>>(a);
   KERNEL_CHECK();
-  if (a.taps > 1) {
-    const long long m = (long long)a.B * (a.taps - 1) * (2 * a.kv_heads * a.dim + a.heads * a.vdim);
-    k_conv_tail<T><<<cdiv(m, 256), 256, 0, s>>>(a);
-    KERNEL_CHECK();
-  }
-  return 0;
+  return conv_tail<T>(a, s);
 }
 template int delta_prep<float>(const DeltaPrepArgs&, cudaStream_t);
 template int delta_prep<bf16>(const DeltaPrepArgs&, cudaStream_t);

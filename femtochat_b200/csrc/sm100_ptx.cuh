@@ -280,3 +280,6 @@ int make_tmap_3d_bf16_sw(CUtensorMap* out, const void* base, uint64_t dim0, uint
                          uint64_t stride1_elems, uint64_t stride2_elems, uint32_t box0, uint32_t box1, int swizzle);
 int make_tmap_2d_bf16(CUtensorMap* out, const void* base, uint64_t dim0, uint64_t dim1, uint64_t stride1_elems,
                       uint32_t box0, uint32_t box1);
+// Any rank up to 5, 128-byte swizzle: strides_elems[i] is the distance of dimension i + 1.  A box may reach past the inner
+// extent: the part outside arrives as zeros, which pads a head's channels to whole 64-wide slabs for free.
+int make_tmap_nd_bf16(CUtensorMap* out, const void* base, int rank, const uint64_t* dims, const uint64_t* strides_elems, const uint32_t* box);
