@@ -44,7 +44,8 @@ template <int DP> struct Item {
   static size_t bytes(int E) { return U + (size_t)(E + 15) / 16 * 16 * C * 4; }
 };
 
-__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+// (an activation: bf16 numbers go in, so the special-function unit's 2^-21 is plenty)
+__device__ __forceinline__ float silu_f(float z) { return z * __fdividef(1.f, 1.f + __expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 __device__ __forceinline__ uint32_t bf2(float lo, float hi) {
@@ -73,21 +74,141 @@ __device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void* p) {
 __device__ __forceinline__ int swz(int row, int col, int width) { return row * width + ((((col >> 3) ^ (row & 7)) << 3) | (col & 7)); }
 
 // ---- local part -------------------------------------------------------------------------------------------------------
-template <int DP, bool DELTA>
-__global__ void __launch_bounds__(LOCAL_THREADS, 1) k_chunk_local(const ChunkArgs a) {
+// eight consecutive channels c .. c + 7 of a row of `size` channels (zeros beyond it)
+__device__ __forceinline__ void load8(const bf16* row, int c, int size, bool vec, float (&f)[8]) {
+  if (vec) {
+    if (c < size) load_vec<bf16, 8>(row + c, f);
+    else
+#pragma unroll
+      for (int e = 0; e < 8; e++) f[e] = 0.f;
+  } else {
+#pragma unroll
+    for (int e = 0; e < 8; e++) f[e] = c + e < size ? __bfloat162float(row[c + e]) : 0.f;
+  }
+}
+__device__ __forceinline__ void split8(const float (&f)[8], uint4& hi, uint4& lo) {
+  split2(f[0], f[1], hi.x, lo.x); split2(f[2], f[3], hi.y, lo.y); split2(f[4], f[5], hi.z, lo.z); split2(f[6], f[7], hi.w, lo.w);
+}
+// Task 0 .. 19 -> block I of 16 rows and first column j0 <= 16 I + 8 of an 8-column tile of the lower triangle
+__device__ __forceinline__ void triangle_task(int task, int& I, int& j0) {
+  I = task < 2 ? 0 : task < 6 ? 1 : task < 12 ? 2 : 3;
+  j0 = (task - I * (I + 1)) * 8;
+}
+__device__ __forceinline__ void zero_above(bf16* tile, int tid) {      // blocks right of the diagonal blocks, high and low
+  for (int i = tid; i < 2 * C * C / 8; i += LOCAL_THREADS) {
+    const int part = i / (C * C / 8), t = i % (C * C / 8) / 8, j = i % 8 * 8;
+    if (j >= (t & ~15) + 16) *reinterpret_cast<uint4*>(tile + part * C * C + swz(t, j, C)) = make_uint4(0, 0, 0, 0);
+  }
+}
+
+// Decayed sum: Q~ = decay^(t+1) q, K^ = decay^(n-1-t) k, U_0 = v and B = (q k^T) decay^(t-j).
+template <int DP>
+__global__ void __launch_bounds__(LOCAL_THREADS) k_chunk_local_sum(const ChunkArgs a) {
   pdl_trigger();
-  constexpr int ST = DP + 8, AT = C + 4;
-  extern __shared__ __align__(16) float sm[];
-  float* sk = sm;                         // [64][ST] k
-  float* sq = sk + C * ST;                // [64][ST] q
-  float* sl = sq + C * ST;                // [64][ST] cumulated log2 decays; later v
-  float* sf = sl + C * ST;                // [64][ST] 2^(L_t - L at the block's start)   (DELTA only, as is A)
-  float* sA = sf + (DELTA ? C * ST : 0);  // [64][AT] diag(beta) A, then scratch of the inverse
-  float* sX = sA + (DELTA ? C * AT : 0);  // [64][AT] the inverse, times diag(beta)
-  float* sB = sX + (DELTA ? C * AT : 0);  // [64][AT] B
-  float* pw = sB + C * AT;                // [65] powers of the decay, or [64] beta
-  float* cw = pw + 72;                    // [3][MAX_TAPS][128] taps
-  int* slow = reinterpret_cast<int*>(cw + (DELTA ? 3 * MAX_TAPS * 128 : 0));   // [4]
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  bf16* tq = reinterpret_cast<bf16*>(smem_raw);    // q, high and low
+  bf16* tk = tq + 2 * C * DP;                      // k
+  __shared__ float pw[C + 1];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int chunk = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
+  const int D = a.dim, E = a.vdim;
+  const int t0 = a.t0 + chunk * C, n = min(C, a.T - t0);
+  const bf16* proj = reinterpret_cast<const bf16*>(a.proj) + ((long long)b * a.T + t0) * a.ldp;
+  char* item = a.ws + (((long long)b * a.heads + h) * gridDim.x + chunk) * a.item_bytes;
+  if (tid <= C) pw[tid] = powf(a.decay[h], (float)tid);
+  __syncthreads();
+  const bool vec = (((D | E) & 7) == 0) && (a.ldp & 7) == 0;
+  bf16* gq = reinterpret_cast<bf16*>(item + Item<DP>::Q);
+  bf16* gk = reinterpret_cast<bf16*>(item + Item<DP>::K);
+  for (int i = tid; i < 2 * C * (DP / 8); i += LOCAL_THREADS) {
+    const int which = i / (C * (DP / 8)), t = i / (DP / 8) % C, c = i % (DP / 8) * 8, o = swz(t, c, DP);
+    float f[8] = {};
+    if (t < n) load8(proj + t * a.ldp + (which ? a.s_k : a.s_q) + h * D, c, D, vec, f);
+#pragma unroll
+    for (int e = 0; e < 8; e++) f[e] = silu_f(f[e]);
+    uint4 hi, lo;
+    split8(f, hi, lo);
+    bf16* st = which ? tk : tq;
+    *reinterpret_cast<uint4*>(st + o) = hi; *reinterpret_cast<uint4*>(st + C * DP + o) = lo;
+    const float p = which ? (t < n ? pw[n - 1 - t] : 0.f) : pw[t + 1];
+#pragma unroll
+    for (int e = 0; e < 8; e++) f[e] *= p;
+    split8(f, hi, lo);
+    bf16* gt = which ? gk : gq;
+    *reinterpret_cast<uint4*>(gt + o) = hi; *reinterpret_cast<uint4*>(gt + C * DP + o) = lo;
+  }
+  float* tu = reinterpret_cast<float*>(item + Item<DP>::U);
+  const int EP8 = (E + 15) / 16 * 2;
+  for (int i = tid; i < C * EP8; i += LOCAL_THREADS) {
+    const int t = i / EP8, e = i % EP8 * 8;
+    float f[8] = {};
+    if (t < n) load8(proj + t * a.ldp + a.s_v + h * E, e, E, vec, f);
+    float* dst = tu + ((e >> 4) * C + t) * 16 + (e & 15);
+    *reinterpret_cast<float4*>(dst) = make_float4(silu_f(f[0]), silu_f(f[1]), silu_f(f[2]), silu_f(f[3]));
+    *reinterpret_cast<float4*>(dst + 4) = make_float4(silu_f(f[4]), silu_f(f[5]), silu_f(f[6]), silu_f(f[7]));
+  }
+  if (tid < DP) reinterpret_cast<float*>(item + Item<DP>::G)[tid] = pw[n];
+  bf16* tb = reinterpret_cast<bf16*>(item + Item<DP>::B);
+  zero_above(tb, tid);
+  __syncthreads();
+  for (int task = warp; task < 20; task += LOCAL_WARPS) {
+    int I, j0;
+    triangle_task(task, I, j0);
+    float acc[3][4] = {};
+#pragma unroll
+    for (int k0 = 0; k0 < DP; k0 += 32) {
+      uint32_t bh[4], bl[4];
+      const int at = swz(j0 + (lane & 7), k0 + 8 * (lane >> 3), DP);
+      ldsm4(bh, tk + at); ldsm4(bl, tk + C * DP + at);
+#pragma unroll
+      for (int k = 0; k < 2; k++) {
+        uint32_t ah[4], al[4];
+        const int aa = swz(16 * I + (lane & 15), k0 + 16 * k + 8 * (lane >> 4), DP);
+        ldsm4(ah, tq + aa); ldsm4(al, tq + C * DP + aa);
+        mma(acc[0], ah, bh[2 * k], bh[2 * k + 1]); mma(acc[1], ah, bl[2 * k], bl[2 * k + 1]); mma(acc[2], al, bh[2 * k], bh[2 * k + 1]);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+      const int t = 16 * I + (lane >> 2) + 8 * e, j = j0 + 2 * (lane & 3);
+      const float x = j <= t ? (acc[0][2 * e] + (acc[1][2 * e] + acc[2][2 * e])) * pw[t - j] : 0.f;
+      const float y = j + 1 <= t ? (acc[0][2 * e + 1] + (acc[1][2 * e + 1] + acc[2][2 * e + 1])) * pw[t - j - 1] : 0.f;
+      uint32_t hi, lo;
+      split2(x, y, hi, lo);
+      const int o = swz(t, j, C);
+      *reinterpret_cast<uint32_t*>(tb + o) = hi; *reinterpret_cast<uint32_t*>(tb + C * C + o) = lo;
+    }
+  }
+}
+
+// Gated delta rule.  The raw inputs of the convolutions lie where the scaled operands and the small matrices go once the
+// convolutions are done.
+template <int DP> struct DeltaSmem {      // offsets in bytes
+  static constexpr int ST = DP + 8, AT = C + 4, ROWS = C + MAX_TAPS - 1;
+  static constexpr int K = 0, Q = K + C * ST * 4, L = Q + C * ST * 4, KF = L + C * ST * 4, QF = KF + 4 * C * DP, A = QF + 4 * C * DP,
+                       X = A + C * AT * 4, V = X + C * AT * 4, BETA = V + C * 128 * 2, SLOW = BETA + C * 4, TOTAL = SLOW + 16;
+  static constexpr int RAW = KF;           // bf16 [3][ROWS][128]
+  static_assert(3 * ROWS * 128 * 2 <= V - RAW, "raw inputs overlap what is live");
+};
+
+template <int DP>
+__global__ void __launch_bounds__(LOCAL_THREADS, 1) k_chunk_local_delta(const ChunkArgs a) {
+  pdl_trigger();
+  typedef DeltaSmem<DP> Sm;
+  constexpr int ST = Sm::ST, AT = Sm::AT;
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  float* sk = reinterpret_cast<float*>(smem_raw + Sm::K);    // [64][ST] k
+  float* sq = reinterpret_cast<float*>(smem_raw + Sm::Q);    // [64][ST] q
+  float* sl = reinterpret_cast<float*>(smem_raw + Sm::L);    // [64][ST] cumulated log2 decays
+  bf16* kf = reinterpret_cast<bf16*>(smem_raw + Sm::KF);     // k times 2^(L_t - L at the block's start), high and low; later K~
+  bf16* qf = reinterpret_cast<bf16*>(smem_raw + Sm::QF);     // q likewise
+  float* sA = reinterpret_cast<float*>(smem_raw + Sm::A);    // [64][AT] diag(beta) A, then scratch of the inverse
+  bf16* xs = reinterpret_cast<bf16*>(smem_raw + Sm::A);      // at the end: the inverse times diag(beta), high and low
+  float* sX = reinterpret_cast<float*>(smem_raw + Sm::X);    // [64][AT] the inverse
+  bf16* sv = reinterpret_cast<bf16*>(smem_raw + Sm::V);      // v [64][128]
+  float* beta = reinterpret_cast<float*>(smem_raw + Sm::BETA);
+  int* slow = reinterpret_cast<int*>(smem_raw + Sm::SLOW);   // [4]
+  bf16* raw = reinterpret_cast<bf16*>(smem_raw + Sm::RAW);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int chunk = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
   const int D = a.dim, E = a.vdim, H = a.heads, qh = h / (H / a.qk_heads);
@@ -97,212 +218,230 @@ __global__ void __launch_bounds__(LOCAL_THREADS, 1) k_chunk_local(const ChunkArg
   const bf16* proj = reinterpret_cast<const bf16*>(a.proj);
   const int G = a.qk_heads, channels = 2 * G * D + H * E, keep = a.taps - 1;
   const bf16* tail = reinterpret_cast<const bf16*>(a.tail_in) + (long long)b * keep * channels;
-  // input of a convolution `back` tokens before token t of this chunk
-  auto input = [&](int t, int back, int seg, int chan) {
-    const int r = t0 + t - back;
-    return __bfloat162float(r >= 0 ? proj[(r0 + t - back) * a.ldp + seg] : tail[(long long)(keep + r) * channels + chan]);
+  // decay logits of this chunk, on their way while the rest is staged: thread -> 4 channels of a token
+  constexpr int GV = C * DP / 4 / LOCAL_THREADS;
+  float4 graw[GV];
+#pragma unroll
+  for (int i = 0; i < GV; i++) {
+    const int t = (i * LOCAL_THREADS + tid) / (DP / 4), d = (i * LOCAL_THREADS + tid) % (DP / 4) * 4;
+    const float* src = a.graw + (r0 + t) * ((long long)H * D) + (long long)h * D + d;
+    graw[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (t < n) {
+      if ((D & 3) == 0) { if (d < D) graw[i] = *reinterpret_cast<const float4*>(src); }
+      else { if (d < D) graw[i].x = src[0]; if (d + 1 < D) graw[i].y = src[1]; if (d + 2 < D) graw[i].z = src[2]; if (d + 3 < D) graw[i].w = src[3]; }
+    }
+  }
+  // raw rows -keep .. 63 of q, k and v: from this call's projections or from the inputs kept of earlier calls
+  const int rows = C + keep;
+  auto source = [&](int which, int r) -> const bf16* {
+    const int t = t0 + r - keep;
+    const int head = which == 2 ? h * E : qh * D;
+    if (t >= 0) return proj + (r0 + r - keep) * a.ldp + (which == 0 ? a.s_q : which == 1 ? a.s_k : a.s_v) + head;
+    return tail + (long long)(keep + t) * channels + (which == 0 ? 0 : which == 1 ? G * D : 2 * G * D) + head;
   };
-  if (DELTA) {
-    for (int i = tid; i < 3 * a.taps * 128; i += LOCAL_THREADS) {
-      const int which = i / (a.taps * 128), j = i / 128 % a.taps, c = i % 128;
-      const float* src = which == 0 ? a.conv_q : which == 1 ? a.conv_k : a.conv_v;
-      const int size = which == 2 ? E : D, head = which == 2 ? h : qh;
-      cw[(which * MAX_TAPS + j) * 128 + c] = c < size ? src[(long long)(head * size + c) * a.taps + j] : 0.f;
+  if (((D | E) & 7) == 0 && (a.ldp & 7) == 0) {
+    for (int i = tid; i < 3 * rows * 16; i += LOCAL_THREADS) {
+      const int which = i / (rows * 16), r = i / 16 % rows, c = i % 16 * 8;
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (r < n + keep && c < (which == 2 ? E : D)) v = *reinterpret_cast<const uint4*>(source(which, r) + c);
+      *reinterpret_cast<uint4*>(raw + (which * Sm::ROWS + r) * 128 + c) = v;
     }
-    if (tid < C) pw[tid] = tid < n ? 1.f / (1.f + expf(-__bfloat162float(proj[(r0 + tid) * a.ldp + a.s_b + h]))) : 0.f;
-    if (tid < 4) slow[tid] = 0;
-    __syncthreads();
-  } else if (tid <= C) {
-    pw[tid] = powf(a.decay[h], (float)tid);
+  } else {
+    for (int i = tid; i < 3 * rows * 128; i += LOCAL_THREADS) {
+      const int which = i / (rows * 128), r = i / 128 % rows, c = i % 128;
+      raw[(which * Sm::ROWS + r) * 128 + c] = r < n + keep && c < (which == 2 ? E : D) ? source(which, r)[c] : __float2bfloat16_rn(0.f);
+    }
   }
-  // q and k: one warp per (token, which)
-  for (int it = warp; it < 2 * C; it += LOCAL_WARPS) {
-    const int t = it >> 1, which = it & 1;
-    float* dst = (which ? sk : sq) + t * ST;
-    float y[DP / 32], ss = 0.f;
+  if (tid < C) beta[tid] = tid < n ? 1.f / (1.f + expf(-__bfloat162float(proj[(r0 + tid) * a.ldp + a.s_b + h]))) : 0.f;
+  if (tid < 4) slow[tid] = 0;
+  const float rate = expf(a.a_log[h]) * LOG2E;
 #pragma unroll
-    for (int i = 0; i < DP / 32; i++) {
-      const int c = i * 32 + lane;
-      y[i] = 0.f;
-      if (t < n && c < D) {
-        const int seg = (which ? a.s_k : a.s_q) + qh * D + c;
-        if (DELTA) {
-          float acc = 0.f;
-          for (int j = 0; j < a.taps; j++)
-            acc += cw[(which * MAX_TAPS + j) * 128 + c] * input(t, keep - j, seg, (which ? G * D : 0) + qh * D + c);
-          y[i] = silu_f(acc);
-          ss += y[i] * y[i];
-        } else {
-          y[i] = silu_f(__bfloat162float(proj[(r0 + t) * a.ldp + seg]));
-        }
-      }
-    }
-    float f = 1.f;
-    if (DELTA) {
-      f = 1.f / sqrtf(warp_sum(ss) + 1e-6f);
-      if (!which) f *= 1.f / sqrtf((float)D);
-    }
+  for (int i = 0; i < GV; i++) {
+    const int t = (i * LOCAL_THREADS + tid) / (DP / 4), d = (i * LOCAL_THREADS + tid) % (DP / 4) * 4;
+    float x[4] = {graw[i].x, graw[i].y, graw[i].z, graw[i].w};
 #pragma unroll
-    for (int i = 0; i < DP / 32; i++) dst[i * 32 + lane] = y[i] * f;
+    for (int e = 0; e < 4; e++) x[e] = t < n && d + e < D ? -rate * softplus_f(x[e] + a.dt_bias[h * D + d + e]) : 0.f;
+    *reinterpret_cast<float4*>(&sl[t * ST + d]) = make_float4(x[0], x[1], x[2], x[3]);
   }
-  if (DELTA) {
-    const float rate = expf(a.a_log[h]) * LOG2E;
-    for (int i = tid; i < C * DP; i += LOCAL_THREADS) {
-      const int t = i / DP, d = i % DP;
-      sl[t * ST + d] = t < n && d < D ? -rate * softplus_f(a.graw[(r0 + t) * ((long long)H * D) + (long long)h * D + d] + a.dt_bias[h * D + d]) : 0.f;
-    }
-    __syncthreads();
-    if (tid < DP) {
-      float acc = 0.f;
-      for (int t = 0; t < C; t++) { acc += sl[t * ST + tid]; sl[t * ST + tid] = acc; }
-    }
-    __syncthreads();
-    for (int i = tid; i < C * DP; i += LOCAL_THREADS) {
-      const int t = i / DP, d = i % DP, first = t & ~15;
-      const float ref = first ? sl[(first - 1) * ST + d] : 0.f;
-      const float x = sl[t * ST + d] - ref;
-      sf[t * ST + d] = fast_exp2(x);
-      if ((t & 15) == 15 && x < -RANGE) slow[t >> 4] = 1;
+  // convolution, silu, unit vectors: a warp takes four consecutive tokens of q, then of k, then of v; a lane two pairs of channels
+  float w[3][4][4];      // the first four taps; further ones are read where they are used
+#pragma unroll
+  for (int which = 0; which < 3; which++) {
+    const float* src = which == 0 ? a.conv_q : which == 1 ? a.conv_k : a.conv_v;
+    const int size = which == 2 ? E : D, head = which == 2 ? h : qh;
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      const int c = (i >> 1) * 64 + 2 * lane + (i & 1);
+#pragma unroll
+      for (int j = 0; j < 4; j++) w[which][i][j] = j < a.taps && c < size ? src[(long long)(head * size + c) * a.taps + j] : 0.f;
     }
   }
   __syncthreads();
-  // A and B: 20 tasks (block of 16 rows, 8 columns), both matrices share the right operand
+  const int tb0 = 4 * warp;
+#pragma unroll
+  for (int which = 0; which < 3; which++) {
+    float x[7][4];
+#pragma unroll
+    for (int r = 0; r < 7; r++)
+      if (r < 3 + min(a.taps, 4)) {
+#pragma unroll
+        for (int p = 0; p < 2; p++) {
+          const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(raw + (which * Sm::ROWS + tb0 + r) * 128 + p * 64 + 2 * lane));
+          x[r][2 * p] = f.x; x[r][2 * p + 1] = f.y;
+        }
+      } else {
+#pragma unroll
+        for (int p = 0; p < 4; p++) x[r][p] = 0.f;
+      }
+#pragma unroll
+    for (int tt = 0; tt < 4; tt++) {
+      const int t = tb0 + tt;
+      float y[4], ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < 4; i++) {
+        float acc = 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; j++) acc = fmaf(w[which][i][j], x[tt + j][i], acc);
+        if (a.taps > 4) {
+          const int c = (i >> 1) * 64 + 2 * lane + (i & 1), size = which == 2 ? E : D, head = which == 2 ? h : qh;
+          const float* src = which == 0 ? a.conv_q : which == 1 ? a.conv_k : a.conv_v;
+          if (c < size)
+            for (int j = 4; j < a.taps; j++)
+              acc = fmaf(src[(long long)(head * size + c) * a.taps + j], __bfloat162float(raw[(which * Sm::ROWS + t + j) * 128 + c]), acc);
+        }
+        y[i] = t < n ? silu_f(acc) : 0.f;      // padding channels: zero
+        ss += y[i] * y[i];
+      }
+      if (which == 2) {
+#pragma unroll
+        for (int p = 0; p < 2; p++) *reinterpret_cast<uint32_t*>(sv + swz(t, p * 64 + 2 * lane, 128)) = bf2(y[2 * p], y[2 * p + 1]);
+      } else {
+        float f = 1.f / sqrtf(warp_sum(ss) + 1e-6f);
+        if (which == 0) f *= 1.f / sqrtf((float)D);
+        float* dst = (which ? sk : sq) + t * ST + 2 * lane;
+#pragma unroll
+        for (int p = 0; p < DP / 64; p++) *reinterpret_cast<float2*>(dst + p * 64) = make_float2(y[2 * p] * f, y[2 * p + 1] * f);
+      }
+    }
+  }
+  // cumulated decays: inside each block of 16 tokens, then over the blocks before it
+  const int blk = tid / DP, dcol = tid % DP;
+  if (blk < 4) {
+    float acc = 0.f;
+#pragma unroll
+    for (int t = 0; t < 16; t++) { acc += sl[(16 * blk + t) * ST + dcol]; sl[(16 * blk + t) * ST + dcol] = acc; }
+  }
+  __syncthreads();                    // the raw inputs have been read as well
+  for (int i = tid; i < C * DP / 2; i += LOCAL_THREADS) {
+    const int t = i / (DP / 2), d = i % (DP / 2) * 2, at = t * ST + d, o = swz(t, d, DP);
+    const float2 x = *reinterpret_cast<const float2*>(&sl[at]), k = *reinterpret_cast<const float2*>(&sk[at]), q = *reinterpret_cast<const float2*>(&sq[at]);
+    const float2 f = make_float2(fast_exp2(x.x), fast_exp2(x.y));
+    if ((t & 15) == 15 && fminf(x.x, x.y) < -RANGE) slow[t >> 4] = 1;
+    uint32_t hi, lo;
+    split2(k.x * f.x, k.y * f.y, hi, lo);
+    *reinterpret_cast<uint32_t*>(kf + o) = hi; *reinterpret_cast<uint32_t*>(kf + C * DP + o) = lo;
+    split2(q.x * f.x, q.y * f.y, hi, lo);
+    *reinterpret_cast<uint32_t*>(qf + o) = hi; *reinterpret_cast<uint32_t*>(qf + C * DP + o) = lo;
+  }
+  __syncthreads();
+  if (blk < 4 && blk > 0) {
+    float before = 0.f;
+    for (int k = 0; k < blk; k++) before += sl[(16 * k + 15) * ST + dcol];
+    // the last row of a block is still its own sum while other threads read it: it is finished below
+#pragma unroll
+    for (int t = 0; t < 15; t++) sl[(16 * blk + t) * ST + dcol] += before;
+  }
+  __syncthreads();
+  if (tid < DP) {
+    float acc = sl[15 * ST + tid];
+#pragma unroll
+    for (int k = 1; k < 4; k++) { acc += sl[(16 * k + 15) * ST + tid]; sl[(16 * k + 15) * ST + tid] = acc; }
+  }
+  bf16* tb = reinterpret_cast<bf16*>(item + Item<DP>::B);
+  zero_above(tb, tid);
+  for (int i = tid; i < C * C; i += LOCAL_THREADS) {            // right of the diagonal blocks
+    const int t = i / C, j = i % C;
+    if (j >= (t & ~15) + 16) { sA[t * AT + j] = 0.f; sX[t * AT + j] = 0.f; }
+  }
+  __syncthreads();
+  // A and B: both matrices share the right operand, k_j times 2^(L at the row block's start - L_j)
+  const int g = lane >> 2, c2 = 2 * (lane & 3);
   for (int task = warp; task < 20; task += LOCAL_WARPS) {
-    const int I = task < 2 ? 0 : task < 6 ? 1 : task < 12 ? 2 : 3;
-    const int j0 = (task - I * (I + 1)) * 8;                    // first column
-    const int g = lane >> 2, c2 = 2 * (lane & 3);
-    if (DELTA && j0 >= 16 * I && slow[I]) continue;             // pair by pair below
+    int I, j0;
+    triangle_task(task, I, j0);
+    if (j0 >= 16 * I && slow[I]) continue;                      // pair by pair below
     float aA[3][4] = {}, aB[3][4] = {};
-    const int j = j0 + g, ra = 16 * I + g;
+    const int j = j0 + g;
+    const float* ref = sl + (16 * I - 1) * ST;
+#pragma unroll 4
     for (int k0 = 0; k0 < DP; k0 += 16) {
-      float2 r[2];
+      uint32_t bh[2], bl[2];
 #pragma unroll
       for (int e = 0; e < 2; e++) {
         const int d = k0 + e * 8 + c2;
-        r[e] = *reinterpret_cast<const float2*>(&sk[j * ST + d]);
-        if (DELTA) {
-          const float2 l = *reinterpret_cast<const float2*>(&sl[j * ST + d]);
-          const float2 ref = I ? *reinterpret_cast<const float2*>(&sl[(16 * I - 1) * ST + d]) : make_float2(0.f, 0.f);
-          r[e].x *= fast_exp2(ref.x - l.x); r[e].y *= fast_exp2(ref.y - l.y);
-        }
+        float2 r = *reinterpret_cast<const float2*>(&sk[j * ST + d]);
+        const float2 l = *reinterpret_cast<const float2*>(&sl[j * ST + d]);
+        const float2 lr = I ? *reinterpret_cast<const float2*>(ref + d) : make_float2(0.f, 0.f);
+        r.x *= fast_exp2(lr.x - l.x); r.y *= fast_exp2(lr.y - l.y);
+        split2(r.x, r.y, bh[e], bl[e]);
       }
-      uint32_t bh[2], bl[2];
-      split2(r[0].x, r[0].y, bh[0], bl[0]); split2(r[1].x, r[1].y, bh[1], bl[1]);
       uint32_t kh[4], kl[4], qh_[4], ql[4];
-#pragma unroll
-      for (int e = 0; e < 4; e++) {
-        const int at = (ra + (e & 1) * 8) * ST + k0 + (e >> 1) * 8 + c2;
-        float2 q = *reinterpret_cast<const float2*>(&sq[at]);
-        if (DELTA) {
-          const float2 f = *reinterpret_cast<const float2*>(&sf[at]);
-          float2 k = *reinterpret_cast<const float2*>(&sk[at]);
-          split2(k.x * f.x, k.y * f.y, kh[e], kl[e]);
-          q.x *= f.x; q.y *= f.y;
-        }
-        split2(q.x, q.y, qh_[e], ql[e]);
-      }
-      if (DELTA) { mma(aA[0], kh, bh[0], bh[1]); mma(aA[1], kh, bl[0], bl[1]); mma(aA[2], kl, bh[0], bh[1]); }
+      const int aa = swz(16 * I + (lane & 15), k0 + 8 * (lane >> 4), DP);
+      ldsm4(kh, kf + aa); ldsm4(kl, kf + C * DP + aa); ldsm4(qh_, qf + aa); ldsm4(ql, qf + C * DP + aa);
+      mma(aA[0], kh, bh[0], bh[1]); mma(aA[1], kh, bl[0], bl[1]); mma(aA[2], kl, bh[0], bh[1]);
       mma(aB[0], qh_, bh[0], bh[1]); mma(aB[1], qh_, bl[0], bl[1]); mma(aB[2], ql, bh[0], bh[1]);
     }
 #pragma unroll
-    for (int e = 0; e < 4; e++) {
-      const int t = ra + (e >> 1) * 8, jj = j0 + c2 + (e & 1);
-      const float vb = aB[0][e] + (aB[1][e] + aB[2][e]);
-      if (DELTA) {
-        const float va = aA[0][e] + (aA[1][e] + aA[2][e]);
-        sA[t * AT + jj] = jj < t ? va * pw[t] : 0.f;
-        sB[t * AT + jj] = jj <= t ? vb : 0.f;
-      } else {
-        sB[t * AT + jj] = jj <= t ? vb * pw[t - jj] : 0.f;
+    for (int e = 0; e < 2; e++) {
+      const int t = 16 * I + g + 8 * e, jj = j0 + c2;
+      float va[2], vb[2];
+#pragma unroll
+      for (int i = 0; i < 2; i++) {
+        va[i] = jj + i < t ? (aA[0][2 * e + i] + (aA[1][2 * e + i] + aA[2][2 * e + i])) * beta[t] : 0.f;
+        vb[i] = jj + i <= t ? aB[0][2 * e + i] + (aB[1][2 * e + i] + aB[2][2 * e + i]) : 0.f;
       }
+      *reinterpret_cast<float2*>(&sA[t * AT + jj]) = make_float2(va[0], va[1]);
+      uint32_t hi, lo;
+      split2(vb[0], vb[1], hi, lo);
+      const int o = swz(t, jj, C);
+      *reinterpret_cast<uint32_t*>(tb + o) = hi; *reinterpret_cast<uint32_t*>(tb + C * C + o) = lo;
     }
   }
-  for (int i = tid; i < C * C; i += LOCAL_THREADS) {            // right of the diagonal blocks
-    const int t = i / C, j = i % C;
-    if (j >= (t & ~15) + 16) { sB[t * AT + j] = 0.f; if (DELTA) { sA[t * AT + j] = 0.f; sX[t * AT + j] = 0.f; } }
-  }
-  if (DELTA) {
-    for (int I = 0; I < 4; I++) {
-      if (!slow[I]) continue;
-      for (int i = tid; i < 256; i += LOCAL_THREADS) {
-        const int t = 16 * I + i / 16, j = 16 * I + i % 16;
-        float va = 0.f, vb = 0.f;
-        if (j <= t)
-          for (int d = 0; d < D; d++) {
-            const float f = sk[j * ST + d] * fast_exp2(sl[t * ST + d] - sl[j * ST + d]);
-            va = fmaf(sk[t * ST + d], f, va); vb = fmaf(sq[t * ST + d], f, vb);
-          }
-        sA[t * AT + j] = j < t ? va * pw[t] : 0.f;
-        sB[t * AT + j] = vb;
-      }
+  for (int I = 0; I < 4; I++) {
+    if (!slow[I]) continue;
+    for (int i = tid; i < 256; i += LOCAL_THREADS) {
+      const int t = 16 * I + i / 16, j = 16 * I + i % 16, o = swz(t, j, C);
+      float va = 0.f, vb = 0.f;
+      if (j <= t)
+        for (int d = 0; d < D; d++) {
+          const float f = sk[j * ST + d] * fast_exp2(sl[t * ST + d] - sl[j * ST + d]);
+          va = fmaf(sk[t * ST + d], f, va); vb = fmaf(sq[t * ST + d], f, vb);
+        }
+      sA[t * AT + j] = j < t ? va * beta[t] : 0.f;
+      const bf16 hi = __float2bfloat16_rn(vb);
+      tb[o] = hi; tb[C * C + o] = __float2bfloat16_rn(vb - __bfloat162float(hi));
     }
   }
   __syncthreads();
-  // Q~, K^, B and Gamma_C leave; K~ replaces sf
+  // Q~ and K^ leave; K~ replaces kf
   {
     bf16* tq = reinterpret_cast<bf16*>(item + Item<DP>::Q);
     bf16* tk = reinterpret_cast<bf16*>(item + Item<DP>::K);
     for (int i = tid; i < C * DP / 2; i += LOCAL_THREADS) {
       const int t = i / (DP / 2), d = i % (DP / 2) * 2, at = t * ST + d, o = swz(t, d, DP);
-      float2 q = *reinterpret_cast<const float2*>(&sq[at]), k = *reinterpret_cast<const float2*>(&sk[at]);
-      if (DELTA) {
-        const float2 l = *reinterpret_cast<const float2*>(&sl[at]), lc = *reinterpret_cast<const float2*>(&sl[(C - 1) * ST + d]);
-        const int first = t & ~15;
-        const float2 ref = first ? *reinterpret_cast<const float2*>(&sl[(first - 1) * ST + d]) : make_float2(0.f, 0.f);
-        float2 f = *reinterpret_cast<const float2*>(&sf[at]);
-        f.x *= fast_exp2(ref.x); f.y *= fast_exp2(ref.y);      // Gamma_t
-        q.x *= f.x; q.y *= f.y;
-        *reinterpret_cast<float2*>(&sf[at]) = make_float2(k.x * f.x, k.y * f.y);
-        k.x *= fast_exp2(lc.x - l.x); k.y *= fast_exp2(lc.y - l.y);
-      } else {
-        q.x *= pw[t + 1]; q.y *= pw[t + 1];
-        const float f = t < n ? pw[n - 1 - t] : 0.f;
-        k.x *= f; k.y *= f;
-      }
+      const float2 q = *reinterpret_cast<const float2*>(&sq[at]), k = *reinterpret_cast<const float2*>(&sk[at]);
+      const float2 l = *reinterpret_cast<const float2*>(&sl[at]), lc = *reinterpret_cast<const float2*>(&sl[(C - 1) * ST + d]);
+      const float2 f = make_float2(fast_exp2(l.x), fast_exp2(l.y));                       // Gamma_t
       uint32_t hi, lo;
-      split2(q.x, q.y, hi, lo);
+      split2(k.x * f.x, k.y * f.y, hi, lo);
+      *reinterpret_cast<uint32_t*>(kf + o) = hi; *reinterpret_cast<uint32_t*>(kf + C * DP + o) = lo;
+      split2(q.x * f.x, q.y * f.y, hi, lo);
       *reinterpret_cast<uint32_t*>(tq + o) = hi; *reinterpret_cast<uint32_t*>(tq + C * DP + o) = lo;
-      split2(k.x, k.y, hi, lo);
+      split2(k.x * fast_exp2(lc.x - l.x), k.y * fast_exp2(lc.y - l.y), hi, lo);
       *reinterpret_cast<uint32_t*>(tk + o) = hi; *reinterpret_cast<uint32_t*>(tk + C * DP + o) = lo;
     }
-    bf16* tb = reinterpret_cast<bf16*>(item + Item<DP>::B);
-    for (int i = tid; i < C * C / 2; i += LOCAL_THREADS) {
-      const int t = i / (C / 2), j = i % (C / 2) * 2, o = swz(t, j, C);
-      uint32_t hi, lo;
-      split2(sB[t * AT + j], sB[t * AT + j + 1], hi, lo);
-      *reinterpret_cast<uint32_t*>(tb + o) = hi; *reinterpret_cast<uint32_t*>(tb + C * C + o) = lo;
-    }
-    float* tg = reinterpret_cast<float*>(item + Item<DP>::G);
-    if (tid < DP) tg[tid] = DELTA ? fast_exp2(sl[(C - 1) * ST + tid]) : pw[n];
+    if (tid < DP) reinterpret_cast<float*>(item + Item<DP>::G)[tid] = fast_exp2(sl[(C - 1) * ST + tid]);
   }
-  float* tu = reinterpret_cast<float*>(item + Item<DP>::U);
-  if (!DELTA) {
-    const int EP = (E + 15) / 16 * 16;
-    for (int i = tid; i < C * EP; i += LOCAL_THREADS) {
-      const int t = i / EP, e = i % EP;
-      tu[((e >> 4) * C + t) * 16 + (e & 15)] = t < n && e < E ? silu_f(__bfloat162float(proj[(r0 + t) * a.ldp + a.s_v + h * E + e])) : 0.f;
-    }
-    return;
-  }
-  __syncthreads();
-  // v into sl (E <= 128 <= ST only when DP = 128: rows of 136 floats either way)
-  constexpr int VT = 136;
-  float* sv = sl;      // [64][VT]: with DP = 64 it runs on over sf's first half, which is saved in sq first
-  float* kt = sf;
-  if (DP < 128) {
-    for (int i = tid; i < C * ST; i += LOCAL_THREADS) sq[i] = sf[i];
-    kt = sq;
-    __syncthreads();
-  }
-  for (int it = warp; it < C; it += LOCAL_WARPS)
-    for (int e = lane; e < 128; e += 32) {
-      float acc = 0.f;
-      if (it < n && e < E) {
-        for (int j = 0; j < a.taps; j++) acc += cw[(2 * MAX_TAPS + j) * 128 + e] * input(it, keep - j, a.s_v + h * E + e, 2 * G * D + h * E + e);
-        acc = __bfloat162float(__float2bfloat16_rn(silu_f(acc)));
-      }
-      sv[it * VT + e] = acc;
-    }
   // inverse of I + diag(beta) A: the four 16 x 16 diagonal blocks, then the blocks below them by distance
   if (warp < 4 && lane < 16) {
     const float* m = sA + (16 * warp) * AT + 16 * warp;
@@ -317,12 +456,14 @@ __global__ void __launch_bounds__(LOCAL_THREADS, 1) k_chunk_local(const ChunkArg
     }
   }
   __syncthreads();
+#pragma unroll
   for (int dist = 1; dist < 4; dist++) {
     // Y_IJ = sum_K M_IK X_KJ goes to the free block (J, I) of sA; X_IJ = -X_II Y_IJ
     for (int i = tid; i < (4 - dist) * 256; i += LOCAL_THREADS) {
       const int J = i / 256, I = J + dist, r = i % 256 / 16, c = i % 16;
       float y = 0.f;
-      for (int k = 16 * J; k < 16 * I; k++) y = fmaf(sA[(16 * I + r) * AT + k], sX[k * AT + 16 * J + c], y);
+#pragma unroll 16
+      for (int k = 0; k < 16 * dist; k++) y = fmaf(sA[(16 * I + r) * AT + 16 * J + k], sX[(16 * J + k) * AT + 16 * J + c], y);
       sA[(16 * J + r) * AT + 16 * I + c] = y;
     }
     __syncthreads();
@@ -335,52 +476,61 @@ __global__ void __launch_bounds__(LOCAL_THREADS, 1) k_chunk_local(const ChunkArg
     }
     __syncthreads();
   }
-  for (int i = tid; i < C * C; i += LOCAL_THREADS) sX[i / C * AT + i % C] *= pw[i % C];
+  for (int i = tid; i < C * C / 2; i += LOCAL_THREADS) {
+    const int t = i / (C / 2), j = i % (C / 2) * 2, o = swz(t, j, C);
+    const float2 x = *reinterpret_cast<const float2*>(&sX[t * AT + j]);
+    uint32_t hi, lo;
+    split2(x.x * beta[j], x.y * beta[j + 1], hi, lo);
+    *reinterpret_cast<uint32_t*>(xs + o) = hi; *reinterpret_cast<uint32_t*>(xs + C * C + o) = lo;
+  }
   __syncthreads();
-  // W = X K~ and U_0 = X V: one task per 8 columns
-  const int wt = DP / 8, ut = (E + 15) / 16 * 2;
+  // W = X K~ and U_0 = X V: one task per 16 columns
+  const int wt = DP / 16, ut = (E + 15) / 16;
   bf16* tw = reinterpret_cast<bf16*>(item + Item<DP>::W);
+  float* tu = reinterpret_cast<float*>(item + Item<DP>::U);
   for (int task = warp; task < wt + ut; task += LOCAL_WARPS) {
     const bool is_w = task < wt;
-    const float* src = is_w ? kt : sv;
-    const int ld = is_w ? ST : VT, n0 = (is_w ? task : task - wt) * 8, g = lane >> 2, c2 = 2 * (lane & 3);
-    float acc[4][4] = {}, low[4][4] = {};
+    const int n0 = (is_w ? task : task - wt) * 16;
+    float acc[4][2][4] = {}, low[4][2][4] = {};
 #pragma unroll
     for (int kk = 0; kk < 4; kk++) {
-      uint32_t bh[2], bl[2];
-#pragma unroll
-      for (int e = 0; e < 2; e++) {
-        const int k = 16 * kk + 8 * e + c2;
-        split2(src[k * ld + n0 + g], src[(k + 1) * ld + n0 + g], bh[e], bl[e]);
+      uint32_t bh[4], bl[4];
+      if (is_w) {
+        const int at = swz(16 * kk + (lane & 15), n0 + 8 * (lane >> 4), DP);
+        ldsm4t(bh, kf + at); ldsm4t(bl, kf + C * DP + at);
+      } else {
+        ldsm4t(bh, sv + swz(16 * kk + (lane & 15), n0 + 8 * (lane >> 4), 128));
       }
 #pragma unroll
       for (int m = kk; m < 4; m++) {
         uint32_t ah[4], al[4];
+        const int at = swz(16 * m + (lane & 15), 16 * kk + 8 * (lane >> 4), C);
+        ldsm4(ah, xs + at); ldsm4(al, xs + C * C + at);
 #pragma unroll
-        for (int e = 0; e < 4; e++) {
-          const float2 x = *reinterpret_cast<const float2*>(&sX[(16 * m + g + (e & 1) * 8) * AT + 16 * kk + (e >> 1) * 8 + c2]);
-          split2(x.x, x.y, ah[e], al[e]);
+        for (int i = 0; i < 2; i++) {
+          mma(acc[m][i], ah, bh[2 * i], bh[2 * i + 1]);
+          mma(low[m][i], al, bh[2 * i], bh[2 * i + 1]);
+          if (is_w) mma(low[m][i], ah, bl[2 * i], bl[2 * i + 1]);     // v is a bf16 number
         }
-        mma(acc[m], ah, bh[0], bh[1]);
-        mma(low[m], al, bh[0], bh[1]);
-        if (is_w) mma(low[m], ah, bl[0], bl[1]);     // v is a bf16 number
       }
     }
 #pragma unroll
     for (int m = 0; m < 4; m++)
 #pragma unroll
-      for (int e = 0; e < 2; e++) {
-        const int t = 16 * m + g + 8 * e, d = n0 + c2;
-        const float x = acc[m][2 * e] + low[m][2 * e], y = acc[m][2 * e + 1] + low[m][2 * e + 1];
-        if (is_w) {
-          uint32_t hi, lo;
-          split2(x, y, hi, lo);
-          const int o = swz(t, d, DP);
-          *reinterpret_cast<uint32_t*>(tw + o) = hi; *reinterpret_cast<uint32_t*>(tw + C * DP + o) = lo;
-        } else {
-          *reinterpret_cast<float2*>(&tu[((d >> 4) * C + t) * 16 + (d & 15)]) = make_float2(x, y);
+      for (int i = 0; i < 2; i++)
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+          const int t = 16 * m + g + 8 * e, d = n0 + 8 * i + c2;
+          const float x = acc[m][i][2 * e] + low[m][i][2 * e], y = acc[m][i][2 * e + 1] + low[m][i][2 * e + 1];
+          if (is_w) {
+            uint32_t hi, lo;
+            split2(x, y, hi, lo);
+            const int o = swz(t, d, DP);
+            *reinterpret_cast<uint32_t*>(tw + o) = hi; *reinterpret_cast<uint32_t*>(tw + C * DP + o) = lo;
+          } else {
+            *reinterpret_cast<float2*>(&tu[((d >> 4) * C + t) * 16 + (d & 15)]) = make_float2(x, y);
+          }
         }
-      }
   }
 }
 
@@ -392,12 +542,12 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
   typedef Item<DP> It;
   constexpr int NT = DP / 64;                  // 8-column tiles of the state's rows per warp
   constexpr size_t X0 = DELTA ? 0 : It::Q, XB = It::X_BYTES - X0;      // without A there is no W
-  constexpr size_t UB = (size_t)C * 16 * 4, XS = XB + UB;
+  constexpr size_t UB = (size_t)C * 16 * 4, XS = XB + UB, SLOT = XS > It::Y_BYTES ? XS : It::Y_BYTES;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~(uintptr_t)127);
-  uint8_t* sx = smem;                          // 2 stages of [W, Q~ | U_0 slice]
-  uint8_t* sy = sx + 2 * XS;                   // [K^, B, Gamma_C]
-  bf16* sS = reinterpret_cast<bf16*>(sy + It::Y_BYTES);      // state^T [16][DP], high and low
+  // ring of three half chunks: first half [W, Q~ | U_0 slice], second half [K^, B, Gamma_C]; half i lies in slot i mod 3, and
+  // half i + 3 is fetched as soon as half i has been read
+  bf16* sS = reinterpret_cast<bf16*>(smem + 3 * SLOT);      // state^T [16][DP], high and low
   bf16* sU = sS + 2 * 16 * DP;                 // U^T [16][64], high and low
   uint64_t* bars = reinterpret_cast<uint64_t*>(sU + 2 * 16 * C);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(bars + 3);
@@ -411,22 +561,23 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
     fence_barrier_init();
   }
   __syncthreads();
-  auto load_x = [&](int c) {
-    const char* it = items + (long long)c * a.item_bytes;
-    uint8_t* dst = sx + (c & 1) * XS;
-    mbar_expect_tx(&bars[c & 1], (uint32_t)XS);
-    bulk_load_1d(dst, it + X0, (uint32_t)XB, &bars[c & 1]);
-    bulk_load_1d(dst + XB, it + It::U + eb * UB, (uint32_t)UB, &bars[c & 1]);
+  auto load = [&](int i) {                     // half i
+    if (i >= 2 * a.chunks) return;
+    const char* it = items + (long long)(i >> 1) * a.item_bytes;
+    uint8_t* dst = smem + (i % 3) * SLOT;
+    uint64_t* bar = &bars[i % 3];
+    if (i & 1) {
+      mbar_expect_tx(bar, (uint32_t)It::Y_BYTES);
+      bulk_load_1d(dst, it + It::K, (uint32_t)It::Y_BYTES, bar);
+    } else {
+      mbar_expect_tx(bar, (uint32_t)XS);
+      bulk_load_1d(dst, it + X0, (uint32_t)XB, bar);
+      bulk_load_1d(dst + XB, it + It::U + eb * UB, (uint32_t)UB, bar);
+    }
   };
-  auto load_y = [&](int c) {
-    mbar_expect_tx(&bars[2], (uint32_t)It::Y_BYTES);
-    bulk_load_1d(sy, items + (long long)c * a.item_bytes + It::K, (uint32_t)It::Y_BYTES, &bars[2]);
-  };
-  if (threadIdx.x == 0) {
-    load_x(0);
-    load_y(0);
-    if (a.chunks > 1) load_x(1);
-  }
+  auto half_bar = [&](int i) { return &bars[i % 3]; };
+  auto half_phase = [&](int i) { return (uint32_t)((i / 3) & 1); };
+  if (threadIdx.x == 0) { load(0); load(1); load(2); }
   // the state: rows d0 .. of column e in accumulator fragments, and its two bf16 parts in shared memory
   const int d0 = warp * 8 * NT;
   float S[NT][4];
@@ -453,9 +604,9 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
   bool ok = true;
   int c = 0;
   for (; c < a.chunks; c++) {
-    if (!mbar_wait(&bars[c & 1], (c >> 1) & 1, abort_flag, a.status)) ok = false;
+    if (!mbar_wait(half_bar(2 * c), half_phase(2 * c), abort_flag, a.status)) ok = false;
     if (!__syncthreads_and(ok)) break;         // also: the published state is complete
-    const uint8_t* x = sx + (c & 1) * XS;
+    const uint8_t* x = smem + (2 * c % 3) * SLOT;
     const bf16* tw = reinterpret_cast<const bf16*>(x);
     const bf16* tq = reinterpret_cast<const bf16*>(x + (It::Q - X0));
     const float* u0 = reinterpret_cast<const float*>(x + XB);
@@ -486,9 +637,10 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
       const int at = swz(g + 8 * e, 8 * warp + c2, C);
       *reinterpret_cast<uint32_t*>(sU + at) = hi; *reinterpret_cast<uint32_t*>(sU + 16 * C + at) = lo;
     }
-    if (!mbar_wait(&bars[2], c & 1, abort_flag, a.status)) ok = false;
+    if (!mbar_wait(half_bar(2 * c + 1), half_phase(2 * c + 1), abort_flag, a.status)) ok = false;
     if (!__syncthreads_and(ok)) break;         // U is complete, this chunk's W, Q~ and the old state have been read
-    if (threadIdx.x == 0 && c + 2 < a.chunks) load_x(c + 2);
+    if (threadIdx.x == 0) load(2 * c + 3);
+    const uint8_t* sy = smem + ((2 * c + 1) % 3) * SLOT;
     const bf16* tk = reinterpret_cast<const bf16*>(sy);
     const bf16* tb = reinterpret_cast<const bf16*>(sy + (It::B - It::K));
     const float* gam = reinterpret_cast<const float*>(sy + (It::G - It::K));
@@ -545,12 +697,12 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
         reinterpret_cast<bf16*>(a.o)[((long long)b * a.T + t) * ((long long)H * E) + (long long)h * E + col] = __float2bfloat16_rn(o[0][e] + (o[1][e] + o[2][e]));
     }
     __syncthreads();                           // K^, B have been read
-    if (threadIdx.x == 0 && c + 1 < a.chunks) load_y(c + 1);
+    if (threadIdx.x == 0) load(2 * c + 4);
   }
   if (c < a.chunks) {                          // a wait ran out: let the copies in flight land before the block ends
     if (threadIdx.x == 0)
-      for (int i = 0; i < 3; i++)
-        for (uint32_t it = 0; it < WAIT_LIMIT && !mbar_try_wait(&bars[i], i < 2 ? (((c + ((c ^ i) & 1)) >> 1) & 1) : (c & 1)); ++it) {}
+      for (int i = 2 * c; i < 2 * c + 4 && i < 2 * a.chunks; i++)
+        for (uint32_t it = 0; it < (WAIT_LIMIT >> 2) && !mbar_try_wait(half_bar(i), half_phase(i)); ++it) {}
     return;
   }
 #pragma unroll
@@ -564,13 +716,13 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
 
 template <int DP, bool DELTA> int run(ChunkArgs a, cudaStream_t s) {
   typedef Item<DP> It;
-  const size_t local = 4 * (size_t)((DELTA ? 4 : 3) * C * (DP + 8) + (DELTA ? 3 : 1) * C * (C + 4) + 72 + (DELTA ? 3 * MAX_TAPS * 128 : 0) + 4);
+  const size_t local = DELTA ? DeltaSmem<DP>::TOTAL : 8 * C * DP;
   const size_t x = (DELTA ? It::X_BYTES : It::X_BYTES - It::Q) + (size_t)C * 16 * 4;
-  const size_t scan = 2 * x + It::Y_BYTES + 2 * 16 * DP * 2 + 2 * 16 * C * 2 + 64 + 128;
+  const size_t scan = 3 * std::max(x, It::Y_BYTES) + 2 * 16 * DP * 2 + 2 * 16 * C * 2 + 64 + 128;
   static PerDevice attr;
   const int dev = PerDevice::current();
   if (dev < 0 || !attr.done[dev]) {
-    CUDA_TRY(cudaFuncSetAttribute(k_chunk_local<DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)local));
+    CUDA_TRY(cudaFuncSetAttribute(DELTA ? k_chunk_local_delta<DP> : k_chunk_local_sum<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)local));
     CUDA_TRY(cudaFuncSetAttribute(k_chunk_scan<DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)scan));
     if (dev >= 0) attr.done[dev] = true;
   }
@@ -580,7 +732,7 @@ template <int DP, bool DELTA> int run(ChunkArgs a, cudaStream_t s) {
   if (seg <= 0) return femto_fail(FEMTO_ERR_NOMEM, "chunked recurrence: workspace too small for %d columns of %d heads", a.B, a.heads);
   for (int c0 = 0; c0 < total; c0 += seg) {
     a.t0 = c0 * C; a.chunks = std::min(seg, total - c0);
-    k_chunk_local<DP, DELTA><<<dim3(a.chunks, a.heads, a.B), LOCAL_THREADS, local, s>>>(a);
+    (DELTA ? k_chunk_local_delta<DP> : k_chunk_local_sum<DP>)<<<dim3(a.chunks, a.heads, a.B), LOCAL_THREADS, local, s>>>(a);
     KERNEL_CHECK();
     k_chunk_scan<DP, DELTA><<<dim3(cdiv(a.vdim, 16), a.heads, a.B), SCAN_THREADS, scan, s>>>(a);
     KERNEL_CHECK();
