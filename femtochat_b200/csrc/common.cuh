@@ -114,6 +114,21 @@ struct PerDevice {
 // has no effect when the next kernel is an ordinary launch.
 #ifdef __CUDACC__
 __device__ __forceinline__ void pdl_trigger() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+// Dependent side of a kernel launched with launch_dependent(): nothing an earlier kernel wrote may be read, and nothing an
+// earlier kernel reads may be written, before this.  Returns at once in a kernel that was launched in the ordinary way.
+__device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+// Launches a kernel that calls pdl_wait() in every thread: its blocks may be scheduled while the previous kernel of the
+// stream drains, so the launch latency of a chain of small kernels (a decode step) is hidden.
+template <typename... P, typename... A>
+static inline cudaError_t launch_dependent(void (*kernel)(P...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, A... args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid; cfg.blockDim = block; cfg.dynamicSmemBytes = smem; cfg.stream = s;
+  cudaLaunchAttribute at[1];
+  at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  at[0].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = at; cfg.numAttrs = 1;
+  return cudaLaunchKernelEx(&cfg, kernel, static_cast<P>(args)...);
+}
 #endif
 int device_sm_count();   // multiprocessors of the current device (cached per device)
 
@@ -133,6 +148,7 @@ enum GemmEpi {
   EPI_F32 = 5,      // C_f32 = (beta? C_f32 : 0) + alpha*acc
   EPI_XENT_STATS = 6,   // tensor-core path only: per-row partial (max, sum exp) of softcapped logits; with C set the
                         // logits are also stored there as T
+  EPI_SWIGLU = 7,   // B's columns are groups of 32 gate and 32 up columns in turn: C_T[M][N / 2] = silu(gate) * up
 };
 
 struct GemmArgs {
@@ -150,6 +166,7 @@ struct GemmArgs {
   // square symmetric result: tiles that lie entirely below the diagonal are not computed (the caller mirrors
   // the upper triangle afterwards); honoured by the tensor-core kernel, ignored by the SIMT fallback
   bool upper_only = false;
+  bool any_size = false;   // take the tensor-core kernel for results smaller than one tile as well
   int ring = 0;   // depth of the operand ring of the tensor-core kernel; 0 = the deepest that fits (fewer stages leave
                   // shared memory free for kernels of another stream to run on the same SMs)
   // cross-entropy statistics epilogue

@@ -65,6 +65,8 @@ int decoder_fill(DecoderStack* d, const femto_decoder_config* cfg) {
     l.c.decay_rank = o.decay_rank; l.c.gate_rank = o.gate_rank;
     if (a.mixer == FEMTO_MIXER_LIGHTNING) l.decay.assign(a.h_decay, a.h_decay + a.heads);
     l.c.h_decay = nullptr;
+    if (a.mixer == FEMTO_MIXER_LATENT_ATTENTION)
+      for (int k = 0; k < a.rot_dims / 2; k++) l.freq.push_back((float)pow(a.rot_base, -2.0 * k / a.rot_dims));
   }
   // flat layout, and the derived sizes of every layer
   long long pos = 0;
@@ -154,6 +156,7 @@ void carve(DecoderStack* d, Carver& b) {
       cq = std::max(cq, (size_t)l.qp); q = std::max(q, H * (D + c.rot_dim)); qa = std::max(qa, H * l.ld);
     }
     b.take(l.decay_dev, 4 * H);
+    b.take(l.freq_dev, 4 * l.freq.size() + 4);
     if (l.own != (int)i) continue;
     b.take(l.w_in, es * l.n_in * w); b.take(l.w_o, es * w * H * E);
     if (c.mixer == FEMTO_MIXER_CHANNEL_DELTA) { b.take(l.w_a2, es * H * D * l.ra); b.take(l.w_g2, es * H * E * l.rg); }
@@ -204,8 +207,10 @@ int decoder_create(const femto_decoder_config* cfg, femto_handle** out) {
   Carver real;
   real.base = d->arena;
   carve(d, real);
-  for (auto& l : d->layers)
+  for (auto& l : d->layers) {
+    if (!l.freq.empty()) cudaMemcpy(l.freq_dev, l.freq.data(), 4 * l.freq.size(), cudaMemcpyHostToDevice);
     if (!l.decay.empty()) cudaMemcpy(l.decay_dev, l.decay.data(), 4 * l.decay.size(), cudaMemcpyHostToDevice);
+  }
   femto_handle* h = new femto_handle();
   h->dec = d;
   h->bf = d->bf;
@@ -284,7 +289,7 @@ int decoder_cache_create(femto_handle* h, int max_batch, int max_len, femto_kv_c
     const femto_layer_config& q = l.c;
     if (q.mixer != FEMTO_MIXER_LATENT_ATTENTION) continue;
     exp_bytes = std::max(exp_bytes, es * B * max_len * (size_t)q.heads * (q.dim + q.vdim));
-    c->part_floats = std::max(c->part_floats, (size_t)std::max(64, max_batch * LATENT_FEW) * q.heads * (size_t)(l.lp + 2) * 2);
+    c->part_floats = std::max(c->part_floats, (size_t)std::max(128, max_batch * LATENT_FEW) * q.heads * (size_t)(l.lp + 2) * 2);
   }
   auto lay = [&](Carver& b) {
     for (size_t i = 0; i < d->layers.size(); i++) {
@@ -351,14 +356,22 @@ static int mixer_t(DecoderStack* d, femto_kv_cache* c, int i, const float* theta
     else FEMTO_TRY(recurrence<T>(a, s));
     FEMTO_TRY(S::gated_norm((const T*)d->mixo, theta + l.mix_norm, true, proj + l.s_g, l.n_in, out, R, 1, H * E, eps, s));
   } else if (q.mixer == FEMTO_MIXER_CHANNEL_DELTA) {
-    FEMTO_TRY(rows_linear<T>(d, proj + l.s_a1, l.n_in, l.w_a2, l.ra, d->gd, H * D, R, H * D, l.ra, EPI_F32, s));
-    FEMTO_TRY(rows_linear<T>(d, proj + l.s_g1, l.n_in, l.w_g2, l.rg, d->g2, H * E, R, H * E, l.rg, EPI_STORE, s));
     DeltaPrepArgs p;
     p.proj = proj; p.ldp = l.n_in; p.s_q = l.s_q; p.s_k = l.s_k; p.s_v = l.s_v; p.s_b = l.s_b;
     p.conv_q = theta + l.conv_q; p.conv_k = theta + l.conv_k; p.conv_v = theta + l.conv_v; p.a_log = theta + l.a_log; p.dt_bias = theta + l.dt_bias;
     p.tail_in = st.tail[st.tail_now]; p.tail_out = st.tail[st.tail_now ^ 1];
     p.qn = d->qn; p.kn = d->kn; p.gd = d->gd; p.beta = d->beta; p.vv = d->vv;
     p.B = B; p.T = Tn; p.heads = H; p.kv_heads = q.kv_heads; p.dim = D; p.vdim = E; p.taps = q.conv;
+    if (Tn == 1) {
+      DeltaDecodeArgs t;
+      t.p = p; t.s_a1 = l.s_a1; t.s_g1 = l.s_g1; t.ra = l.ra; t.rg = l.rg; t.w_a2 = l.w_a2; t.w_g2 = l.w_g2; t.S = st.S;
+      t.norm = theta + l.mix_norm; t.eps = eps; t.out = out;
+      FEMTO_TRY(delta_decode<T>(t, s));
+      st.tail_now ^= 1;
+      return rows_linear<T>(d, out, H * E, l.w_o, H * E, d->y, w, R, w, H * E, EPI_STORE, s);
+    }
+    FEMTO_TRY(rows_linear<T>(d, proj + l.s_a1, l.n_in, l.w_a2, l.ra, d->gd, H * D, R, H * D, l.ra, EPI_F32, s));
+    FEMTO_TRY(rows_linear<T>(d, proj + l.s_g1, l.n_in, l.w_g2, l.rg, d->g2, H * E, R, H * E, l.rg, EPI_STORE, s));
     ChunkArgs ca;
     ca.proj = proj; ca.ldp = l.n_in; ca.s_q = l.s_q; ca.s_k = l.s_k; ca.s_v = l.s_v; ca.s_b = l.s_b; ca.conv_q = p.conv_q; ca.conv_k = p.conv_k;
     ca.conv_v = p.conv_v; ca.a_log = p.a_log; ca.dt_bias = p.dt_bias; ca.graw = d->gd; ca.tail_in = p.tail_in; ca.S = st.S; ca.o = d->mixo;
@@ -374,15 +387,15 @@ static int mixer_t(DecoderStack* d, femto_kv_cache* c, int i, const float* theta
     if (!chunked) FEMTO_TRY(recurrence<T>(a, s));
     FEMTO_TRY(S::gated_norm((const T*)d->mixo, theta + l.mix_norm, false, (const T*)d->g2, (long long)H * E, out, R, H, E, eps, s));
   } else {
-    FEMTO_TRY(S::norm_cols(proj + l.s_q, l.n_in, theta + l.dq_norm, (T*)d->cq, l.qp, R, q.q_rank, eps, s));
-    FEMTO_TRY(rows_linear<T>(d, d->cq, l.qp, l.w_uq, l.qp, d->q, H * (D + q.rot_dim), R, H * (D + q.rot_dim), l.qp, EPI_STORE, s));
     LatentArgs a;
     a.q = d->q; a.dkv = proj + l.s_dkv; a.ld_dkv = l.n_in; a.dkv_norm = theta + l.dkv_norm; a.gate = proj + l.s_g; a.ld_gate = l.n_in;
     a.latent = st.latent; a.ld = l.ld; a.lp = l.lp; a.maxT = c->maxT; a.w_kv = l.w_kv; a.kv = c->kv_exp;
     a.qabs = d->qabs; a.part = c->part; a.part_floats = c->part_floats; a.o = out;
     a.B = B; a.T = Tn; a.first = first; a.heads = H; a.dim = D; a.rot_dim = q.rot_dim; a.rot_dims = q.rot_dims; a.vdim = E; a.kv_rank = q.kv_rank;
-    a.scale = q.scale; a.eps = eps; a.rot_base = q.rot_base; a.d = d;
-    FEMTO_TRY(latent_prep<T>(a, s));
+    a.scale = q.scale; a.eps = eps; a.freq = l.freq_dev; a.d = d;
+    a.dq = proj + l.s_q; a.dq_norm = theta + l.dq_norm; a.cq = d->cq; a.q_rank = q.q_rank; a.qp = l.qp;
+    FEMTO_TRY(latent_norms<T>(a, s));
+    FEMTO_TRY(rows_linear<T>(d, d->cq, l.qp, l.w_uq, l.qp, d->q, H * (D + q.rot_dim), R, H * (D + q.rot_dim), l.qp, EPI_STORE, s));
     FEMTO_TRY(latent_attention<T>(a, s));
   }
   return rows_linear<T>(d, out, H * E, l.w_o, H * E, d->y, w, R, w, H * E, EPI_STORE, s);
@@ -404,8 +417,7 @@ static int pass_t(DecoderStack* d, femto_kv_cache* c, const float* theta, const 
     const bool mlp = l.c.ff > 0;
     FEMTO_TRY(S::resid_norm(d->x, (const T*)d->y, theta + l.norm1b, m, mlp ? theta + l.norm2 : next, mlp || next ? (T*)d->hn : nullptr, R, w, eps, s));
     if (mlp) {
-      FEMTO_TRY(rows_linear<T>(d, d->hn, w, l.w_gu, w, d->gu, 2 * l.ffp, R, 2 * l.ffp, w, EPI_STORE, s));
-      FEMTO_TRY(S::gated_mlp((const T*)d->gu, (T*)d->act, R, l.ffp, s));
+      FEMTO_TRY(rows_linear<T>(d, d->hn, w, l.w_gu, w, d->act, l.ffp, R, l.ffp, w, EPI_SWIGLU, s));
       FEMTO_TRY(rows_linear<T>(d, d->act, l.ffp, l.w_down, l.ffp, d->y, w, R, w, l.ffp, EPI_STORE, s));
       FEMTO_TRY(S::resid_norm(d->x, (const T*)d->y, theta + l.norm2b, m, next, next ? (T*)d->hn : nullptr, R, w, eps, s));
     }

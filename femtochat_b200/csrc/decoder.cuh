@@ -15,6 +15,8 @@ struct DecLayer {
   int own = 0;                        // layer that holds the tensors
   std::vector<float> decay;
   float* decay_dev = nullptr;
+  std::vector<float> freq;            // latent attention: rot_base^(-2i/rot_dims)
+  float* freq_dev = nullptr;
   // element offsets into Theta of what is read there in fp32
   long long norm1 = -1, norm1b = -1, norm2 = -1, norm2b = -1, mix_norm = -1, conv_q = -1, conv_k = -1, conv_v = -1,
             a_log = -1, dt_bias = -1, dq_norm = -1, dkv_norm = -1;
@@ -76,8 +78,6 @@ template <typename T> struct DecStream {
   // out[r][g] = rms_norm over each of `groups` runs of `size` of in[r], times w (size, or groups*size when w_all), times sigmoid(gate)
   static int gated_norm(const T* in, const float* w, bool w_all, const T* gate, long long ldg, T* out, int rows, int groups, int size,
                         float eps, cudaStream_t s);
-  // out[r][0..size) = rms_norm(in[r]) w, out[r][size..ldo) = 0
-  static int norm_cols(const T* in, long long ldi, const float* w, T* out, long long ldo, int rows, int size, float eps, cudaStream_t s);
   // act[r][j] = silu(gate) * up from rows of interleaved groups of 32 gate and 32 up columns
   static int gated_mlp(const T* gu, T* act, int rows, int ffp, cudaStream_t s);
 };
@@ -86,8 +86,8 @@ template <typename T>
 int pack_rows(const float* src, int rows, int cols, T* dst, long long ldd, int dst_row, int group, int step, cudaStream_t s);
 
 // ---- products -------------------------------------------------------------------------------------------------------
-// C[M][N] = X[M][K] W[N][K]^T; epi EPI_STORE (compute type) or EPI_F32.  Up to 8 rows stream the weights once through
-// a row-dot kernel, more rows take the tensor-core GEMM.
+// C[M][N] = X[M][K] W[N][K]^T; epi EPI_STORE (compute type), EPI_F32, or EPI_SWIGLU (W holds 2 N rows, groups of 32 gate and
+// 32 up rows in turn; C = silu(gate) * up).  A few rows stream the weights once, more rows take the tensor-core GEMM.
 template <typename T>
 int rows_linear(DecoderStack* d, const void* X, long long ldx, const void* W, long long ldw, void* C, long long ldc, int M, int N, int K,
                 int epi, cudaStream_t s);
@@ -117,6 +117,17 @@ struct DeltaPrepArgs {
 template <typename T> int delta_prep(const DeltaPrepArgs& a, cudaStream_t s);
 template <typename T> int conv_tail(const DeltaPrepArgs& a, cudaStream_t s);   // only the kept inputs
 
+// One token per column: everything between the packed projection and the output projection in one launch.
+struct DeltaDecodeArgs {
+  DeltaPrepArgs p;               // projections, taps and kept inputs (its outputs are unused)
+  int s_a1 = 0, s_g1 = 0, ra = 0, rg = 0;
+  const void *w_a2 = nullptr, *w_g2 = nullptr;
+  float* S = nullptr;
+  const float* norm = nullptr; float eps = 0.f;
+  void* out = nullptr;           // [B][heads * vdim], normed and gated
+};
+template <typename T> int delta_decode(const DeltaDecodeArgs& a, cudaStream_t s);
+
 // The same recurrences for many tokens in bf16 models, chunk by chunk on the tensor cores (chunked_recurrence.cu);
 // convolutions, unit vectors and decays included.
 struct ChunkArgs {
@@ -138,7 +149,7 @@ int chunked_recurrence(const ChunkArgs& a, cudaStream_t s);
 
 // ---- latent attention (latent_attention.cu) -------------------------------------------------------------------------
 struct LatentArgs {
-  void* q = nullptr;             // [rows][heads (dim + rot_dim)], rotated in place by latent_prep
+  void* q = nullptr;             // [rows][heads (dim + rot_dim)], not rotated yet
   const void* dkv = nullptr; long long ld_dkv = 0;     // new rows of W_dkv h (kv_rank, rot_dim)
   const float* dkv_norm = nullptr;
   const void* gate = nullptr; long long ld_gate = 0;   // one logit per head
@@ -149,10 +160,12 @@ struct LatentArgs {
   float* qabs = nullptr; float* part = nullptr; size_t part_floats = 0;
   void* o = nullptr;             // [rows][heads vdim]
   int B = 0, T = 0, first = 0, heads = 0, dim = 0, rot_dim = 0, rot_dims = 0, vdim = 0, kv_rank = 0;
-  float scale = 1.f, eps = 0.f; double rot_base = 1.0;
+  float scale = 1.f, eps = 0.f;
+  const float* freq = nullptr;   // [rot_dims / 2] angle per position
+  const void* dq = nullptr; const float* dq_norm = nullptr; void* cq = nullptr; int q_rank = 0, qp = 0;   // query latent
   DecoderStack* d = nullptr;
 };
-template <typename T> int latent_prep(const LatentArgs& a, cudaStream_t s);
+template <typename T> int latent_norms(const LatentArgs& a, cudaStream_t s);   // query latent -> cq, new rows -> cache
 template <typename T> int latent_attention(const LatentArgs& a, cudaStream_t s);
 bool latent_attention_tc_supported(const LatentArgs& a);       // latent_attention_sm100.cu: the prompt's attention on the tensor cores
 int latent_attention_tc(const LatentArgs& a, cudaStream_t s);

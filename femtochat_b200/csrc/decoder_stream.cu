@@ -26,6 +26,7 @@ __global__ void __launch_bounds__(RT) k_dec_embed(const T* __restrict__ table, c
                                                   int base, int vocab, const float* __restrict__ w, float* __restrict__ x,
                                                   T* __restrict__ h, int d, float eps, unsigned int* status) {
   pdl_trigger();
+  pdl_wait();
   const int row = blockIdx.x;
   int tk = tokens[(long long)(row / T_) * ld_tok + row % T_] - base;
   if (tk < 0 || tk >= vocab) { if (threadIdx.x == 0) atomicOr(status, ST_BAD_TOKEN); tk = min(max(tk, 0), vocab - 1); }
@@ -45,6 +46,7 @@ template <typename T, int NV>
 __global__ void __launch_bounds__(RT) k_resid_norm(float* __restrict__ x, const T* __restrict__ y, const float* __restrict__ w_post,
                                                    float m, const float* __restrict__ w_pre, T* __restrict__ h, int d, float eps) {
   pdl_trigger();
+  pdl_wait();
   const long long base = (long long)blockIdx.x * d;
   if constexpr (NV > 0) {
     float f[NV][4], r[NV][4];
@@ -120,6 +122,7 @@ template <typename T>
 __global__ void __launch_bounds__(RT) k_gather_norm(const float* __restrict__ x, const int* __restrict__ want, int stride,
                                                     const float* __restrict__ w, T* __restrict__ h, int d, float eps) {
   pdl_trigger();
+  pdl_wait();
   const int i = blockIdx.x;
   const float* src = x + (long long)(want ? want[i] : (i + 1) * stride - 1) * d;
   float ss = 0.f;
@@ -134,6 +137,7 @@ __global__ void __launch_bounds__(256) k_gated_norm(const T* __restrict__ in, co
                                                     const T* __restrict__ gate, long long ldg, T* __restrict__ out, long long n,
                                                     int groups, int size, float eps) {
   pdl_trigger();
+  pdl_wait();
   const long long it = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   if (it >= n) return;
   const int lane = threadIdx.x & 31, g = (int)(it % groups);
@@ -160,21 +164,9 @@ __global__ void __launch_bounds__(256) k_gated_norm(const T* __restrict__ in, co
 }
 
 template <typename T>
-__global__ void __launch_bounds__(256) k_norm_cols(const T* __restrict__ in, long long ldi, const float* __restrict__ w, T* __restrict__ out,
-                                                   long long ldo, int rows, int size, float eps) {
-  pdl_trigger();
-  const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (row >= rows) return;
-  const T* a = in + (long long)row * ldi;
-  float ss = 0.f;
-  for (int c = lane; c < size; c += 32) { const float f = to_f<T>(a[c]); ss += f * f; }
-  const float inv = 1.f / sqrtf(warp_sum(ss) / size + eps);
-  for (int c = lane; c < ldo; c += 32) out[(long long)row * ldo + c] = from_f<T>(c < size ? to_f<T>(a[c]) * inv * w[c] : 0.f);
-}
-
-template <typename T>
 __global__ void __launch_bounds__(256) k_gated_mlp(const T* __restrict__ gu, T* __restrict__ act, long long n, int ffp) {
   pdl_trigger();
+  pdl_wait();
   constexpr int V = VecN<T>::n;
   const long long i = ((long long)blockIdx.x * 256 + threadIdx.x) * V;
   if (i >= n) return;
@@ -198,52 +190,110 @@ __global__ void __launch_bounds__(256) k_pack_rows(const float* __restrict__ src
   dst[(long long)(dst_row + (r / group) * step + r % group) * ldd + c] = from_f<T>(src[i]);
 }
 
-// C[m][n] = sum_k X[m][k] W[n][k] for M <= 8 rows: one warp per output column, 16-byte loads of W, X in shared memory.
-// Every weight is read exactly once.
+// C[m][n] = sum_k X[m][k] W[n][k] for a few rows, any size: one warp per output column.  GATED: column n is
+// silu(row n of the gate weights) * row n of the up weights, which alternate in groups of 32 rows.
 constexpr int RL_ROWS = 8;
-template <typename T, int MR, bool VEC>
+template <typename T, bool GATED>
 __global__ void __launch_bounds__(256) k_rows_linear(const T* __restrict__ X, long long ldx, const T* __restrict__ W, long long ldw,
                                                      void* __restrict__ C, long long ldc, int M, int N, int K, int f32_out) {
   pdl_trigger();
+  pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n = blockIdx.x * 8 + warp;
   if (n >= N) return;
-  const T* wr = W + (long long)n * ldw;
-  float acc[MR];
+  const T* wr = W + (long long)(GATED ? (n >> 5) * 64 + (n & 31) : n) * ldw;
+  float acc[RL_ROWS] = {}, up[RL_ROWS] = {};
+  for (int k = lane; k < K; k += 32) {
+    const float w = to_f<T>(wr[k]), u = GATED ? to_f<T>(wr[32 * ldw + k]) : 0.f;
 #pragma unroll
-  for (int m = 0; m < MR; m++) acc[m] = 0.f;
-  if constexpr (VEC) {
-    constexpr int V = VecN<T>::n;
-#pragma unroll 4
-    for (int k = lane * V; k < K; k += 32 * V) {
-      float w[V];
-      load_vec<T, V>(wr + k, w);
-#pragma unroll
-      for (int m = 0; m < MR; m++) {
-        if (m < M) {
-          float x[V];
-          load_vec<T, V>(X + m * ldx + k, x);
-#pragma unroll
-          for (int e = 0; e < V; e++) acc[m] = fmaf(x[e], w[e], acc[m]);
-        }
+    for (int m = 0; m < RL_ROWS; m++)
+      if (m < M) {
+        const float x = to_f<T>(X[m * ldx + k]);
+        acc[m] = fmaf(x, w, acc[m]);
+        if (GATED) up[m] = fmaf(x, u, up[m]);
       }
-    }
-  } else {
-    for (int k = lane; k < K; k += 32) {
-      const float w = to_f<T>(wr[k]);
-#pragma unroll
-      for (int m = 0; m < MR; m++)
-        if (m < M) acc[m] = fmaf(to_f<T>(X[m * ldx + k]), w, acc[m]);
-    }
   }
 #pragma unroll
-  for (int m = 0; m < MR; m++) {
+  for (int m = 0; m < RL_ROWS; m++) {
     if (m >= M) break;
-    const float v = warp_sum(acc[m]);
+    float v = warp_sum(acc[m]);
+    if (GATED) v = v * sigmoid_f(v) * warp_sum(up[m]);
     if (lane == 0) {
       if (f32_out) reinterpret_cast<float*>(C)[m * ldc + n] = v;
       else reinterpret_cast<T*>(C)[m * ldc + n] = from_f<T>(v);
     }
+  }
+}
+
+// The same in bf16 as a stream of the weights through the tensor cores: a block owns 16 output columns (32 weight rows when
+// GATED), its eight warps share K.  The weights are the 16-row operand, the rows of X the 8-column operand, so every
+// weight is loaded once, straight into the fragment that uses it: a lane takes 16 consecutive bytes of a row, and since X
+// is read in the same order the permutation of K inside a step does not matter.  The first weights are on their way
+// before the kernel waits for its predecessor.
+template <int NT, bool GATED>
+__global__ void __launch_bounds__(256) k_rows_mma(const bf16* __restrict__ X, long long ldx, const bf16* __restrict__ W, long long ldw,
+                                                  void* __restrict__ C, long long ldc, int M, int N, int K, int f32_out) {
+  pdl_trigger();
+  constexpr int RT = GATED ? 2 : 1, U = 4;      // U steps of 256 k are loaded ahead
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c8 = (lane & 3) * 8;
+  const int n0 = blockIdx.x * 16;
+  const bf16* wp[2 * RT];
+#pragma unroll
+  for (int i = 0; i < 2; i++) {
+    const int n = min(n0 + g + 8 * i, N - 1), r = GATED ? (n >> 5) * 64 + (n & 31) : n;
+    wp[i] = W + (long long)r * ldw;
+    if (GATED) wp[2 + i] = W + (long long)(r + 32) * ldw;
+  }
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  uint4 w[U][2 * RT];
+  auto fetch = [&](int u, int k) {
+#pragma unroll
+    for (int i = 0; i < 2 * RT; i++) w[u][i] = k < K ? __ldg(reinterpret_cast<const uint4*>(wp[i] + k)) : zero;
+  };
+  const int kb = warp * 32 + c8;
+#pragma unroll
+  for (int u = 0; u < U; u++) fetch(u, kb + u * 256);
+  pdl_wait();
+  float acc[RT][NT][4] = {};
+  for (int k0 = kb; k0 < K + c8; k0 += U * 256) {       // the four lanes of a row leave together
+#pragma unroll
+    for (int u = 0; u < U; u++) {
+      const int k = k0 + u * 256;
+      uint4 x[NT];
+#pragma unroll
+      for (int t = 0; t < NT; t++) x[t] = k < K && 8 * t + g < M ? *reinterpret_cast<const uint4*>(X + (8 * t + g) * ldx + k) : zero;
+#pragma unroll
+      for (int i = 0; i < RT; i++)
+#pragma unroll
+        for (int t = 0; t < NT; t++) {
+          float* d = acc[i][t];
+          const uint4 a = w[u][2 * i], b = w[u][2 * i + 1];
+          asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a.x), "r"(b.x), "r"(a.y), "r"(b.y), "r"(x[t].x), "r"(x[t].y));
+          asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a.z), "r"(b.z), "r"(a.w), "r"(b.w), "r"(x[t].z), "r"(x[t].w));
+        }
+      fetch(u, k + U * 256);
+    }
+  }
+  // sum over the warps in order
+  __shared__ float red[8][RT][8 * NT][16 + 1];
+#pragma unroll
+  for (int i = 0; i < RT; i++)
+#pragma unroll
+    for (int t = 0; t < NT; t++)
+#pragma unroll
+      for (int e = 0; e < 4; e++) red[warp][i][8 * t + 2 * (lane & 3) + (e & 1)][g + 8 * (e >> 1)] = acc[i][t][e];
+  __syncthreads();
+  for (int o = threadIdx.x; o < 16 * 8 * NT; o += 256) {
+    const int m = o >> 4, j = o & 15;
+    if (m >= M || n0 + j >= N) continue;
+    float v = 0.f, up = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; i++) { v += red[i][0][m][j]; if (GATED) up += red[i][RT - 1][m][j]; }
+    if (GATED) v = v * sigmoid_f(v) * up;
+    if (f32_out) reinterpret_cast<float*>(C)[m * ldc + n0 + j] = v;
+    else reinterpret_cast<bf16*>(C)[m * ldc + n0 + j] = __float2bfloat16_rn(v);
   }
 }
 
@@ -252,7 +302,7 @@ __global__ void __launch_bounds__(256) k_rows_linear(const T* __restrict__ X, lo
 template <typename T>
 int DecStream<T>::embed(const T* table, const int* tokens, int ld_tok, int B, int T_, int base, int vocab, const float* w, float* x, T* h,
                         int d, float eps, unsigned int* status, cudaStream_t s) {
-  k_dec_embed<T><<<B * T_, RT, 0, s>>>(table, tokens, ld_tok, T_, base, vocab, w, x, h, d, eps, status);
+  CUDA_TRY(launch_dependent(k_dec_embed<T>, B * T_, RT, 0, s, table, tokens, ld_tok, T_, base, vocab, w, x, h, d, eps, status));
   KERNEL_CHECK();
   return 0;
 }
@@ -261,16 +311,16 @@ int DecStream<T>::resid_norm(float* x, const T* y, const float* w_post, float m,
                              cudaStream_t s) {
   const bool vec = (d & 3) == 0 && aligned16(x) && aligned16(y) && aligned16(w_post) && (!h || (aligned16(w_pre) && aligned16(h)));
   const int nv = vec ? cdiv(d, RT * 4) : 0;
-  if (nv == 1) k_resid_norm<T, 1><<<rows, RT, 0, s>>>(x, y, w_post, m, w_pre, h, d, eps);
-  else if (nv == 2) k_resid_norm<T, 2><<<rows, RT, 0, s>>>(x, y, w_post, m, w_pre, h, d, eps);
-  else if (nv == 3 || nv == 4) k_resid_norm<T, 4><<<rows, RT, 0, s>>>(x, y, w_post, m, w_pre, h, d, eps);
-  else k_resid_norm<T, 0><<<rows, RT, 0, s>>>(x, y, w_post, m, w_pre, h, d, eps);
+  if (nv == 1) CUDA_TRY(launch_dependent(k_resid_norm<T, 1>, rows, RT, 0, s, x, y, w_post, m, w_pre, h, d, eps));
+  else if (nv == 2) CUDA_TRY(launch_dependent(k_resid_norm<T, 2>, rows, RT, 0, s, x, y, w_post, m, w_pre, h, d, eps));
+  else if (nv == 3 || nv == 4) CUDA_TRY(launch_dependent(k_resid_norm<T, 4>, rows, RT, 0, s, x, y, w_post, m, w_pre, h, d, eps));
+  else CUDA_TRY(launch_dependent(k_resid_norm<T, 0>, rows, RT, 0, s, x, y, w_post, m, w_pre, h, d, eps));
   KERNEL_CHECK();
   return 0;
 }
 template <typename T>
 int DecStream<T>::gather_norm(const float* x, const int* want, int stride, const float* w, T* h, int n, int d, float eps, cudaStream_t s) {
-  k_gather_norm<T><<<n, RT, 0, s>>>(x, want, stride, w, h, d, eps);
+  CUDA_TRY(launch_dependent(k_gather_norm<T>, n, RT, 0, s, x, want, stride, w, h, d, eps));
   KERNEL_CHECK();
   return 0;
 }
@@ -280,21 +330,15 @@ int DecStream<T>::gated_norm(const T* in, const float* w, bool w_all, const T* g
   const long long n = (long long)rows * groups;
   constexpr int V = VecN<T>::n;
   if (size % V == 0 && ldg % V == 0 && aligned16(in) && aligned16(gate) && aligned16(out))
-    k_gated_norm<T, V><<<cdiv(n, 8), 256, 0, s>>>(in, w, w_all, gate, ldg, out, n, groups, size, eps);
+    CUDA_TRY(launch_dependent(k_gated_norm<T, V>, cdiv(n, 8), 256, 0, s, in, w, (int)w_all, gate, ldg, out, n, groups, size, eps));
   else
-    k_gated_norm<T, 1><<<cdiv(n, 8), 256, 0, s>>>(in, w, w_all, gate, ldg, out, n, groups, size, eps);
-  KERNEL_CHECK();
-  return 0;
-}
-template <typename T>
-int DecStream<T>::norm_cols(const T* in, long long ldi, const float* w, T* out, long long ldo, int rows, int size, float eps, cudaStream_t s) {
-  k_norm_cols<T><<<cdiv(rows, 8), 256, 0, s>>>(in, ldi, w, out, ldo, rows, size, eps);
+    CUDA_TRY(launch_dependent(k_gated_norm<T, 1>, cdiv(n, 8), 256, 0, s, in, w, (int)w_all, gate, ldg, out, n, groups, size, eps));
   KERNEL_CHECK();
   return 0;
 }
 template <typename T> int DecStream<T>::gated_mlp(const T* gu, T* act, int rows, int ffp, cudaStream_t s) {
   const long long n = (long long)rows * ffp;
-  k_gated_mlp<T><<<cdiv(n, 256 * VecN<T>::n), 256, 0, s>>>(gu, act, n, ffp);
+  CUDA_TRY(launch_dependent(k_gated_mlp<T>, cdiv(n, 256 * VecN<T>::n), 256, 0, s, gu, act, n, ffp));
   KERNEL_CHECK();
   return 0;
 }
@@ -311,28 +355,43 @@ int pack_rows(const float* src, int rows, int cols, T* dst, long long ldd, int d
 template int pack_rows<float>(const float*, int, int, float*, long long, int, int, int, cudaStream_t);
 template int pack_rows<bf16>(const float*, int, int, bf16*, long long, int, int, int, cudaStream_t);
 
+// Up to ROWS_STREAM rows in bf16 with aligned operands (RL_ROWS otherwise) stream the weights; more rows are a GEMM.
+constexpr int ROWS_STREAM = 32;
+
 template <typename T>
 int rows_linear(DecoderStack* d, const void* X, long long ldx, const void* W, long long ldw, void* C, long long ldc, int M, int N, int K,
                 int epi, cudaStream_t s) {
-  if (M <= RL_ROWS) {
-    constexpr int V = VecN<T>::n;
-    const bool vec = K % V == 0 && ldx % V == 0 && ldw % V == 0 && aligned16(X) && aligned16(W);
-    const int grid = cdiv(N, 8), f32 = epi == EPI_F32;
-#define LAUNCH(MR, VEC) k_rows_linear<T, MR, VEC><<<grid, 256, 0, s>>>((const T*)X, ldx, (const T*)W, ldw, C, ldc, M, N, K, f32)
-    if (!vec) LAUNCH(8, false);
-    else if (M == 1) LAUNCH(1, true);
-    else if (M == 2) LAUNCH(2, true);
-    else if (M <= 4) LAUNCH(4, true);
-    else LAUNCH(8, true);
+  const int f32 = epi == EPI_F32;
+  if constexpr (sizeof(T) == 2) {
+    if (M <= ROWS_STREAM && ((K | ldx | ldw) & 7) == 0 && aligned16(X) && aligned16(W)) {
+      const int grid = cdiv(N, 16);
+#define LAUNCH(NT) CUDA_TRY(epi == EPI_SWIGLU ? launch_dependent(k_rows_mma<NT, true>, grid, 256, 0, s, (const bf16*)X, ldx, (const bf16*)W, ldw, C, ldc, M, N, K, f32) \
+                                              : launch_dependent(k_rows_mma<NT, false>, grid, 256, 0, s, (const bf16*)X, ldx, (const bf16*)W, ldw, C, ldc, M, N, K, f32))
+      if (M <= 8) LAUNCH(1);
+      else if (M <= 16) LAUNCH(2);
+      else LAUNCH(4);
 #undef LAUNCH
+      KERNEL_CHECK();
+      return 0;
+    }
+  }
+  if (M <= RL_ROWS) {
+    if (epi == EPI_SWIGLU) CUDA_TRY(launch_dependent(k_rows_linear<T, true>, cdiv(N, 8), 256, 0, s, (const T*)X, ldx, (const T*)W, ldw, C, ldc, M, N, K, f32));
+    else CUDA_TRY(launch_dependent(k_rows_linear<T, false>, cdiv(N, 8), 256, 0, s, (const T*)X, ldx, (const T*)W, ldw, C, ldc, M, N, K, f32));
     KERNEL_CHECK();
     return 0;
   }
   GemmArgs g;
   g.ws = d->gemm_ws; g.ws_bytes = d->gemm_ws_bytes; g.status = d->status;
   g.A = X; g.lda = ldx; g.a_kmajor = true; g.B = W; g.ldb = ldw; g.b_kmajor = true;
-  g.C = C; g.ldc = ldc; g.M = M; g.N = N; g.K = K; g.epi = epi; g.beta = 0.f;
-  return gemm<T>(g, s);
+  g.C = C; g.ldc = ldc; g.M = M; g.N = N; g.K = K; g.epi = epi; g.beta = 0.f; g.any_size = true;
+  if (epi != EPI_SWIGLU) return gemm<T>(g, s);
+  // g.N counts the weight rows, gate and up together; the result is half as wide
+  g.N = 2 * N;
+  if (sizeof(T) == 2 && gemm_tc_supported(g)) return gemm<T>(g, s);
+  g.epi = EPI_STORE; g.C = d->gu; g.ldc = 2 * N;
+  FEMTO_TRY(gemm<T>(g, s));
+  return DecStream<T>::gated_mlp((const T*)d->gu, (T*)C, M, N, s);
 }
 template int rows_linear<float>(DecoderStack*, const void*, long long, const void*, long long, void*, long long, int, int, int, int, cudaStream_t);
 template int rows_linear<bf16>(DecoderStack*, const void*, long long, const void*, long long, void*, long long, int, int, int, int, cudaStream_t);

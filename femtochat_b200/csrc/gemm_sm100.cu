@@ -179,7 +179,8 @@ __device__ __forceinline__ void bf16_chunk(const GemmArgs& g, float (&v)[32], in
   }
 }
 
-template <bool A_K, bool B_K, bool PAIR>
+// ACT: the instantiation for EPI_SWIGLU, kept apart so that the other epilogues keep their registers.
+template <bool A_K, bool B_K, bool PAIR, bool ACT = false>
 __global__ void __launch_bounds__(NTHREADS, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                const __grid_constant__ CUtensorMap tmC, const TcParams p) {
@@ -383,6 +384,28 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
         }
         tmem_ld_wait();
         const int nc = n0 + c * 32;
+        if constexpr (ACT) {
+          // chunks come in pairs of 32 gate and 32 up columns; both are taken at the first
+          if (nc >= g.N || (ci & 1)) continue;
+          uint32_t up[32];
+          tmem_ld32(taddr + c * 32 + 32, up);
+          tmem_ld_wait();
+          if (!row_ok) continue;
+          bf16* dst = reinterpret_cast<bf16*>(g.C) + (long long)bz * g.strideC + (long long)m * g.ldc + nc / 2;
+#pragma unroll
+          for (int j = 0; j < 32; j += 8) {
+            uint4 q;
+            __nv_bfloat162* hq = reinterpret_cast<__nv_bfloat162*>(&q);
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+              const float x = __uint_as_float(r[j + 2 * e]), y = __uint_as_float(r[j + 2 * e + 1]);
+              hq[e] = __floats2bfloat162_rn(x * __fdividef(1.f, 1.f + __expf(-x)) * __uint_as_float(up[j + 2 * e]),
+                                            y * __fdividef(1.f, 1.f + __expf(-y)) * __uint_as_float(up[j + 2 * e + 1]));
+            }
+            *reinterpret_cast<uint4*>(dst + j) = q;
+          }
+          continue;
+        }
         const bool tma_out = p.tma_store != 0 && p.splits == 1 && g.epi != EPI_F32;
         if (nc >= g.N || (!row_ok && !tma_out)) continue;   // on the TMA path the whole warp stays together
         uint8_t* sbuf = tma_out ? store_stage + (warp - 2) * 4096 : nullptr;
@@ -642,7 +665,10 @@ int make_tmap_2d_bf16(CUtensorMap* out, const void* base, uint64_t dim0, uint64_
 }
 
 bool gemm_tc_supported(const GemmArgs& g) {
-  if (g.M < BM || g.N < BN || g.K < BK) return false;
+  // smaller results than one tile go to the SIMT kernel unless the caller asks for the tensor cores (tiles are clipped and
+  // zero-filled by the copies either way)
+  if (g.any_size ? g.M < 1 || g.N < 1 || g.K < 8 : g.M < BM || g.N < BN || g.K < BK) return false;
+  if (g.epi == EPI_SWIGLU && (!g.a_kmajor || !g.b_kmajor || (g.N & 63) || (g.ldc & 7) || !g.C || !aligned16(g.C))) return false;
   if ((g.lda & 7) || (g.ldb & 7) || (g.strideA & 7) || (g.strideB & 7)) return false;
   if (!aligned16(g.A) || !aligned16(g.B)) return false;
   // the contiguous extent of an M/N-major operand must cover whole 16-byte units
@@ -764,6 +790,7 @@ static int launch_tc(const GemmArgs& g, const CUtensorMap& tmA, const CUtensorMa
   const int dev = PerDevice::current();
   if (dev < 0 || !attr.done[dev]) {
     CUDA_TRY(cudaFuncSetAttribute(gemm_tc_kernel<true, true, PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, G::SMEM_BYTES));
+    CUDA_TRY(cudaFuncSetAttribute(gemm_tc_kernel<true, true, PAIR, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, G::SMEM_BYTES));
     CUDA_TRY(cudaFuncSetAttribute(gemm_tc_kernel<true, false, PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, G::SMEM_BYTES));
     CUDA_TRY(cudaFuncSetAttribute(gemm_tc_kernel<false, true, PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, G::SMEM_BYTES));
     CUDA_TRY(cudaFuncSetAttribute(gemm_tc_kernel<false, false, PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, G::SMEM_BYTES));
@@ -781,7 +808,8 @@ static int launch_tc(const GemmArgs& g, const CUtensorMap& tmA, const CUtensorMa
   at[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = at; cfg.numAttrs = pdl ? 2 : 1;
   cudaError_t e;
-  if (g.a_kmajor && g.b_kmajor) e = cudaLaunchKernelEx(&cfg, gemm_tc_kernel<true, true, PAIR>, tmA, tmB, tmC, p);
+  if (g.epi == EPI_SWIGLU) e = cudaLaunchKernelEx(&cfg, gemm_tc_kernel<true, true, PAIR, true>, tmA, tmB, tmC, p);
+  else if (g.a_kmajor && g.b_kmajor) e = cudaLaunchKernelEx(&cfg, gemm_tc_kernel<true, true, PAIR>, tmA, tmB, tmC, p);
   else if (g.a_kmajor) e = cudaLaunchKernelEx(&cfg, gemm_tc_kernel<true, false, PAIR>, tmA, tmB, tmC, p);
   else if (g.b_kmajor) e = cudaLaunchKernelEx(&cfg, gemm_tc_kernel<false, true, PAIR>, tmA, tmB, tmC, p);
   else e = cudaLaunchKernelEx(&cfg, gemm_tc_kernel<false, false, PAIR>, tmA, tmB, tmC, p);
@@ -861,7 +889,7 @@ int gemm_tc_bf16(const GemmArgs& g, cudaStream_t s) {
 
   CUtensorMap tmC = tmA;
   p.tma_store = 0;
-  const bool bf16_out = g.epi != EPI_F32 && (g.epi != EPI_XENT_STATS || g.C != nullptr);
+  const bool bf16_out = g.epi != EPI_F32 && g.epi != EPI_SWIGLU && (g.epi != EPI_XENT_STATS || g.C != nullptr);
   if (bf16_out && splits == 1 && (g.ldc & 7) == 0 && (g.strideC & 7) == 0 && aligned16(g.C)) {
     FEMTO_TRY(make_tmap_3d_bf16_sw(&tmC, g.C, g.N, g.M, nb, g.ldc, g.strideC, 64, 32, 3));
     p.tma_store = 1;

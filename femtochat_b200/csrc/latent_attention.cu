@@ -8,41 +8,90 @@
 
 namespace {
 
-// ---- new rows: latent norm, rotations -------------------------------------------------------------------------------
-// One warp per token row.
+// ---- new rows ---------------------------------------------------------------------------------------------------------
+// out[0 .. ldo) = rms_norm(in[0 .. size)) w, then zeros; by one warp
+template <typename T, int V>
+__device__ __forceinline__ void warp_norm(const T* __restrict__ in, const float* __restrict__ w, T* __restrict__ out, int ldo, int size,
+                                          float eps, int lane) {
+  float ss = 0.f;
+#pragma unroll 4
+  for (int c = lane * V; c < size; c += 32 * V) {
+    float f[V];
+    load_vec<T, V>(in + c, f);
+#pragma unroll
+    for (int e = 0; e < V; e++) ss += f[e] * f[e];
+  }
+  const float inv = 1.f / sqrtf(warp_sum(ss) / size + eps);
+#pragma unroll 4
+  for (int c = lane * V; c < ldo; c += 32 * V) {
+    float f[V] = {};
+    if (c < size) load_vec<T, V>(in + c, f);
+#pragma unroll
+    for (int e = 0; e < V; e++) f[e] = c + e < size ? f[e] * inv * w[c + e] : 0.f;
+    store_vec<T, V>(out + c, f);
+  }
+}
+__device__ __forceinline__ void rotate(float u, float v, float pos, float freq, float& a, float& b) {
+  float sn, cs;
+  sincosf(pos * freq, &sn, &cs);
+  a = u * cs - v * sn;
+  b = v * cs + u * sn;
+}
+
+// One warp per (row, part): part 0 norms the query latent, part 1 norms the latent and rotates the shared key part into
+// the cache.
 template <typename T>
-__global__ void __launch_bounds__(256) k_latent_prep(const LatentArgs a) {
+__global__ void __launch_bounds__(256) k_latent_norms(const LatentArgs a) {
   pdl_trigger();
-  const long long row = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (row >= (long long)a.B * a.T) return;
-  const int lane = threadIdx.x & 31;
+  pdl_wait();
+  constexpr int V = VecN<T>::n;
+  const long long it = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (it >= 2LL * a.B * a.T) return;
+  const int lane = threadIdx.x & 31, part = (int)(it & 1);
+  const long long row = it >> 1;
+  if (part == 0) {
+    const T* src = reinterpret_cast<const T*>(a.dq) + row * a.ld_dkv;
+    T* dst = reinterpret_cast<T*>(a.cq) + row * a.qp;
+    if (a.q_rank % V == 0) warp_norm<T, V>(src, a.dq_norm, dst, a.qp, a.q_rank, a.eps, lane);
+    else warp_norm<T, 1>(src, a.dq_norm, dst, a.qp, a.q_rank, a.eps, lane);
+    return;
+  }
   const int b = (int)(row / a.T), t = (int)(row % a.T);
   const T* src = reinterpret_cast<const T*>(a.dkv) + row * a.ld_dkv;
   T* dst = reinterpret_cast<T*>(a.latent) + ((long long)b * a.maxT + a.first + t) * a.ld;
-  float ss = 0.f;
-  for (int c = lane; c < a.kv_rank; c += 32) { const float f = to_f<T>(src[c]); ss += f * f; }
-  const float inv = 1.f / sqrtf(warp_sum(ss) / a.kv_rank + a.eps);
-  for (int c = lane; c < a.kv_rank; c += 32) dst[c] = from_f<T>(to_f<T>(src[c]) * inv * a.dkv_norm[c]);
-  const int half = a.rot_dims / 2, hd = a.dim + a.rot_dim;
-  const float pos = (float)(a.first + t);
+  if (a.kv_rank % V == 0) warp_norm<T, V>(src, a.dkv_norm, dst, a.lp, a.kv_rank, a.eps, lane);
+  else warp_norm<T, 1>(src, a.dkv_norm, dst, a.lp, a.kv_rank, a.eps, lane);
+  const int half = a.rot_dims / 2;
   src += a.kv_rank;
   dst += a.lp;
-  T* q = reinterpret_cast<T*>(a.q) + row * (long long)a.heads * hd + a.dim;
   for (int i = lane; i < half; i += 32) {
-    const float f = (float)pow(a.rot_base, -2.0 * i / a.rot_dims);
-    float sn, cs;
-    sincosf(pos * f, &sn, &cs);
-    const float u = to_f<T>(src[i]), v = to_f<T>(src[i + half]);
-    dst[i] = from_f<T>(u * cs - v * sn);
-    dst[i + half] = from_f<T>(v * cs + u * sn);
-    for (int h = 0; h < a.heads; h++) {
-      T* qh = q + (long long)h * hd;
-      const float qu = to_f<T>(qh[i]), qv = to_f<T>(qh[i + half]);
-      qh[i] = from_f<T>(qu * cs - qv * sn);
-      qh[i + half] = from_f<T>(qv * cs + qu * sn);
-    }
+    float u, v;
+    rotate(to_f<T>(src[i]), to_f<T>(src[i + half]), (float)(a.first + t), a.freq[i], u, v);
+    dst[i] = from_f<T>(u);
+    dst[i + half] = from_f<T>(v);
   }
   for (int i = a.rot_dims + lane; i < a.rot_dim; i += 32) dst[i] = src[i];
+}
+
+// q in place, for prompts: a thread rotates one pair of every head of its row.
+template <typename T>
+__global__ void __launch_bounds__(256) k_rotate_q(const LatentArgs a) {
+  pdl_trigger();
+  pdl_wait();
+  const int half = a.rot_dims / 2, hd = a.dim + a.rot_dim;
+  const long long it = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (it >= (long long)a.B * a.T * half) return;
+  const int i = (int)(it % half);
+  const long long row = it / half;
+  float sn, cs;
+  sincosf((float)(a.first + (int)(row % a.T)) * a.freq[i], &sn, &cs);
+  T* q = reinterpret_cast<T*>(a.q) + row * (long long)a.heads * hd + a.dim;
+#pragma unroll 4
+  for (int h = 0; h < a.heads; h++, q += hd) {
+    const float u = to_f<T>(q[i]), v = to_f<T>(q[i + half]);
+    q[i] = from_f<T>(u * cs - v * sn);
+    q[i + half] = from_f<T>(v * cs + u * sn);
+  }
 }
 
 // ---- a prompt: expanded keys and values -----------------------------------------------------------------------------
@@ -128,26 +177,206 @@ __global__ void __launch_bounds__(128) k_latent_attn_simt(const LatentArgs a, in
 }
 
 // ---- a few tokens: attention in the latent space ----------------------------------------------------------------------
-// qabs[row][head] = [W_uk^T q (kv_rank), zeros up to lp, rotated q (rot_dim), zeros up to ld]
+// qabs[row][head] = [W_uk^T q (kv_rank), zeros up to lp, rotated q (rot_dim), zeros up to ld].  A thread owns one 16-byte
+// group of latent channels and one slice of the head's channels.
 template <typename T>
-__global__ void __launch_bounds__(256) k_absorb_q(const LatentArgs a) {
+__global__ void __launch_bounds__(1024) k_absorb_q(const LatentArgs a) {
   pdl_trigger();
-  extern __shared__ float qs[];
-  const int h = blockIdx.y, hd = a.dim + a.rot_dim;
-  const long long row = blockIdx.z;
+  pdl_wait();
+  constexpr int V = VecN<T>::n;
+  extern __shared__ float sm[];
+  const int h = blockIdx.x, hd = a.dim + a.rot_dim, tid = threadIdx.x;
+  const long long row = blockIdx.y;
+  float* qs = sm;                     // [hd]
+  float* part = sm + hd;              // [slices][lp]
   const T* q = reinterpret_cast<const T*>(a.q) + (row * a.heads + h) * hd;
-  for (int i = threadIdx.x; i < hd; i += 256) qs[i] = to_f<T>(q[i]);
+  for (int i = tid; i < hd; i += 1024) qs[i] = to_f<T>(q[i]);
   __syncthreads();
-  const int c = blockIdx.x * 256 + threadIdx.x;
-  if (c >= a.ld) return;
-  float acc = 0.f;
-  if (c < a.kv_rank) {
-    const T* w = reinterpret_cast<const T*>(a.w_kv) + (long long)h * a.dim * a.lp + c;
-    for (int d = 0; d < a.dim; d++) acc = fmaf(qs[d], to_f<T>(w[(long long)d * a.lp]), acc);
-  } else if (c >= a.lp && c < a.lp + a.rot_dim) {
-    acc = qs[a.dim + c - a.lp];
+  const int groups = a.lp / V, slices = 1024 / groups, per = (a.dim + slices - 1) / slices;
+  const int gr = tid % groups, sl = tid / groups;
+  if (sl < slices) {
+    float acc[V] = {};
+    const int d1 = min(a.dim, (sl + 1) * per);
+    const T* w = reinterpret_cast<const T*>(a.w_kv) + (long long)h * a.dim * a.lp + gr * V;
+#pragma unroll 8
+    for (int d = sl * per; d < d1; d++) {
+      float f[V];
+      load_vec<T, V>(w + (long long)d * a.lp, f);
+#pragma unroll
+      for (int e = 0; e < V; e++) acc[e] = fmaf(qs[d], f[e], acc[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < V; e++) part[sl * a.lp + gr * V + e] = acc[e];
   }
-  a.qabs[(row * a.heads + h) * a.ld + c] = acc;
+  __syncthreads();
+  float* dst = a.qabs + (row * a.heads + h) * a.ld;
+  const int half = a.rot_dims / 2;
+  for (int c = tid; c < a.ld; c += 1024) {
+    float x = 0.f;
+    if (c < a.lp) {
+      for (int k = 0; k < slices; k++) x += part[k * a.lp + c];
+    } else if (c < a.lp + a.rot_dim) {
+      const int i = c - a.lp;
+      const float* qr = qs + a.dim;
+      x = qr[i];
+      if (i < a.rot_dims) {
+        float u, v;
+        const int k = i < half ? i : i - half;
+        rotate(qr[k], qr[k + half], (float)(a.first + (int)(row % a.T)), a.freq[k], u, v);
+        x = round_to<T>(i < half ? u : v);
+      }
+    }
+    dst[c] = x;
+  }
+}
+
+// The tensor-core form for bf16 caches.  grid (heads / 16, splits, rows): 16 heads are the rows of one mma tile; the cached
+// rows arrive in tiles of `KT` through two shared-memory buffers (16-byte units of row r permuted by r & 7) and serve as
+// keys (read as they lie) and as values (read transposed).  Queries and softmax weights are sums of two bf16 numbers, so
+// scores and weights keep fp32 accuracy.
+__device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)) : "memory");
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)) : "memory");
+}
+__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ int swz(int row, int col, int width) { return row * width + ((((col >> 3) ^ (row & 7)) << 3) | (col & 7)); }
+
+template <int NP>      // pairs of 8-channel tiles of the result per warp: lp <= 128 NP
+__global__ void __launch_bounds__(256) k_latent_decode_mma(const LatentArgs a, int splits, int tiles_per, int KT, int width) {
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ __align__(16) uint8_t raw[];
+  bf16* rows = reinterpret_cast<bf16*>(raw);            // 2 x [KT][width]
+  bf16* qh = rows + 2 * KT * width;                     // [16][width] high, low
+  bf16* ph = qh + 2 * 16 * width;                       // [16][64] high, low
+  float* ss = reinterpret_cast<float*>(ph + 2 * 16 * 64);   // [16][KT + 4]
+  float* sal = ss + 16 * (KT + 4);                      // [16] rescale factor of this tile
+  float* sml = sal + 16;                                // [16][2] running max and sum
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c2 = 2 * (lane & 3);
+  const int h0 = blockIdx.x * 16, sp = blockIdx.y;
+  const long long row = blockIdx.z;
+  const int b = (int)(row / a.T), n = a.first + (int)(row % a.T) + 1;      // keys this query sees
+  const int ntiles = (n + KT - 1) / KT, tb = sp * tiles_per, te = min(ntiles, tb + tiles_per);
+  const bf16* lat = reinterpret_cast<const bf16*>(a.latent) + (long long)b * a.maxT * a.ld;
+  const int units = a.ld / 8;
+  auto load = [&](int tile) {
+    bf16* dst = rows + (tile & 1) * KT * width;
+    for (int i = tid; i < KT * units; i += 256) {
+      const int r = i / units, c = i % units * 8, key = tile * KT + r;
+      const uint32_t to = smem_addr(dst + swz(r, c, width));
+      if (key < n) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(to), "l"(lat + (long long)key * a.ld + c) : "memory");
+      else *reinterpret_cast<uint4*>(dst + swz(r, c, width)) = make_uint4(0, 0, 0, 0);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (tb < te) load(tb);
+  // queries, and zeros in the columns that pad a row to whole groups of 64
+  for (int i = tid; i < 16 * width / 2; i += 256) {
+    const int r = i / (width / 2), c = i % (width / 2) * 2;
+    float x = 0.f, y = 0.f;
+    if (h0 + r < a.heads && c < a.ld) {
+      const float2 f = *reinterpret_cast<const float2*>(a.qabs + (row * a.heads + h0 + r) * a.ld + c);
+      x = f.x; y = f.y;
+    }
+    const __nv_bfloat162 hi = __floats2bfloat162_rn(x, y);
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(x - __bfloat162float(hi.x), y - __bfloat162float(hi.y));
+    const int o = swz(r, c, width);
+    *reinterpret_cast<__nv_bfloat162*>(qh + o) = hi;
+    *reinterpret_cast<__nv_bfloat162*>(qh + 16 * width + o) = lo;
+  }
+  const int pad = width - a.ld;
+  if (pad)
+    for (int i = tid; i < 2 * KT * pad / 8; i += 256) {
+      const int r = i / (pad / 8), c = a.ld + i % (pad / 8) * 8;
+      *reinterpret_cast<uint4*>(rows + (r / KT) * KT * width + swz(r % KT, c, width)) = make_uint4(0, 0, 0, 0);
+    }
+  if (KT < 64)
+    for (int i = tid; i < 2 * 16 * 64 / 8; i += 256) *reinterpret_cast<uint4*>(ph + i * 8) = make_uint4(0, 0, 0, 0);
+  if (tid < 16) { sml[2 * tid] = -INFINITY; sml[2 * tid + 1] = 0.f; }
+  float o[NP][2][4] = {};
+  for (int tile = tb; tile < te; tile++) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                   // the tile is complete, the other buffer free
+    if (tile + 1 < te) load(tile + 1);
+    const bf16* kt = rows + (tile & 1) * KT * width;
+    if (warp * 8 < KT) {               // scores of eight keys
+      float s[2][4] = {};
+#pragma unroll 2
+      for (int k = 0; k < width; k += 32) {
+        uint32_t kb[4];
+        ldsm4(kb, kt + swz(8 * warp + (lane & 7), k + 8 * (lane >> 3), width));
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+          uint32_t ah[4], al[4];
+          const int at = swz(lane & 15, k + 16 * i + 8 * (lane >> 4), width);
+          ldsm4(ah, qh + at); ldsm4(al, qh + 16 * width + at);
+          mma16816(s[0], ah, kb[2 * i], kb[2 * i + 1]);
+          mma16816(s[1], al, kb[2 * i], kb[2 * i + 1]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const int key = 8 * warp + c2 + (e & 1);
+        ss[(g + 8 * (e >> 1)) * (KT + 4) + key] = tile * KT + key < n ? (s[0][e] + s[1][e]) * a.scale : -INFINITY;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 2; i++) {      // softmax of two heads per warp
+      const int r = 2 * warp + i;
+      const float x0 = lane < KT ? ss[r * (KT + 4) + lane] : -INFINITY, x1 = lane + 32 < KT ? ss[r * (KT + 4) + lane + 32] : -INFINITY;
+      const float m = sml[2 * r], mn = fmaxf(m, warp_max(fmaxf(x0, x1)));      // finite: the first key of a tile is always seen
+      const float p0 = __expf(x0 - mn), p1 = __expf(x1 - mn), f = __expf(m - mn);
+      const float l = warp_sum(p0 + p1);
+      const bf16 h0b = __float2bfloat16_rn(p0), h1b = __float2bfloat16_rn(p1);
+      const int o0 = swz(r, lane, 64), o1 = swz(r, lane + 32, 64);
+      ph[o0] = h0b; ph[16 * 64 + o0] = __float2bfloat16_rn(p0 - __bfloat162float(h0b));
+      if (KT > 32) { ph[o1] = h1b; ph[16 * 64 + o1] = __float2bfloat16_rn(p1 - __bfloat162float(h1b)); }
+      __syncwarp();
+      if (lane == 0) { sal[r] = f; sml[2 * r] = mn; sml[2 * r + 1] = sml[2 * r + 1] * f + l; }
+    }
+    __syncthreads();
+    const float f0 = sal[g], f1 = sal[g + 8];
+#pragma unroll
+    for (int j = 0; j < NP; j++)
+#pragma unroll
+      for (int i = 0; i < 2; i++) { o[j][i][0] *= f0; o[j][i][1] *= f0; o[j][i][2] *= f1; o[j][i][3] *= f1; }
+    for (int k = 0; k < KT; k += 16) {
+      uint32_t ah[4], al[4];
+      const int at = swz(lane & 15, k + 8 * (lane >> 4), 64);
+      ldsm4(ah, ph + at); ldsm4(al, ph + 16 * 64 + at);
+#pragma unroll
+      for (int j = 0; j < NP; j++) {
+        const int c = (j * 8 + warp) * 16;
+        if (c >= a.lp) continue;
+        uint32_t vb[4];
+        ldsm4t(vb, kt + swz(k + (lane & 15), c + 8 * (lane >> 4), width));
+#pragma unroll
+        for (int i = 0; i < 2; i++) { mma16816(o[j][i], ah, vb[2 * i], vb[2 * i + 1]); mma16816(o[j][i], al, vb[2 * i], vb[2 * i + 1]); }
+      }
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int e = 0; e < 2; e++) {
+    const int h = h0 + g + 8 * e;
+    if (h >= a.heads) continue;
+    float* dst = a.part + ((row * a.heads + h) * splits + sp) * (a.lp + 2);
+    if (warp == 0 && (lane & 3) == 0) { dst[0] = sml[2 * (g + 8 * e)]; dst[1] = sml[2 * (g + 8 * e) + 1]; }
+#pragma unroll
+    for (int j = 0; j < NP; j++)
+#pragma unroll
+      for (int i = 0; i < 2; i++) {
+        const int c = (j * 8 + warp) * 16 + 8 * i + c2;
+        if (c < a.lp) *reinterpret_cast<float2*>(dst + 2 + c) = make_float2(o[j][i][2 * e], o[j][i][2 * e + 1]);
+      }
+  }
 }
 
 // grid (heads / 8, splits, rows): a block takes one contiguous range of the cached rows, staged 32 at a time in shared
@@ -156,6 +385,7 @@ constexpr int LP_MAX = 32;   // kv_rank <= 1024
 template <typename T, int PER>
 __global__ void __launch_bounds__(256) k_latent_decode(const LatentArgs a, int splits) {
   pdl_trigger();
+  pdl_wait();
   extern __shared__ float sm[];
   const int P = a.ld + 1;
   float* rows = sm;               // [32][P]
@@ -203,39 +433,57 @@ __global__ void __launch_bounds__(256) k_latent_decode(const LatentArgs a, int s
   for (int i = 0; i < PER; i++) if (i * 32 + lane < a.lp) dst[2 + i * 32 + lane] = o[i];
 }
 
-// grid (heads, rows): combine the splits in order, then W_uv and the head's gate.
+// grid (vdim / 32, heads, rows): combine the splits in order, then 32 rows of W_uv and the head's gate.
 template <typename T>
-__global__ void __launch_bounds__(256) k_latent_decode_out(const LatentArgs a, int splits) {
+__global__ void __launch_bounds__(1024) k_latent_decode_out(const LatentArgs a, int splits) {
   pdl_trigger();
-  extern __shared__ float oc[];   // [lp]
-  const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const long long row = blockIdx.y;
-  const float* p = a.part + (row * a.heads + h) * (long long)splits * (a.lp + 2);
-  float M = -INFINITY, L = 0.f;
-  for (int s = 0; s < splits; s++) M = fmaxf(M, p[(long long)s * (a.lp + 2)]);
-  for (int s = 0; s < splits; s++) {
-    const float ms = p[(long long)s * (a.lp + 2)];
-    if (ms != -INFINITY) L += p[(long long)s * (a.lp + 2) + 1] * expf(ms - M);
-  }
-  const float inv = 1.f / L;
-  for (int c = threadIdx.x; c < a.lp; c += 256) {
-    float acc = 0.f;
-    for (int s = 0; s < splits; s++) {
-      const float ms = p[(long long)s * (a.lp + 2)];
-      if (ms != -INFINITY) acc += p[(long long)s * (a.lp + 2) + 2 + c] * expf(ms - M);
+  pdl_wait();
+  constexpr int V = VecN<T>::n;
+  extern __shared__ float sm[];
+  float* oc = sm;                 // [lp], then [halves][lp] partial sums
+  float* ws = oc + 2 * a.lp;      // [splits]
+  __shared__ float total;
+  const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
+  const long long row = blockIdx.z;
+  const int ldp = a.lp + 2;
+  const float* p = a.part + (row * a.heads + h) * (long long)splits * ldp;
+  if (warp == 0) {
+    float M = -INFINITY, L = 0.f;
+    for (int s = lane; s < splits; s += 32) M = fmaxf(M, p[(long long)s * ldp]);
+    M = warp_max(M);
+    for (int s = lane; s < splits; s += 32) {
+      const float ms = p[(long long)s * ldp], w = ms == -INFINITY ? 0.f : expf(ms - M);
+      ws[s] = w;
+      L += w * p[(long long)s * ldp + 1];
     }
-    oc[c] = acc * inv;
+    L = warp_sum(L);
+    if (lane == 0) total = L;
   }
   __syncthreads();
-  const float g = to_f<T>(reinterpret_cast<const T*>(a.gate)[row * a.ld_gate + h]);
-  const float f = 1.f / (1.f + expf(-g));
-  const T* w = reinterpret_cast<const T*>(a.w_kv) + (long long)(a.heads * a.dim + h * a.vdim) * a.lp;
-  for (int e = warp; e < a.vdim; e += 8) {
+  const int per = (splits + 1) / 2;
+  for (int i = tid; i < 2 * a.lp; i += 1024) {
+    const int c = i % a.lp, half = i / a.lp, s1 = min(splits, (half + 1) * per);
     float acc = 0.f;
-    for (int c = lane; c < a.kv_rank; c += 32) acc = fmaf(to_f<T>(w[(long long)e * a.lp + c]), oc[c], acc);
-    acc = warp_sum(acc);
-    if (lane == 0) reinterpret_cast<T*>(a.o)[row * (long long)a.heads * a.vdim + (long long)h * a.vdim + e] = from_f<T>(acc * f);
+#pragma unroll 8
+    for (int s = half * per; s < s1; s++) acc = fmaf(ws[s], ws[s] == 0.f ? 0.f : p[(long long)s * ldp + 2 + c], acc);
+    oc[i] = acc;
   }
+  __syncthreads();
+  const int e = blockIdx.x * 32 + warp;
+  if (e >= a.vdim) return;
+  const float g = to_f<T>(reinterpret_cast<const T*>(a.gate)[row * a.ld_gate + h]);
+  const float f = 1.f / (total * (1.f + expf(-g)));
+  const T* w = reinterpret_cast<const T*>(a.w_kv) + ((long long)a.heads * a.dim + (long long)h * a.vdim + e) * a.lp;
+  float acc = 0.f;
+#pragma unroll 2
+  for (int c = lane * V; c < a.lp; c += 32 * V) {
+    float x[V];
+    load_vec<T, V>(w + c, x);
+#pragma unroll
+    for (int k = 0; k < V; k++) acc = fmaf(x[k], oc[c + k] + oc[a.lp + c + k], acc);
+  }
+  acc = warp_sum(acc);
+  if (lane == 0) reinterpret_cast<T*>(a.o)[row * (long long)a.heads * a.vdim + (long long)h * a.vdim + e] = from_f<T>(acc * f);
 }
 
 // Opt-in to more than 48 KB of dynamic shared memory, once per kernel and device.
@@ -247,44 +495,80 @@ template <typename K> int allow_smem(K kernel, size_t bytes) {
 
 }  // namespace
 
-template <typename T> int latent_prep(const LatentArgs& a, cudaStream_t s) {
-  k_latent_prep<T><<<cdiv((long long)a.B * a.T, 8), 256, 0, s>>>(a);
+template <typename T> int latent_norms(const LatentArgs& a, cudaStream_t s) {
+  CUDA_TRY(launch_dependent(k_latent_norms<T>, cdiv(2LL * a.B * a.T, 8), 256, 0, s, a));
   KERNEL_CHECK();
   return 0;
 }
-template int latent_prep<float>(const LatentArgs&, cudaStream_t);
-template int latent_prep<bf16>(const LatentArgs&, cudaStream_t);
+template int latent_norms<float>(const LatentArgs&, cudaStream_t);
+template int latent_norms<bf16>(const LatentArgs&, cudaStream_t);
 
-template <typename T> int latent_attention(const LatentArgs& a, cudaStream_t s) {
+// A few new tokens per column: queries into the latent space, attention over the cached rows, back out.
+template <typename T> static int latent_decode(const LatentArgs& a, cudaStream_t s) {
+  constexpr int V = VecN<T>::n;
   const int N = a.first + a.T, rows = a.B * a.T;
-  if (a.vdim > 256 || a.dim + a.rot_dim > 512 || a.lp > 32 * LP_MAX)
-    return femto_fail(FEMTO_ERR_UNSUPPORTED, "latent attention: dim %d + %d, vdim %d, rank %d", a.dim, a.rot_dim, a.vdim, a.kv_rank);
-  if (a.T <= LATENT_FEW) {
-    k_absorb_q<T><<<dim3(cdiv(a.ld, 256), a.heads, rows), 256, (a.dim + a.rot_dim) * 4, s>>>(a);
-    KERNEL_CHECK();
+  const size_t absorb = 4 * (size_t)(a.dim + a.rot_dim + 1024 / (a.lp / V) * a.lp);
+  FEMTO_TRY(allow_smem(k_absorb_q<T>, absorb));
+  CUDA_TRY(launch_dependent(k_absorb_q<T>, dim3(a.heads, rows), 1024, absorb, s, a));
+  KERNEL_CHECK();
+  int splits = 0;
+  const auto fits = [&](int n) { return (size_t)rows * a.heads * n * (a.lp + 2) <= a.part_floats; };
+  bool done = false;
+  if constexpr (sizeof(T) == 2) {
+    const int width = round_up(a.ld, 64), blocks = cdiv(a.heads, 16) * rows;
+    auto bytes = [&](int kt) { return (size_t)2 * kt * width * 2 + 2 * 16 * width * 2 + 2 * 16 * 64 * 2 + 4 * (16 * (kt + 4) + 48); };
+    const int KT = bytes(64) <= 227 * 1024 ? 64 : 32;
+    if (bytes(KT) <= 227 * 1024) {
+      const int tiles = cdiv(N, KT);
+      // as many splits as fill the device once, each of at least two tiles
+      int per = std::max(std::min(2, tiles), cdiv(tiles, std::max(1, device_sm_count() / blocks)));
+      while (!fits(cdiv(tiles, per))) per++;
+      splits = cdiv(tiles, per);
+#define LAUNCH(NP) do { FEMTO_TRY(allow_smem(k_latent_decode_mma<NP>, bytes(KT))); \
+      CUDA_TRY(launch_dependent(k_latent_decode_mma<NP>, dim3(cdiv(a.heads, 16), splits, rows), 256, bytes(KT), s, a, splits, per, KT, width)); } while (0)
+      if (a.lp <= 128) LAUNCH(1);
+      else if (a.lp <= 256) LAUNCH(2);
+      else if (a.lp <= 512) LAUNCH(4);
+      else LAUNCH(8);
+#undef LAUNCH
+      done = true;
+    }
+  }
+  if (!done) {
     const int blocks = cdiv(a.heads, 8) * rows;
-    int splits = std::max(1, std::min({LATENT_MAX_SPLITS, cdiv(N, 64), cdiv(2 * device_sm_count(), blocks)}));
-    while (splits > 1 && (size_t)rows * a.heads * splits * (a.lp + 2) > a.part_floats) splits--;
+    splits = std::max(1, std::min({LATENT_MAX_SPLITS, cdiv(N, 64), cdiv(2 * device_sm_count(), blocks)}));
+    while (splits > 1 && !fits(splits)) splits--;
     const size_t smem = 4 * (size_t)(32 * (a.ld + 1) + 8 * a.ld);
     const int per = cdiv(a.lp, 32);
     const dim3 grid(cdiv(a.heads, 8), splits, rows);
-#define LAUNCH(PER) do { FEMTO_TRY(allow_smem(k_latent_decode<T, PER>, smem)); k_latent_decode<T, PER><<<grid, 256, smem, s>>>(a, splits); } while (0)
+#define LAUNCH(PER) do { FEMTO_TRY(allow_smem(k_latent_decode<T, PER>, smem)); CUDA_TRY(launch_dependent(k_latent_decode<T, PER>, grid, 256, smem, s, a, splits)); } while (0)
     if (per <= 4) LAUNCH(4);
     else if (per <= 8) LAUNCH(8);
     else if (per <= 16) LAUNCH(16);
     else LAUNCH(32);
 #undef LAUNCH
+  }
+  KERNEL_CHECK();
+  CUDA_TRY(launch_dependent(k_latent_decode_out<T>, dim3(cdiv(a.vdim, 32), a.heads, rows), 1024, 4 * (size_t)(2 * a.lp + splits), s, a, splits));
+  KERNEL_CHECK();
+  return 0;
+}
+
+template <typename T> int latent_attention(const LatentArgs& a, cudaStream_t s) {
+  const int N = a.first + a.T, rows = a.B * a.T;
+  if (a.vdim > 256 || a.dim + a.rot_dim > 512 || a.lp > 32 * LP_MAX)
+    return femto_fail(FEMTO_ERR_UNSUPPORTED, "latent attention: dim %d + %d, vdim %d, rank %d", a.dim, a.rot_dim, a.vdim, a.kv_rank);
+  if (a.T <= LATENT_FEW) return latent_decode<T>(a, s);
+  if (a.rot_dims > 0) {
+    CUDA_TRY(launch_dependent(k_rotate_q<T>, cdiv((long long)rows * (a.rot_dims / 2), 256), 256, 0, s, a));
     KERNEL_CHECK();
-    k_latent_decode_out<T><<<dim3(a.heads, rows), 256, a.lp * 4, s>>>(a, splits);
-    KERNEL_CHECK();
-    return 0;
   }
   // keys and values of all N tokens of every column: [N][lp] x [heads (dim + vdim)][lp]^T
   const int wide = a.heads * (a.dim + a.vdim);
   GemmArgs g;
   g.ws = a.d->gemm_ws; g.ws_bytes = a.d->gemm_ws_bytes; g.status = a.d->status;
   g.A = a.latent; g.lda = a.ld; g.strideA = (long long)a.maxT * a.ld; g.B = a.w_kv; g.ldb = a.lp; g.strideB = 0;
-  g.C = a.kv; g.ldc = wide; g.strideC = (long long)a.maxT * wide; g.M = N; g.N = wide; g.K = a.lp; g.epi = EPI_STORE;
+  g.C = a.kv; g.ldc = wide; g.strideC = (long long)a.maxT * wide; g.M = N; g.N = wide; g.K = a.lp; g.epi = EPI_STORE; g.any_size = true;
   for (int b = 0; b < a.B; b++) {
     FEMTO_TRY(gemm<T>(g, s));
     g.A = reinterpret_cast<const T*>(g.A) + g.strideA;

@@ -15,6 +15,7 @@ template <int NI> struct Tile { static constexpr int TOK = NI >= 8 ? 8 : 16; }; 
 template <typename T, bool DELTA, int NI>
 __global__ void __launch_bounds__(256) k_recurrence(const RecurrenceArgs a) {
   pdl_trigger();
+  pdl_wait();
   constexpr int DP = 32 * NI, TT = Tile<NI>::TOK;
   __shared__ __align__(16) float sq[TT][DP], sk[TT][DP], sg[DELTA ? TT : 1][DELTA ? DP : 4], sv[TT][32], sb[TT];
   const int h = blockIdx.y, b = blockIdx.z;
@@ -111,6 +112,7 @@ __device__ __forceinline__ float conv_input(const DeltaPrepArgs& a, int b, int t
 template <typename T>
 __global__ void __launch_bounds__(256) k_delta_prep(const DeltaPrepArgs a) {
   pdl_trigger();
+  pdl_wait();
   const int units = 2 * a.kv_heads + 2 * a.heads;
   const long long it = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   if (it >= (long long)a.B * a.T * units) return;
@@ -170,6 +172,7 @@ __global__ void __launch_bounds__(256) k_delta_prep(const DeltaPrepArgs a) {
 template <typename T>
 __global__ void __launch_bounds__(256) k_conv_tail(const DeltaPrepArgs a) {
   pdl_trigger();
+  pdl_wait();
   const int G = a.kv_heads, D = a.dim, channels = 2 * G * D + a.heads * a.vdim, keep = a.taps - 1;
   const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
   if (i >= (long long)a.B * keep * channels) return;
@@ -180,12 +183,152 @@ __global__ void __launch_bounds__(256) k_conv_tail(const DeltaPrepArgs a) {
                                                : reinterpret_cast<const T*>(a.tail_in)[((long long)b * keep + keep + r) * channels + chan];
 }
 
+// ---- one token -----------------------------------------------------------------------------------------------------------
+// The whole mixer between the packed projection and the output projection for one new token: convolutions, unit vectors,
+// both low-rank projections, state update, read-out, norm and gate.  One block per (head, column).
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+
+template <typename T> __device__ __forceinline__ float row_dot(const T* __restrict__ w, const float* x, int n, int lane) {
+  constexpr int V = VecN<T>::n;      // rows are padded to multiples of 8 with zeros
+  float acc = 0.f;
+  for (int c = lane * V; c < n; c += 32 * V) {
+    float f[V];
+    load_vec<T, V>(w + c, f);
+#pragma unroll
+    for (int e = 0; e < V; e++) acc = fmaf(f[e], x[c + e], acc);
+  }
+  return warp_sum(acc);
+}
+
+template <typename T, int NI>
+__global__ void __launch_bounds__(1024) k_delta_decode(const DeltaDecodeArgs a) {
+  pdl_trigger();
+  pdl_wait();
+  constexpr int DP = 32 * NI;
+  const DeltaPrepArgs& p = a.p;
+  extern __shared__ __align__(16) float sm[];
+  float *sq = sm, *sk = sq + DP, *sg = sk + DP, *sv = sg + DP, *so = sv + p.vdim, *sz = so + p.vdim, *sa = sz + p.vdim, *sb = sa + a.ra;
+  __shared__ float red[32], f_q, f_k;
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int H = p.heads, G = p.kv_heads, D = p.dim, E = p.vdim, n = p.taps, keep = n - 1;
+  const int qh = h / (H / G), channels = 2 * G * D + H * E;
+  const T* proj = reinterpret_cast<const T*>(p.proj) + (long long)b * p.ldp;
+  const T* tin = reinterpret_cast<const T*>(p.tail_in) + (long long)b * keep * channels;
+  T* tout = reinterpret_cast<T*>(p.tail_out) + (long long)b * keep * channels;
+  for (int i = tid; i < a.ra; i += 1024) sa[i] = to_f<T>(proj[a.s_a1 + i]);
+  for (int i = tid; i < a.rg; i += 1024) sb[i] = to_f<T>(proj[a.s_g1 + i]);
+  for (int i = tid; i < 2 * DP + E; i += 1024) {
+    const int which = i < DP ? 0 : i < 2 * DP ? 1 : 2, c = which == 2 ? i - 2 * DP : i - which * DP;
+    const int size = which == 2 ? E : D, head = which == 2 ? h : qh;
+    float y = 0.f;
+    if (c < size) {
+      const int at = head * size + c, chan = (which == 0 ? 0 : which == 1 ? G * D : 2 * G * D) + at;
+      const float* taps = (which == 0 ? p.conv_q : which == 1 ? p.conv_k : p.conv_v) + (long long)at * n;
+      const T now = proj[(which == 0 ? p.s_q : which == 1 ? p.s_k : p.s_v) + at];
+      const bool writes = which == 2 || h % (H / G) == 0;      // the heads of a group share q and k
+      float acc = 0.f;
+      for (int j = 0; j < keep; j++) {
+        const T x = tin[(long long)j * channels + chan];
+        acc = fmaf(taps[j], to_f<T>(x), acc);
+        if (writes && j > 0) tout[(long long)(j - 1) * channels + chan] = x;
+      }
+      if (writes && keep > 0) tout[(long long)(keep - 1) * channels + chan] = now;
+      y = silu_f(fmaf(taps[keep], to_f<T>(now), acc));
+      if (which == 2) y = round_to<T>(y);
+    }
+    (which == 0 ? sq : which == 1 ? sk : sv)[c] = y;
+  }
+  __syncthreads();
+  if (warp < 2) {
+    const float* x = warp ? sk : sq;
+    float ss = 0.f;
+    for (int c = lane; c < D; c += 32) ss += x[c] * x[c];
+    ss = 1.f / sqrtf(warp_sum(ss) + 1e-6f);
+    if (lane == 0) { if (warp) f_k = ss; else f_q = ss * (1.f / sqrtf((float)D)); }
+  }
+  const float rate = expf(p.a_log[h]);
+#pragma unroll 4
+  for (int i = warp; i < D + E; i += 32) {
+    const bool decay = i < D;
+    const int c = decay ? i : i - D, r = decay ? a.ra : a.rg;
+    const T* w = reinterpret_cast<const T*>(decay ? a.w_a2 : a.w_g2) + (long long)(h * (decay ? D : E) + c) * r;
+    const float z = row_dot<T>(w, decay ? sa : sb, r, lane);
+    if (lane == 0) {
+      if (decay) sg[c] = expf(-rate * softplus_f(z + p.dt_bias[h * D + c]));
+      else sz[c] = sigmoid_f(round_to<T>(z));
+    }
+  }
+  for (int c = D + tid; c < DP; c += 1024) sg[c] = 0.f;
+  __syncthreads();
+  const float beta = sigmoid_f(to_f<T>(proj[p.s_b + h])), fk = f_k, fq = f_q;
+  const int sub = tid & 7;
+  const bool vec = (D & 3) == 0;
+  for (int e = tid >> 3; e < (E + 127) / 128 * 128; e += 128) {
+    float* Sp = a.S + (((long long)b * H + h) * E + min(e, E - 1)) * D;
+    float s[NI][4], dot = 0.f;
+#pragma unroll
+    for (int i = 0; i < NI; i++) {
+      const int d = 4 * (sub + 8 * i);
+      if (vec) {
+        const float4 v = d < D && e < E ? *reinterpret_cast<const float4*>(Sp + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+        s[i][0] = v.x; s[i][1] = v.y; s[i][2] = v.z; s[i][3] = v.w;
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; j++) s[i][j] = d + j < D && e < E ? Sp[d + j] : 0.f;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NI; i++)
+#pragma unroll
+      for (int j = 0; j < 4; j++) {
+        const int d = 4 * (sub + 8 * i) + j;
+        s[i][j] *= sg[d];
+        dot = fmaf(s[i][j], sk[d] * fk, dot);
+      }
+    dot += __shfl_xor_sync(0xffffffffu, dot, 1); dot += __shfl_xor_sync(0xffffffffu, dot, 2); dot += __shfl_xor_sync(0xffffffffu, dot, 4);
+    const float u = beta * ((e < E ? sv[e] : 0.f) - dot);
+    float o = 0.f;
+#pragma unroll
+    for (int i = 0; i < NI; i++)
+#pragma unroll
+      for (int j = 0; j < 4; j++) {
+        const int d = 4 * (sub + 8 * i) + j;
+        s[i][j] = fmaf(sk[d] * fk, u, s[i][j]);
+        o = fmaf(s[i][j], sq[d] * fq, o);
+      }
+    o += __shfl_xor_sync(0xffffffffu, o, 1); o += __shfl_xor_sync(0xffffffffu, o, 2); o += __shfl_xor_sync(0xffffffffu, o, 4);
+    if (e < E) {
+#pragma unroll
+      for (int i = 0; i < NI; i++) {
+        const int d = 4 * (sub + 8 * i);
+        if (vec) {
+          if (d < D) *reinterpret_cast<float4*>(Sp + d) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; j++) if (d + j < D) Sp[d + j] = s[i][j];
+        }
+      }
+      if (sub == 0) so[e] = round_to<T>(o);
+    }
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < E; c += 1024) ss += so[c] * so[c];
+  ss = warp_sum(ss);
+  if (lane == 0) red[warp] = ss;
+  __syncthreads();
+  ss = warp_sum(red[lane]);
+  const float inv = 1.f / sqrtf(ss / E + a.eps);
+  T* out = reinterpret_cast<T*>(a.out) + ((long long)b * H + h) * E;
+  for (int c = tid; c < E; c += 1024) out[c] = from_f<T>(so[c] * inv * a.norm[c] * sz[c]);
+}
+
 }  // namespace
 
 template <typename T> int recurrence(const RecurrenceArgs& a, cudaStream_t s) {
   const dim3 grid(cdiv(a.vdim, 32), a.heads, a.B);
   const bool delta = a.beta != nullptr;
-#define LAUNCH(NI) if (delta) k_recurrence<T, true, NI><<<grid, 256, 0, s>>>(a); else k_recurrence<T, false, NI><<<grid, 256, 0, s>>>(a)
+#define LAUNCH(NI) if (delta) CUDA_TRY(launch_dependent(k_recurrence<T, true, NI>, grid, 256, 0, s, a)); else CUDA_TRY(launch_dependent(k_recurrence<T, false, NI>, grid, 256, 0, s, a))
   if (a.dim <= 32) { LAUNCH(1); }
   else if (a.dim <= 64) { LAUNCH(2); }
   else if (a.dim <= 128) { LAUNCH(4); }
@@ -201,7 +344,7 @@ template int recurrence<bf16>(const RecurrenceArgs&, cudaStream_t);
 template <typename T> int conv_tail(const DeltaPrepArgs& a, cudaStream_t s) {
   if (a.taps <= 1) return 0;
   const long long m = (long long)a.B * (a.taps - 1) * (2 * a.kv_heads * a.dim + a.heads * a.vdim);
-  k_conv_tail<T><<<cdiv(m, 256), 256, 0, s>>>(a);
+  CUDA_TRY(launch_dependent(k_conv_tail<T>, cdiv(m, 256), 256, 0, s, a));
   KERNEL_CHECK();
   return 0;
 }
@@ -211,9 +354,27 @@ template int conv_tail<bf16>(const DeltaPrepArgs&, cudaStream_t);
 template <typename T> int delta_prep(const DeltaPrepArgs& a, cudaStream_t s) {
   if (a.dim > 256 || a.vdim > 256) return femto_fail(FEMTO_ERR_UNSUPPORTED, "delta rule: dim %d / vdim %d > 256", a.dim, a.vdim);
   const long long n = (long long)a.B * a.T * (2 * a.kv_heads + 2 * a.heads);
-  k_delta_prep<T><<<cdiv(n, 8), 256, 0, s>>>(a);
+  CUDA_TRY(launch_dependent(k_delta_prep<T>, cdiv(n, 8), 256, 0, s, a));
   KERNEL_CHECK();
   return conv_tail<T>(a, s);
 }
 template int delta_prep<float>(const DeltaPrepArgs&, cudaStream_t);
 template int delta_prep<bf16>(const DeltaPrepArgs&, cudaStream_t);
+
+template <typename T> int delta_decode(const DeltaDecodeArgs& a, cudaStream_t s) {
+  const dim3 grid(a.p.heads, a.p.B);
+  const int ni = a.p.dim <= 32 ? 1 : a.p.dim <= 64 ? 2 : a.p.dim <= 128 ? 4 : 8;
+  if (a.p.dim > 256 || a.p.vdim > 256) return femto_fail(FEMTO_ERR_UNSUPPORTED, "delta rule: dim %d / vdim %d > 256", a.p.dim, a.p.vdim);
+  const size_t smem = 4 * (size_t)(3 * 32 * ni + 3 * a.p.vdim + a.ra + a.rg);
+  if (smem > 48 * 1024) return femto_fail(FEMTO_ERR_UNSUPPORTED, "delta rule: ranks %d and %d are too large", a.ra, a.rg);
+#define LAUNCH(NI) CUDA_TRY(launch_dependent(k_delta_decode<T, NI>, grid, 1024, smem, s, a))
+  if (ni == 1) LAUNCH(1);
+  else if (ni == 2) LAUNCH(2);
+  else if (ni == 4) LAUNCH(4);
+  else LAUNCH(8);
+#undef LAUNCH
+  KERNEL_CHECK();
+  return 0;
+}
+template int delta_decode<float>(const DeltaDecodeArgs&, cudaStream_t);
+template int delta_decode<bf16>(const DeltaDecodeArgs&, cudaStream_t);
