@@ -389,6 +389,20 @@ def run_ours(args):
         dist.destroy_process_group()
 
 
+def run_serve(args):
+    """`--serve`: one JSON line with prefill and decode tokens/s of both model families at each size."""
+    from femtochat_b200 import serve_bench
+    clocks = ClockSampler(0)
+    clocks.start()
+    sizes = [serve_bench.run(s) for s in args.serve_sizes.split(",")]
+    first = sizes[0]["Virolorn"][0]
+    print(json.dumps(dict(metric="prefill tokens/sec", value=first["prefill_tokens_per_s"], unit="tokens/s", n_gpus=1,
+                          higher_is_better=True, dtype="bf16", data="synthetic", vs_baseline=None,
+                          config=dict(workload="prefill of a prompt and decode steps after it, random weights, whole calls timed with CUDA events",
+                                      l2="weights, caches and activations of a call exceed L2"),
+                          sizes=sizes, clocks=clocks.stop())), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -414,7 +428,14 @@ def main():
     ap.add_argument("--phases", action="store_true",
                     help="N > 1: after the bench line, time reverse pass / gradient sum / update separately for the "
                          "owner-sharded and the replicated update (stderr)")
+    ap.add_argument("--serve", action="store_true",
+                    help="instead of the training step: prefill and decode throughput of a Virolorn model (layers listed one by "
+                         "one) beside the GPT at equal size, random weights, one GPU")
+    ap.add_argument("--serve-sizes", default="d20,w2560", help="with --serve: sizes of femtochat_b200/serve_bench.py")
     args = ap.parse_args()
+    if args.serve:
+        run_serve(args)
+        return
     if args.warmup < 3 and args.impl == "ours":
         args.warmup = 3
     if args.impl == "reference":

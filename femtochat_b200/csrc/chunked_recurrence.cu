@@ -46,7 +46,15 @@ template <int DP> struct Item {
 
 // (an activation: bf16 numbers go in, so the special-function unit's 2^-21 is plenty)
 __device__ __forceinline__ float silu_f(float z) { return z * __fdividef(1.f, 1.f + __expf(-z)); }
-__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// log(1 + e^z) = max(z, 0) + log(1 + x), x = e^-|z| in (0, 1], with log(1 + x) = 2 artanh(s), s = x / (2 + x) <= 1/3: eight terms
+// of the artanh series leave a relative error of 3e-9
+__device__ __forceinline__ float softplus_f(float z) {
+  const float x = expf(-fabsf(z)), s = __fdividef(x, 2.f + x), t = s * s;
+  float p = 1.f / 15.f;
+  p = fmaf(p, t, 1.f / 13.f); p = fmaf(p, t, 1.f / 11.f); p = fmaf(p, t, 1.f / 9.f); p = fmaf(p, t, 1.f / 7.f);
+  p = fmaf(p, t, 1.f / 5.f); p = fmaf(p, t, 1.f / 3.f); p = fmaf(p, t, 1.f);
+  return fmaf(2.f * s, p, fmaxf(z, 0.f));
+}
 
 __device__ __forceinline__ uint32_t bf2(float lo, float hi) {
   __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
@@ -181,12 +189,26 @@ __global__ void __launch_bounds__(LOCAL_THREADS) k_chunk_local_sum(const ChunkAr
   }
 }
 
+// d (16 x 8) += A (16 x 16) B (16 x 8), both fp32 in shared memory with pitch ld; by one warp
+__device__ __forceinline__ void block_product(float (&d)[4], const float* A, const float* B, int ld, int lane) {
+  const int g = lane >> 2, c2 = 2 * (lane & 3);
+  uint32_t ah[4], al[4], bh[2], bl[2];
+#pragma unroll
+  for (int e = 0; e < 4; e++) {
+    const float2 x = *reinterpret_cast<const float2*>(&A[(g + (e & 1) * 8) * ld + (e >> 1) * 8 + c2]);
+    split2(x.x, x.y, ah[e], al[e]);
+  }
+#pragma unroll
+  for (int e = 0; e < 2; e++) split2(B[(8 * e + c2) * ld + g], B[(8 * e + c2 + 1) * ld + g], bh[e], bl[e]);
+  mma(d, ah, bl[0], bl[1]); mma(d, al, bh[0], bh[1]); mma(d, ah, bh[0], bh[1]);
+}
+
 // Gated delta rule.  The raw inputs of the convolutions lie where the scaled operands and the small matrices go once the
 // convolutions are done.
 template <int DP> struct DeltaSmem {      // offsets in bytes
   static constexpr int ST = DP + 8, AT = C + 4, ROWS = C + MAX_TAPS - 1;
   static constexpr int K = 0, Q = K + C * ST * 4, L = Q + C * ST * 4, KF = L + C * ST * 4, QF = KF + 4 * C * DP, A = QF + 4 * C * DP,
-                       X = A + C * AT * 4, V = X + C * AT * 4, BETA = V + C * 128 * 2, SLOW = BETA + C * 4, TOTAL = SLOW + 16;
+                       X = A + C * AT * 4, V = X + C * AT * 4, CW = V + C * 128 * 2, BETA = CW + 3 * 128 * 16, SLOW = BETA + C * 4, TOTAL = SLOW + 16;
   static constexpr int RAW = KF;           // bf16 [3][ROWS][128]
   static_assert(3 * ROWS * 128 * 2 <= V - RAW, "raw inputs overlap what is live");
 };
@@ -206,6 +228,7 @@ __global__ void __launch_bounds__(LOCAL_THREADS, 1) k_chunk_local_delta(const Ch
   bf16* xs = reinterpret_cast<bf16*>(smem_raw + Sm::A);      // at the end: the inverse times diag(beta), high and low
   float* sX = reinterpret_cast<float*>(smem_raw + Sm::X);    // [64][AT] the inverse
   bf16* sv = reinterpret_cast<bf16*>(smem_raw + Sm::V);      // v [64][128]
+  float4* cw = reinterpret_cast<float4*>(smem_raw + Sm::CW); // [3][128] first four taps of every channel
   float* beta = reinterpret_cast<float*>(smem_raw + Sm::BETA);
   int* slow = reinterpret_cast<int*>(smem_raw + Sm::SLOW);   // [4]
   bf16* raw = reinterpret_cast<bf16*>(smem_raw + Sm::RAW);
@@ -240,17 +263,33 @@ __global__ void __launch_bounds__(LOCAL_THREADS, 1) k_chunk_local_delta(const Ch
     return tail + (long long)(keep + t) * channels + (which == 0 ? 0 : which == 1 ? G * D : 2 * G * D) + head;
   };
   if (((D | E) & 7) == 0 && (a.ldp & 7) == 0) {
-    for (int i = tid; i < 3 * rows * 16; i += LOCAL_THREADS) {
-      const int which = i / (rows * 16), r = i / 16 % rows, c = i % 16 * 8;
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (r < n + keep && c < (which == 2 ? E : D)) v = *reinterpret_cast<const uint4*>(source(which, r) + c);
-      *reinterpret_cast<uint4*>(raw + (which * Sm::ROWS + r) * 128 + c) = v;
-    }
+    const int c = tid % 16 * 8;
+#pragma unroll
+    for (int which = 0; which < 3; which++)
+#pragma unroll
+      for (int i = 0; i < 3; i++) {
+        const int r = tid / 16 + i * (LOCAL_THREADS / 16);
+        if (r >= rows) break;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (r < n + keep && c < (which == 2 ? E : D)) v = *reinterpret_cast<const uint4*>(source(which, r) + c);
+        *reinterpret_cast<uint4*>(raw + (which * Sm::ROWS + r) * 128 + c) = v;
+      }
   } else {
     for (int i = tid; i < 3 * rows * 128; i += LOCAL_THREADS) {
       const int which = i / (rows * 128), r = i / 128 % rows, c = i % 128;
       raw[(which * Sm::ROWS + r) * 128 + c] = r < n + keep && c < (which == 2 ? E : D) ? source(which, r)[c] : __float2bfloat16_rn(0.f);
     }
+  }
+  if (tid < 3 * 128) {
+    const int which = tid / 128, c = tid % 128;
+    const float* src = which == 0 ? a.conv_q : which == 1 ? a.conv_k : a.conv_v;
+    float w[4] = {};
+    if (c < (which == 2 ? E : D)) {
+      src += (long long)((which == 2 ? h * E : qh * D) + c) * a.taps;
+#pragma unroll
+      for (int j = 0; j < 4; j++) if (j < a.taps) w[j] = src[j];
+    }
+    cw[tid] = make_float4(w[0], w[1], w[2], w[3]);
   }
   if (tid < C) beta[tid] = tid < n ? 1.f / (1.f + expf(-__bfloat162float(proj[(r0 + tid) * a.ldp + a.s_b + h]))) : 0.f;
   if (tid < 4) slow[tid] = 0;
@@ -263,35 +302,23 @@ __global__ void __launch_bounds__(LOCAL_THREADS, 1) k_chunk_local_delta(const Ch
     for (int e = 0; e < 4; e++) x[e] = t < n && d + e < D ? -rate * softplus_f(x[e] + a.dt_bias[h * D + d + e]) : 0.f;
     *reinterpret_cast<float4*>(&sl[t * ST + d]) = make_float4(x[0], x[1], x[2], x[3]);
   }
-  // convolution, silu, unit vectors: a warp takes four consecutive tokens of q, then of k, then of v; a lane two pairs of channels
-  float w[3][4][4];      // the first four taps; further ones are read where they are used
-#pragma unroll
-  for (int which = 0; which < 3; which++) {
-    const float* src = which == 0 ? a.conv_q : which == 1 ? a.conv_k : a.conv_v;
-    const int size = which == 2 ? E : D, head = which == 2 ? h : qh;
-#pragma unroll
-    for (int i = 0; i < 4; i++) {
-      const int c = (i >> 1) * 64 + 2 * lane + (i & 1);
-#pragma unroll
-      for (int j = 0; j < 4; j++) w[which][i][j] = j < a.taps && c < size ? src[(long long)(head * size + c) * a.taps + j] : 0.f;
-    }
-  }
   __syncthreads();
+  // convolution, silu, unit vectors: a warp takes four consecutive tokens of q, then of k, then of v; a lane two pairs of channels
   const int tb0 = 4 * warp;
-#pragma unroll
+  const float q_scale = rsqrtf((float)D);
+#pragma unroll 1
   for (int which = 0; which < 3; which++) {
     float x[7][4];
+    float4 w[4];
+#pragma unroll
+    for (int i = 0; i < 4; i++) w[i] = cw[which * 128 + (i >> 1) * 64 + 2 * lane + (i & 1)];
 #pragma unroll
     for (int r = 0; r < 7; r++)
-      if (r < 3 + min(a.taps, 4)) {
 #pragma unroll
-        for (int p = 0; p < 2; p++) {
-          const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(raw + (which * Sm::ROWS + tb0 + r) * 128 + p * 64 + 2 * lane));
-          x[r][2 * p] = f.x; x[r][2 * p + 1] = f.y;
-        }
-      } else {
-#pragma unroll
-        for (int p = 0; p < 4; p++) x[r][p] = 0.f;
+      for (int p = 0; p < 2; p++) {
+        float2 f = make_float2(0.f, 0.f);
+        if (r < 3 + a.taps) f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(raw + (which * Sm::ROWS + tb0 + r) * 128 + p * 64 + 2 * lane));
+        x[r][2 * p] = f.x; x[r][2 * p + 1] = f.y;
       }
 #pragma unroll
     for (int tt = 0; tt < 4; tt++) {
@@ -299,9 +326,8 @@ __global__ void __launch_bounds__(LOCAL_THREADS, 1) k_chunk_local_delta(const Ch
       float y[4], ss = 0.f;
 #pragma unroll
       for (int i = 0; i < 4; i++) {
-        float acc = 0.f;
-#pragma unroll
-        for (int j = 0; j < 4; j++) acc = fmaf(w[which][i][j], x[tt + j][i], acc);
+        float acc = w[i].x * x[tt][i];
+        acc = fmaf(w[i].y, x[tt + 1][i], acc); acc = fmaf(w[i].z, x[tt + 2][i], acc); acc = fmaf(w[i].w, x[tt + 3][i], acc);
         if (a.taps > 4) {
           const int c = (i >> 1) * 64 + 2 * lane + (i & 1), size = which == 2 ? E : D, head = which == 2 ? h : qh;
           const float* src = which == 0 ? a.conv_q : which == 1 ? a.conv_k : a.conv_v;
@@ -316,8 +342,7 @@ __global__ void __launch_bounds__(LOCAL_THREADS, 1) k_chunk_local_delta(const Ch
 #pragma unroll
         for (int p = 0; p < 2; p++) *reinterpret_cast<uint32_t*>(sv + swz(t, p * 64 + 2 * lane, 128)) = bf2(y[2 * p], y[2 * p + 1]);
       } else {
-        float f = 1.f / sqrtf(warp_sum(ss) + 1e-6f);
-        if (which == 0) f *= 1.f / sqrtf((float)D);
+        const float f = rsqrtf(warp_sum(ss) + 1e-6f) * (which ? 1.f : q_scale);
         float* dst = (which ? sk : sq) + t * ST + 2 * lane;
 #pragma unroll
         for (int p = 0; p < DP / 64; p++) *reinterpret_cast<float2*>(dst + p * 64) = make_float2(y[2 * p] * f, y[2 * p + 1] * f);
@@ -456,23 +481,22 @@ __global__ void __launch_bounds__(LOCAL_THREADS, 1) k_chunk_local_delta(const Ch
     }
   }
   __syncthreads();
+  // X_IJ = -X_II sum_K M_IK X_KJ, one warp per (block, half of its columns); the inner sum goes to the free block (J, I) of sA
 #pragma unroll
   for (int dist = 1; dist < 4; dist++) {
-    // Y_IJ = sum_K M_IK X_KJ goes to the free block (J, I) of sA; X_IJ = -X_II Y_IJ
-    for (int i = tid; i < (4 - dist) * 256; i += LOCAL_THREADS) {
-      const int J = i / 256, I = J + dist, r = i % 256 / 16, c = i % 16;
-      float y = 0.f;
-#pragma unroll 16
-      for (int k = 0; k < 16 * dist; k++) y = fmaf(sA[(16 * I + r) * AT + 16 * J + k], sX[(16 * J + k) * AT + 16 * J + c], y);
-      sA[(16 * J + r) * AT + 16 * I + c] = y;
-    }
-    __syncthreads();
-    for (int i = tid; i < (4 - dist) * 256; i += LOCAL_THREADS) {
-      const int J = i / 256, I = J + dist, r = i % 256 / 16, c = i % 16;
-      float x = 0.f;
+    const int J = warp >> 1, I = J + dist, nh = (warp & 1) * 8;
+    if (I < 4) {
+      float y[4] = {};
 #pragma unroll
-      for (int k = 0; k < 16; k++) x = fmaf(sX[(16 * I + r) * AT + 16 * I + k], sA[(16 * J + k) * AT + 16 * I + c], x);
-      sX[(16 * I + r) * AT + 16 * J + c] = -x;
+      for (int k = 0; k < dist; k++)
+        block_product(y, sA + 16 * I * AT + 16 * (J + k), sX + 16 * (J + k) * AT + 16 * J + nh, AT, lane);
+#pragma unroll
+      for (int e = 0; e < 2; e++) *reinterpret_cast<float2*>(&sA[(16 * J + g + 8 * e) * AT + 16 * I + nh + c2]) = make_float2(y[2 * e], y[2 * e + 1]);
+      __syncwarp();
+      float x[4] = {};
+      block_product(x, sX + 16 * I * AT + 16 * I, sA + 16 * J * AT + 16 * I + nh, AT, lane);
+#pragma unroll
+      for (int e = 0; e < 2; e++) *reinterpret_cast<float2*>(&sX[(16 * I + g + 8 * e) * AT + 16 * J + nh + c2]) = make_float2(-x[2 * e], -x[2 * e + 1]);
     }
     __syncthreads();
   }
@@ -535,24 +559,26 @@ __global__ void __launch_bounds__(LOCAL_THREADS, 1) k_chunk_local_delta(const Ch
 }
 
 // ---- scan over the chunks -----------------------------------------------------------------------------------------------
-// One block: 16 columns of one head's state.  Warp w computes U and O of tokens 8w .. 8w+7 and owns 1/8 of the state's rows.
-template <int DP, bool DELTA>
+// One block: MT tiles of 16 columns of one head's state.  Warp w computes U and O of tokens 8w .. 8w+7 and owns 1/8 of the
+// state's rows.  Two tiles per block read the chunk's operands from shared memory once for both (its bandwidth is the limit);
+// one tile gives more blocks when there are few heads.
+template <int DP, bool DELTA, int MT>
 __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs a) {
   pdl_trigger();
   typedef Item<DP> It;
   constexpr int NT = DP / 64;                  // 8-column tiles of the state's rows per warp
   constexpr size_t X0 = DELTA ? 0 : It::Q, XB = It::X_BYTES - X0;      // without A there is no W
-  constexpr size_t UB = (size_t)C * 16 * 4, XS = XB + UB, SLOT = XS > It::Y_BYTES ? XS : It::Y_BYTES;
+  constexpr size_t SLOT = XB > It::Y_BYTES ? XB : It::Y_BYTES;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~(uintptr_t)127);
-  // ring of three half chunks: first half [W, Q~ | U_0 slice], second half [K^, B, Gamma_C]; half i lies in slot i mod 3, and
-  // half i + 3 is fetched as soon as half i has been read
-  bf16* sS = reinterpret_cast<bf16*>(smem + 3 * SLOT);      // state^T [16][DP], high and low
-  bf16* sU = sS + 2 * 16 * DP;                 // U^T [16][64], high and low
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sU + 2 * 16 * C);
+  // ring of three half chunks: first half [W, Q~], second half [K^, B, Gamma_C]; half i lies in slot i mod 3, and half i + 3
+  // is fetched as soon as half i has been read
+  bf16* sS = reinterpret_cast<bf16*>(smem + 3 * SLOT);      // state^T [MT][16][DP], high and low
+  bf16* sU = sS + MT * 2 * 16 * DP;            // U^T [MT][16][64], high and low
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sU + MT * 2 * 16 * C);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(bars + 3);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c2 = 2 * (lane & 3);
-  const int eb = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
+  const int e0 = blockIdx.x * MT * 16, h = blockIdx.y, b = blockIdx.z;
   const int D = a.dim, E = a.vdim, H = a.heads;
   const char* items = a.ws + ((long long)b * H + h) * a.chunks * a.item_bytes;
   if (threadIdx.x == 0) {
@@ -564,42 +590,52 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
   auto load = [&](int i) {                     // half i
     if (i >= 2 * a.chunks) return;
     const char* it = items + (long long)(i >> 1) * a.item_bytes;
-    uint8_t* dst = smem + (i % 3) * SLOT;
     uint64_t* bar = &bars[i % 3];
-    if (i & 1) {
-      mbar_expect_tx(bar, (uint32_t)It::Y_BYTES);
-      bulk_load_1d(dst, it + It::K, (uint32_t)It::Y_BYTES, bar);
-    } else {
-      mbar_expect_tx(bar, (uint32_t)XS);
-      bulk_load_1d(dst, it + X0, (uint32_t)XB, bar);
-      bulk_load_1d(dst + XB, it + It::U + eb * UB, (uint32_t)UB, bar);
-    }
+    mbar_expect_tx(bar, (uint32_t)(i & 1 ? It::Y_BYTES : XB));
+    bulk_load_1d(smem + (i % 3) * SLOT, it + (i & 1 ? It::K : X0), (uint32_t)(i & 1 ? It::Y_BYTES : XB), bar);
   };
   auto half_bar = [&](int i) { return &bars[i % 3]; };
   auto half_phase = [&](int i) { return (uint32_t)((i / 3) & 1); };
   if (threadIdx.x == 0) { load(0); load(1); load(2); }
+  // U_0 of this thread's tokens and columns, one chunk ahead
+  float u0[MT][2][2];
+  auto fetch_u0 = [&](int c) {
+    const float* src = reinterpret_cast<const float*>(items + (long long)c * a.item_bytes + It::U);
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+      for (int e = 0; e < 2; e++)
+#pragma unroll
+        for (int i = 0; i < 2; i++)
+          u0[m][e][i] = e0 + 16 * m < E ? __ldg(src + ((long long)(e0 / 16 + m) * C + 8 * warp + c2 + i) * 16 + g + 8 * e) : 0.f;
+  };
+  fetch_u0(0);
   // the state: rows d0 .. of column e in accumulator fragments, and its two bf16 parts in shared memory
   const int d0 = warp * 8 * NT;
-  float S[NT][4];
+  float S[MT][NT][4];
   auto publish = [&]() {
 #pragma unroll
-    for (int i = 0; i < NT; i++)
+    for (int m = 0; m < MT; m++)
 #pragma unroll
-      for (int e = 0; e < 2; e++) {
-        uint32_t hi, lo;
-        split2(S[i][2 * e], S[i][2 * e + 1], hi, lo);
-        const int o = swz(g + 8 * e, d0 + 8 * i + c2, DP);
-        *reinterpret_cast<uint32_t*>(sS + o) = hi; *reinterpret_cast<uint32_t*>(sS + 16 * DP + o) = lo;
-      }
+      for (int i = 0; i < NT; i++)
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+          uint32_t hi, lo;
+          split2(S[m][i][2 * e], S[m][i][2 * e + 1], hi, lo);
+          bf16* o = sS + m * 32 * DP + swz(g + 8 * e, d0 + 8 * i + c2, DP);
+          *reinterpret_cast<uint32_t*>(o) = hi; *reinterpret_cast<uint32_t*>(o + 16 * DP) = lo;
+        }
   };
   auto state_at = [&](int e, int d) { return a.S + (((long long)b * H + h) * E + e) * D + d; };
 #pragma unroll
-  for (int i = 0; i < NT; i++)
+  for (int m = 0; m < MT; m++)
 #pragma unroll
-    for (int e = 0; e < 4; e++) {
-      const int col = eb * 16 + g + 8 * (e >> 1), d = d0 + 8 * i + c2 + (e & 1);
-      S[i][e] = col < E && d < D ? *state_at(col, d) : 0.f;
-    }
+    for (int i = 0; i < NT; i++)
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const int col = e0 + 16 * m + g + 8 * (e >> 1), d = d0 + 8 * i + c2 + (e & 1);
+        S[m][i][e] = col < E && d < D ? *state_at(col, d) : 0.f;
+      }
   publish();
   bool ok = true;
   int c = 0;
@@ -609,8 +645,7 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
     const uint8_t* x = smem + (2 * c % 3) * SLOT;
     const bf16* tw = reinterpret_cast<const bf16*>(x);
     const bf16* tq = reinterpret_cast<const bf16*>(x + (It::Q - X0));
-    const float* u0 = reinterpret_cast<const float*>(x + XB);
-    float u[3][4] = {}, o[3][4] = {};
+    float u[MT][3][4] = {}, o[MT][3][4] = {};
 #pragma unroll
     for (int k0 = 0; k0 < DP; k0 += 32) {
       // operand rows are tokens 8 warp + 0..7, four 8-channel units (two k steps) per load
@@ -619,52 +654,63 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
       if (DELTA) { ldsm4(wh, tw + at); ldsm4(wl, tw + C * DP + at); }
       ldsm4(qh, tq + at); ldsm4(ql, tq + C * DP + at);
 #pragma unroll
-      for (int k = 0; k < 2; k++) {
-        uint32_t sh[4], sl[4];
-        const int as = swz(lane & 15, k0 + 16 * k + 8 * (lane >> 4), DP);
-        ldsm4(sh, sS + as); ldsm4(sl, sS + 16 * DP + as);
-        if (DELTA) { mma(u[0], sh, wh[2 * k], wh[2 * k + 1]); mma(u[1], sh, wl[2 * k], wl[2 * k + 1]); mma(u[2], sl, wh[2 * k], wh[2 * k + 1]); }
-        mma(o[0], sh, qh[2 * k], qh[2 * k + 1]); mma(o[1], sh, ql[2 * k], ql[2 * k + 1]); mma(o[2], sl, qh[2 * k], qh[2 * k + 1]);
+      for (int k = 0; k < 2; k++)
+#pragma unroll
+        for (int m = 0; m < MT; m++) {
+          uint32_t sh[4], sl[4];
+          const bf16* as = sS + m * 32 * DP + swz(lane & 15, k0 + 16 * k + 8 * (lane >> 4), DP);
+          ldsm4(sh, as); ldsm4(sl, as + 16 * DP);
+          if (DELTA) { mma(u[m][0], sh, wh[2 * k], wh[2 * k + 1]); mma(u[m][1], sh, wl[2 * k], wl[2 * k + 1]); mma(u[m][2], sl, wh[2 * k], wh[2 * k + 1]); }
+          mma(o[m][0], sh, qh[2 * k], qh[2 * k + 1]); mma(o[m][1], sh, ql[2 * k], ql[2 * k + 1]); mma(o[m][2], sl, qh[2 * k], qh[2 * k + 1]);
+        }
+    }
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+      for (int e = 0; e < 2; e++) {
+        float v[2];
+#pragma unroll
+        for (int i = 0; i < 2; i++) v[i] = u0[m][e][i] - (DELTA ? u[m][0][2 * e + i] + (u[m][1][2 * e + i] + u[m][2][2 * e + i]) : 0.f);
+        uint32_t hi, lo;
+        split2(v[0], v[1], hi, lo);
+        bf16* to = sU + m * 32 * C + swz(g + 8 * e, 8 * warp + c2, C);
+        *reinterpret_cast<uint32_t*>(to) = hi; *reinterpret_cast<uint32_t*>(to + 16 * C) = lo;
       }
-    }
-#pragma unroll
-    for (int e = 0; e < 2; e++) {
-      float v[2];
-#pragma unroll
-      for (int i = 0; i < 2; i++) v[i] = u0[(8 * warp + c2 + i) * 16 + g + 8 * e] - (DELTA ? u[0][2 * e + i] + (u[1][2 * e + i] + u[2][2 * e + i]) : 0.f);
-      uint32_t hi, lo;
-      split2(v[0], v[1], hi, lo);
-      const int at = swz(g + 8 * e, 8 * warp + c2, C);
-      *reinterpret_cast<uint32_t*>(sU + at) = hi; *reinterpret_cast<uint32_t*>(sU + 16 * C + at) = lo;
-    }
     if (!mbar_wait(half_bar(2 * c + 1), half_phase(2 * c + 1), abort_flag, a.status)) ok = false;
     if (!__syncthreads_and(ok)) break;         // U is complete, this chunk's W, Q~ and the old state have been read
     if (threadIdx.x == 0) load(2 * c + 3);
+    if (c + 1 < a.chunks) fetch_u0(c + 1);
     const uint8_t* sy = smem + ((2 * c + 1) % 3) * SLOT;
     const bf16* tk = reinterpret_cast<const bf16*>(sy);
     const bf16* tb = reinterpret_cast<const bf16*>(sy + (It::B - It::K));
     const float* gam = reinterpret_cast<const float*>(sy + (It::G - It::K));
-    uint32_t uh[4][4], ul[4][4];
+    float low[MT][NT][4] = {};
 #pragma unroll
-    for (int k = 0; k < 4; k++) {
-      const int at = swz(lane & 15, 16 * k + 8 * (lane >> 4), C);
-      ldsm4(uh[k], sU + at); ldsm4(ul[k], sU + 16 * C + at);
+    for (int i = 0; i < NT; i++) {
+      const float2 f = *reinterpret_cast<const float2*>(&gam[d0 + 8 * i + c2]);
+#pragma unroll
+      for (int m = 0; m < MT; m++) { S[m][i][0] *= f.x; S[m][i][1] *= f.y; S[m][i][2] *= f.x; S[m][i][3] *= f.y; }
     }
-    float low[NT][4] = {};
-#pragma unroll
-    for (int i = 0; i < NT; i++)
-#pragma unroll
-      for (int e = 0; e < 4; e++) S[i][e] *= gam[d0 + 8 * i + c2 + (e & 1)];
 #pragma unroll
     for (int k = 0; k < 4; k += 2) {
-      uint32_t bh[4], bl[4];
+      uint32_t uh[MT][2][4], ul[MT][2][4];
+#pragma unroll
+      for (int m = 0; m < MT; m++)
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+          const bf16* at = sU + m * 32 * C + swz(lane & 15, 16 * (k + i) + 8 * (lane >> 4), C);
+          ldsm4(uh[m][i], at); ldsm4(ul[m][i], at + 16 * C);
+        }
       if (16 * k <= 8 * warp + 7) {            // later tokens do not reach these
+        uint32_t bh[4], bl[4];
         const int at = swz(8 * warp + (lane & 7), 16 * k + 8 * (lane >> 3), C);
         ldsm4(bh, tb + at); ldsm4(bl, tb + C * C + at);
 #pragma unroll
-        for (int i = 0; i < 2; i++) {
-          mma(o[0], uh[k + i], bh[2 * i], bh[2 * i + 1]); mma(o[1], uh[k + i], bl[2 * i], bl[2 * i + 1]); mma(o[2], ul[k + i], bh[2 * i], bh[2 * i + 1]);
-        }
+        for (int m = 0; m < MT; m++)
+#pragma unroll
+          for (int i = 0; i < 2; i++) {
+            mma(o[m][0], uh[m][i], bh[2 * i], bh[2 * i + 1]); mma(o[m][1], uh[m][i], bl[2 * i], bl[2 * i + 1]); mma(o[m][2], ul[m][i], bh[2 * i], bh[2 * i + 1]);
+          }
       }
 #pragma unroll
       for (int i = 0; i < 2; i++) {
@@ -678,24 +724,30 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
           kl[0] = kh[2]; kl[1] = kh[3];
         }
 #pragma unroll
-        for (int j = 0; j < NT; j++) {
-          mma(S[j], uh[k + i], kh[2 * j], kh[2 * j + 1]);
-          mma(low[j], uh[k + i], kl[2 * j], kl[2 * j + 1]); mma(low[j], ul[k + i], kh[2 * j], kh[2 * j + 1]);
-        }
+        for (int m = 0; m < MT; m++)
+#pragma unroll
+          for (int j = 0; j < NT; j++) {
+            mma(S[m][j], uh[m][i], kh[2 * j], kh[2 * j + 1]);
+            mma(low[m][j], uh[m][i], kl[2 * j], kl[2 * j + 1]); mma(low[m][j], ul[m][i], kh[2 * j], kh[2 * j + 1]);
+          }
       }
     }
 #pragma unroll
-    for (int i = 0; i < NT; i++)
+    for (int m = 0; m < MT; m++)
 #pragma unroll
-      for (int e = 0; e < 4; e++) S[i][e] += low[i][e];
+      for (int i = 0; i < NT; i++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) S[m][i][e] += low[m][i][e];
     publish();
     const int t0 = a.t0 + c * C + 8 * warp + c2;
 #pragma unroll
-    for (int e = 0; e < 4; e++) {
-      const int t = t0 + (e & 1), col = eb * 16 + g + 8 * (e >> 1);
-      if (t < a.T && col < E)
-        reinterpret_cast<bf16*>(a.o)[((long long)b * a.T + t) * ((long long)H * E) + (long long)h * E + col] = __float2bfloat16_rn(o[0][e] + (o[1][e] + o[2][e]));
-    }
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const int t = t0 + (e & 1), col = e0 + 16 * m + g + 8 * (e >> 1);
+        if (t < a.T && col < E)
+          reinterpret_cast<bf16*>(a.o)[((long long)b * a.T + t) * ((long long)H * E) + (long long)h * E + col] = __float2bfloat16_rn(o[m][0][e] + (o[m][1][e] + o[m][2][e]));
+      }
     __syncthreads();                           // K^, B have been read
     if (threadIdx.x == 0) load(2 * c + 4);
   }
@@ -706,24 +758,27 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
     return;
   }
 #pragma unroll
-  for (int i = 0; i < NT; i++)
+  for (int m = 0; m < MT; m++)
 #pragma unroll
-    for (int e = 0; e < 4; e++) {
-      const int col = eb * 16 + g + 8 * (e >> 1), d = d0 + 8 * i + c2 + (e & 1);
-      if (col < E && d < D) *state_at(col, d) = S[i][e];
-    }
+    for (int i = 0; i < NT; i++)
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const int col = e0 + 16 * m + g + 8 * (e >> 1), d = d0 + 8 * i + c2 + (e & 1);
+        if (col < E && d < D) *state_at(col, d) = S[m][i][e];
+      }
 }
 
 template <int DP, bool DELTA> int run(ChunkArgs a, cudaStream_t s) {
   typedef Item<DP> It;
   const size_t local = DELTA ? DeltaSmem<DP>::TOTAL : 8 * C * DP;
-  const size_t x = (DELTA ? It::X_BYTES : It::X_BYTES - It::Q) + (size_t)C * 16 * 4;
-  const size_t scan = 3 * std::max(x, It::Y_BYTES) + 2 * 16 * DP * 2 + 2 * 16 * C * 2 + 64 + 128;
+  const size_t x = DELTA ? It::X_BYTES : It::X_BYTES - It::Q;
+  const auto scan = [&](int mt) { return 3 * std::max(x, It::Y_BYTES) + (size_t)mt * (2 * 16 * DP * 2 + 2 * 16 * C * 2) + 64 + 128; };
   static PerDevice attr;
   const int dev = PerDevice::current();
   if (dev < 0 || !attr.done[dev]) {
     CUDA_TRY(cudaFuncSetAttribute(DELTA ? k_chunk_local_delta<DP> : k_chunk_local_sum<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)local));
-    CUDA_TRY(cudaFuncSetAttribute(k_chunk_scan<DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)scan));
+    CUDA_TRY(cudaFuncSetAttribute(k_chunk_scan<DP, DELTA, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)scan(1)));
+    CUDA_TRY(cudaFuncSetAttribute(k_chunk_scan<DP, DELTA, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)scan(2)));
     if (dev >= 0) attr.done[dev] = true;
   }
   a.item_bytes = (It::bytes(a.vdim) + 127) / 128 * 128;
@@ -734,7 +789,10 @@ template <int DP, bool DELTA> int run(ChunkArgs a, cudaStream_t s) {
     a.t0 = c0 * C; a.chunks = std::min(seg, total - c0);
     (DELTA ? k_chunk_local_delta<DP> : k_chunk_local_sum<DP>)<<<dim3(a.chunks, a.heads, a.B), LOCAL_THREADS, local, s>>>(a);
     KERNEL_CHECK();
-    k_chunk_scan<DP, DELTA><<<dim3(cdiv(a.vdim, 16), a.heads, a.B), SCAN_THREADS, scan, s>>>(a);
+    if (cdiv(a.vdim, 32) * a.heads * a.B >= device_sm_count())
+      k_chunk_scan<DP, DELTA, 2><<<dim3(cdiv(a.vdim, 32), a.heads, a.B), SCAN_THREADS, scan(2), s>>>(a);
+    else
+      k_chunk_scan<DP, DELTA, 1><<<dim3(cdiv(a.vdim, 16), a.heads, a.B), SCAN_THREADS, scan(1), s>>>(a);
     KERNEL_CHECK();
   }
   return 0;

@@ -5,6 +5,7 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 #include <stdio.h>
+#include <stdlib.h>
 
 #include "../../include/femto.h"
 
@@ -126,7 +127,8 @@ static inline cudaError_t launch_dependent(void (*kernel)(P...), dim3 grid, dim3
   cudaLaunchAttribute at[1];
   at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
   at[0].val.programmaticStreamSerializationAllowed = 1;
-  cfg.attrs = at; cfg.numAttrs = 1;
+  static const bool off = [] { const char* e = getenv("FEMTO_PDL"); return e && e[0] == '0'; }();   // measurement aid: fully serialised
+  cfg.attrs = at; cfg.numAttrs = off ? 0 : 1;
   return cudaLaunchKernelEx(&cfg, kernel, static_cast<P>(args)...);
 }
 #endif

@@ -465,7 +465,7 @@ __global__ void __launch_bounds__(1024) k_latent_decode_out(const LatentArgs a, 
     const int c = i % a.lp, half = i / a.lp, s1 = min(splits, (half + 1) * per);
     float acc = 0.f;
 #pragma unroll 8
-    for (int s = half * per; s < s1; s++) acc = fmaf(ws[s], ws[s] == 0.f ? 0.f : p[(long long)s * ldp + 2 + c], acc);
+    for (int s = half * per; s < s1; s++) acc = fmaf(ws[s], p[(long long)s * ldp + 2 + c], acc);   // an empty split holds zeros
     oc[i] = acc;
   }
   __syncthreads();
@@ -520,8 +520,8 @@ template <typename T> static int latent_decode(const LatentArgs& a, cudaStream_t
     const int KT = bytes(64) <= 227 * 1024 ? 64 : 32;
     if (bytes(KT) <= 227 * 1024) {
       const int tiles = cdiv(N, KT);
-      // as many splits as fill the device once, each of at least two tiles
-      int per = std::max(std::min(2, tiles), cdiv(tiles, std::max(1, device_sm_count() / blocks)));
+      // as many splits as fill the device once
+      int per = std::max(1, cdiv(tiles, std::max(1, device_sm_count() / blocks)));
       while (!fits(cdiv(tiles, per))) per++;
       splits = cdiv(tiles, per);
 #define LAUNCH(NP) do { FEMTO_TRY(allow_smem(k_latent_decode_mma<NP>, bytes(KT))); \

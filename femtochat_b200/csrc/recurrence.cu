@@ -227,10 +227,16 @@ __global__ void __launch_bounds__(1024) k_delta_decode(const DeltaDecodeArgs a) 
       const T now = proj[(which == 0 ? p.s_q : which == 1 ? p.s_k : p.s_v) + at];
       const bool writes = which == 2 || h % (H / G) == 0;      // the heads of a group share q and k
       float acc = 0.f;
-      for (int j = 0; j < keep; j++) {
-        const T x = tin[(long long)j * channels + chan];
-        acc = fmaf(taps[j], to_f<T>(x), acc);
-        if (writes && j > 0) tout[(long long)(j - 1) * channels + chan] = x;
+      for (int j0 = 0; j0 < keep; j0 += 4) {          // four loads in flight before the first store
+        T x[4];
+#pragma unroll
+        for (int j = 0; j < 4; j++) if (j0 + j < keep) x[j] = tin[(long long)(j0 + j) * channels + chan];
+#pragma unroll
+        for (int j = 0; j < 4; j++)
+          if (j0 + j < keep) {
+            acc = fmaf(taps[j0 + j], to_f<T>(x[j]), acc);
+            if (writes && j0 + j > 0) tout[(long long)(j0 + j - 1) * channels + chan] = x[j];
+          }
       }
       if (writes && keep > 0) tout[(long long)(keep - 1) * channels + chan] = now;
       y = silu_f(fmaf(taps[keep], to_f<T>(now), acc));
@@ -253,12 +259,13 @@ __global__ void __launch_bounds__(1024) k_delta_decode(const DeltaDecodeArgs a) 
     const int c = decay ? i : i - D, r = decay ? a.ra : a.rg;
     const T* w = reinterpret_cast<const T*>(decay ? a.w_a2 : a.w_g2) + (long long)(h * (decay ? D : E) + c) * r;
     const float z = row_dot<T>(w, decay ? sa : sb, r, lane);
-    if (lane == 0) {
-      if (decay) sg[c] = expf(-rate * softplus_f(z + p.dt_bias[h * D + c]));
-      else sz[c] = sigmoid_f(round_to<T>(z));
-    }
+    if (lane == 0) (decay ? sg : sz)[c] = z;
   }
-  for (int c = D + tid; c < DP; c += 1024) sg[c] = 0.f;
+  __syncthreads();
+  for (int i = tid; i < DP + E; i += 1024) {
+    if (i < DP) sg[i] = i < D ? expf(-rate * softplus_f(sg[i] + p.dt_bias[h * D + i])) : 0.f;
+    else sz[i - DP] = sigmoid_f(round_to<T>(sz[i - DP]));
+  }
   __syncthreads();
   const float beta = sigmoid_f(to_f<T>(proj[p.s_b + h])), fk = f_k, fq = f_q;
   const int sub = tid & 7;
