@@ -105,7 +105,7 @@ int decoder_fill(DecoderStack* d, const femto_decoder_config* cfg) {
       l.conv_q = put(x + "q.conv", G * D, c.conv); l.conv_k = put(x + "k.conv", G * D, c.conv); l.conv_v = put(x + "v.conv", H * E, c.conv);
       l.a_log = put(x + "A_log", H, 0); l.dt_bias = put(x + "dt_bias", H * D, 0); l.mix_norm = put(x + "norm", E, 0);
     } else {
-      l.qp = round_up(c.q_rank, 8); l.lp = round_up(c.kv_rank, 8); l.ld = round_up(l.lp + c.rot_dim, 8);
+      l.qp = round_up(c.q_rank, 8); l.dp = round_up(c.dim, 8); l.lp = round_up(c.kv_rank, 8); l.ld = round_up(l.lp + c.rot_dim, 8);
       l.s_q = seg(c.q_rank); l.s_dkv = seg(c.kv_rank + c.rot_dim); l.s_g = seg(H);
       put(x + "dq", c.q_rank, w); put(x + "dkv", c.kv_rank + c.rot_dim, w); put(x + "g", H, w);
       put(x + "uq", H * (D + c.rot_dim), c.q_rank); put(x + "uk", H * D, c.kv_rank); put(x + "uv", H * E, c.kv_rank);
@@ -160,12 +160,12 @@ void carve(DecoderStack* d, Carver& b) {
     if (l.own != (int)i) continue;
     b.take(l.w_in, es * l.n_in * w); b.take(l.w_o, es * w * H * E);
     if (c.mixer == FEMTO_MIXER_CHANNEL_DELTA) { b.take(l.w_a2, es * H * D * l.ra); b.take(l.w_g2, es * H * E * l.rg); }
-    if (c.mixer == FEMTO_MIXER_LATENT_ATTENTION) { b.take(l.w_uq, es * H * (D + c.rot_dim) * l.qp); b.take(l.w_kv, es * H * (D + E) * l.lp); }
+    if (c.mixer == FEMTO_MIXER_LATENT_ATTENTION) { b.take(l.w_uq, es * H * (D + c.rot_dim) * l.qp); b.take(l.w_kv, es * H * (D + E) * l.lp); b.take(l.w_ukt, es * H * l.lp * l.dp); }
     if (c.ff > 0) { b.take(l.w_gu, es * 2 * l.ffp * w); b.take(l.w_down, es * w * l.ffp); }
   }
   for (auto& l : d->layers) {
     const DecLayer& o = d->layers[l.own];
-    l.w_in = o.w_in; l.w_o = o.w_o; l.w_a2 = o.w_a2; l.w_g2 = o.w_g2; l.w_uq = o.w_uq; l.w_kv = o.w_kv; l.w_gu = o.w_gu; l.w_down = o.w_down;
+    l.w_in = o.w_in; l.w_o = o.w_o; l.w_a2 = o.w_a2; l.w_g2 = o.w_g2; l.w_uq = o.w_uq; l.w_kv = o.w_kv; l.w_ukt = o.w_ukt; l.w_gu = o.w_gu; l.w_down = o.w_down;
   }
   b.take(d->tok0, 4 * R); b.take(d->want, 4 * R);
   b.take(d->x, 4 * R * w); b.take(d->hn, es * R * w); b.take(d->y, es * R * w);
@@ -174,7 +174,8 @@ void carve(DecoderStack* d, Carver& b) {
   b.take(d->qn, 4 * R * qk); b.take(d->kn, 4 * R * qk); b.take(d->gd, 4 * R * hd); b.take(d->beta, 4 * R * heads);
   b.take(d->vv, es * R * vv); b.take(d->g2, es * R * g2);
   b.take(d->cq, es * R * cq); b.take(d->q, es * R * q);
-  b.take(d->qabs, 4 * std::min(R, (size_t)d->cfg.max_batch * LATENT_FEW) * qa);
+  const size_t few = std::min(R, (size_t)d->cfg.max_batch * LATENT_FEW);
+  b.take(d->qabs, 4 * few * qa); b.take(d->oc, es * few * qa);
   size_t items = 0;
   for (const auto& l : d->layers)
     if (d->bf && l.c.mixer != FEMTO_MIXER_LATENT_ATTENTION && l.c.dim <= 128 && l.c.vdim <= 128)
@@ -251,6 +252,7 @@ template <typename T> static int refresh_t(DecoderStack* d, const float* theta, 
       FEMTO_TRY(pack(x + "dq", l.w_in, w, l.s_q, all, 0)); FEMTO_TRY(pack(x + "dkv", l.w_in, w, l.s_dkv, all, 0));
       FEMTO_TRY(pack(x + "g", l.w_in, w, l.s_g, all, 0));
       FEMTO_TRY(pack(x + "uq", l.w_uq, l.qp, 0, all, 0));
+      FEMTO_TRY(pack_transposed<T>(theta + find(x + "uk")->offset, c.heads, c.dim, c.kv_rank, (T*)l.w_ukt, l.dp, l.lp, s));
       FEMTO_TRY(pack(x + "uk", l.w_kv, l.lp, 0, all, 0)); FEMTO_TRY(pack(x + "uv", l.w_kv, l.lp, c.heads * c.dim, all, 0));
     } else {
       FEMTO_TRY(pack(x + "q", l.w_in, w, l.s_q, all, 0)); FEMTO_TRY(pack(x + "k", l.w_in, w, l.s_k, all, 0));
@@ -389,7 +391,7 @@ static int mixer_t(DecoderStack* d, femto_kv_cache* c, int i, const float* theta
   } else {
     LatentArgs a;
     a.q = d->q; a.dkv = proj + l.s_dkv; a.ld_dkv = l.n_in; a.dkv_norm = theta + l.dkv_norm; a.gate = proj + l.s_g; a.ld_gate = l.n_in;
-    a.latent = st.latent; a.ld = l.ld; a.lp = l.lp; a.maxT = c->maxT; a.w_kv = l.w_kv; a.kv = c->kv_exp;
+    a.latent = st.latent; a.ld = l.ld; a.lp = l.lp; a.maxT = c->maxT; a.w_kv = l.w_kv; a.w_ukt = l.w_ukt; a.dp = l.dp; a.oc = d->oc; a.kv = c->kv_exp;
     a.qabs = d->qabs; a.part = c->part; a.part_floats = c->part_floats; a.o = out;
     a.B = B; a.T = Tn; a.first = first; a.heads = H; a.dim = D; a.rot_dim = q.rot_dim; a.rot_dims = q.rot_dims; a.vdim = E; a.kv_rank = q.kv_rank;
     a.scale = q.scale; a.eps = eps; a.freq = l.freq_dev; a.d = d;

@@ -21,12 +21,12 @@ struct DecLayer {
   long long norm1 = -1, norm1b = -1, norm2 = -1, norm2b = -1, mix_norm = -1, conv_q = -1, conv_k = -1, conv_v = -1,
             a_log = -1, dt_bias = -1, dq_norm = -1, dkv_norm = -1;
   // packed compute-type weights, row-major [out][in]
-  void *w_in = nullptr, *w_o = nullptr, *w_a2 = nullptr, *w_g2 = nullptr, *w_uq = nullptr, *w_kv = nullptr, *w_gu = nullptr,
+  void *w_in = nullptr, *w_o = nullptr, *w_a2 = nullptr, *w_g2 = nullptr, *w_uq = nullptr, *w_kv = nullptr, *w_ukt = nullptr, *w_gu = nullptr,
        *w_down = nullptr;
   int n_in = 0;                       // columns of proj
   int s_q = 0, s_k = 0, s_v = 0, s_g = 0, s_b = 0, s_a1 = 0, s_g1 = 0, s_dkv = 0;   // segment starts
   int ra = 0, rg = 0;                 // decay_rank / gate_rank rounded up to 8
-  int qp = 0, lp = 0, ld = 0;         // q_rank, kv_rank rounded up to 8; pitch of a cached latent row
+  int qp = 0, lp = 0, ld = 0, dp = 0; // q_rank, kv_rank rounded up to 8; pitch of a cached latent row; dim rounded up to 8
   int ffp = 0;                        // ff rounded up to 32: the feed-forward's products are this wide
   int qk_heads() const { return c.mixer == FEMTO_MIXER_CHANNEL_DELTA ? c.kv_heads : c.heads; }
 };
@@ -49,6 +49,7 @@ struct DecoderStack {
   float *qn = nullptr, *kn = nullptr, *gd = nullptr, *beta = nullptr;
   void *vv = nullptr, *g2 = nullptr, *cq = nullptr, *q = nullptr;
   float* qabs = nullptr;              // latent attention, few rows: queries in the latent space
+  void* oc = nullptr;                 // and results there
   char* chunk_ws = nullptr;           // chunked recurrences: operands of the chunks of one segment
   size_t chunk_ws_bytes = 0;
   void* gemm_ws = nullptr;
@@ -83,6 +84,8 @@ template <typename T> struct DecStream {
 };
 // weight packing: dst[(r / group) * step + r % group + dst_row][c] = src[r][c], c < cols (dst pitch ldd)
 template <typename T>
+int pack_transposed(const float* src, int batch, int rows, int cols, T* dst, int ld_rows, int ld_cols, cudaStream_t s);   // dst[b][c][r] = src[b][r][c]
+template <typename T>
 int pack_rows(const float* src, int rows, int cols, T* dst, long long ldd, int dst_row, int group, int step, cudaStream_t s);
 
 // ---- products -------------------------------------------------------------------------------------------------------
@@ -91,6 +94,17 @@ int pack_rows(const float* src, int rows, int cols, T* dst, long long ldd, int d
 template <typename T>
 int rows_linear(DecoderStack* d, const void* X, long long ldx, const void* W, long long ldw, void* C, long long ldc, int M, int N, int K,
                 int epi, cudaStream_t s);
+
+// The streaming kernel by itself (bf16, aligned, at most ROWS_STREAM rows), as a batch over heads: element strides between the
+// heads' operands, and optionally one gate logit per (row, head) whose sigmoid multiplies the result.
+constexpr int ROWS_STREAM = 32;
+struct RowsBatch {
+  long long x = 0, w = 0, c = 0;
+  const bf16* gate = nullptr;
+  long long ld_gate = 0;
+};
+int rows_stream(const bf16* X, long long ldx, const bf16* W, long long ldw, void* C, long long ldc, int M, int N, int K, int epi, int batch,
+                const RowsBatch& bt, cudaStream_t s);
 
 // ---- recurrences (recurrence.cu) ------------------------------------------------------------------------------------
 struct RecurrenceArgs {
@@ -156,6 +170,9 @@ struct LatentArgs {
   void* latent = nullptr;        // cache [maxB][maxT][ld]
   int ld = 0, lp = 0, maxT = 0;
   const void* w_kv = nullptr;    // [heads dim + heads vdim][lp]
+  const void* w_ukt = nullptr;   // [heads][lp][dp]: the key up-projection transposed, dim padded to dp
+  int dp = 0;
+  void* oc = nullptr;            // [rows][heads][lp] attention results in the latent space
   void* kv = nullptr;            // expanded keys and values, [B][maxT][heads (dim + vdim)]
   float* qabs = nullptr; float* part = nullptr; size_t part_floats = 0;
   void* o = nullptr;             // [rows][heads vdim]

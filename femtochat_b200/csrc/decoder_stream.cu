@@ -131,34 +131,41 @@ __global__ void __launch_bounds__(RT) k_gather_norm(const float* __restrict__ x,
   for (int c = threadIdx.x; c < d; c += RT) h[(long long)i * d + c] = from_f<T>(src[c] * inv * w[c]);
 }
 
-// One warp per (row, group).
-template <typename T, int V>
+// LG lanes per (row, group).
+template <typename T, int V, int LG>
 __global__ void __launch_bounds__(256) k_gated_norm(const T* __restrict__ in, const float* __restrict__ w, int w_all,
                                                     const T* __restrict__ gate, long long ldg, T* __restrict__ out, long long n,
                                                     int groups, int size, float eps) {
   pdl_trigger();
   pdl_wait();
-  const long long it = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (it >= n) return;
-  const int lane = threadIdx.x & 31, g = (int)(it % groups);
+  const int lane = threadIdx.x & (LG - 1);
+  long long it = (long long)blockIdx.x * (256 / LG) + threadIdx.x / LG;
+  const bool live = it < n;
+  if (!live) it = n - 1;
+  const int g = (int)(it % groups);
   const long long row = it / groups;
   const T* a = in + it * size;
   const T* gt = gate + row * ldg + (long long)g * size;
   const float* wg = w + (w_all ? (long long)g * size : 0);
   float ss = 0.f;
-  for (int c = lane * V; c < size; c += 32 * V) {
+#pragma unroll 4
+  for (int c = lane * V; c < size; c += LG * V) {
     float f[V];
     load_vec<T, V>(a + c, f);
 #pragma unroll
     for (int e = 0; e < V; e++) ss += f[e] * f[e];
   }
-  const float inv = 1.f / sqrtf(warp_sum(ss) / size + eps);
-  for (int c = lane * V; c < size; c += 32 * V) {
+#pragma unroll
+  for (int o = LG / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float inv = 1.f / sqrtf(ss / size + eps);
+  if (!live) return;
+#pragma unroll 4
+  for (int c = lane * V; c < size; c += LG * V) {
     float f[V], z[V];
     load_vec<T, V>(a + c, f);
     load_vec<T, V>(gt + c, z);
 #pragma unroll
-    for (int e = 0; e < V; e++) f[e] = f[e] * inv * wg[c + e] * sigmoid_f(z[e]);
+    for (int e = 0; e < V; e++) f[e] = f[e] * inv * wg[c + e] * (sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-z[e])) : sigmoid_f(z[e]));
     store_vec<T, V>(out + it * size + c, f);
   }
 }
@@ -188,6 +195,16 @@ __global__ void __launch_bounds__(256) k_pack_rows(const float* __restrict__ src
   if (i >= n) return;
   const int r = (int)(i / cols), c = (int)(i % cols);
   dst[(long long)(dst_row + (r / group) * step + r % group) * ldd + c] = from_f<T>(src[i]);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) k_pack_transposed(const float* __restrict__ src, long long n, int rows, int cols, T* __restrict__ dst,
+                                                         int ld_rows, int ld_cols) {
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= n) return;
+  const int c = (int)(i % cols), r = (int)(i / cols % rows);
+  const long long b = i / cols / rows;
+  dst[(b * ld_cols + c) * ld_rows + r] = from_f<T>(src[i]);
 }
 
 // C[m][n] = sum_k X[m][k] W[n][k] for a few rows, any size: one warp per output column.  GATED: column n is
@@ -232,8 +249,10 @@ __global__ void __launch_bounds__(256) k_rows_linear(const T* __restrict__ X, lo
 // before the kernel waits for its predecessor.
 template <int NT, bool GATED>
 __global__ void __launch_bounds__(256) k_rows_mma(const bf16* __restrict__ X, long long ldx, const bf16* __restrict__ W, long long ldw,
-                                                  void* __restrict__ C, long long ldc, int M, int N, int K, int f32_out) {
+                                                  void* __restrict__ C, long long ldc, int M, int N, int K, int f32_out, const RowsBatch bt) {
   pdl_trigger();
+  X += blockIdx.y * bt.x;
+  W += blockIdx.y * bt.w;
   constexpr int RT = GATED ? 2 : 1, U = 4;      // U steps of 256 k are loaded ahead
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c8 = (lane & 3) * 8;
   const int n0 = blockIdx.x * 16;
@@ -292,8 +311,10 @@ __global__ void __launch_bounds__(256) k_rows_mma(const bf16* __restrict__ X, lo
 #pragma unroll
     for (int i = 0; i < 8; i++) { v += red[i][0][m][j]; if (GATED) up += red[i][RT - 1][m][j]; }
     if (GATED) v = v * sigmoid_f(v) * up;
-    if (f32_out) reinterpret_cast<float*>(C)[m * ldc + n0 + j] = v;
-    else reinterpret_cast<bf16*>(C)[m * ldc + n0 + j] = __float2bfloat16_rn(v);
+    if (bt.gate) v *= sigmoid_f(__bfloat162float(bt.gate[m * bt.ld_gate + blockIdx.y]));
+    const long long at = m * ldc + blockIdx.y * bt.c + n0 + j;
+    if (f32_out) reinterpret_cast<float*>(C)[at] = v;
+    else reinterpret_cast<bf16*>(C)[at] = __float2bfloat16_rn(v);
   }
 }
 
@@ -329,10 +350,13 @@ int DecStream<T>::gated_norm(const T* in, const float* w, bool w_all, const T* g
                              float eps, cudaStream_t s) {
   const long long n = (long long)rows * groups;
   constexpr int V = VecN<T>::n;
-  if (size % V == 0 && ldg % V == 0 && aligned16(in) && aligned16(gate) && aligned16(out))
-    CUDA_TRY(launch_dependent(k_gated_norm<T, V>, cdiv(n, 8), 256, 0, s, in, w, (int)w_all, gate, ldg, out, n, groups, size, eps));
-  else
-    CUDA_TRY(launch_dependent(k_gated_norm<T, 1>, cdiv(n, 8), 256, 0, s, in, w, (int)w_all, gate, ldg, out, n, groups, size, eps));
+  const bool vec = size % V == 0 && ldg % V == 0 && aligned16(in) && aligned16(gate) && aligned16(out);
+#define LAUNCH(VV, LG) CUDA_TRY(launch_dependent(k_gated_norm<T, VV, LG>, cdiv(n, 256 / LG), 256, 0, s, in, w, (int)w_all, gate, ldg, out, n, groups, size, eps))
+  if (!vec) LAUNCH(1, 32);
+  else if (size <= 8 * V) LAUNCH(V, 8);
+  else if (size <= 16 * V) LAUNCH(V, 16);
+  else LAUNCH(V, 32);
+#undef LAUNCH
   KERNEL_CHECK();
   return 0;
 }
@@ -356,25 +380,37 @@ template int pack_rows<float>(const float*, int, int, float*, long long, int, in
 template int pack_rows<bf16>(const float*, int, int, bf16*, long long, int, int, int, cudaStream_t);
 
 // Up to ROWS_STREAM rows in bf16 with aligned operands (RL_ROWS otherwise) stream the weights; more rows are a GEMM.
-constexpr int ROWS_STREAM = 32;
+int rows_stream(const bf16* X, long long ldx, const bf16* W, long long ldw, void* C, long long ldc, int M, int N, int K, int epi, int batch,
+                const RowsBatch& bt, cudaStream_t s) {
+  const dim3 grid(cdiv(N, 16), batch);
+  const int f32 = epi == EPI_F32;
+#define LAUNCH(NT) CUDA_TRY(epi == EPI_SWIGLU ? launch_dependent(k_rows_mma<NT, true>, grid, 256, 0, s, X, ldx, W, ldw, C, ldc, M, N, K, f32, bt) \
+                                              : launch_dependent(k_rows_mma<NT, false>, grid, 256, 0, s, X, ldx, W, ldw, C, ldc, M, N, K, f32, bt))
+  if (M <= 8) LAUNCH(1);
+  else if (M <= 16) LAUNCH(2);
+  else LAUNCH(4);
+#undef LAUNCH
+  KERNEL_CHECK();
+  return 0;
+}
+
+template <typename T>
+int pack_transposed(const float* src, int batch, int rows, int cols, T* dst, int ld_rows, int ld_cols, cudaStream_t s) {
+  const long long n = (long long)batch * rows * cols;
+  k_pack_transposed<T><<<cdiv(n, 256), 256, 0, s>>>(src, n, rows, cols, dst, ld_rows, ld_cols);
+  KERNEL_CHECK();
+  return 0;
+}
+template int pack_transposed<float>(const float*, int, int, int, float*, int, int, cudaStream_t);
+template int pack_transposed<bf16>(const float*, int, int, int, bf16*, int, int, cudaStream_t);
 
 template <typename T>
 int rows_linear(DecoderStack* d, const void* X, long long ldx, const void* W, long long ldw, void* C, long long ldc, int M, int N, int K,
                 int epi, cudaStream_t s) {
   const int f32 = epi == EPI_F32;
-  if constexpr (sizeof(T) == 2) {
-    if (M <= ROWS_STREAM && ((K | ldx | ldw) & 7) == 0 && aligned16(X) && aligned16(W)) {
-      const int grid = cdiv(N, 16);
-#define LAUNCH(NT) CUDA_TRY(epi == EPI_SWIGLU ? launch_dependent(k_rows_mma<NT, true>, grid, 256, 0, s, (const bf16*)X, ldx, (const bf16*)W, ldw, C, ldc, M, N, K, f32) \
-                                              : launch_dependent(k_rows_mma<NT, false>, grid, 256, 0, s, (const bf16*)X, ldx, (const bf16*)W, ldw, C, ldc, M, N, K, f32))
-      if (M <= 8) LAUNCH(1);
-      else if (M <= 16) LAUNCH(2);
-      else LAUNCH(4);
-#undef LAUNCH
-      KERNEL_CHECK();
-      return 0;
-    }
-  }
+  if constexpr (sizeof(T) == 2)
+    if (M <= ROWS_STREAM && ((K | ldx | ldw) & 7) == 0 && aligned16(X) && aligned16(W))
+      return rows_stream((const bf16*)X, ldx, (const bf16*)W, ldw, C, ldc, M, N, K, epi, 1, RowsBatch(), s);
   if (M <= RL_ROWS) {
     if (epi == EPI_SWIGLU) CUDA_TRY(launch_dependent(k_rows_linear<T, true>, cdiv(N, 8), 256, 0, s, (const T*)X, ldx, (const T*)W, ldw, C, ldc, M, N, K, f32));
     else CUDA_TRY(launch_dependent(k_rows_linear<T, false>, cdiv(N, 8), 256, 0, s, (const T*)X, ldx, (const T*)W, ldw, C, ldc, M, N, K, f32));

@@ -73,24 +73,32 @@ __global__ void __launch_bounds__(256) k_latent_norms(const LatentArgs a) {
   for (int i = a.rot_dims + lane; i < a.rot_dim; i += 32) dst[i] = src[i];
 }
 
-// q in place, for prompts: a thread rotates one pair of every head of its row.
-template <typename T>
+// q in place, for prompts: a thread rotates V neighbouring pairs of every head of its row (V = 2 needs even offsets).
+template <typename T, int V>
 __global__ void __launch_bounds__(256) k_rotate_q(const LatentArgs a) {
   pdl_trigger();
   pdl_wait();
-  const int half = a.rot_dims / 2, hd = a.dim + a.rot_dim;
+  struct __align__(V * sizeof(T)) Vec { T v[V]; };
+  const int half = a.rot_dims / 2, hd = a.dim + a.rot_dim, per = half / V;
   const long long it = (long long)blockIdx.x * 256 + threadIdx.x;
-  if (it >= (long long)a.B * a.T * half) return;
-  const int i = (int)(it % half);
-  const long long row = it / half;
-  float sn, cs;
-  sincosf((float)(a.first + (int)(row % a.T)) * a.freq[i], &sn, &cs);
+  if (it >= (long long)a.B * a.T * per) return;
+  const int i = (int)(it % per) * V;
+  const long long row = it / per;
+  float sn[V], cs[V];
+#pragma unroll
+  for (int e = 0; e < V; e++) sincosf((float)(a.first + (int)(row % a.T)) * a.freq[i + e], &sn[e], &cs[e]);
   T* q = reinterpret_cast<T*>(a.q) + row * (long long)a.heads * hd + a.dim;
-#pragma unroll 4
+#pragma unroll 8
   for (int h = 0; h < a.heads; h++, q += hd) {
-    const float u = to_f<T>(q[i]), v = to_f<T>(q[i + half]);
-    q[i] = from_f<T>(u * cs - v * sn);
-    q[i + half] = from_f<T>(v * cs + u * sn);
+    Vec u = *reinterpret_cast<const Vec*>(q + i), v = *reinterpret_cast<const Vec*>(q + i + half);
+#pragma unroll
+    for (int e = 0; e < V; e++) {
+      const float x = to_f<T>(u.v[e]), y = to_f<T>(v.v[e]);
+      u.v[e] = from_f<T>(x * cs[e] - y * sn[e]);
+      v.v[e] = from_f<T>(y * cs[e] + x * sn[e]);
+    }
+    *reinterpret_cast<Vec*>(q + i) = u;
+    *reinterpret_cast<Vec*>(q + i + half) = v;
   }
 }
 
@@ -233,7 +241,8 @@ __global__ void __launch_bounds__(1024) k_absorb_q(const LatentArgs a) {
 // The tensor-core form for bf16 caches.  grid (heads / 16, splits, rows): 16 heads are the rows of one mma tile; the cached
 // rows arrive in tiles of `KT` through two shared-memory buffers (16-byte units of row r permuted by r & 7) and serve as
 // keys (read as they lie) and as values (read transposed).  Queries and softmax weights are sums of two bf16 numbers, so
-// scores and weights keep fp32 accuracy.
+// scores and weights keep fp32 accuracy.  For the scores the warps share the channels, so a warp's part of the queries
+// stays in registers for the whole kernel and shared memory is read once; their partial sums meet in shared memory.
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)) : "memory");
@@ -247,16 +256,17 @@ __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], 
 }
 __device__ __forceinline__ int swz(int row, int col, int width) { return row * width + ((((col >> 3) ^ (row & 7)) << 3) | (col & 7)); }
 
-template <int NP>      // pairs of 8-channel tiles of the result per warp: lp <= 128 NP
+// NK: 16-channel steps per warp (width <= 128 NK); NP: pairs of 8-channel tiles of the result per warp (lp <= 128 NP)
+template <int NK, int NP>
 __global__ void __launch_bounds__(256) k_latent_decode_mma(const LatentArgs a, int splits, int tiles_per, int KT, int width) {
   pdl_trigger();
   pdl_wait();
   extern __shared__ __align__(16) uint8_t raw[];
+  const int SP = KT + 4;
   bf16* rows = reinterpret_cast<bf16*>(raw);            // 2 x [KT][width]
-  bf16* qh = rows + 2 * KT * width;                     // [16][width] high, low
-  bf16* ph = qh + 2 * 16 * width;                       // [16][64] high, low
-  float* ss = reinterpret_cast<float*>(ph + 2 * 16 * 64);   // [16][KT + 4]
-  float* sal = ss + 16 * (KT + 4);                      // [16] rescale factor of this tile
+  bf16* ph = rows + 2 * KT * width;                     // [16][64] high, low
+  float* ss = reinterpret_cast<float*>(ph + 2 * 16 * 64);   // [8 warps][16][SP]
+  float* sal = ss + 8 * 16 * SP;                        // [16] rescale factor of this tile
   float* sml = sal + 16;                                // [16][2] running max and sum
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c2 = 2 * (lane & 3);
   const int h0 = blockIdx.x * 16, sp = blockIdx.y;
@@ -276,28 +286,50 @@ __global__ void __launch_bounds__(256) k_latent_decode_mma(const LatentArgs a, i
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   if (tb < te) load(tb);
-  // queries, and zeros in the columns that pad a row to whole groups of 64
-  for (int i = tid; i < 16 * width / 2; i += 256) {
-    const int r = i / (width / 2), c = i % (width / 2) * 2;
-    float x = 0.f, y = 0.f;
-    if (h0 + r < a.heads && c < a.ld) {
-      const float2 f = *reinterpret_cast<const float2*>(a.qabs + (row * a.heads + h0 + r) * a.ld + c);
-      x = f.x; y = f.y;
+  // the rotated parts of the queries, through shared memory that the scores use later
+  float* qr = ss;                                       // [16][rot_dim]
+  const int half = a.rot_dims / 2, rest = a.rot_dim - half;       // a thread makes both entries of a pair, or passes one on
+  for (int i = tid; i < 16 * rest; i += 256) {
+    const int r = i / rest, k = i % rest, h = h0 + r;
+    if (h >= a.heads) continue;
+    const bf16* q = reinterpret_cast<const bf16*>(a.q) + (row * a.heads + h) * (a.dim + a.rot_dim) + a.dim;
+    if (k < half) {
+      float u, v;
+      rotate(__bfloat162float(q[k]), __bfloat162float(q[k + half]), (float)(n - 1), a.freq[k], u, v);
+      qr[r * a.rot_dim + k] = round_to<bf16>(u);
+      qr[r * a.rot_dim + k + half] = round_to<bf16>(v);
+    } else {
+      qr[r * a.rot_dim + k + half] = __bfloat162float(q[k + half]);
     }
-    const __nv_bfloat162 hi = __floats2bfloat162_rn(x, y);
-    const __nv_bfloat162 lo = __floats2bfloat162_rn(x - __bfloat162float(hi.x), y - __bfloat162float(hi.y));
-    const int o = swz(r, c, width);
-    *reinterpret_cast<__nv_bfloat162*>(qh + o) = hi;
-    *reinterpret_cast<__nv_bfloat162*>(qh + 16 * width + o) = lo;
   }
+  __syncthreads();
+  // this warp's steps of the queries: latent channels from qabs, then the rotated part, zeros in the padding
+  uint32_t qa[NK][4], ql[NK][4];
+#pragma unroll
+  for (int s = 0; s < NK; s++)
+#pragma unroll
+    for (int e = 0; e < 4; e++) {
+      const int r = g + 8 * (e & 1), h = h0 + r, c = (warp + 8 * s) * 16 + 8 * (e >> 1) + c2;
+      float2 f = make_float2(0.f, 0.f);
+      if (h < a.heads) {
+        if (c < a.lp) {
+          f = *reinterpret_cast<const float2*>(a.qabs + (row * a.heads + h) * a.lp + c);
+        } else {
+          if (c < a.lp + a.rot_dim) f.x = qr[r * a.rot_dim + c - a.lp];
+          if (c + 1 < a.lp + a.rot_dim) f.y = qr[r * a.rot_dim + c + 1 - a.lp];
+        }
+      }
+      const __nv_bfloat162 hi = __floats2bfloat162_rn(f.x, f.y);
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(f.x - __bfloat162float(hi.x), f.y - __bfloat162float(hi.y));
+      qa[s][e] = *reinterpret_cast<const uint32_t*>(&hi);
+      ql[s][e] = *reinterpret_cast<const uint32_t*>(&lo);
+    }
   const int pad = width - a.ld;
   if (pad)
     for (int i = tid; i < 2 * KT * pad / 8; i += 256) {
       const int r = i / (pad / 8), c = a.ld + i % (pad / 8) * 8;
       *reinterpret_cast<uint4*>(rows + (r / KT) * KT * width + swz(r % KT, c, width)) = make_uint4(0, 0, 0, 0);
     }
-  if (KT < 64)
-    for (int i = tid; i < 2 * 16 * 64 / 8; i += 256) *reinterpret_cast<uint4*>(ph + i * 8) = make_uint4(0, 0, 0, 0);
   if (tid < 16) { sml[2 * tid] = -INFINITY; sml[2 * tid + 1] = 0.f; }
   float o[NP][2][4] = {};
   for (int tile = tb; tile < te; tile++) {
@@ -305,32 +337,36 @@ __global__ void __launch_bounds__(256) k_latent_decode_mma(const LatentArgs a, i
     __syncthreads();                   // the tile is complete, the other buffer free
     if (tile + 1 < te) load(tile + 1);
     const bf16* kt = rows + (tile & 1) * KT * width;
-    if (warp * 8 < KT) {               // scores of eight keys
+    for (int j = 0; j < KT; j += 16) { // partial scores of 16 keys
       float s[2][4] = {};
-#pragma unroll 2
-      for (int k = 0; k < width; k += 32) {
+#pragma unroll
+      for (int k = 0; k < NK; k++) {
+        const int c = (warp + 8 * k) * 16;
+        if (c >= width) break;
         uint32_t kb[4];
-        ldsm4(kb, kt + swz(8 * warp + (lane & 7), k + 8 * (lane >> 3), width));
+        ldsm4(kb, kt + swz(j + (lane & 7) + 8 * (lane >> 4), c + 8 * ((lane >> 3) & 1), width));
 #pragma unroll
-        for (int i = 0; i < 2; i++) {
-          uint32_t ah[4], al[4];
-          const int at = swz(lane & 15, k + 16 * i + 8 * (lane >> 4), width);
-          ldsm4(ah, qh + at); ldsm4(al, qh + 16 * width + at);
-          mma16816(s[0], ah, kb[2 * i], kb[2 * i + 1]);
-          mma16816(s[1], al, kb[2 * i], kb[2 * i + 1]);
-        }
+        for (int i = 0; i < 2; i++) { mma16816(s[i], qa[k], kb[2 * i], kb[2 * i + 1]); mma16816(s[i], ql[k], kb[2 * i], kb[2 * i + 1]); }
       }
 #pragma unroll
-      for (int e = 0; e < 4; e++) {
-        const int key = 8 * warp + c2 + (e & 1);
-        ss[(g + 8 * (e >> 1)) * (KT + 4) + key] = tile * KT + key < n ? (s[0][e] + s[1][e]) * a.scale : -INFINITY;
-      }
+      for (int i = 0; i < 2; i++)
+#pragma unroll
+        for (int e = 0; e < 2; e++)
+          *reinterpret_cast<float2*>(&ss[(warp * 16 + g + 8 * e) * SP + j + 8 * i + c2]) = make_float2(s[i][2 * e], s[i][2 * e + 1]);
     }
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < 2; i++) {      // softmax of two heads per warp
       const int r = 2 * warp + i;
-      const float x0 = lane < KT ? ss[r * (KT + 4) + lane] : -INFINITY, x1 = lane + 32 < KT ? ss[r * (KT + 4) + lane + 32] : -INFINITY;
+      float x0 = 0.f, x1 = 0.f;
+#pragma unroll
+      for (int k = 0; k < 8; k++) {
+        x0 += ss[(k * 16 + r) * SP + lane];
+        if (KT > 32) x1 += ss[(k * 16 + r) * SP + lane + 32];
+      }
+      const int key = tile * KT + lane;
+      x0 = key < n ? x0 * a.scale : -INFINITY;
+      x1 = KT > 32 && key + 32 < n ? x1 * a.scale : -INFINITY;
       const float m = sml[2 * r], mn = fmaxf(m, warp_max(fmaxf(x0, x1)));      // finite: the first key of a tile is always seen
       const float p0 = __expf(x0 - mn), p1 = __expf(x1 - mn), f = __expf(m - mn);
       const float l = warp_sum(p0 + p1);
@@ -376,6 +412,43 @@ __global__ void __launch_bounds__(256) k_latent_decode_mma(const LatentArgs a, i
         const int c = (j * 8 + warp) * 16 + 8 * i + c2;
         if (c < a.lp) *reinterpret_cast<float2*>(dst + 2 + c) = make_float2(o[j][i][2 * e], o[j][i][2 * e + 1]);
       }
+  }
+}
+
+// grid (heads, rows): the splits of a head in order, normalised, as bf16 rows for the value up-projection.
+__global__ void __launch_bounds__(1024) k_latent_combine(const LatentArgs a, int splits) {
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ float sm[];
+  float* ws = sm;                 // [splits]
+  float* half1 = sm + splits;     // [lp]
+  const int h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, ldp = a.lp + 2;
+  const long long row = blockIdx.y;
+  const float* p = a.part + (row * a.heads + h) * (long long)splits * ldp;
+  if (tid < 32) {
+    float M = -INFINITY, L = 0.f;
+    for (int s = lane; s < splits; s += 32) { const float m = p[(long long)s * ldp]; ws[s] = m; M = fmaxf(M, m); }
+    M = warp_max(M);
+    for (int s = lane; s < splits; s += 32) {
+      const float w = ws[s] == -INFINITY ? 0.f : expf(ws[s] - M);
+      L += w * p[(long long)s * ldp + 1];
+      ws[s] = w;
+    }
+    L = 1.f / warp_sum(L);
+    for (int s = lane; s < splits; s += 32) ws[s] *= L;
+  }
+  __syncthreads();
+  const int part = tid >> 9, per = (splits + 1) / 2, s1 = min(splits, (part + 1) * per);
+  for (int c0 = 0; c0 < a.lp; c0 += 512) {
+    const int c = c0 + (tid & 511);
+    float acc = 0.f;
+    if (c < a.lp) {
+#pragma unroll 8
+      for (int s = part * per; s < s1; s++) acc = fmaf(ws[s], p[(long long)s * ldp + 2 + c], acc);   // an empty split holds zeros
+      if (part) half1[c] = acc;
+    }
+    __syncthreads();
+    if (!part && c < a.lp) reinterpret_cast<bf16*>(a.oc)[(row * a.heads + h) * a.lp + c] = __float2bfloat16_rn(acc + half1[c]);
   }
 }
 
@@ -504,50 +577,70 @@ template int latent_norms<float>(const LatentArgs&, cudaStream_t);
 template int latent_norms<bf16>(const LatentArgs&, cudaStream_t);
 
 // A few new tokens per column: queries into the latent space, attention over the cached rows, back out.
+static int latent_decode_tc(const LatentArgs& a, cudaStream_t s, bool& done) {
+  const int N = a.first + a.T, rows = a.B * a.T, H = a.heads, hd = a.dim + a.rot_dim;
+  const int width = round_up(a.ld, 64), nk = cdiv(width, 128), np = cdiv(a.lp, 128);
+  auto bytes = [&](int kt) { return (size_t)2 * kt * width * 2 + 2 * 16 * 64 * 2 + 4 * (size_t)(8 * 16 * (kt + 4) + 48); };
+  const int KT = bytes(64) <= 227 * 1024 ? 64 : 32;
+  // the rotated queries (16 x rot_dim) pass through the space of the scores
+  done = bytes(KT) <= 227 * 1024 && (hd & 7) == 0 && (a.dim & 7) == 0 && nk <= 9 && a.rot_dim <= 8 * (KT + 4);
+  if (!done) return 0;
+  const bf16* q = (const bf16*)a.q;
+  for (int r0 = 0; r0 < rows; r0 += ROWS_STREAM) {      // qabs[row][head] = W_uk^T q
+    RowsBatch bt;
+    bt.x = hd; bt.w = (long long)a.lp * a.dp; bt.c = a.lp;
+    FEMTO_TRY(rows_stream(q + (long long)r0 * H * hd, (long long)H * hd, (const bf16*)a.w_ukt, a.dp, a.qabs + (long long)r0 * H * a.lp, (long long)H * a.lp,
+                          std::min(ROWS_STREAM, rows - r0), a.lp, a.dim, EPI_F32, H, bt, s));
+  }
+  const int tiles = cdiv(N, KT), blocks = cdiv(H, 16) * rows;
+  int per = std::max(1, cdiv(tiles, std::max(1, device_sm_count() / blocks)));      // as many splits as fill the device once
+  while ((size_t)rows * H * cdiv(tiles, per) * (a.lp + 2) > a.part_floats) per++;
+  const int splits = cdiv(tiles, per);
+#define LAUNCH(NK, NP) do { FEMTO_TRY(allow_smem(k_latent_decode_mma<NK, NP>, bytes(KT))); \
+  CUDA_TRY(launch_dependent(k_latent_decode_mma<NK, NP>, dim3(cdiv(H, 16), splits, rows), 256, bytes(KT), s, a, splits, per, KT, width)); } while (0)
+  if (nk <= 1) LAUNCH(1, 1);
+  else if (nk <= 2) LAUNCH(2, 2);
+  else if (nk <= 3) LAUNCH(3, 3);
+  else if (nk <= 5 && np <= 4) LAUNCH(5, 4);
+  else LAUNCH(9, 8);
+#undef LAUNCH
+  KERNEL_CHECK();
+  CUDA_TRY(launch_dependent(k_latent_combine, dim3(H, rows), 1024, 4 * (size_t)(splits + a.lp), s, a, splits));
+  KERNEL_CHECK();
+  for (int r0 = 0; r0 < rows; r0 += ROWS_STREAM) {      // o[row][head] = W_uv oc sigmoid(gate)
+    RowsBatch bt;
+    bt.x = a.lp; bt.w = (long long)a.vdim * a.lp; bt.c = a.vdim;
+    bt.gate = (const bf16*)a.gate + (long long)r0 * a.ld_gate; bt.ld_gate = a.ld_gate;
+    FEMTO_TRY(rows_stream((const bf16*)a.oc + (long long)r0 * H * a.lp, (long long)H * a.lp, (const bf16*)a.w_kv + (long long)H * a.dim * a.lp, a.lp,
+                          (bf16*)a.o + (long long)r0 * H * a.vdim, (long long)H * a.vdim, std::min(ROWS_STREAM, rows - r0), a.vdim, a.lp, EPI_STORE, H, bt, s));
+  }
+  return 0;
+}
+
 template <typename T> static int latent_decode(const LatentArgs& a, cudaStream_t s) {
+  if constexpr (sizeof(T) == 2) {
+    bool done = false;
+    FEMTO_TRY(latent_decode_tc(a, s, done));
+    if (done) return 0;
+  }
   constexpr int V = VecN<T>::n;
   const int N = a.first + a.T, rows = a.B * a.T;
   const size_t absorb = 4 * (size_t)(a.dim + a.rot_dim + 1024 / (a.lp / V) * a.lp);
   FEMTO_TRY(allow_smem(k_absorb_q<T>, absorb));
   CUDA_TRY(launch_dependent(k_absorb_q<T>, dim3(a.heads, rows), 1024, absorb, s, a));
   KERNEL_CHECK();
-  int splits = 0;
-  const auto fits = [&](int n) { return (size_t)rows * a.heads * n * (a.lp + 2) <= a.part_floats; };
-  bool done = false;
-  if constexpr (sizeof(T) == 2) {
-    const int width = round_up(a.ld, 64), blocks = cdiv(a.heads, 16) * rows;
-    auto bytes = [&](int kt) { return (size_t)2 * kt * width * 2 + 2 * 16 * width * 2 + 2 * 16 * 64 * 2 + 4 * (16 * (kt + 4) + 48); };
-    const int KT = bytes(64) <= 227 * 1024 ? 64 : 32;
-    if (bytes(KT) <= 227 * 1024) {
-      const int tiles = cdiv(N, KT);
-      // as many splits as fill the device once
-      int per = std::max(1, cdiv(tiles, std::max(1, device_sm_count() / blocks)));
-      while (!fits(cdiv(tiles, per))) per++;
-      splits = cdiv(tiles, per);
-#define LAUNCH(NP) do { FEMTO_TRY(allow_smem(k_latent_decode_mma<NP>, bytes(KT))); \
-      CUDA_TRY(launch_dependent(k_latent_decode_mma<NP>, dim3(cdiv(a.heads, 16), splits, rows), 256, bytes(KT), s, a, splits, per, KT, width)); } while (0)
-      if (a.lp <= 128) LAUNCH(1);
-      else if (a.lp <= 256) LAUNCH(2);
-      else if (a.lp <= 512) LAUNCH(4);
-      else LAUNCH(8);
-#undef LAUNCH
-      done = true;
-    }
-  }
-  if (!done) {
-    const int blocks = cdiv(a.heads, 8) * rows;
-    splits = std::max(1, std::min({LATENT_MAX_SPLITS, cdiv(N, 64), cdiv(2 * device_sm_count(), blocks)}));
-    while (splits > 1 && !fits(splits)) splits--;
-    const size_t smem = 4 * (size_t)(32 * (a.ld + 1) + 8 * a.ld);
-    const int per = cdiv(a.lp, 32);
-    const dim3 grid(cdiv(a.heads, 8), splits, rows);
+  const int blocks = cdiv(a.heads, 8) * rows;
+  int splits = std::max(1, std::min({LATENT_MAX_SPLITS, cdiv(N, 64), cdiv(2 * device_sm_count(), blocks)}));
+  while (splits > 1 && (size_t)rows * a.heads * splits * (a.lp + 2) > a.part_floats) splits--;
+  const size_t smem = 4 * (size_t)(32 * (a.ld + 1) + 8 * a.ld);
+  const int per = cdiv(a.lp, 32);
+  const dim3 grid(cdiv(a.heads, 8), splits, rows);
 #define LAUNCH(PER) do { FEMTO_TRY(allow_smem(k_latent_decode<T, PER>, smem)); CUDA_TRY(launch_dependent(k_latent_decode<T, PER>, grid, 256, smem, s, a, splits)); } while (0)
-    if (per <= 4) LAUNCH(4);
-    else if (per <= 8) LAUNCH(8);
-    else if (per <= 16) LAUNCH(16);
-    else LAUNCH(32);
+  if (per <= 4) LAUNCH(4);
+  else if (per <= 8) LAUNCH(8);
+  else if (per <= 16) LAUNCH(16);
+  else LAUNCH(32);
 #undef LAUNCH
-  }
   KERNEL_CHECK();
   CUDA_TRY(launch_dependent(k_latent_decode_out<T>, dim3(cdiv(a.vdim, 32), a.heads, rows), 1024, 4 * (size_t)(2 * a.lp + splits), s, a, splits));
   KERNEL_CHECK();
@@ -560,7 +653,10 @@ template <typename T> int latent_attention(const LatentArgs& a, cudaStream_t s) 
     return femto_fail(FEMTO_ERR_UNSUPPORTED, "latent attention: dim %d + %d, vdim %d, rank %d", a.dim, a.rot_dim, a.vdim, a.kv_rank);
   if (a.T <= LATENT_FEW) return latent_decode<T>(a, s);
   if (a.rot_dims > 0) {
-    CUDA_TRY(launch_dependent(k_rotate_q<T>, cdiv((long long)rows * (a.rot_dims / 2), 256), 256, 0, s, a));
+    if (a.rot_dims % 4 == 0 && a.dim % 2 == 0 && a.rot_dim % 2 == 0)
+      CUDA_TRY(launch_dependent(k_rotate_q<T, 2>, cdiv((long long)rows * (a.rot_dims / 4), 256), 256, 0, s, a));
+    else
+      CUDA_TRY(launch_dependent(k_rotate_q<T, 1>, cdiv((long long)rows * (a.rot_dims / 2), 256), 256, 0, s, a));
     KERNEL_CHECK();
   }
   // keys and values of all N tokens of every column: [N][lp] x [heads (dim + vdim)][lp]^T
