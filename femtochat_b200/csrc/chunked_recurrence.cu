@@ -783,7 +783,15 @@ template <int DP, bool DELTA> int run(ChunkArgs a, cudaStream_t s) {
   }
   a.item_bytes = (It::bytes(a.vdim) + 127) / 128 * 128;
   const int total = cdiv(a.T, C);
-  const int seg = (int)std::min<long long>(total, (long long)a.ws_bytes / ((long long)a.item_bytes * a.B * a.heads));
+  const int most = (int)std::min<long long>(total, (long long)a.ws_bytes / ((long long)a.item_bytes * a.B * a.heads));
+  // the local part runs one block per SM: of the segment lengths that fit, the one that needs the fewest waves in all
+  int seg = most;
+  long long best = -1;
+  for (int n = most; n > most / 2; n--) {
+    const auto waves = [&](int chunks) { return (long long)cdiv((long long)chunks * a.heads * a.B, device_sm_count()); };
+    const long long w = total / n * waves(n) + (total % n ? waves(total % n) : 0);
+    if (best < 0 || w < best) { best = w; seg = n; }
+  }
   if (seg <= 0) return femto_fail(FEMTO_ERR_NOMEM, "chunked recurrence: workspace too small for %d columns of %d heads", a.B, a.heads);
   for (int c0 = 0; c0 < total; c0 += seg) {
     a.t0 = c0 * C; a.chunks = std::min(seg, total - c0);

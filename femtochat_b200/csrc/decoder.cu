@@ -180,8 +180,8 @@ void carve(DecoderStack* d, Carver& b) {
   for (const auto& l : d->layers)
     if (d->bf && l.c.mixer != FEMTO_MIXER_LATENT_ATTENTION && l.c.dim <= 128 && l.c.vdim <= 128)
       items = std::max(items, chunked_recurrence_item_bytes(l.c.dim, l.c.vdim) * l.c.heads * d->cfg.max_batch);
-  // the chunks of a segment go through memory once between the two kernels: a segment that stays in L2, at least one chunk
-  const size_t chunks = items ? std::max<size_t>(1, std::min<size_t>(((size_t)80 << 20) / items, R / d->cfg.max_batch / 64 + 1)) : 0;
+  // operands of the chunks of one segment, at least one chunk of every column
+  const size_t chunks = items ? std::max<size_t>(1, std::min<size_t>(((size_t)160 << 20) / items, R / d->cfg.max_batch / 64 + 1)) : 0;
   d->chunk_ws_bytes = items * chunks;
   b.take(d->chunk_ws, d->chunk_ws_bytes);
   d->gemm_ws_bytes = (size_t)64 << 20;
