@@ -568,7 +568,9 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
   typedef Item<DP> It;
   constexpr int NT = DP / 64;                  // 8-column tiles of the state's rows per warp
   constexpr size_t X0 = DELTA ? 0 : It::Q, XB = It::X_BYTES - X0;      // without A there is no W
-  constexpr size_t SLOT = XB > It::Y_BYTES ? XB : It::Y_BYTES;
+  // with one tile U_0 travels with W and Q~; with two the ring has no room for it and each thread loads its own, a chunk ahead
+  constexpr bool RING_U = MT == 1;
+  constexpr size_t UB = (size_t)C * 16 * 4, XS = XB + (RING_U ? UB : 0), SLOT = XS > It::Y_BYTES ? XS : It::Y_BYTES;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~(uintptr_t)127);
   // ring of three half chunks: first half [W, Q~], second half [K^, B, Gamma_C]; half i lies in slot i mod 3, and half i + 3
@@ -591,13 +593,14 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
     if (i >= 2 * a.chunks) return;
     const char* it = items + (long long)(i >> 1) * a.item_bytes;
     uint64_t* bar = &bars[i % 3];
-    mbar_expect_tx(bar, (uint32_t)(i & 1 ? It::Y_BYTES : XB));
+    mbar_expect_tx(bar, (uint32_t)(i & 1 ? It::Y_BYTES : XS));
     bulk_load_1d(smem + (i % 3) * SLOT, it + (i & 1 ? It::K : X0), (uint32_t)(i & 1 ? It::Y_BYTES : XB), bar);
+    if (RING_U && !(i & 1)) bulk_load_1d(smem + (i % 3) * SLOT + XB, it + It::U + blockIdx.x * UB, (uint32_t)UB, bar);
   };
   auto half_bar = [&](int i) { return &bars[i % 3]; };
   auto half_phase = [&](int i) { return (uint32_t)((i / 3) & 1); };
   if (threadIdx.x == 0) { load(0); load(1); load(2); }
-  // U_0 of this thread's tokens and columns, one chunk ahead
+  // U_0 of this thread's tokens and columns
   float u0[MT][2][2];
   auto fetch_u0 = [&](int c) {
     const float* src = reinterpret_cast<const float*>(items + (long long)c * a.item_bytes + It::U);
@@ -609,7 +612,7 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
         for (int i = 0; i < 2; i++)
           u0[m][e][i] = e0 + 16 * m < E ? __ldg(src + ((long long)(e0 / 16 + m) * C + 8 * warp + c2 + i) * 16 + g + 8 * e) : 0.f;
   };
-  fetch_u0(0);
+  if (!RING_U) fetch_u0(0);
   // the state: rows d0 .. of column e in accumulator fragments, and its two bf16 parts in shared memory
   const int d0 = warp * 8 * NT;
   float S[MT][NT][4];
@@ -645,6 +648,13 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
     const uint8_t* x = smem + (2 * c % 3) * SLOT;
     const bf16* tw = reinterpret_cast<const bf16*>(x);
     const bf16* tq = reinterpret_cast<const bf16*>(x + (It::Q - X0));
+    if (RING_U) {
+      const float* src = reinterpret_cast<const float*>(x + XB);
+#pragma unroll
+      for (int e = 0; e < 2; e++)
+#pragma unroll
+        for (int i = 0; i < 2; i++) u0[0][e][i] = src[(8 * warp + c2 + i) * 16 + g + 8 * e];
+    }
     float u[MT][3][4] = {}, o[MT][3][4] = {};
 #pragma unroll
     for (int k0 = 0; k0 < DP; k0 += 32) {
@@ -679,7 +689,7 @@ __global__ void __launch_bounds__(SCAN_THREADS, 1) k_chunk_scan(const ChunkArgs 
     if (!mbar_wait(half_bar(2 * c + 1), half_phase(2 * c + 1), abort_flag, a.status)) ok = false;
     if (!__syncthreads_and(ok)) break;         // U is complete, this chunk's W, Q~ and the old state have been read
     if (threadIdx.x == 0) load(2 * c + 3);
-    if (c + 1 < a.chunks) fetch_u0(c + 1);
+    if (!RING_U && c + 1 < a.chunks) fetch_u0(c + 1);
     const uint8_t* sy = smem + ((2 * c + 1) % 3) * SLOT;
     const bf16* tk = reinterpret_cast<const bf16*>(sy);
     const bf16* tb = reinterpret_cast<const bf16*>(sy + (It::B - It::K));
@@ -772,7 +782,7 @@ template <int DP, bool DELTA> int run(ChunkArgs a, cudaStream_t s) {
   typedef Item<DP> It;
   const size_t local = DELTA ? DeltaSmem<DP>::TOTAL : 8 * C * DP;
   const size_t x = DELTA ? It::X_BYTES : It::X_BYTES - It::Q;
-  const auto scan = [&](int mt) { return 3 * std::max(x, It::Y_BYTES) + (size_t)mt * (2 * 16 * DP * 2 + 2 * 16 * C * 2) + 64 + 128; };
+  const auto scan = [&](int mt) { return 3 * std::max(x + (mt == 1 ? (size_t)C * 64 : 0), It::Y_BYTES) + (size_t)mt * (2 * 16 * DP * 2 + 2 * 16 * C * 2) + 64 + 128; };
   static PerDevice attr;
   const int dev = PerDevice::current();
   if (dev < 0 || !attr.done[dev]) {
