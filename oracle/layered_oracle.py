@@ -1,4 +1,4 @@
-"""Plain restatement, on the CPU, of the decoders whose configuration lists their layers one by one (Virolorn).
+"""Plain restatement, on the CPU, of the decoders whose configuration lists their layers one by one (Virolorn, Zurevik).
 
 One function per mechanism, written from its equations and token by token wherever the mechanism is a recurrence.  It is
 slow on purpose and shares no code with the product: only `tests/` use it.  All arithmetic is in the dtype of the tensors
@@ -148,16 +148,111 @@ def latent_attention(h, w, m, eps, state):
     return o.reshape(T, H * E) @ w["o"].T
 
 
+def sees(i, j, size, keep_first=0):
+    """A sliding window of `size` tokens, itself included, and the first `keep_first` tokens of the sequence."""
+    return j <= i and (i - j < size or j < keep_first)
+
+
+def windowed_attention(q, k, v, scale, first, size, keep_first=0, sink=None):
+    """q [T, H, D] at positions first .., k [N, G, D], v [N, G, E]; query head h reads key/value head h // (H / G).  `sink` [H]:
+    one more term exp(sink) in the denominator."""
+    T, H, per = q.shape[0], q.shape[1], q.shape[1] // k.shape[1]
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for t in range(T):
+        see = torch.tensor([j for j in range(k.shape[0]) if sees(first + t, j, size, keep_first)])
+        for h in range(H):
+            s = (k[see, h // per] @ q[t, h]) * scale
+            top = s.max() if sink is None else torch.maximum(s.max(), sink[h])
+            e = torch.exp(s - top)
+            total = e.sum() if sink is None else e.sum() + torch.exp(sink[h] - top)
+            out[t, h] = (e / total) @ v[see, h // per]
+    return out
+
+
+def differential_lambda(w, diff):
+    return torch.exp((w["lq1"] * w["lk1"]).sum()) - torch.exp((w["lq2"] * w["lk2"]).sum()) + diff
+
+
+def append_kv(state, k, v):
+    """Adds rows to a layer's cached keys and values; returns (position of the first new row, all keys, all values)."""
+    first = state["k"].shape[0] if "k" in state else 0
+    state["k"] = torch.cat([state["k"], k]) if first else k
+    state["v"] = torch.cat([state["v"], v]) if first else v
+    return first
+
+
+def differential_attention(h, w, m, eps, state):
+    T, H, G, D, E = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q = rms_norm((h @ w["q"].T).view(T, H, 2, D), w["q.norm"], eps)
+    k = rms_norm((h @ w["k"].T).view(T, G, 2, D), w["k.norm"], eps)
+    first = append_kv(state, k, (h @ w["v"].T).view(T, G, E))
+    a = [windowed_attention(q[:, :, i], state["k"][:, :, i], state["v"], m["scale"], first, m["mask"]["size"], m["mask"]["keep_first"])
+         for i in range(2)]
+    o = a[0] - differential_lambda(w, m["diff"]) * a[1]
+    o = rms_norm(o, None, eps) * (1.0 - m["diff"])
+    return (o.reshape(T, H * E) * torch.sigmoid(h @ w["g"].T)) @ w["o"].T
+
+
+def sink_attention(h, w, m, eps, state, shared=None):
+    """`shared`: the state of the layer whose keys and values this one reads (that layer has added its rows already)."""
+    T, H, G, D, E = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q = (h @ w["q"].T + w["q.b"]).view(T, H, D)
+    if shared is None:
+        append_kv(state, (h @ w["k"].T + w["k.b"]).view(T, G, D), (h @ w["v"].T + w["v.b"]).view(T, G, E))
+        shared = state
+    o = windowed_attention(q, shared["k"], shared["v"], m["scale"], shared["k"].shape[0] - T, m["mask"]["size"], sink=w["sink"])
+    o = o * torch.sigmoid(h @ w["g"].T)[:, :, None]
+    return o.reshape(T, H * E) @ w["o"].T
+
+
 def gated_mlp(h, w):
     return (silu(h @ w["gate"].T) * (h @ w["up"].T)) @ w["down"].T
 
 
-MIXERS = dict(lightning=lightning, channel_delta=channel_delta, latent_attention=latent_attention)
+def route(z, top):
+    """The `top` largest logits of every row: (expert indices, softmax over the chosen ones)."""
+    best = torch.sort(z, dim=-1, descending=True, stable=True).indices[:, :top]
+    s = torch.gather(z, 1, best)
+    e = torch.exp(s - s.max(-1, keepdim=True).values)
+    return best, e / e.sum(-1, keepdim=True)
+
+
+def expert_mlp(h, up, down):
+    return torch.clamp(h @ up.T, min=0) ** 2 @ down.T
+
+
+def mixture_mlp(h, w, top):
+    best, weight = route(h @ w["router"].T + w["router.b"], top)
+    out = torch.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, p in zip(best[t].tolist(), weight[t]):
+            out[t] = out[t] + p * expert_mlp(h[t:t + 1], w[f"e{e}.up"], w[f"e{e}.down"])[0]
+    return out
+
+
+MIXERS = dict(lightning=lightning, channel_delta=channel_delta, latent_attention=latent_attention, attention=differential_attention,
+              attention_2=sink_attention)
 
 
 # ---- the model -----------------------------------------------------------------------------------------------------
 def _sub(weights, prefix):
     return {n[len(prefix):]: t for n, t in weights.items() if n.startswith(prefix)}
+
+
+def sandwich_layer(x, w, layer, eps, mult, mix):
+    """A norm before and after each sublayer, one after the other."""
+    x = x + mult * rms_norm(mix(rms_norm(x, w["norm1"], eps)), w["norm1b"], eps)
+    if layer["mlp"] is not None:
+        x = x + mult * rms_norm(gated_mlp(rms_norm(x, w["norm2"], eps), _sub(w, "mlp.")), w["norm2b"], eps)
+    return x
+
+
+def parallel_layer(x, w, layer, eps, mix):
+    """Mixer and feed-forward side by side, each behind a norm of its own."""
+    y = mix(rms_norm(x, w["norm1"], eps))
+    if layer["mlp"] is not None:
+        y = y + mixture_mlp(rms_norm(x, w["norm2"], eps), _sub(w, "mlp."), layer["mlp"]["router"]["top"])
+    return x + y
 
 
 class Sequence:
@@ -170,33 +265,40 @@ class Sequence:
         self.residuals = []           # the residual stream after every layer of the last call
 
     def feed(self, tokens):
-        cfg, eps, m = self.cfg, self.cfg["norm"]["eps"], self.cfg["residual_mult"]
-        x = self.w["embed"][torch.as_tensor(tokens, dtype=torch.long)]
+        cfg, eps = self.cfg, self.cfg["norm"]["eps"]
+        x = self.w["embed"][torch.as_tensor(tokens, dtype=torch.long)] * cfg.get("embedding", {}).get("scale", 1.0)
         self.residuals = []
         for i, layer in enumerate(cfg["layers"]):
             own = i
             while cfg["layers"][own].get("weights_of") is not None:
                 own = cfg["layers"][own]["weights_of"]
-            w = _sub(self.w, f"l{own}.")
-            y = MIXERS[layer["type"]](rms_norm(x, w["norm1"], eps), _sub(w, "mix."), layer["mixer"], eps, self.state[i])
-            x = x + m * rms_norm(y, w["norm1b"], eps)
-            if layer["mlp"] is not None:
-                y = gated_mlp(rms_norm(x, w["norm2"], eps), _sub(w, "mlp."))
-                x = x + m * rms_norm(y, w["norm2b"], eps)
+            w, m = _sub(self.w, f"l{own}."), layer["mixer"]
+            shared = {} if m.get("kv_from") is None else dict(shared=self.state[m["kv_from"]])
+            mix = lambda h: MIXERS[layer["type"]](h, _sub(w, "mix."), m, eps, self.state[i], **shared)
+            if cfg["architecture"] == "Zurevik":
+                x = parallel_layer(x, w, layer, eps, mix)
+            else:
+                x = sandwich_layer(x, w, layer, eps, cfg["residual_mult"], mix)
             self.residuals.append(x)
-        return rms_norm(x, self.w["final.norm"], eps) @ self.w["embed"].T
+        z = rms_norm(x, self.w["final.norm"], eps) @ self.w["head" if "head" in self.w else "embed"].T
+        cap = cfg.get("logit_softcap")
+        return z if cap is None else cap * torch.tanh(z / cap)
 
 
 # ---- small random models for the tests -------------------------------------------------------------------------------
 def tensor_shapes(cfg, decay_rank=8, gate_rank=8):
     """name -> shape of every tensor of a model; the two low-rank projections' ranks exist only as shapes."""
     d, out = cfg["width"], {"embed": (cfg["vocab"], cfg["width"]), "final.norm": (cfg["width"],)}
+    if cfg["architecture"] == "Zurevik":
+        out["head"] = out["embed"]
     for i, layer in enumerate(cfg["layers"]):
         if layer.get("weights_of") is not None:
             continue
         m, p = layer["mixer"], f"l{i}."
         x = p + "mix."
-        out[p + "norm1"] = out[p + "norm1b"] = (d,)
+        out[p + "norm1"] = (d,)
+        if cfg["architecture"] == "Virolorn":
+            out[p + "norm1b"] = (d,)
         if layer["type"] == "lightning":
             H, D, E = m["heads"], m["dim"], m["vdim"]
             out.update({x + "q": (H * D, d), x + "k": (H * D, d), x + "v": (H * E, d), x + "g": (H * E, d),
@@ -207,11 +309,26 @@ def tensor_shapes(cfg, decay_rank=8, gate_rank=8):
                         x + "v": (H * E, d), x + "v.conv": (H * E, n), x + "b": (H, d), x + "A_log": (H,), x + "norm": (E,),
                         x + "a1": (decay_rank, d), x + "a2": (H * D, decay_rank), x + "dt_bias": (H * D,),
                         x + "g1": (gate_rank, d), x + "g2": (H * E, gate_rank), x + "o": (d, H * E)})
+        elif layer["type"] == "attention":
+            H, G, D, E = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            out.update({x + "q": (H * 2 * D, d), x + "k": (G * 2 * D, d), x + "v": (G * E, d), x + "q.norm": (D,), x + "k.norm": (D,),
+                        x + "g": (H * E, d), x + "o": (d, H * E)})
+            out.update({x + n: (D,) for n in ("lq1", "lk1", "lq2", "lk2")})
+        elif layer["type"] == "attention_2":
+            H, G, D, E = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            out.update({x + "q": (H * D, d), x + "q.b": (H * D,), x + "sink": (H,), x + "g": (H, d), x + "o": (d, H * E)})
+            if m.get("kv_from") is None:
+                out.update({x + "k": (G * D, d), x + "k.b": (G * D,), x + "v": (G * E, d), x + "v.b": (G * E,)})
         else:
             H, D, R, E, L, Q = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"]
             out.update({x + "dq": (Q, d), x + "dq.norm": (Q,), x + "uq": (H * (D + R), Q), x + "dkv": (L + R, d),
                         x + "dkv.norm": (L,), x + "uk": (H * D, L), x + "uv": (H * E, L), x + "g": (H, d), x + "o": (d, H * E)})
-        if layer["mlp"] is not None:
+        if layer["mlp"] is not None and layer["mlp"]["kind"] == "moe":
+            f, n = layer["mlp"]["expert"]["ff"], layer["mlp"]["router"]["experts"]
+            out.update({p + "norm2": (d,), p + "mlp.router": (n, d), p + "mlp.router.b": (n,)})
+            for e in range(n):
+                out.update({p + f"mlp.e{e}.up": (f, d), p + f"mlp.e{e}.down": (d, f)})
+        elif layer["mlp"] is not None:
             f = layer["mlp"]["ff"]
             out[p + "norm2"] = out[p + "norm2b"] = (d,)
             out.update({p + "mlp.gate": (f, d), p + "mlp.up": (f, d), p + "mlp.down": (d, f)})
@@ -231,6 +348,10 @@ def random_weights(cfg, seed=0, decay_rank=8, gate_rank=8):
             t = 0.5 * r
         elif leaf == "dt_bias":
             t = r - 2.0
+        elif leaf in ("sink", "b") and len(shape) == 1:
+            t = r
+        elif leaf in ("lq1", "lk1", "lq2", "lk2"):
+            t = 0.6 * r / math.sqrt(shape[0]) ** 0.5
         elif leaf == "conv":
             t = r / math.sqrt(shape[1])
         elif name == "embed":
