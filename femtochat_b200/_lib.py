@@ -46,13 +46,16 @@ class OptimizerConfig(C.Structure):
 class LayerConfigC(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("mixer", "weights_of", "heads", "kv_heads", "dim", "vdim", "conv", "decay_rank", "gate_rank",
                                          "q_rank", "kv_rank", "rot_dim", "rot_dims", "ff")] + [
-        ("scale", C.c_float), ("rot_base", C.c_double), ("h_decay", C.POINTER(C.c_float))]
+        ("scale", C.c_float), ("rot_base", C.c_double), ("h_decay", C.POINTER(C.c_float))] + [
+        (n, C.c_int32) for n in ("maps", "window", "keep_first", "kv_from", "qkv_bias", "qk_norm", "sink", "gate")] + [
+        ("diff", C.c_float), ("experts", C.c_int32), ("top", C.c_int32)]
 
 
 class DecoderConfigC(C.Structure):
     _fields_ = [("vocab", C.c_int32), ("width", C.c_int32), ("n_layer", C.c_int32), ("compute_dtype", C.c_int32), ("index_base", C.c_int32),
                 ("max_batch", C.c_int32), ("max_rows", C.c_int32), ("norm_eps", C.c_float), ("residual_mult", C.c_float),
-                ("h_layers", C.POINTER(LayerConfigC))]
+                ("h_layers", C.POINTER(LayerConfigC)), ("block", C.c_int32), ("untied", C.c_int32), ("embed_scale", C.c_float),
+                ("logit_softcap", C.c_float)]
 
 
 class DecoderTensorC(C.Structure):

@@ -168,6 +168,12 @@ struct GemmArgs {
   // square symmetric result: tiles that lie entirely below the diagonal are not computed (the caller mirrors
   // the upper triangle afterwards); honoured by the tensor-core kernel, ignored by the SIMT fallback
   bool upper_only = false;
+  // Grouped product (EPI_STORE, EPI_RELU2; batch 1): the rows of A come in runs of group_rows (128 or 256) rows, run i is
+  // multiplied by matrix groups[1 + i] of B (strideB apart), and only the first groups[0] runs hold anything.  Device memory:
+  // the host knows no more than the largest number of runs, M / group_rows.
+  const int* groups = nullptr;
+  int group_rows = 0, n_groups = 0;   // n_groups: matrices in B
+  const float* bias = nullptr;   // [N] added to the columns before the store (EPI_STORE)
   bool any_size = false;   // take the tensor-core kernel for results smaller than one tile as well
   int ring = 0;   // depth of the operand ring of the tensor-core kernel; 0 = the deepest that fits (fewer stages leave
                   // shared memory free for kernels of another stream to run on the same SMs)

@@ -17,6 +17,7 @@ static int check_layer(const femto_decoder_config& cfg, int i) {
   NEED(c.heads > 0 && c.dim > 0 && c.vdim > 0, "heads, dim and vdim must be positive");
   NEED(c.ff >= 0, "ff is negative");
   NEED(c.weights_of < cfg.n_layer && c.weights_of != i, "weights_of names no other layer");
+  if (c.experts) NEED(c.ff > 0 && moe_supported(c.experts, c.top), "a mixture needs 1 to 1024 experts, of which a token uses 1 to 32, and their ff");
   switch (c.mixer) {
     case FEMTO_MIXER_LIGHTNING:
       NEED(c.h_decay != nullptr, "lightning attention needs one decay per head");
@@ -33,6 +34,19 @@ static int check_layer(const femto_decoder_config& cfg, int i) {
       NEED(c.rot_dims >= 0 && c.rot_dims <= c.rot_dim && c.rot_dims % 2 == 0, "rot_dims must be even and at most rot_dim");
       NEED(c.kv_rank <= 1024 && c.vdim <= 256 && c.dim + c.rot_dim <= 512, "kv_rank above 1024, vdim above 256 or dim + rot_dim above 512 is not supported");
       break;
+    case FEMTO_MIXER_ATTENTION:
+      NEED(c.kv_heads > 0 && c.heads % c.kv_heads == 0, "heads must be a multiple of kv_heads");
+      NEED(c.maps == 1 || c.maps == 2, "maps must be 1 or 2");
+      NEED(c.window > 0 && c.keep_first >= 0, "window must be positive and keep_first not negative");
+      NEED(c.gate >= FEMTO_GATE_NONE && c.gate <= FEMTO_GATE_ELEMENT, "unknown gate");
+      NEED(c.dim <= 256 && c.vdim <= 256, "dim or vdim above 256 is not supported");
+      if (c.kv_from >= 0) {
+        NEED(c.kv_from < i, "kv_from must name an earlier layer");
+        const femto_layer_config& o = cfg.h_layers[c.kv_from];
+        NEED(o.mixer == FEMTO_MIXER_ATTENTION && o.kv_from < 0, "kv_from must name an attention layer with keys and values of its own");
+        NEED(o.kv_heads == c.kv_heads && o.dim == c.dim && o.vdim == c.vdim && o.maps == c.maps, "differs in its key or value sizes from the layer named by kv_from");
+      }
+      break;
     default: return femto_fail(FEMTO_ERR_ARG, "layer %d: unknown mixer %d", i, c.mixer);
   }
 #undef NEED
@@ -44,6 +58,7 @@ int decoder_fill(DecoderStack* d, const femto_decoder_config* cfg) {
   if (cfg->vocab <= 0 || cfg->width <= 0 || cfg->n_layer <= 0) return femto_fail(FEMTO_ERR_ARG, "vocab, width and n_layer must be positive");
   if (cfg->compute_dtype != FEMTO_F32 && cfg->compute_dtype != FEMTO_BF16) return femto_fail(FEMTO_ERR_ARG, "compute_dtype must be FEMTO_F32 or FEMTO_BF16");
   if (cfg->index_base != 0 && cfg->index_base != 1) return femto_fail(FEMTO_ERR_ARG, "index_base must be 0 or 1");
+  if (cfg->block != FEMTO_BLOCK_SANDWICH && cfg->block != FEMTO_BLOCK_PARALLEL) return femto_fail(FEMTO_ERR_ARG, "unknown block %d", cfg->block);
   d->cfg = *cfg;
   d->layer_cfg.assign(cfg->h_layers, cfg->h_layers + cfg->n_layer);
   d->cfg.h_layers = d->layer_cfg.data();
@@ -60,7 +75,8 @@ int decoder_fill(DecoderStack* d, const femto_decoder_config* cfg) {
     }
     const femto_layer_config &a = l.c, &o = d->layer_cfg[l.own];
     if (a.mixer != o.mixer || a.heads != o.heads || a.kv_heads != o.kv_heads || a.dim != o.dim || a.vdim != o.vdim || a.conv != o.conv ||
-        a.q_rank != o.q_rank || a.kv_rank != o.kv_rank || a.rot_dim != o.rot_dim || a.ff != o.ff)
+        a.q_rank != o.q_rank || a.kv_rank != o.kv_rank || a.rot_dim != o.rot_dim || a.ff != o.ff || a.maps != o.maps || a.qkv_bias != o.qkv_bias ||
+        a.qk_norm != o.qk_norm || a.sink != o.sink || a.gate != o.gate || (a.kv_from < 0) != (o.kv_from < 0) || a.diff != o.diff || a.experts != o.experts)
       return femto_fail(FEMTO_ERR_SHAPE, "layer %d differs in its sizes from layer %d, whose weights it uses", i, l.own);
     l.c.decay_rank = o.decay_rank; l.c.gate_rank = o.gate_rank;
     if (a.mixer == FEMTO_MIXER_LIGHTNING) l.decay.assign(a.h_decay, a.h_decay + a.heads);
@@ -81,17 +97,19 @@ int decoder_fill(DecoderStack* d, const femto_decoder_config* cfg) {
     return t.offset;
   };
   const long long w = cfg->width;
+  const bool sandwich = cfg->block == FEMTO_BLOCK_SANDWICH;
   d->off_embed = take("embed", cfg->vocab, w);
   for (int i = 0; i < cfg->n_layer; i++) {
     DecLayer& l = d->layers[i];
     const femto_layer_config& c = l.c;
     const long long H = c.heads, D = c.dim, E = c.vdim, G = c.kv_heads;
     auto seg = [&](long long n) { const int at = l.n_in; l.n_in += round_up((int)n, 8); return at; };
-    l.ffp = round_up(c.ff, 32);
+    l.ffp = round_up(c.ff, c.experts ? 8 : 32);
     const std::string p = "l" + std::to_string(i) + ".", x = p + "mix.";
     const bool mine = l.own == i;
     auto put = [&](const std::string& name, long long rows, long long cols) { return mine ? take(name, rows, cols) : -1LL; };
-    l.norm1 = put(p + "norm1", w, 0); l.norm1b = put(p + "norm1b", w, 0);
+    l.norm1 = put(p + "norm1", w, 0);
+    if (sandwich) l.norm1b = put(p + "norm1b", w, 0);
     if (c.mixer == FEMTO_MIXER_LIGHTNING) {
       l.s_q = seg(H * D); l.s_k = seg(H * D); l.s_v = seg(H * E); l.s_g = seg(H * E);
       put(x + "q", H * D, w); put(x + "k", H * D, w); put(x + "v", H * E, w); put(x + "g", H * E, w);
@@ -104,6 +122,25 @@ int decoder_fill(DecoderStack* d, const femto_decoder_config* cfg) {
       put(x + "a2", H * D, c.decay_rank); put(x + "g2", H * E, c.gate_rank);
       l.conv_q = put(x + "q.conv", G * D, c.conv); l.conv_k = put(x + "k.conv", G * D, c.conv); l.conv_v = put(x + "v.conv", H * E, c.conv);
       l.a_log = put(x + "A_log", H, 0); l.dt_bias = put(x + "dt_bias", H * D, 0); l.mix_norm = put(x + "norm", E, 0);
+    } else if (c.mixer == FEMTO_MIXER_ATTENTION) {
+      // q and the gate are columns of proj; keys and values go from the same product straight to the cache
+      const long long M = c.maps;
+      const bool own_kv = c.kv_from < 0;
+      l.s_q = seg(H * M * D);
+      if (c.gate != FEMTO_GATE_NONE) l.s_g = seg(c.gate == FEMTO_GATE_HEAD ? H : H * E);
+      l.vo = round_up((int)(G * M * D), 8);
+      l.n_kv = l.vo + round_up((int)(G * E), 8);
+      l.kv_layer = own_kv ? i : c.kv_from;
+      put(x + "q", H * M * D, w);
+      if (own_kv) { put(x + "k", G * M * D, w); put(x + "v", G * E, w); }
+      if (c.qkv_bias) {
+        l.q_bias = put(x + "q.b", H * M * D, 0);
+        if (own_kv) { l.k_bias = put(x + "k.b", G * M * D, 0); l.v_bias = put(x + "v.b", G * E, 0); }
+      }
+      if (c.qk_norm) { l.q_norm = put(x + "q.norm", D, 0); if (own_kv) l.k_norm = put(x + "k.norm", D, 0); }
+      if (M == 2) { l.lq1 = put(x + "lq1", D, 0); l.lk1 = put(x + "lk1", D, 0); l.lq2 = put(x + "lq2", D, 0); l.lk2 = put(x + "lk2", D, 0); }
+      if (c.sink) l.sink = put(x + "sink", H, 0);
+      if (c.gate != FEMTO_GATE_NONE) put(x + "g", c.gate == FEMTO_GATE_HEAD ? H : H * E, w);
     } else {
       l.qp = round_up(c.q_rank, 8); l.dp = round_up(c.dim, 8); l.lp = round_up(c.kv_rank, 8); l.ld = round_up(l.lp + c.rot_dim, 8);
       l.s_q = seg(c.q_rank); l.s_dkv = seg(c.kv_rank + c.rot_dim); l.s_g = seg(H);
@@ -113,15 +150,28 @@ int decoder_fill(DecoderStack* d, const femto_decoder_config* cfg) {
     }
     put(x + "o", w, H * E);
     if (c.ff > 0) {
-      l.norm2 = put(p + "norm2", w, 0); l.norm2b = put(p + "norm2b", w, 0);
-      put(p + "mlp.gate", c.ff, w); put(p + "mlp.up", c.ff, w); put(p + "mlp.down", w, c.ff);
+      l.norm2 = put(p + "norm2", w, 0);
+      if (sandwich) l.norm2b = put(p + "norm2b", w, 0);
+      if (c.experts) {
+        put(p + "mlp.router", c.experts, w);
+        l.router_bias = put(p + "mlp.router.b", c.experts, 0);
+        for (int e = 0; e < c.experts; e++) {
+          const std::string x2 = p + "mlp.e" + std::to_string(e);
+          put(x2 + ".up", c.ff, w); put(x2 + ".down", w, c.ff);
+        }
+      } else {
+        put(p + "mlp.gate", c.ff, w); put(p + "mlp.up", c.ff, w); put(p + "mlp.down", w, c.ff);
+      }
     }
   }
   for (auto& l : d->layers) {
     const DecLayer& o = d->layers[l.own];
     l.norm1 = o.norm1; l.norm1b = o.norm1b; l.norm2 = o.norm2; l.norm2b = o.norm2b; l.mix_norm = o.mix_norm; l.conv_q = o.conv_q;
     l.conv_k = o.conv_k; l.conv_v = o.conv_v; l.a_log = o.a_log; l.dt_bias = o.dt_bias; l.dq_norm = o.dq_norm; l.dkv_norm = o.dkv_norm;
+    l.q_norm = o.q_norm; l.k_norm = o.k_norm; l.sink = o.sink; l.q_bias = o.q_bias; l.k_bias = o.k_bias; l.v_bias = o.v_bias;
+    l.lq1 = o.lq1; l.lk1 = o.lk1; l.lq2 = o.lq2; l.lk2 = o.lk2; l.router_bias = o.router_bias;
   }
+  if (cfg->untied) take("head", cfg->vocab, w);
   d->off_final = take("final.norm", w, 0);
   d->nparams = pos;
   return 0;
@@ -143,6 +193,10 @@ void carve(DecoderStack* d, Carver& b) {
   const size_t es = d->bf ? 2 : 4, R = d->cfg.max_rows, w = d->cfg.width;
   b.take(d->status, 256);
   b.take(d->embed, es * d->cfg.vocab * w);
+  d->head = d->embed;
+  if (d->cfg.untied) b.take(d->head, es * d->cfg.vocab * w);
+  size_t moe_pairs = 0, experts = 0, slots_w = 0, slots_ff = 0, runs = 0;
+  bool dense = false;
   size_t n_in = 0, mix = 0, ff = 0, qk = 0, hd = 0, heads = 0, g2 = 0, cq = 0, q = 0, qa = 0, vv = 0;
   for (size_t i = 0; i < d->layers.size(); i++) {
     DecLayer& l = d->layers[i];
@@ -155,20 +209,42 @@ void carve(DecoderStack* d, Carver& b) {
     if (c.mixer == FEMTO_MIXER_LATENT_ATTENTION) {
       cq = std::max(cq, (size_t)l.qp); q = std::max(q, H * (D + c.rot_dim)); qa = std::max(qa, H * l.ld);
     }
+    if (c.ff > 0 && !c.experts) dense = true;
+    if (c.experts) {
+      for (const int gr : {128, 256}) {
+        const size_t slots = moe_max_slots(R, c.experts, c.top, gr);
+        slots_w = std::max(slots_w, slots); slots_ff = std::max(slots_ff, slots * l.ffp); runs = std::max(runs, slots / gr);
+      }
+      moe_pairs = std::max(moe_pairs, R * c.top); experts = std::max(experts, (size_t)c.experts);
+    }
     b.take(l.decay_dev, 4 * H);
     b.take(l.freq_dev, 4 * l.freq.size() + 4);
     if (l.own != (int)i) continue;
-    b.take(l.w_in, es * l.n_in * w); b.take(l.w_o, es * w * H * E);
+    const bool own_kv = c.mixer == FEMTO_MIXER_ATTENTION && c.kv_from < 0;
+    b.take(l.w_in, es * (l.n_in + (own_kv ? l.n_kv : 0)) * w); b.take(l.w_o, es * w * H * E);
+    if (c.mixer == FEMTO_MIXER_ATTENTION) {
+      if (c.qkv_bias) b.take(l.bias, 4 * (size_t)(l.n_in + l.n_kv));
+      b.take(l.lambda, 4);
+    }
     if (c.mixer == FEMTO_MIXER_CHANNEL_DELTA) { b.take(l.w_a2, es * H * D * l.ra); b.take(l.w_g2, es * H * E * l.rg); }
     if (c.mixer == FEMTO_MIXER_LATENT_ATTENTION) { b.take(l.w_uq, es * H * (D + c.rot_dim) * l.qp); b.take(l.w_kv, es * H * (D + E) * l.lp); b.take(l.w_ukt, es * H * l.lp * l.dp); }
-    if (c.ff > 0) { b.take(l.w_gu, es * 2 * l.ffp * w); b.take(l.w_down, es * w * l.ffp); }
+    if (c.experts) {
+      b.take(l.w_router, es * c.experts * w); b.take(l.w_gu, es * c.experts * l.ffp * w); b.take(l.w_down, es * c.experts * w * l.ffp);
+    } else if (c.ff > 0) { b.take(l.w_gu, es * 2 * l.ffp * w); b.take(l.w_down, es * w * l.ffp); }
   }
   for (auto& l : d->layers) {
     const DecLayer& o = d->layers[l.own];
     l.w_in = o.w_in; l.w_o = o.w_o; l.w_a2 = o.w_a2; l.w_g2 = o.w_g2; l.w_uq = o.w_uq; l.w_kv = o.w_kv; l.w_ukt = o.w_ukt; l.w_gu = o.w_gu; l.w_down = o.w_down;
+    l.w_router = o.w_router; l.bias = o.bias; l.lambda = o.lambda;
   }
   b.take(d->tok0, 4 * R); b.take(d->want, 4 * R);
   b.take(d->x, 4 * R * w); b.take(d->hn, es * R * w); b.take(d->y, es * R * w);
+  if (d->cfg.block == FEMTO_BLOCK_PARALLEL) { b.take(d->hn2, es * R * w); if (dense) b.take(d->y2, es * R * w); }
+  b.take(d->moe_z, 4 * R * round_up((int)experts, 4)); b.take(d->moe_weight, 4 * moe_pairs); b.take(d->moe_expert, 4 * moe_pairs);
+  b.take(d->moe_slot, 4 * moe_pairs); b.take(d->moe_counts, 4 * experts); b.take(d->moe_groups, 4 * (runs + 1));
+  const size_t few_pairs = experts ? (size_t)ROWS_STREAM * 32 : 0;
+  b.take(d->moe_lists, 4 * (1 + 4 * few_pairs));
+  b.take(d->moe_x, es * slots_w * w); b.take(d->moe_act, es * slots_ff); b.take(d->moe_out, es * slots_w * w);
   b.take(d->proj, es * R * n_in); b.take(d->mixo, es * R * mix); b.take(d->mixg, es * R * mix);
   b.take(d->gu, es * R * 2 * ff); b.take(d->act, es * R * ff);
   b.take(d->qn, 4 * R * qk); b.take(d->kn, 4 * R * qk); b.take(d->gd, 4 * R * hd); b.take(d->beta, 4 * R * heads);
@@ -243,12 +319,25 @@ template <typename T> static int refresh_t(DecoderStack* d, const float* theta, 
   };
   const int all = 1 << 30;
   FEMTO_TRY(pack("embed", d->embed, w, 0, all, 0));
+  if (d->cfg.untied) FEMTO_TRY(pack("head", d->head, w, 0, all, 0));
   for (size_t i = 0; i < d->layers.size(); i++) {
     DecLayer& l = d->layers[i];
     if (l.own != (int)i) continue;
     const femto_layer_config& c = l.c;
     const std::string p = "l" + std::to_string(i) + ".", x = p + "mix.";
-    if (c.mixer == FEMTO_MIXER_LATENT_ATTENTION) {
+    if (c.mixer == FEMTO_MIXER_ATTENTION) {
+      FEMTO_TRY(pack(x + "q", l.w_in, w, l.s_q, all, 0));
+      if (c.gate != FEMTO_GATE_NONE) FEMTO_TRY(pack(x + "g", l.w_in, w, l.s_g, all, 0));
+      if (c.kv_from < 0) { FEMTO_TRY(pack(x + "k", l.w_in, w, l.n_in, all, 0)); FEMTO_TRY(pack(x + "v", l.w_in, w, l.n_in + l.vo, all, 0)); }
+      if (c.qkv_bias) {
+        auto put_bias = [&](long long off, int at, int n) {
+          return cudaMemcpyAsync(l.bias + at, theta + off, 4 * (size_t)n, cudaMemcpyDeviceToDevice, s);
+        };
+        CUDA_TRY(put_bias(l.q_bias, l.s_q, c.heads * c.maps * c.dim));
+        if (c.kv_from < 0) { CUDA_TRY(put_bias(l.k_bias, l.n_in, c.kv_heads * c.maps * c.dim)); CUDA_TRY(put_bias(l.v_bias, l.n_in + l.vo, c.kv_heads * c.vdim)); }
+      }
+      if (c.maps == 2) FEMTO_TRY(diff_lambda(theta + l.lq1, theta + l.lk1, theta + l.lq2, theta + l.lk2, c.dim, c.diff, l.lambda, s));
+    } else if (c.mixer == FEMTO_MIXER_LATENT_ATTENTION) {
       FEMTO_TRY(pack(x + "dq", l.w_in, w, l.s_q, all, 0)); FEMTO_TRY(pack(x + "dkv", l.w_in, w, l.s_dkv, all, 0));
       FEMTO_TRY(pack(x + "g", l.w_in, w, l.s_g, all, 0));
       FEMTO_TRY(pack(x + "uq", l.w_uq, l.qp, 0, all, 0));
@@ -266,7 +355,13 @@ template <typename T> static int refresh_t(DecoderStack* d, const float* theta, 
       }
     }
     FEMTO_TRY(pack(x + "o", l.w_o, c.heads * c.vdim, 0, all, 0));
-    if (c.ff > 0) {   // groups of 32 gate rows and 32 up rows alternate, so that one epilogue sees both of a column
+    if (c.experts) {
+      FEMTO_TRY(pack(p + "mlp.router", l.w_router, w, 0, all, 0));
+      for (int e = 0; e < c.experts; e++) {
+        const std::string x2 = p + "mlp.e" + std::to_string(e);
+        FEMTO_TRY(pack(x2 + ".up", l.w_gu, w, e * l.ffp, all, 0)); FEMTO_TRY(pack(x2 + ".down", l.w_down, l.ffp, e * w, all, 0));
+      }
+    } else if (c.ff > 0) {   // groups of 32 gate rows and 32 up rows alternate, so that one epilogue sees both of a column
       FEMTO_TRY(pack(p + "mlp.gate", l.w_gu, w, 0, 32, 64)); FEMTO_TRY(pack(p + "mlp.up", l.w_gu, w, 32, 32, 64));
       FEMTO_TRY(pack(p + "mlp.down", l.w_down, l.ffp, 0, all, 0));
     }
@@ -289,6 +384,7 @@ int decoder_cache_create(femto_handle* h, int max_batch, int max_len, femto_kv_c
   size_t exp_bytes = 0;
   for (auto& l : d->layers) {
     const femto_layer_config& q = l.c;
+    if (q.mixer == FEMTO_MIXER_ATTENTION) c->part_floats = std::max(c->part_floats, window_attention_part_floats(max_batch, q.heads, q.maps, q.vdim));
     if (q.mixer != FEMTO_MIXER_LATENT_ATTENTION) continue;
     exp_bytes = std::max(exp_bytes, es * B * max_len * (size_t)q.heads * (q.dim + q.vdim));
     c->part_floats = std::max(c->part_floats, (size_t)std::max(128, max_batch * LATENT_FEW) * q.heads * (size_t)(l.lp + 2) * 2);
@@ -298,7 +394,10 @@ int decoder_cache_create(femto_handle* h, int max_batch, int max_len, femto_kv_c
       const DecLayer& l = d->layers[i];
       const femto_layer_config& q = l.c;
       LayerState& s = c->state[i];
-      if (q.mixer != FEMTO_MIXER_LATENT_ATTENTION) { s.S_bytes = 4 * B * q.heads * q.dim * q.vdim; b.take(s.S, s.S_bytes); }
+      if (q.mixer == FEMTO_MIXER_ATTENTION) {
+        s.ld = l.n_kv;
+        if (q.kv_from < 0) b.take(s.kv, es * B * max_len * l.n_kv);
+      } else if (q.mixer != FEMTO_MIXER_LATENT_ATTENTION) { s.S_bytes = 4 * B * q.heads * q.dim * q.vdim; b.take(s.S, s.S_bytes); }
       if (q.mixer == FEMTO_MIXER_CHANNEL_DELTA) {
         s.tail_bytes = es * B * (q.conv - 1) * (2 * (size_t)q.kv_heads * q.dim + (size_t)q.heads * q.vdim);
         b.take(s.tail[0], s.tail_bytes); b.take(s.tail[1], s.tail_bytes);
@@ -345,8 +444,25 @@ static int mixer_t(DecoderStack* d, femto_kv_cache* c, int i, const float* theta
   const int R = B * Tn, w = d->cfg.width, H = q.heads, D = q.dim, E = q.vdim;
   const float eps = d->cfg.norm_eps;
   T* proj = (T*)d->proj;
-  FEMTO_TRY(rows_linear<T>(d, d->hn, w, l.w_in, w, proj, l.n_in, R, l.n_in, w, EPI_STORE, s));
   T* out = (T*)d->mixg;
+  if (q.mixer == FEMTO_MIXER_ATTENTION) {
+    const LayerState& src = c->state[l.kv_layer];
+    const bool own_kv = l.kv_layer == i;
+    RowsOut ro;
+    ro.bias = l.bias;
+    if (own_kv) { ro.n2 = l.n_in; ro.T2 = Tn; ro.C2 = (T*)src.kv + (long long)first * src.ld; ro.ld2 = src.ld; ro.stride2 = (long long)c->maxT * src.ld; }
+    FEMTO_TRY(rows_linear<T>(d, d->hn, w, l.w_in, w, proj, l.n_in, R, l.n_in + (own_kv ? l.n_kv : 0), w, EPI_STORE, s, ro));
+    WindowAttnArgs a;
+    a.q = proj + l.s_q; a.ldq = l.n_in; a.kv = src.kv; a.ld = src.ld; a.vo = l.vo; a.maxT = c->maxT;
+    a.gate = proj + l.s_g; a.ld_gate = l.n_in; a.gate_mode = q.gate; a.o = out;
+    a.B = B; a.T = Tn; a.first = first; a.heads = H; a.kv_heads = q.kv_heads; a.dim = D; a.vdim = E; a.maps = q.maps; a.window = q.window; a.keep = q.keep_first;
+    a.scale = q.scale; a.eps = eps; a.out_scale = 1.f - q.diff; a.sink = q.sink ? theta + l.sink : nullptr; a.lambda = l.lambda;
+    a.part = c->part; a.part_floats = c->part_floats; a.status = d->status;
+    if (q.qk_norm) FEMTO_TRY(qk_norm<T>(a, theta + l.q_norm, own_kv ? theta + l.k_norm : nullptr, own_kv, s));
+    FEMTO_TRY(window_attention<T>(a, s));
+    return rows_linear<T>(d, out, H * E, l.w_o, H * E, d->y, w, R, w, H * E, EPI_STORE, s);
+  }
+  FEMTO_TRY(rows_linear<T>(d, d->hn, w, l.w_in, w, proj, l.n_in, R, l.n_in, w, EPI_STORE, s));
   if (q.mixer == FEMTO_MIXER_LIGHTNING) {
     ChunkArgs ca;
     ca.proj = proj; ca.ldp = l.n_in; ca.s_q = l.s_q; ca.s_k = l.s_k; ca.s_v = l.s_v; ca.decay = l.decay_dev; ca.S = st.S; ca.o = d->mixo;
@@ -403,6 +519,48 @@ static int mixer_t(DecoderStack* d, femto_kv_cache* c, int i, const float* theta
   return rows_linear<T>(d, out, H * E, l.w_o, H * E, d->y, w, R, w, H * E, EPI_STORE, s);
 }
 
+// The feed-forward of R rows h: one row each in y, or, with experts, the rows that MoeRows names.
+template <typename T>
+static int feed_forward(DecoderStack* d, const DecLayer& l, const float* theta, const void* h, void* y, int R, MoeRows& mr, cudaStream_t s) {
+  const int w = d->cfg.width;
+  const femto_layer_config& q = l.c;
+  if (!q.experts) {
+    FEMTO_TRY(rows_linear<T>(d, h, w, l.w_gu, w, d->act, l.ffp, R, l.ffp, w, EPI_SWIGLU, s));
+    return rows_linear<T>(d, d->act, l.ffp, l.w_down, l.ffp, y, w, R, w, l.ffp, EPI_STORE, s);
+  }
+  MoeArgs a;
+  a.ldz = round_up(q.experts, 4);
+  FEMTO_TRY(rows_linear<T>(d, h, w, l.w_router, w, d->moe_z, a.ldz, R, q.experts, w, EPI_F32, s));
+  a.z = d->moe_z; a.bias = theta + l.router_bias; a.rows = R; a.experts = q.experts; a.top = q.top; a.width = w;
+  a.h = h; a.weight = d->moe_weight; a.expert = d->moe_expert; a.slot = d->moe_slot; a.counts = d->moe_counts; a.groups = d->moe_groups;
+  a.lists = d->moe_lists; a.xs = d->moe_x;
+  mr.out = d->moe_out; mr.weight = d->moe_weight; mr.top = q.top;
+  if constexpr (sizeof(T) == 2) {
+    if (R <= ROWS_STREAM && (w & 7) == 0) {
+      a.max_lists = std::min(q.experts, R * q.top);
+      FEMTO_TRY(moe_choose_few(a, s));
+      RowsBatch bt;
+      bt.lists = d->moe_lists; bt.max_lists = a.max_lists; bt.x_div = q.top; bt.w = (long long)l.ffp * w;
+      FEMTO_TRY(rows_stream((const bf16*)h, w, (const bf16*)l.w_gu, w, d->moe_act, l.ffp, R, l.ffp, w, EPI_RELU2, a.max_lists, bt, s));
+      bt.x_div = 1;
+      FEMTO_TRY(rows_stream((const bf16*)d->moe_act, l.ffp, (const bf16*)l.w_down, l.ffp, d->moe_out, w, R, w, l.ffp, EPI_STORE, a.max_lists, bt, s));
+      return 0;
+    }
+  }
+  a.group_rows = moe_group_rows(R, q.experts, q.top);
+  FEMTO_TRY(moe_sort<T>(a, s));
+  mr.slot = d->moe_slot;
+  GemmArgs g;
+  g.ws = d->gemm_ws; g.ws_bytes = d->gemm_ws_bytes; g.status = d->status; g.any_size = true;
+  g.groups = d->moe_groups; g.group_rows = a.group_rows; g.n_groups = q.experts;
+  g.M = (int)moe_max_slots(R, q.experts, q.top, a.group_rows);
+  g.A = d->moe_x; g.lda = w; g.B = l.w_gu; g.ldb = w; g.strideB = (long long)l.ffp * w; g.C = d->moe_act; g.ldc = l.ffp;
+  g.N = l.ffp; g.K = w; g.epi = EPI_RELU2;
+  FEMTO_TRY(gemm<T>(g, s));
+  g.A = d->moe_act; g.lda = l.ffp; g.B = l.w_down; g.ldb = l.ffp; g.C = d->moe_out; g.ldc = w; g.N = w; g.K = l.ffp; g.epi = EPI_STORE;
+  return gemm<T>(g, s);
+}
+
 // Tokens [t0, t0 + Tn) of every column.
 template <typename T>
 static int pass_t(DecoderStack* d, femto_kv_cache* c, const float* theta, const int* tokens, int ld_tok, int B, int Tn, float* residuals,
@@ -410,18 +568,33 @@ static int pass_t(DecoderStack* d, femto_kv_cache* c, const float* theta, const 
   typedef DecStream<T> S;
   const int R = B * Tn, w = d->cfg.width, L = d->cfg.n_layer;
   const float eps = d->cfg.norm_eps, m = d->cfg.residual_mult;
-  FEMTO_TRY(S::embed((const T*)d->embed, tokens, ld_tok, B, Tn, d->cfg.index_base, d->cfg.vocab, theta + d->layers[0].norm1, d->x, (T*)d->hn,
-                     w, eps, d->status, s));
+  const bool parallel = d->cfg.block == FEMTO_BLOCK_PARALLEL;
+  // what follows layer i - 1: the norms of layer i, none after the last
+  auto norms_of = [&](int i) {
+    NextNorms<T> n;
+    if (i == L) return n;
+    n.w = theta + d->layers[i].norm1; n.h = (T*)d->hn;
+    if (parallel && d->layers[i].c.ff > 0) { n.w2 = theta + d->layers[i].norm2; n.h2 = (T*)d->hn2; }
+    return n;
+  };
+  FEMTO_TRY(S::embed((const T*)d->embed, tokens, ld_tok, B, Tn, d->cfg.index_base, d->cfg.vocab, d->cfg.embed_scale, d->x, norms_of(0), w, eps,
+                     d->status, s));
   for (int i = 0; i < L; i++) {
     const DecLayer& l = d->layers[i];
-    FEMTO_TRY(mixer_t<T>(d, c, i, theta, B, Tn, c->len, s));
-    const float* next = i + 1 < L ? theta + d->layers[i + 1].norm1 : nullptr;
     const bool mlp = l.c.ff > 0;
-    FEMTO_TRY(S::resid_norm(d->x, (const T*)d->y, theta + l.norm1b, m, mlp ? theta + l.norm2 : next, mlp || next ? (T*)d->hn : nullptr, R, w, eps, s));
-    if (mlp) {
-      FEMTO_TRY(rows_linear<T>(d, d->hn, w, l.w_gu, w, d->act, l.ffp, R, l.ffp, w, EPI_SWIGLU, s));
-      FEMTO_TRY(rows_linear<T>(d, d->act, l.ffp, l.w_down, l.ffp, d->y, w, R, w, l.ffp, EPI_STORE, s));
-      FEMTO_TRY(S::resid_norm(d->x, (const T*)d->y, theta + l.norm2b, m, next, next ? (T*)d->hn : nullptr, R, w, eps, s));
+    const NextNorms<T> next = norms_of(i + 1);
+    MoeRows mr;
+    FEMTO_TRY(mixer_t<T>(d, c, i, theta, B, Tn, c->len, s));
+    if (parallel) {
+      if (mlp) FEMTO_TRY(feed_forward<T>(d, l, theta, d->hn2, d->y2, R, mr, s));
+      FEMTO_TRY(S::parallel_resid(d->x, (const T*)d->y, mlp && !l.c.experts ? (const T*)d->y2 : nullptr, mr, next, R, w, eps, s));
+    } else {
+      FEMTO_TRY(S::resid_norm(d->x, (const T*)d->y, theta + l.norm1b, m, mlp ? theta + l.norm2 : next.w, mlp || next.h ? (T*)d->hn : nullptr, R, w, eps, s));
+      if (mlp) {
+        FEMTO_TRY(feed_forward<T>(d, l, theta, d->hn, d->y, R, mr, s));
+        if (l.c.experts) FEMTO_TRY(moe_combine<T>(mr, (T*)d->y, R, w, s));
+        FEMTO_TRY(S::resid_norm(d->x, (const T*)d->y, theta + l.norm2b, m, next.w, next.h, R, w, eps, s));
+      }
     }
     if (residuals) CUDA_TRY(cudaMemcpyAsync(residuals + (size_t)i * R * w, d->x, 4 * (size_t)R * w, cudaMemcpyDeviceToDevice, s));
   }
@@ -433,7 +606,9 @@ template <typename T>
 static int logits_t(DecoderStack* d, const float* theta, const int* want, int stride, int n, float* out, cudaStream_t s) {
   const int w = d->cfg.width;
   FEMTO_TRY(DecStream<T>::gather_norm(d->x, want, stride, theta + d->off_final, (T*)d->hn, n, w, d->cfg.norm_eps, s));
-  return rows_linear<T>(d, d->hn, w, d->embed, w, out, d->cfg.vocab, n, d->cfg.vocab, w, EPI_F32, s);
+  RowsOut ro;
+  ro.softcap = d->cfg.logit_softcap;
+  return rows_linear<T>(d, d->hn, w, d->head, w, out, d->cfg.vocab, n, d->cfg.vocab, w, EPI_F32, s, ro);
 }
 
 int decoder_step(femto_handle* h, femto_kv_cache* c, const float* theta, const int* tokens, int B, int T, const int* h_want, int n_want,

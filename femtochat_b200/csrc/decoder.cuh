@@ -19,15 +19,19 @@ struct DecLayer {
   float* freq_dev = nullptr;
   // element offsets into Theta of what is read there in fp32
   long long norm1 = -1, norm1b = -1, norm2 = -1, norm2b = -1, mix_norm = -1, conv_q = -1, conv_k = -1, conv_v = -1,
-            a_log = -1, dt_bias = -1, dq_norm = -1, dkv_norm = -1;
+            a_log = -1, dt_bias = -1, dq_norm = -1, dkv_norm = -1, q_norm = -1, k_norm = -1, sink = -1, q_bias = -1, k_bias = -1, v_bias = -1,
+            lq1 = -1, lk1 = -1, lq2 = -1, lk2 = -1, router_bias = -1;
   // packed compute-type weights, row-major [out][in]
   void *w_in = nullptr, *w_o = nullptr, *w_a2 = nullptr, *w_g2 = nullptr, *w_uq = nullptr, *w_kv = nullptr, *w_ukt = nullptr, *w_gu = nullptr,
-       *w_down = nullptr;
+       *w_down = nullptr, *w_router = nullptr;      // experts: w_gu [experts][ffp][width] (up), w_down [experts][width][ffp]
   int n_in = 0;                       // columns of proj
+  int n_kv = 0, vo = 0;               // attention: columns of a cached row, which follow those of proj in w_in; where the values start
+  int kv_layer = 0;                   // attention: layer whose cache holds the keys and values
+  float *bias = nullptr, *lambda = nullptr;   // attention: [n_in + n_kv]; one number
   int s_q = 0, s_k = 0, s_v = 0, s_g = 0, s_b = 0, s_a1 = 0, s_g1 = 0, s_dkv = 0;   // segment starts
   int ra = 0, rg = 0;                 // decay_rank / gate_rank rounded up to 8
   int qp = 0, lp = 0, ld = 0, dp = 0; // q_rank, kv_rank rounded up to 8; pitch of a cached latent row; dim rounded up to 8
-  int ffp = 0;                        // ff rounded up to 32: the feed-forward's products are this wide
+  int ffp = 0;                        // ff rounded up to 32 (experts: to 8): the feed-forward's products are this wide
   int qk_heads() const { return c.mixer == FEMTO_MIXER_CHANNEL_DELTA ? c.kv_heads : c.heads; }
 };
 
@@ -40,16 +44,21 @@ struct DecoderStack {
   bool bf = false, weights_valid = false;
   char* arena = nullptr;
   unsigned int* status = nullptr;
-  void* embed = nullptr;              // [vocab][width] compute type: input table and output head
+  void* embed = nullptr;              // [vocab][width] compute type: input table
+  void* head = nullptr;               // output head (the same table when tied)
   // workspace of one internal pass of up to max_rows tokens
   int* tok0 = nullptr;
   int* want = nullptr;                // [max_rows]
   float* x = nullptr;                 // residual stream, fp32
-  void *hn = nullptr, *y = nullptr, *proj = nullptr, *mixo = nullptr, *mixg = nullptr, *gu = nullptr, *act = nullptr;
+  void *hn = nullptr, *hn2 = nullptr, *y = nullptr, *y2 = nullptr, *proj = nullptr, *mixo = nullptr, *mixg = nullptr, *gu = nullptr, *act = nullptr;
   float *qn = nullptr, *kn = nullptr, *gd = nullptr, *beta = nullptr;
   void *vv = nullptr, *g2 = nullptr, *cq = nullptr, *q = nullptr;
   float* qabs = nullptr;              // latent attention, few rows: queries in the latent space
   void* oc = nullptr;                 // and results there
+  // experts: router logits, choices, places, counts, runs, lists of a few rows' choices; sorted inputs and results
+  float *moe_z = nullptr, *moe_weight = nullptr;
+  int *moe_expert = nullptr, *moe_slot = nullptr, *moe_counts = nullptr, *moe_groups = nullptr, *moe_lists = nullptr;
+  void *moe_x = nullptr, *moe_act = nullptr, *moe_out = nullptr;
   char* chunk_ws = nullptr;           // chunked recurrences: operands of the chunks of one segment
   size_t chunk_ws_bytes = 0;
   void* gemm_ws = nullptr;
@@ -66,10 +75,22 @@ int decoder_cache_create(femto_handle* h, int max_batch, int max_len, femto_kv_c
 int decoder_cache_reset(femto_kv_cache* c, cudaStream_t s);
 
 // ---- streaming kernels (decoder_stream.cu) ------------------------------------------------------------------------
+// What the experts made of a row: out[slot ? slot[p] : p] for the pairs p = row * top + k, with their weights.
+struct MoeRows {
+  const void* out = nullptr;
+  const int* slot = nullptr;
+  const float* weight = nullptr;
+  int top = 0;
+};
+// The norms that follow a sum: h = rms_norm(x) w and, with h2, h2 = rms_norm(x) w2 (h may be NULL: none)
+template <typename T> struct NextNorms { const float* w = nullptr; T* h = nullptr; const float* w2 = nullptr; T* h2 = nullptr; };
 template <typename T> struct DecStream {
-  // x = table[token] (fp32), h = rms_norm(x) w
-  static int embed(const T* table, const int* tokens, int ld_tok, int B, int T_, int base, int vocab, const float* w, float* x,
-                   T* h, int d, float eps, unsigned int* status, cudaStream_t s);
+  // x = scale * table[token] (fp32), then the norms
+  static int embed(const T* table, const int* tokens, int ld_tok, int B, int T_, int base, int vocab, float scale, float* x,
+                   const NextNorms<T>& n, int d, float eps, unsigned int* status, cudaStream_t s);
+  // x += y + (y2, or the weighted sum of the experts' rows, or nothing), then the norms
+  static int parallel_resid(float* x, const T* y, const T* y2, const MoeRows& m, const NextNorms<T>& n, int rows, int d, float eps,
+                            cudaStream_t s);
   // x += m rms_norm(y) w_post;  h = rms_norm(x) w_pre (skipped when h is NULL)
   static int resid_norm(float* x, const T* y, const float* w_post, float m, const float* w_pre, T* h, int rows, int d, float eps,
                         cudaStream_t s);
@@ -91,9 +112,17 @@ int pack_rows(const float* src, int rows, int cols, T* dst, long long ldd, int d
 // ---- products -------------------------------------------------------------------------------------------------------
 // C[M][N] = X[M][K] W[N][K]^T; epi EPI_STORE (compute type), EPI_F32, or EPI_SWIGLU (W holds 2 N rows, groups of 32 gate and
 // 32 up rows in turn; C = silu(gate) * up).  A few rows stream the weights once, more rows take the tensor-core GEMM.
+struct RowsOut {
+  const float* bias = nullptr;   // [N], added to the sums
+  float softcap = 0.f;           // EPI_F32: cap tanh(c / cap) when not 0
+  // columns n2 and up (0: none) go elsewhere: column n of row m to C2 + (m / T2) * stride2 + (m % T2) * ld2 + n - n2
+  int n2 = 0, T2 = 1;
+  void* C2 = nullptr;
+  long long ld2 = 0, stride2 = 0;
+};
 template <typename T>
 int rows_linear(DecoderStack* d, const void* X, long long ldx, const void* W, long long ldw, void* C, long long ldc, int M, int N, int K,
-                int epi, cudaStream_t s);
+                int epi, cudaStream_t s, const RowsOut& out = RowsOut());
 
 // The streaming kernel by itself (bf16, aligned, at most ROWS_STREAM rows), as a batch over heads: element strides between the
 // heads' operands, and optionally one gate logit per (row, head) whose sigmoid multiplies the result.
@@ -102,6 +131,11 @@ struct RowsBatch {
   long long x = 0, w = 0, c = 0;
   const bf16* gate = nullptr;
   long long ld_gate = 0;
+  RowsOut out;
+  // Experts: the batch are the lists of k_moe_choose_few (lists[0] of them, each expert, start, length); list entry p is row
+  // p / x_div of X and row p of C; EPI_RELU2 squares the positive part of the result.
+  const int* lists = nullptr;
+  int max_lists = 0, x_div = 1;
 };
 int rows_stream(const bf16* X, long long ldx, const bf16* W, long long ldw, void* C, long long ldc, int M, int N, int K, int epi, int batch,
                 const RowsBatch& bt, cudaStream_t s);
@@ -184,7 +218,49 @@ struct LatentArgs {
 };
 template <typename T> int latent_norms(const LatentArgs& a, cudaStream_t s);   // query latent -> cq, new rows -> cache
 template <typename T> int latent_attention(const LatentArgs& a, cudaStream_t s);
-bool latent_attention_tc_supported(const LatentArgs& a);       // latent_attention_sm100.cu: the prompt's attention on the tensor cores
+bool latent_attention_tc_supported(const LatentArgs& a);       // slab_attention_sm100.cu: the prompt's attention on the tensor cores
 int latent_attention_tc(const LatentArgs& a, cudaStream_t s);
+
+// ---- attention over cached keys and values (window_attention.cu; prompts in bf16: slab_attention_sm100.cu) --------------
+struct WindowAttnArgs {
+  const void* q = nullptr; long long ldq = 0;          // [rows][heads][maps][dim]
+  const void* kv = nullptr;      // cache [maxB][maxT][ld]: keys [kv_heads][maps][dim], from column vo on values [kv_heads][vdim]
+  int ld = 0, vo = 0, maxT = 0;
+  const void* gate = nullptr; long long ld_gate = 0; int gate_mode = FEMTO_GATE_NONE;   // [rows][heads] or [rows][heads vdim]
+  void* o = nullptr;             // [rows][heads vdim]
+  int B = 0, T = 0, first = 0, heads = 0, kv_heads = 0, dim = 0, vdim = 0, maps = 1, window = 0, keep = 0;
+  float scale = 1.f, eps = 0.f, out_scale = 1.f;
+  const float* sink = nullptr;   // [heads]
+  const float* lambda = nullptr; // two maps: (a1 - lambda a2) / rms * out_scale
+  float* part = nullptr; size_t part_floats = 0;
+  unsigned int* status = nullptr;
+};
+template <typename T> int qk_norm(const WindowAttnArgs& a, const float* wq, const float* wk, bool with_k, cudaStream_t s);   // in place
+template <typename T> int window_attention(const WindowAttnArgs& a, cudaStream_t s);
+int diff_lambda(const float* lq1, const float* lk1, const float* lq2, const float* lk2, int dim, float diff, float* out, cudaStream_t s);
+size_t window_attention_part_floats(int max_batch, int heads, int maps, int vdim);
+bool window_attention_tc_supported(const WindowAttnArgs& a);
+int window_attention_tc(const WindowAttnArgs& a, cudaStream_t s);
+constexpr int ATTN_FEW = 8;            // columns with at most this many new tokens take the split-key kernels
+
+// ---- mixture of experts (moe.cu) -------------------------------------------------------------------------------------
+struct MoeArgs {
+  const float* z = nullptr; long long ldz = 0;         // router logits [rows][ldz], without the bias
+  const float* bias = nullptr;
+  int rows = 0, experts = 0, top = 0, width = 0, group_rows = 0, max_lists = 0;
+  const void* h = nullptr;       // [rows][width]
+  float* weight = nullptr; int *expert = nullptr, *slot = nullptr;   // [rows * top]
+  int* counts = nullptr;         // [experts]
+  int* groups = nullptr;         // runs of the sorted rows: their number, then the expert of each
+  int* lists = nullptr;          // few rows: number of lists, (expert, start, length) of each, from 1 + 3 max_lists on the pairs
+  void* xs = nullptr;            // sorted inputs
+};
+bool moe_supported(int experts, int top);
+int moe_group_rows(long long rows, int experts, int top);
+long long moe_max_slots(long long rows, int experts, int top, int group_rows);
+template <typename T> int moe_sort(const MoeArgs& a, cudaStream_t s);
+int moe_choose_few(const MoeArgs& a, cudaStream_t s);
+template <typename T> int moe_combine(const MoeRows& m, T* y, int rows, int d, cudaStream_t s);
+
 constexpr int LATENT_FEW = 8;          // columns with at most this many new tokens attend in the latent space
 constexpr int LATENT_MAX_SPLITS = 64;

@@ -1,6 +1,7 @@
 // HBM-streaming kernels of the layer-listing decoders: embedding, norms around each sublayer with the fp32 residual
 // sum, gated norms, the feed-forward's gate, weight packing, and the product of a few rows with a [out][in] weight.
 #include "decoder.cuh"
+#include "streaming.cuh"
 
 namespace {
 
@@ -23,8 +24,8 @@ constexpr int RT = 256;   // threads of a row kernel: one row per block
 
 template <typename T>
 __global__ void __launch_bounds__(RT) k_dec_embed(const T* __restrict__ table, const int* __restrict__ tokens, int ld_tok, int T_,
-                                                  int base, int vocab, const float* __restrict__ w, float* __restrict__ x,
-                                                  T* __restrict__ h, int d, float eps, unsigned int* status) {
+                                                  int base, int vocab, float scale, float* __restrict__ x, const NextNorms<T> nn, int d,
+                                                  float eps, unsigned int* status) {
   pdl_trigger();
   pdl_wait();
   const int row = blockIdx.x;
@@ -32,12 +33,118 @@ __global__ void __launch_bounds__(RT) k_dec_embed(const T* __restrict__ table, c
   if (tk < 0 || tk >= vocab) { if (threadIdx.x == 0) atomicOr(status, ST_BAD_TOKEN); tk = min(max(tk, 0), vocab - 1); }
   const T* src = table + (long long)tk * d;
   float ss = 0.f;
-  for (int c = threadIdx.x; c < d; c += RT) { const float f = to_f<T>(src[c]); ss += f * f; }
+  for (int c = threadIdx.x; c < d; c += RT) { const float f = to_f<T>(src[c]) * scale; ss += f * f; }
   const float inv = 1.f / sqrtf(block_sum(ss) / d + eps);
   for (int c = threadIdx.x; c < d; c += RT) {
-    const float f = to_f<T>(src[c]);
-    x[(long long)row * d + c] = f;
-    h[(long long)row * d + c] = from_f<T>(f * inv * w[c]);
+    const float f = to_f<T>(src[c]) * scale;
+    const long long at = (long long)row * d + c;
+    x[at] = f;
+    nn.h[at] = from_f<T>(f * inv * nn.w[c]);
+    if (nn.h2) nn.h2[at] = from_f<T>(f * inv * nn.w2[c]);
+  }
+}
+
+template <typename T> __device__ __forceinline__ void load4(const T* p, float (&f)[4]) {
+  if constexpr (sizeof(T) == 4) {
+    const float4 q = *reinterpret_cast<const float4*>(p);
+    f[0] = q.x; f[1] = q.y; f[2] = q.z; f[3] = q.w;
+  } else {
+    const uint2 q = *reinterpret_cast<const uint2*>(p);
+    const bf16* h = reinterpret_cast<const bf16*>(&q);
+#pragma unroll
+    for (int e = 0; e < 4; e++) f[e] = __bfloat162float(h[e]);
+  }
+}
+template <typename T> __device__ __forceinline__ void store4(T* p, float a, float b, float c, float d) {
+  if constexpr (sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
+  } else {
+    uint2 q;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&q);
+    h[0] = __floats2bfloat162_rn(a, b); h[1] = __floats2bfloat162_rn(c, d);
+    *reinterpret_cast<uint2*>(p) = q;
+  }
+}
+
+// NV 4-element vectors per thread stay in registers between the sum and the norms (NV = 0: any width, through memory).
+template <typename T, int NV>
+__global__ void __launch_bounds__(RT) k_parallel_resid(float* __restrict__ x, const T* __restrict__ y, const T* __restrict__ y2, const MoeRows m,
+                                                       const NextNorms<T> nn, int d, float eps) {
+  pdl_trigger();
+  pdl_wait();
+  const long long row = blockIdx.x, base = row * d;
+  auto expert_row = [&](int k, float& w) {
+    const long long p = row * m.top + k;
+    w = m.weight[p];
+    return reinterpret_cast<const T*>(m.out) + (m.slot ? m.slot[p] : p) * (long long)d;
+  };
+  float ss = 0.f;
+  if constexpr (NV > 0) {
+    float r[NV][4], f[4];
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+      const int c = (i * RT + threadIdx.x) * 4;
+      if (c >= d) continue;
+      load4<T>(y + base + c, r[i]);
+      if (y2) {
+        load4<T>(y2 + base + c, f);
+#pragma unroll
+        for (int e = 0; e < 4; e++) r[i][e] += f[e];
+      }
+    }
+#pragma unroll 4
+    for (int k = 0; k < m.top; k++) {
+      float w;
+      const T* o = expert_row(k, w);
+#pragma unroll
+      for (int i = 0; i < NV; i++) {
+        const int c = (i * RT + threadIdx.x) * 4;
+        if (c >= d) continue;
+        load4<T>(o + c, f);
+#pragma unroll
+        for (int e = 0; e < 4; e++) r[i][e] = fmaf(w, f[e], r[i][e]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+      const int c = (i * RT + threadIdx.x) * 4;
+      if (c >= d) continue;
+      load4<float>(x + base + c, f);
+#pragma unroll
+      for (int e = 0; e < 4; e++) { r[i][e] += f[e]; ss += r[i][e] * r[i][e]; }
+      store4<float>(x + base + c, r[i][0], r[i][1], r[i][2], r[i][3]);
+    }
+    if (!nn.h) return;
+    const float inv = 1.f / sqrtf(block_sum(ss) / d + eps);
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+      const int c = (i * RT + threadIdx.x) * 4;
+      if (c >= d) continue;
+      load4<float>(nn.w + c, f);
+      store4<T>(nn.h + base + c, r[i][0] * inv * f[0], r[i][1] * inv * f[1], r[i][2] * inv * f[2], r[i][3] * inv * f[3]);
+      if (!nn.h2) continue;
+      load4<float>(nn.w2 + c, f);
+      store4<T>(nn.h2 + base + c, r[i][0] * inv * f[0], r[i][1] * inv * f[1], r[i][2] * inv * f[2], r[i][3] * inv * f[3]);
+    }
+  } else {
+    for (int c = threadIdx.x; c < d; c += RT) {
+      float r = to_f<T>(y[base + c]) + (y2 ? to_f<T>(y2[base + c]) : 0.f);
+      for (int k = 0; k < m.top; k++) {
+        float w;
+        const T* o = expert_row(k, w);
+        r = fmaf(w, to_f<T>(o[c]), r);
+      }
+      r += x[base + c];
+      x[base + c] = r;
+      ss += r * r;
+    }
+    if (!nn.h) return;
+    const float inv = 1.f / sqrtf(block_sum(ss) / d + eps);
+    for (int c = threadIdx.x; c < d; c += RT) {
+      const float r = x[base + c] * inv;
+      nn.h[base + c] = from_f<T>(r * nn.w[c]);
+      if (nn.h2) nn.h2[base + c] = from_f<T>(r * nn.w2[c]);
+    }
   }
 }
 
@@ -212,7 +319,7 @@ __global__ void __launch_bounds__(256) k_pack_transposed(const float* __restrict
 constexpr int RL_ROWS = 8;
 template <typename T, bool GATED>
 __global__ void __launch_bounds__(256) k_rows_linear(const T* __restrict__ X, long long ldx, const T* __restrict__ W, long long ldw,
-                                                     void* __restrict__ C, long long ldc, int M, int N, int K, int f32_out) {
+                                                     void* __restrict__ C, long long ldc, int M, int N, int K, int f32_out, const RowsOut out) {
   pdl_trigger();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -236,7 +343,10 @@ __global__ void __launch_bounds__(256) k_rows_linear(const T* __restrict__ X, lo
     float v = warp_sum(acc[m]);
     if (GATED) v = v * sigmoid_f(v) * warp_sum(up[m]);
     if (lane == 0) {
-      if (f32_out) reinterpret_cast<float*>(C)[m * ldc + n] = v;
+      if (out.bias) v += out.bias[n];
+      if (out.softcap != 0.f) v = out.softcap * tanhf(v / out.softcap);
+      if (out.n2 && n >= out.n2) reinterpret_cast<T*>(out.C2)[(m / out.T2) * out.stride2 + (m % out.T2) * out.ld2 + n - out.n2] = from_f<T>(v);
+      else if (f32_out) reinterpret_cast<float*>(C)[m * ldc + n] = v;
       else reinterpret_cast<T*>(C)[m * ldc + n] = from_f<T>(v);
     }
   }
@@ -246,13 +356,24 @@ __global__ void __launch_bounds__(256) k_rows_linear(const T* __restrict__ X, lo
 // GATED), its eight warps share K.  The weights are the 16-row operand, the rows of X the 8-column operand, so every
 // weight is loaded once, straight into the fragment that uses it: a lane takes 16 consecutive bytes of a row, and since X
 // is read in the same order the permutation of K inside a step does not matter.  The first weights are on their way
-// before the kernel waits for its predecessor.
-template <int NT, bool GATED>
+// before the kernel waits for its predecessor.  LISTS: the rows of a block are one list of k_moe_choose_few, its weights those
+// of the list's expert.
+template <int NT, bool GATED, bool LISTS>
 __global__ void __launch_bounds__(256) k_rows_mma(const bf16* __restrict__ X, long long ldx, const bf16* __restrict__ W, long long ldw,
-                                                  void* __restrict__ C, long long ldc, int M, int N, int K, int f32_out, const RowsBatch bt) {
+                                                  void* __restrict__ C, long long ldc, int M, int N, int K, int epi, const RowsBatch bt) {
   pdl_trigger();
-  X += blockIdx.y * bt.x;
-  W += blockIdx.y * bt.w;
+  const int* list = nullptr;
+  if constexpr (LISTS) {
+    pdl_wait();
+    if ((int)blockIdx.y >= bt.lists[0]) return;
+    const int* g = bt.lists + 1 + 3 * blockIdx.y;
+    W += g[0] * bt.w;
+    list = bt.lists + 1 + 3 * bt.max_lists + g[1];
+    M = g[2];
+  } else {
+    X += blockIdx.y * bt.x;
+    W += blockIdx.y * bt.w;
+  }
   constexpr int RT = GATED ? 2 : 1, U = 4;      // U steps of 256 k are loaded ahead
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c8 = (lane & 3) * 8;
   const int n0 = blockIdx.x * 16;
@@ -272,7 +393,13 @@ __global__ void __launch_bounds__(256) k_rows_mma(const bf16* __restrict__ X, lo
   const int kb = warp * 32 + c8;
 #pragma unroll
   for (int u = 0; u < U; u++) fetch(u, kb + u * 256);
-  pdl_wait();
+  if (!LISTS) pdl_wait();
+  const bf16* xp[NT];          // this lane's rows of X
+#pragma unroll
+  for (int t = 0; t < NT; t++) {
+    const int m = 8 * t + g;
+    xp[t] = X + (m < M ? (LISTS ? list[m] / bt.x_div : m) : 0) * ldx;
+  }
   float acc[RT][NT][4] = {};
   for (int k0 = kb; k0 < K + c8; k0 += U * 256) {       // the four lanes of a row leave together
 #pragma unroll
@@ -280,7 +407,7 @@ __global__ void __launch_bounds__(256) k_rows_mma(const bf16* __restrict__ X, lo
       const int k = k0 + u * 256;
       uint4 x[NT];
 #pragma unroll
-      for (int t = 0; t < NT; t++) x[t] = k < K && 8 * t + g < M ? *reinterpret_cast<const uint4*>(X + (8 * t + g) * ldx + k) : zero;
+      for (int t = 0; t < NT; t++) x[t] = k < K && 8 * t + g < M ? *reinterpret_cast<const uint4*>(xp[t] + k) : zero;
 #pragma unroll
       for (int i = 0; i < RT; i++)
 #pragma unroll
@@ -312,8 +439,17 @@ __global__ void __launch_bounds__(256) k_rows_mma(const bf16* __restrict__ X, lo
     for (int i = 0; i < 8; i++) { v += red[i][0][m][j]; if (GATED) up += red[i][RT - 1][m][j]; }
     if (GATED) v = v * sigmoid_f(v) * up;
     if (bt.gate) v *= sigmoid_f(__bfloat162float(bt.gate[m * bt.ld_gate + blockIdx.y]));
-    const long long at = m * ldc + blockIdx.y * bt.c + n0 + j;
-    if (f32_out) reinterpret_cast<float*>(C)[at] = v;
+    const int n = n0 + j;
+    const RowsOut& out = bt.out;
+    if (out.bias) v += out.bias[n];
+    if (out.softcap != 0.f) v = out.softcap * tanhf(v / out.softcap);
+    if (epi == EPI_RELU2) { v = fmaxf(v, 0.f); v *= v; }
+    if (out.n2 && n >= out.n2) {
+      reinterpret_cast<bf16*>(out.C2)[(m / out.T2) * out.stride2 + (m % out.T2) * out.ld2 + n - out.n2] = __float2bfloat16_rn(v);
+      continue;
+    }
+    const long long at = LISTS ? list[m] * ldc + n : m * ldc + blockIdx.y * bt.c + n;
+    if (epi == EPI_F32) reinterpret_cast<float*>(C)[at] = v;
     else reinterpret_cast<bf16*>(C)[at] = __float2bfloat16_rn(v);
   }
 }
@@ -321,9 +457,25 @@ __global__ void __launch_bounds__(256) k_rows_mma(const bf16* __restrict__ X, lo
 }  // namespace
 
 template <typename T>
-int DecStream<T>::embed(const T* table, const int* tokens, int ld_tok, int B, int T_, int base, int vocab, const float* w, float* x, T* h,
-                        int d, float eps, unsigned int* status, cudaStream_t s) {
-  CUDA_TRY(launch_dependent(k_dec_embed<T>, B * T_, RT, 0, s, table, tokens, ld_tok, T_, base, vocab, w, x, h, d, eps, status));
+int DecStream<T>::embed(const T* table, const int* tokens, int ld_tok, int B, int T_, int base, int vocab, float scale, float* x,
+                        const NextNorms<T>& n, int d, float eps, unsigned int* status, cudaStream_t s) {
+  CUDA_TRY(launch_dependent(k_dec_embed<T>, B * T_, RT, 0, s, table, tokens, ld_tok, T_, base, vocab, scale, x, n, d, eps, status));
+  KERNEL_CHECK();
+  return 0;
+}
+template <typename T>
+int DecStream<T>::parallel_resid(float* x, const T* y, const T* y2, const MoeRows& m, const NextNorms<T>& n, int rows, int d, float eps,
+                                 cudaStream_t s) {
+  bool vec = (d & 3) == 0;
+  for (const void* p : {(const void*)x, (const void*)y, (const void*)y2, m.out, (const void*)n.w, (const void*)n.h, (const void*)n.w2, (const void*)n.h2})
+    vec = vec && aligned16(p);
+  const int nv = vec ? cdiv(d, RT * 4) : 0;
+#define LAUNCH(NV) CUDA_TRY(launch_dependent(k_parallel_resid<T, NV>, rows, RT, 0, s, x, y, y2, m, n, d, eps))
+  if (nv == 1) LAUNCH(1);
+  else if (nv == 2) LAUNCH(2);
+  else if (nv == 3 || nv == 4) LAUNCH(4);
+  else LAUNCH(0);
+#undef LAUNCH
   KERNEL_CHECK();
   return 0;
 }
@@ -383,9 +535,9 @@ template int pack_rows<bf16>(const float*, int, int, bf16*, long long, int, int,
 int rows_stream(const bf16* X, long long ldx, const bf16* W, long long ldw, void* C, long long ldc, int M, int N, int K, int epi, int batch,
                 const RowsBatch& bt, cudaStream_t s) {
   const dim3 grid(cdiv(N, 16), batch);
-  const int f32 = epi == EPI_F32;
-#define LAUNCH(NT) CUDA_TRY(epi == EPI_SWIGLU ? launch_dependent(k_rows_mma<NT, true>, grid, 256, 0, s, X, ldx, W, ldw, C, ldc, M, N, K, f32, bt) \
-                                              : launch_dependent(k_rows_mma<NT, false>, grid, 256, 0, s, X, ldx, W, ldw, C, ldc, M, N, K, f32, bt))
+#define LAUNCH(NT) CUDA_TRY(bt.lists          ? launch_dependent(k_rows_mma<NT, false, true>, grid, 256, 0, s, X, ldx, W, ldw, C, ldc, M, N, K, epi, bt) \
+                            : epi == EPI_SWIGLU ? launch_dependent(k_rows_mma<NT, true, false>, grid, 256, 0, s, X, ldx, W, ldw, C, ldc, M, N, K, epi, bt) \
+                                                : launch_dependent(k_rows_mma<NT, false, false>, grid, 256, 0, s, X, ldx, W, ldw, C, ldc, M, N, K, epi, bt))
   if (M <= 8) LAUNCH(1);
   else if (M <= 16) LAUNCH(2);
   else LAUNCH(4);
@@ -406,22 +558,40 @@ template int pack_transposed<bf16>(const float*, int, int, int, bf16*, int, int,
 
 template <typename T>
 int rows_linear(DecoderStack* d, const void* X, long long ldx, const void* W, long long ldw, void* C, long long ldc, int M, int N, int K,
-                int epi, cudaStream_t s) {
+                int epi, cudaStream_t s, const RowsOut& out) {
   const int f32 = epi == EPI_F32;
   if constexpr (sizeof(T) == 2)
-    if (M <= ROWS_STREAM && ((K | ldx | ldw) & 7) == 0 && aligned16(X) && aligned16(W))
-      return rows_stream((const bf16*)X, ldx, (const bf16*)W, ldw, C, ldc, M, N, K, epi, 1, RowsBatch(), s);
+    if (M <= ROWS_STREAM && ((K | ldx | ldw) & 7) == 0 && aligned16(X) && aligned16(W)) {
+      RowsBatch bt;
+      bt.out = out;
+      return rows_stream((const bf16*)X, ldx, (const bf16*)W, ldw, C, ldc, M, N, K, epi, 1, bt, s);
+    }
   if (M <= RL_ROWS) {
-    if (epi == EPI_SWIGLU) CUDA_TRY(launch_dependent(k_rows_linear<T, true>, cdiv(N, 8), 256, 0, s, (const T*)X, ldx, (const T*)W, ldw, C, ldc, M, N, K, f32));
-    else CUDA_TRY(launch_dependent(k_rows_linear<T, false>, cdiv(N, 8), 256, 0, s, (const T*)X, ldx, (const T*)W, ldw, C, ldc, M, N, K, f32));
+    if (epi == EPI_SWIGLU) CUDA_TRY(launch_dependent(k_rows_linear<T, true>, cdiv(N, 8), 256, 0, s, (const T*)X, ldx, (const T*)W, ldw, C, ldc, M, N, K, f32, out));
+    else CUDA_TRY(launch_dependent(k_rows_linear<T, false>, cdiv(N, 8), 256, 0, s, (const T*)X, ldx, (const T*)W, ldw, C, ldc, M, N, K, f32, out));
     KERNEL_CHECK();
     return 0;
   }
   GemmArgs g;
   g.ws = d->gemm_ws; g.ws_bytes = d->gemm_ws_bytes; g.status = d->status;
   g.A = X; g.lda = ldx; g.a_kmajor = true; g.B = W; g.ldb = ldw; g.b_kmajor = true;
-  g.C = C; g.ldc = ldc; g.M = M; g.N = N; g.K = K; g.epi = epi; g.beta = 0.f; g.any_size = true;
-  if (epi != EPI_SWIGLU) return gemm<T>(g, s);
+  g.C = C; g.ldc = ldc; g.M = M; g.N = N; g.K = K; g.epi = epi; g.beta = 0.f; g.any_size = true; g.bias = out.bias;
+  if (out.n2) {      // two products: this part, and for every column of tokens the rest
+    g.N = out.n2;
+    FEMTO_TRY(gemm<T>(g, s));
+    g.B = (const T*)W + out.n2 * ldw; g.N = N - out.n2; g.M = out.T2; g.ldc = out.ld2;
+    if (g.bias) g.bias += out.n2;
+    for (int b = 0; b < M / out.T2; b++) {
+      g.A = (const T*)X + (long long)b * out.T2 * ldx;
+      g.C = (T*)out.C2 + b * out.stride2;
+      FEMTO_TRY(gemm<T>(g, s));
+    }
+    return 0;
+  }
+  if (epi != EPI_SWIGLU) {
+    FEMTO_TRY(gemm<T>(g, s));
+    return out.softcap != 0.f ? softcap_inplace((float*)C, (long long)M * ldc, s, out.softcap) : 0;
+  }
   // g.N counts the weight rows, gate and up together; the result is half as wide
   g.N = 2 * N;
   if (sizeof(T) == 2 && gemm_tc_supported(g)) return gemm<T>(g, s);
@@ -429,5 +599,5 @@ int rows_linear(DecoderStack* d, const void* X, long long ldx, const void* W, lo
   FEMTO_TRY(gemm<T>(g, s));
   return DecStream<T>::gated_mlp((const T*)d->gu, (T*)C, M, N, s);
 }
-template int rows_linear<float>(DecoderStack*, const void*, long long, const void*, long long, void*, long long, int, int, int, int, cudaStream_t);
-template int rows_linear<bf16>(DecoderStack*, const void*, long long, const void*, long long, void*, long long, int, int, int, int, cudaStream_t);
+template int rows_linear<float>(DecoderStack*, const void*, long long, const void*, long long, void*, long long, int, int, int, int, cudaStream_t, const RowsOut&);
+template int rows_linear<bf16>(DecoderStack*, const void*, long long, const void*, long long, void*, long long, int, int, int, int, cudaStream_t, const RowsOut&);

@@ -12,9 +12,15 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(GemmArgs g) {
   __shared__ float As[TK][TM + 1];
   __shared__ float Bs[TK][TN + 1];
   const int bz = blockIdx.z;
-  const T* A = reinterpret_cast<const T*>(g.A) + (long long)bz * g.strideA;
-  const T* B = reinterpret_cast<const T*>(g.B) + (long long)bz * g.strideB;
   const int m0 = blockIdx.y * TM, n0 = blockIdx.x * TN;
+  int bb = bz;
+  if (g.groups) {      // runs of rows are multiples of TM
+    const int run = m0 / g.group_rows;
+    if (run >= g.groups[0]) return;
+    bb = g.groups[1 + run];
+  }
+  const T* A = reinterpret_cast<const T*>(g.A) + (long long)bz * g.strideA;
+  const T* B = reinterpret_cast<const T*>(g.B) + (long long)bb * g.strideB;
   const int tid = threadIdx.x;
   const int tx = tid % 16, ty = tid / 16;
   float acc[4][4];
@@ -73,7 +79,7 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(GemmArgs g) {
       if (n >= g.N) continue;
       float v = acc[i][j];
       switch (g.epi) {
-        case EPI_STORE: C[(long long)m * g.ldc + n] = from_f<T>(v); break;
+        case EPI_STORE: C[(long long)m * g.ldc + n] = from_f<T>(g.bias ? v + g.bias[n] : v); break;
         case EPI_RESID:
           C[(long long)m * g.ldc + n] = from_f<T>(to_f<T>(aux[(long long)m * g.ldaux + n]) + v);
           break;

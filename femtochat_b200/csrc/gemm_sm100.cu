@@ -55,13 +55,13 @@ struct TcParams {
 // Tile rasterisation: groups of GROUP_M row-tiles are walked column by column, so one wave of CTAs
 // covers a roughly square patch of the output (16 x 9 tiles) and re-reads neither operand from HBM.
 constexpr int GROUP_M = 16;
-__device__ __forceinline__ void tile_coords(const TcParams& p, int t, int& bz, int& mt, int& nt) {
-  const int per = p.tiles_m * p.tiles_n;
+__device__ __forceinline__ void tile_coords(const TcParams& p, int tiles_m, int t, int& bz, int& mt, int& nt) {
+  const int per = tiles_m * p.tiles_n;
   bz = t / per;
   const int pid = t % per;
   const int width = GROUP_M * p.tiles_n;
   const int first_m = (pid / width) * GROUP_M;
-  const int gsz = min(p.tiles_m - first_m, GROUP_M);
+  const int gsz = min(tiles_m - first_m, GROUP_M);
   mt = first_m + (pid % width) % gsz;
   nt = (pid % width) / gsz;
 }
@@ -150,6 +150,18 @@ __device__ __forceinline__ void bf16_chunk(const GemmArgs& g, float (&v)[32], in
       for (int j = 0; j < 32; j++) a[j] = (nc + j < g.N) ? __bfloat162float(aux[j]) : 0.f;
     }
   }
+  if (EPI == EPI_STORE && g.bias != nullptr) {
+    if (full_chunk) {
+#pragma unroll
+      for (int j = 0; j < 32; j += 4) {
+        const float4 q = __ldg(reinterpret_cast<const float4*>(g.bias + nc + j));
+        v[j] += q.x; v[j + 1] += q.y; v[j + 2] += q.z; v[j + 3] += q.w;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 32; j++) if (nc + j < g.N) v[j] += __ldg(g.bias + nc + j);
+    }
+  }
   const float alpha = g.alpha, beta = g.beta;
 #pragma unroll
   for (int j = 0; j < 32; j++) {
@@ -232,12 +244,19 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
   grid_launch_dependents();
   grid_dependency_wait();
 
+  // a grouped product has as many row-tiles as the device counted
+  int tiles_m = p.tiles_m, total_units = p.total_units;
+  if (g.groups) {
+    tiles_m = min(tiles_m, g.groups[0] * (g.group_rows / TILE_M));
+    total_units = tiles_m * p.tiles_n;
+  }
+
   auto unit_coords = [&](int u, int& bz, int& mt, int& nt, int& kb0, int& kb1) {
     // split-major: all tiles of one k-range run together, so the 148 CTAs stream the same rows of
     // both operands through L2 at the same time
-    const int ntile = p.tiles_m * p.tiles_n * p.g.batch;
+    const int ntile = tiles_m * p.tiles_n * p.g.batch;
     const int s = u / ntile;
-    tile_coords(p, u % ntile, bz, mt, nt);
+    tile_coords(p, tiles_m, u % ntile, bz, mt, nt);
     kb0 = s * p.kb_per_split;
     kb1 = min(p.kblocks, kb0 + p.kb_per_split);
   };
@@ -248,12 +267,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       int stage = 0; uint32_t phase = 0;
       uint32_t issued_mask = 0, last_parity = 0;
       bool ok = true;
-      for (int u = first_unit; u < p.total_units && ok; u += unit_step) {
+      for (int u = first_unit; u < total_units && ok; u += unit_step) {
         int bz, mt, nt, kb0, kb1;
         unit_coords(u, bz, mt, nt, kb0, kb1);
         if (below_diagonal(g, mt, nt, TILE_M)) continue;
         const int m0 = mt * TILE_M + rank * BM;           // first row of A this CTA loads
         const int n0 = nt * BN + rank * G::BN_LOCAL;      // first column of B this CTA loads (its half, in a pair)
+        const int bb = g.groups ? __ldg(g.groups + 1 + mt * TILE_M / g.group_rows) : bz;   // which matrix of B
         for (int kb = kb0; kb < kb1; kb++) {
           if (!mbar_wait(&empty[stage], phase ^ 1, abort_flag, g.status)) { ok = false; break; }
           uint8_t* sa = smem + stage * STAGE_BYTES;
@@ -263,7 +283,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             if (rank == 0) mbar_expect_tx(&full[stage], 2 * STAGE_BYTES);
             if (A_K) tma_load_3d_pair(sa, &tmA, &full[stage], kb * BK, m0, bz);
             else tma_load_4d_pair(sa, &tmA, &full[stage], 0, kb * BK, m0 / 64, bz);
-            if (B_K) tma_load_3d_pair(sb, &tmB, &full[stage], kb * BK, n0, bz);
+            if (B_K) tma_load_3d_pair(sb, &tmB, &full[stage], kb * BK, n0, bb);
             else tma_load_4d_pair(sb, &tmB, &full[stage], 0, kb * BK, n0 / 64, bz);
           } else {
           mbar_expect_tx(&full[stage], STAGE_BYTES);
@@ -276,7 +296,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             for (int j = 0; j < BM / 64; j++) tma_load_3d(sa + j * 8192, &tmA, &full[stage], mt * BM + j * 64, kb * BK, bz);
           }
           if (B_K) {
-            tma_load_3d(sb, &tmB, &full[stage], kb * BK, nt * BN, bz);
+            tma_load_3d(sb, &tmB, &full[stage], kb * BK, nt * BN, bb);
           } else if (p.b_slabs) {
             tma_load_4d(sb, &tmB, &full[stage], 0, kb * BK, nt * (BN / 64), bz);
           } else {
@@ -304,7 +324,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       int stage = 0; uint32_t phase = 0;
       int acc = 0; uint32_t acc_phase = 0;
       bool ok = true;
-      for (int u = first_unit; u < p.total_units && ok; u += unit_step) {
+      for (int u = first_unit; u < total_units && ok; u += unit_step) {
         int bz, mt, nt, kb0, kb1;
         unit_coords(u, bz, mt, nt, kb0, kb1);
         if (below_diagonal(g, mt, nt, TILE_M)) continue;
@@ -340,7 +360,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
     const int half = (warp - 2) >> 2;    // the two warps of a quadrant take alternate pairs of 32-column chunks
     const int row_in_tile = quad * 32 + lane;
     int acc = 0; uint32_t acc_phase = 0;
-    for (int u = first_unit; u < p.total_units; u += unit_step) {
+    for (int u = first_unit; u < total_units; u += unit_step) {
       int bz, mt, nt, kb0, kb1;
       unit_coords(u, bz, mt, nt, kb0, kb1);
       if (below_diagonal(g, mt, nt, TILE_M)) continue;
@@ -528,7 +548,7 @@ __global__ void __launch_bounds__(256) gemm_tc_reduce_kernel(const TcParams p) {
   const int c = blockIdx.x & 7, half_id = (blockIdx.x >> 3) % slots, tile = (blockIdx.x >> 3) / slots;
   const int ntile = p.tiles_m * p.tiles_n * g.batch;
   int bz, mt, nt;
-  tile_coords(p, tile, bz, mt, nt);
+  tile_coords(p, p.tiles_m, tile, bz, mt, nt);
   const int tile_m = p.pair ? 2 * BM : BM;
 #pragma unroll
   for (int it = 0; it < 4; it++) {
@@ -676,6 +696,7 @@ bool gemm_tc_supported(const GemmArgs& g) {
   if (!g.b_kmajor && (g.N & 7)) return false;
   if (g.a_kmajor && (g.K & 7)) return false;
   if (g.b_kmajor && (g.K & 7)) return false;
+  if (g.groups && (g.batch != 1 || !g.b_kmajor || !g.a_kmajor || (g.epi != EPI_STORE && g.epi != EPI_RELU2) || g.group_rows % BM || g.M % g.group_rows)) return false;
   if (g.epi == EPI_F32) {
     if (!g.ws) return false;
   } else if (g.epi == EPI_XENT_STATS) {
@@ -830,12 +851,13 @@ int gemm_tc_bf16(const GemmArgs& g, cudaStream_t s) {
     const char* e = getenv("FEMTO_GEMM_PAIR");
     g_pair_mode = (e && e[0] == '0') ? 0 : 1;
   }
-  bool pair = (g_pair_mode != 0) && g.M >= 2 * BM && sms >= 2;
+  bool pair = (g_pair_mode != 0) && g.M >= 2 * BM && sms >= 2 && (!g.groups || g.group_rows % (2 * BM) == 0);
+  const int nbB = g.groups ? g.n_groups : nb;      // matrices of B
   if (pair) {
     if (g.a_kmajor) pair = make_tmap_3d_bf16(&tmA, g.A, g.K, g.M, nb, g.lda, g.strideA, 64, BM) == 0;
     else pair = make_tmap_4d_slabs_bf16(&tmA, g.A, g.M, g.K, nb, g.lda, g.strideA, BK, BM / 64) == 0;
     if (pair) {
-      if (g.b_kmajor) pair = make_tmap_3d_bf16(&tmB, g.B, g.K, g.N, nb, g.ldb, g.strideB, 64, BN / 2) == 0;
+      if (g.b_kmajor) pair = make_tmap_3d_bf16(&tmB, g.B, g.K, g.N, nbB, g.ldb, g.strideB, 64, BN / 2) == 0;
       else pair = make_tmap_4d_slabs_bf16(&tmB, g.B, g.N, g.K, nb, g.ldb, g.strideB, BK, BN / 128) == 0;
     }
     if (pair) { p.a_slabs = !g.a_kmajor; p.b_slabs = !g.b_kmajor; }
@@ -882,7 +904,7 @@ int gemm_tc_bf16(const GemmArgs& g, cudaStream_t s) {
     if (g.a_kmajor) FEMTO_TRY(make_tmap_3d_bf16(&tmA, g.A, g.K, g.M, nb, g.lda, g.strideA, 64, BM));
     else if (make_tmap_4d_slabs_bf16(&tmA, g.A, g.M, g.K, nb, g.lda, g.strideA, BK, BM / 64) == 0) p.a_slabs = 1;
     else FEMTO_TRY(make_tmap_3d_bf16(&tmA, g.A, g.M, g.K, nb, g.lda, g.strideA, 64, BK));
-    if (g.b_kmajor) FEMTO_TRY(make_tmap_3d_bf16(&tmB, g.B, g.K, g.N, nb, g.ldb, g.strideB, 64, BN));
+    if (g.b_kmajor) FEMTO_TRY(make_tmap_3d_bf16(&tmB, g.B, g.K, g.N, nbB, g.ldb, g.strideB, 64, BN));
     else if (make_tmap_4d_slabs_bf16(&tmB, g.B, g.N, g.K, nb, g.ldb, g.strideB, BK, BN / 64) == 0) p.b_slabs = 1;
     else FEMTO_TRY(make_tmap_3d_bf16(&tmB, g.B, g.N, g.K, nb, g.ldb, g.strideB, 64, BK));
   }

@@ -13,6 +13,7 @@ struct LayerState {
   size_t tail_bytes = 0;                // a step reads one and writes the other, so blocks of one launch do not race
   int tail_now = 0;
   void* latent = nullptr;      // [maxB][maxT][ld]: latent and rotated key part of every token, compute type
+  void* kv = nullptr;          // [maxB][maxT][ld]: keys and values of every token, compute type
   int ld = 0;
 };
 

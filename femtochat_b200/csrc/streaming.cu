@@ -1091,15 +1091,15 @@ int xent_dlogit_inplace(void* logits_bf16, long long ld, const float* lse_rows, 
   return 0;
 }
 namespace {
-// z = 15 tanh(x / 15) in place (src/gpt.jl:12)
-__global__ void __launch_bounds__(256) k_softcap(float* __restrict__ x, long long n) {
+// z = cap tanh(x / cap) in place (src/gpt.jl:12)
+__global__ void __launch_bounds__(256) k_softcap(float* __restrict__ x, long long n, float cap, float inv) {
   pdl_trigger();
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
-    x[i] = 15.f * tanhf(x[i] * (1.f / 15.f));
+    x[i] = cap * tanhf(x[i] * inv);
 }
 }  // namespace
-int softcap_inplace(float* x, long long n, cudaStream_t s) {
-  k_softcap<<<(int)std::min<long long>(cdiv(n, 256), 148 * 16), 256, 0, s>>>(x, n);
+int softcap_inplace(float* x, long long n, cudaStream_t s, float cap) {
+  k_softcap<<<(int)std::min<long long>(cdiv(n, 256), 148 * 16), 256, 0, s>>>(x, n, cap, 1.f / cap);
   KERNEL_CHECK();
   return 0;
 }

@@ -12,7 +12,7 @@ from .decoder import Decoder
 from .gpt import GPT
 from .weights import SafeTensors
 
-MODELS = {"GPT": GPT, "Virolorn": Decoder}
+MODELS = {"GPT": GPT, "Virolorn": Decoder, "Zurevik": Decoder}
 
 
 def register(architecture: str, cls) -> None:

@@ -142,14 +142,25 @@ int32_t femto_decode_step(femto_handle* h, femto_kv_cache* c, const float* theta
                           const int32_t* positions, int32_t B, float* logits_out, void* stream);
 
 /* ---- decoders that list their layers ------------------------------------------------------------------------------ */
-/* A decoder-only model given as a list of layers, each a token mixer and an optional gated feed-forward, with an RMS norm
- * before and after both:  x += m norm1b(mixer(norm1(x))),  x += m norm2b(mlp(norm2(x)));  the residual stream x is fp32 in
- * every build.  No counterpart in the reference: the handle is a femto_handle like any other, and
- * femto_refresh_weights, femto_kv_cache_*, femto_prefill, femto_decode_step, femto_status_word, femto_launch_count and
- * femto_destroy take it; calls that train do not (FEMTO_ERR_UNSUPPORTED).  The model "Virolorn" is built of these. */
+/* A decoder-only model given as a list of layers, each a token mixer and an optional feed-forward, arranged in one of two
+ * ways (block):
+ *   FEMTO_BLOCK_SANDWICH  x += m norm1b(mixer(norm1(x))),  x += m norm2b(mlp(norm2(x)))
+ *   FEMTO_BLOCK_PARALLEL  x += mixer(norm1(x)) + mlp(norm2(x)), both of the same x
+ * All norms are RMS norms; the residual stream x is fp32 in every build.  No counterpart in the reference: the handle is a
+ * femto_handle like any other, and femto_refresh_weights, femto_kv_cache_*, femto_prefill, femto_decode_step,
+ * femto_status_word, femto_launch_count and femto_destroy take it; calls that train do not (FEMTO_ERR_UNSUPPORTED).
+ * The models "Virolorn" and "Zurevik" are built of these. */
 #define FEMTO_MIXER_LIGHTNING 1        /* S <- decay_h S + k v^T, o = S^T q, one constant decay per head */
 #define FEMTO_MIXER_CHANNEL_DELTA 2    /* gated delta rule with a data-dependent decay per head and key channel */
 #define FEMTO_MIXER_LATENT_ATTENTION 3 /* softmax attention over a cached low-rank latent plus one rotated key part */
+#define FEMTO_MIXER_ATTENTION 4        /* softmax attention over cached keys and values, in a sliding window */
+
+#define FEMTO_BLOCK_SANDWICH 0
+#define FEMTO_BLOCK_PARALLEL 1
+
+#define FEMTO_GATE_NONE 0
+#define FEMTO_GATE_HEAD 1              /* one sigmoid per head on the head's output */
+#define FEMTO_GATE_ELEMENT 2           /* one per entry of the concatenated heads */
 
 typedef struct femto_layer_config {
   int32_t mixer;       /* FEMTO_MIXER_* */
@@ -158,10 +169,19 @@ typedef struct femto_layer_config {
   int32_t conv;        /* CHANNEL_DELTA: taps of the causal convolutions on q, k and v */
   int32_t decay_rank, gate_rank;      /* CHANNEL_DELTA: inner sizes of the two low-rank projections */
   int32_t q_rank, kv_rank, rot_dim, rot_dims; /* LATENT_ATTENTION; the first rot_dims of the rot_dim part are rotated */
-  int32_t ff;          /* inner size of the gated feed-forward, 0 = the layer has none */
-  float scale;         /* LATENT_ATTENTION: factor on the scores */
+  int32_t ff;          /* inner size of the feed-forward (of one expert), 0 = the layer has none */
+  float scale;         /* LATENT_ATTENTION, ATTENTION: factor on the scores */
   double rot_base;     /* LATENT_ATTENTION: pair i turns by position * rot_base^(-2i/rot_dims) */
   const float* h_decay; /* LIGHTNING: [heads], host memory, read during the call */
+  /* ATTENTION.  maps = 2 is differential attention: q and k hold two maps per head ([map 1, map 2], dim each), the result is
+   * (a1 - lambda a2) / rms * (1 - diff) with lambda = exp(lq1.lk1) - exp(lq2.lk2) + diff.  Position i sees j <= i with
+   * i - j < window or j < keep_first.  kv_from: -1, or the earlier layer whose cached keys and values this one reads. */
+  int32_t maps, window, keep_first, kv_from;
+  int32_t qkv_bias, qk_norm, sink;    /* biases of q, k, v; RMS norms of q and k per head and map; exp(sink_h) in the denominator */
+  int32_t gate;                       /* FEMTO_GATE_* */
+  float diff;
+  int32_t experts, top; /* feed-forward: 0 = one gated feed-forward; else `top` of `experts`, W_down relu(W_up h)^2 each, weighted by
+                           the softmax over the chosen router logits */
 } femto_layer_config;
 
 typedef struct femto_decoder_config {
@@ -172,6 +192,10 @@ typedef struct femto_decoder_config {
   int32_t max_rows;      /* tokens (over all columns) that one internal pass takes; longer prompts are fed in portions */
   float norm_eps, residual_mult;
   const femto_layer_config* h_layers; /* [n_layer], host memory */
+  int32_t block;         /* FEMTO_BLOCK_* */
+  int32_t untied;        /* 1: the output head is a tensor of its own ("head"), 0: the embedding */
+  float embed_scale;     /* factor on the embedding rows as they enter */
+  float logit_softcap;   /* logits <- cap tanh(logits / cap); 0 = none */
 } femto_decoder_config;
 
 /* One tensor of the flat fp32 parameter vector: a weight is row-major [rows][cols] = [out][in]. */
