@@ -221,8 +221,13 @@ def expert_mlp(h, up, down):
     return torch.clamp(h @ up.T, min=0) ** 2 @ down.T
 
 
-def mixture_mlp(h, w, top):
-    best, weight = route(h @ w["router"].T + w["router.b"], top)
+def mixture_mlp(h, w, top, margins=None):
+    """`margins` collects, per row, the gap between the last logit that was chosen and the first that was not."""
+    z = h @ w["router"].T + w["router.b"]
+    best, weight = route(z, top)
+    if margins is not None and top < z.shape[1]:
+        s = torch.sort(z, dim=-1, descending=True).values
+        margins.append(s[:, top - 1] - s[:, top])
     out = torch.zeros_like(h)
     for t in range(h.shape[0]):
         for e, p in zip(best[t].tolist(), weight[t]):
@@ -239,19 +244,23 @@ def _sub(weights, prefix):
     return {n[len(prefix):]: t for n, t in weights.items() if n.startswith(prefix)}
 
 
-def sandwich_layer(x, w, layer, eps, mult, mix):
+def feed_forward(h, w, mlp, margins=None):
+    return gated_mlp(h, w) if mlp["kind"] == "dense" else mixture_mlp(h, w, mlp["router"]["top"], margins)
+
+
+def sandwich_layer(x, w, layer, eps, mult, mix, margins=None):
     """A norm before and after each sublayer, one after the other."""
     x = x + mult * rms_norm(mix(rms_norm(x, w["norm1"], eps)), w["norm1b"], eps)
     if layer["mlp"] is not None:
-        x = x + mult * rms_norm(gated_mlp(rms_norm(x, w["norm2"], eps), _sub(w, "mlp.")), w["norm2b"], eps)
+        x = x + mult * rms_norm(feed_forward(rms_norm(x, w["norm2"], eps), _sub(w, "mlp."), layer["mlp"], margins), w["norm2b"], eps)
     return x
 
 
-def parallel_layer(x, w, layer, eps, mix):
+def parallel_layer(x, w, layer, eps, mix, margins=None):
     """Mixer and feed-forward side by side, each behind a norm of its own."""
     y = mix(rms_norm(x, w["norm1"], eps))
     if layer["mlp"] is not None:
-        y = y + mixture_mlp(rms_norm(x, w["norm2"], eps), _sub(w, "mlp."), layer["mlp"]["router"]["top"])
+        y = y + feed_forward(rms_norm(x, w["norm2"], eps), _sub(w, "mlp."), layer["mlp"], margins)
     return x + y
 
 
@@ -263,11 +272,12 @@ class Sequence:
         self.w = {n: t.to(dtype) for n, t in weights.items()}
         self.state = [dict() for _ in config["layers"]]
         self.residuals = []           # the residual stream after every layer of the last call
+        self.margins = []             # of the last call's routers
 
     def feed(self, tokens):
         cfg, eps = self.cfg, self.cfg["norm"]["eps"]
         x = self.w["embed"][torch.as_tensor(tokens, dtype=torch.long)] * cfg.get("embedding", {}).get("scale", 1.0)
-        self.residuals = []
+        self.residuals, self.margins = [], []
         for i, layer in enumerate(cfg["layers"]):
             own = i
             while cfg["layers"][own].get("weights_of") is not None:
@@ -276,9 +286,9 @@ class Sequence:
             shared = {} if m.get("kv_from") is None else dict(shared=self.state[m["kv_from"]])
             mix = lambda h: MIXERS[layer["type"]](h, _sub(w, "mix."), m, eps, self.state[i], **shared)
             if cfg["architecture"] == "Zurevik":
-                x = parallel_layer(x, w, layer, eps, mix)
+                x = parallel_layer(x, w, layer, eps, mix, self.margins)
             else:
-                x = sandwich_layer(x, w, layer, eps, cfg["residual_mult"], mix)
+                x = sandwich_layer(x, w, layer, eps, cfg["residual_mult"], mix, self.margins)
             self.residuals.append(x)
         z = rms_norm(x, self.w["final.norm"], eps) @ self.w["head" if "head" in self.w else "embed"].T
         cap = cfg.get("logit_softcap")
@@ -326,11 +336,15 @@ def tensor_shapes(cfg, decay_rank=8, gate_rank=8):
         if layer["mlp"] is not None and layer["mlp"]["kind"] == "moe":
             f, n = layer["mlp"]["expert"]["ff"], layer["mlp"]["router"]["experts"]
             out.update({p + "norm2": (d,), p + "mlp.router": (n, d), p + "mlp.router.b": (n,)})
+            if cfg["architecture"] == "Virolorn":
+                out[p + "norm2b"] = (d,)
             for e in range(n):
                 out.update({p + f"mlp.e{e}.up": (f, d), p + f"mlp.e{e}.down": (d, f)})
         elif layer["mlp"] is not None:
             f = layer["mlp"]["ff"]
-            out[p + "norm2"] = out[p + "norm2b"] = (d,)
+            out[p + "norm2"] = (d,)
+            if cfg["architecture"] == "Virolorn":
+                out[p + "norm2b"] = (d,)
             out.update({p + "mlp.gate": (f, d), p + "mlp.up": (f, d), p + "mlp.down": (d, f)})
     return out
 

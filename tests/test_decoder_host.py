@@ -109,7 +109,7 @@ def test_safetensors_round_trip_and_format(tmp_path):
 
 
 def test_registry(tmp_path):
-    assert fb.MODELS["Virolorn"] is fb.Decoder and fb.MODELS["GPT"] is fb.GPT
+    assert fb.MODELS["Virolorn"] is fb.MODELS["Zurevik"] is fb.Decoder and fb.MODELS["GPT"] is fb.GPT
     (tmp_path / "config.json").write_text(json.dumps(dict(architecture="Nothing")))
     with pytest.raises(ValueError, match="unknown architecture"):
         fb.load_model(str(tmp_path))
@@ -129,3 +129,77 @@ def test_no_cpu_fallback():
     c = fb.DecoderConfig.from_json(cfg, lo.tensor_shapes(cfg, *ranks))
     with pytest.raises(_lib.FemtoError, match="no CUDA device"):
         fb.DecoderState(c, 1)
+
+
+# ---- windows, sinks, differential attention, mixtures of experts ------------------------------------------------------
+@pytest.mark.parametrize("name", ["differential", "sinks", "sinks, shared keys"])
+def test_oracle_portions_of_windowed_layers(name):
+    cfg, ranks = dc.SINGLE[name]
+    w, t = lo.random_weights(cfg, 1, *ranks), dc.tokens(60, cfg["vocab"])
+    whole = lo.Sequence(cfg, w).feed(t)
+    for cuts in ((2, 5, 2), (1,) * 59, (21,)):
+        s, at, out = lo.Sequence(cfg, w), 0, []
+        for n in cuts + (99,):
+            out.append(s.feed(t[at:at + n])) if at < 60 else None
+            at += n
+        assert (torch.cat(out) - whole).abs().max() < 1e-10
+
+
+def test_oracle_windowed_attention_against_masked_softmax():
+    g = torch.Generator().manual_seed(6)
+    r = lambda *s: torch.randn(*s, generator=g, dtype=torch.float64)
+    N, T, H, G, D, E, size, keep = 23, 9, 4, 2, 5, 3, 6, 2
+    q, k, v, sink = r(T, H, D), r(N, G, D), r(N, G, E), r(H)
+    i, j = torch.arange(N - T, N)[:, None], torch.arange(N)[None, :]
+    see = (j <= i) & ((i - j < size) | (j < keep))
+    kk, vv = k.repeat_interleave(H // G, 1), v.repeat_interleave(H // G, 1)
+    s = torch.einsum("thd,nhd->htn", q, kk) * 0.7
+    s = s.masked_fill(~see, -torch.inf)
+    p = torch.softmax(torch.cat([s, sink[:, None, None].expand(H, T, 1)], -1), -1)[..., :-1]
+    assert torch.allclose(lo.windowed_attention(q, k, v, 0.7, N - T, size, keep, sink), torch.einsum("htn,nhe->the", p, vv))
+    assert torch.allclose(lo.windowed_attention(q, k, v, 0.7, N - T, size, keep), torch.einsum("htn,nhe->the", torch.softmax(s, -1), vv))
+    # an unreachable sink changes nothing, an overwhelming one leaves nothing
+    assert torch.allclose(lo.windowed_attention(q, k, v, 0.7, N - T, size, keep, sink - 100), lo.windowed_attention(q, k, v, 0.7, N - T, size, keep))
+    assert lo.windowed_attention(q, k, v, 0.7, N - T, size, keep, sink + 100).abs().max() < 1e-30
+
+
+def test_oracle_routing():
+    best, weight = lo.route(torch.tensor([[1.0, 3.0, 3.0, -2.0], [0.0, -1.0, 5.0, 4.0]], dtype=torch.float64), 2)
+    assert best.tolist() == [[1, 2], [2, 3]] and torch.allclose(weight[0], torch.tensor([0.5, 0.5], dtype=torch.float64))
+    assert torch.allclose(weight[1], torch.softmax(torch.tensor([5.0, 4.0], dtype=torch.float64), 0))
+
+
+@pytest.mark.parametrize("name", sorted(dc.EXPERTS))
+def test_layout_of_mixtures(name):
+    cfg = dc.EXPERTS[name]
+    shapes = lo.tensor_shapes(cfg)
+    assert {n: s.shape for n, s in fb.decoder_layout(fb.DecoderConfig.from_json(cfg, shapes)).items()} == shapes
+
+
+def test_a_layer_that_reads_anothers_keys_has_none():
+    lay = fb.decoder_layout(fb.DecoderConfig.from_json(dc.ZMIXED, lo.tensor_shapes(dc.ZMIXED)))
+    assert "l0.mix.k" in lay and "l0.mix.v.b" in lay and "l2.mix.q.b" in lay and "head" in lay
+    assert not any(n.startswith(("l2.mix.k", "l2.mix.v")) or n.endswith("norm1b") for n in lay)
+
+
+def test_bad_windowed_configurations_are_refused():
+    def layout(*layers, **kw):
+        return fb.decoder_layout(fb.DecoderConfig.from_json(dc.zurevik(*layers, **kw), {}))
+    with pytest.raises(_lib.FemtoError, match="multiple of kv_heads"):
+        layout(dc.differential(heads=3, kv_heads=2))
+    with pytest.raises(_lib.FemtoError, match="earlier layer"):
+        layout(dc.sinks(kv_from=1), dc.sinks())
+    with pytest.raises(_lib.FemtoError, match="of its own"):
+        layout(dc.sinks(), dc.sinks(kv_from=0), dc.sinks(kv_from=1))
+    with pytest.raises(_lib.FemtoError, match="key or value sizes"):
+        layout(dc.sinks(), dc.sinks(kv_from=0, vdim=24))
+    with pytest.raises(_lib.FemtoError, match="window"):
+        layout(dc.sinks(size=0))
+    with pytest.raises(_lib.FemtoError, match="256"):
+        layout(dc.differential(dim=300))
+    with pytest.raises(_lib.FemtoError, match="experts"):
+        layout(dc.sinks(mlp=dc.moe(experts=3, top=4)))
+    with pytest.raises(ValueError, match="unknown mixer"):
+        layout(dc.lightning())
+    with pytest.raises(ValueError, match="unknown feed-forward"):
+        layout(dc.sinks(mlp=dict(kind="spline")))
