@@ -390,7 +390,7 @@ def run_ours(args):
 
 
 def run_serve(args):
-    """`--serve`: one JSON line with prefill and decode tokens/s of both model families at each size."""
+    """`--serve`: one JSON line with prefill and decode tokens/s of every model at each size."""
     from femtochat_b200 import serve_bench
     clocks = ClockSampler(0)
     clocks.start()
@@ -431,8 +431,8 @@ def main():
                     help="N > 1: after the bench line, time reverse pass / gradient sum / update separately for the "
                          "owner-sharded and the replicated update (stderr)")
     ap.add_argument("--serve", action="store_true",
-                    help="instead of the training step: prefill and decode throughput of a Virolorn model (layers listed one by "
-                         "one) beside the GPT at equal size, random weights, one GPU")
+                    help="instead of the training step: prefill and decode throughput of the models that list their layers "
+                         "(Virolorn, Zurevik) beside the GPT at equal size, random weights, one GPU")
     ap.add_argument("--serve-sizes", default="d20,w2560", help="with --serve: sizes of femtochat_b200/serve_bench.py")
     args = ap.parse_args()
     if args.serve:

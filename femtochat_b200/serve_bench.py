@@ -1,4 +1,5 @@
-"""Prefill and decode throughput of a layer-listing decoder beside the framework's GPT at equal size, random weights.
+"""Prefill and decode throughput of the layer-listing decoders beside the framework's GPT at equal size, random weights: the
+GPT with full attention (Virolorn's counterpart) and with the window that Zurevik's layers have.
 
 Times are CUDA events around whole calls of the public entry points (`extend` / `prefill` / `decode_step`), after warm-up;
 every call reads weights and caches larger than L2.  `--kernels` lists where a call's device time goes."""
@@ -13,6 +14,8 @@ SIZES = {
     "w2560": dict(width=2560, n_layer=12, ff=6912, heads=20, kv_heads=10, q_rank=1536, kv_rank=512, vocab=65536),
 }
 MIX = ("lightning", "channel_delta", "channel_delta", "latent_attention")
+WINDOW, KEEP, EXPERTS, TOP = 1024, 4, 8, 2      # Zurevik: two experts of 2 x width, the weights a token uses in the GPT's 4 x width
+MODELS = ("Virolorn", "Zurevik", "GPT", "GPT window")
 
 
 def decoder_config(s, mix=MIX):
@@ -31,11 +34,24 @@ def decoder_config(s, mix=MIX):
     return fb.DecoderConfig(vocab_size=s["vocab"], width=s["width"], norm_eps=1e-6, residual_mult=0.5, layers=layers)
 
 
-def random_decoder(s, mix=MIX, max_rows=16384):
+def zurevik_config(s):
+    import femtochat_b200 as fb
+    layers = []
+    for i in range(s["n_layer"]):
+        kw = dict(mixer="attention", heads=s["heads"], kv_heads=s["kv_heads"], vdim=128, window=WINDOW, ff=2 * s["width"], experts=EXPERTS, top=TOP)
+        if i % 4 < 2:       # the second reads the keys and values of the first
+            layers.append(fb.LayerConfig(dim=128, scale=128 ** -0.5, qkv_bias=True, sink=True, gate="head", kv_from=i - 1 if i % 4 else None, **kw))
+        else:
+            layers.append(fb.LayerConfig(dim=64, scale=64 ** -0.5, maps=2, qk_norm=True, gate="element", diff=0.5, keep_first=KEEP, **kw))
+    return fb.DecoderConfig(vocab_size=s["vocab"], width=s["width"], norm_eps=1e-6, layers=layers, block="parallel", untied=True,
+                            embed_scale=1.0, logit_softcap=15.0)
+
+
+def random_decoder(s, cfg=None, max_rows=16384):
     import torch
     import femtochat_b200 as fb
     from femtochat_b200 import _lib
-    cfg = decoder_config(s, mix)
+    cfg = cfg or decoder_config(s)
     lay = fb.decoder_layout(cfg)
     theta = torch.zeros(int(_lib.lib().femto_decoder_nparams(cfg.c_struct())), device="cuda")
     g = torch.Generator(device="cuda").manual_seed(1)
@@ -44,6 +60,8 @@ def random_decoder(s, mix=MIX, max_rows=16384):
         leaf = name.rsplit(".", 1)[-1]
         if leaf.startswith("norm"):
             v.fill_(1.0)
+        elif leaf in ("sink", "b", "lq1", "lk1", "lq2", "lk2"):
+            v.normal_(0.0, 0.1, generator=g)
         elif leaf == "dt_bias":
             v.normal_(-3.0, 1.0, generator=g)
         elif leaf == "A_log":
@@ -53,15 +71,15 @@ def random_decoder(s, mix=MIX, max_rows=16384):
     return fb.Decoder(fb.Params(theta, delta=False), cfg, lay, compute_type="bfloat16", max_rows=max_rows)
 
 
-def random_gpt(s, T):
+def random_gpt(s, T, window=None):
     import torch
     import femtochat_b200 as fb
     cfg = fb.GPTConfig(sequence_len=T, max_document_tokens=16384, vocab_size=s["vocab"], n_layer=s["n_layer"], n_head=s["heads"],
-                       n_kv_head=s["kv_heads"], n_embed=s["width"], window_pattern="L")
+                       n_kv_head=s["kv_heads"], n_embed=s["width"], window_pattern="L" if window is None else "S")
     lay = fb.parameter_layout(cfg)
     theta = torch.empty(lay.nparams, device="cuda")
     fb.initialize_(theta, lay, seed=1, all_nonzero=True)
-    return fb.GPT(fb.Params(theta, delta=False), cfg, lay, compute_type="bfloat16")
+    return fb.GPT(fb.Params(theta, delta=False), cfg, lay, compute_type="bfloat16", **({"short_window": window} if window else {}))
 
 
 def timed(fn, iters, warm=3):
@@ -113,13 +131,18 @@ def measure(model, B, T, vocab, n_decode=32, kernels=False):
     return out
 
 
-def run(size="d20", shapes=((1, 8192), (8, 2048)), kernels=False, which=("Virolorn", "GPT")):
+def run(size="d20", shapes=((1, 8192), (8, 2048)), kernels=False, which=MODELS):
     import torch
     s, out = SIZES[size], dict(size=size)
     for name in which:
         out[name] = []
         for B, T in shapes:
-            model = random_decoder(s, max_rows=B * T) if name == "Virolorn" else random_gpt(s, T + 192)
+            if name == "Zurevik":
+                model = random_decoder(s, zurevik_config(s), max_rows=B * T)
+            elif name == "Virolorn":
+                model = random_decoder(s, max_rows=B * T)
+            else:
+                model = random_gpt(s, T + 192, WINDOW if name == "GPT window" else None)
             if kernels:
                 print(f"== {name} {size}")
             out[name].append(measure(model, B, T, s["vocab"], kernels=kernels))
@@ -135,7 +158,7 @@ def main():
     ap.add_argument("--size", default="d20", choices=sorted(SIZES))
     ap.add_argument("--kernels", action="store_true")
     ap.add_argument("--shapes", default="1x8192,8x2048")
-    ap.add_argument("--which", default="Virolorn,GPT")
+    ap.add_argument("--which", default=",".join(MODELS))
     a = ap.parse_args()
     shapes = [tuple(int(v) for v in x.split("x")) for x in a.shapes.split(",")]
     print(json.dumps(run(a.size, shapes, a.kernels, a.which.split(","))))
