@@ -1,19 +1,20 @@
 // A prompt's attention for the layer-listing decoders on the sm_100a tensor cores: causal from position `first` on, for any
-// query/key and value sizes that are multiples of 8.  The structure is that of the GPT's forward kernel
-// (attention_sm100.cu): one CTA owns 128 queries of one head, a TMA warp streams key and value tiles of 128 tokens, one
-// thread issues S = Q K^T into one of two TMEM buffers, another O += P V with P read back from TMEM, and two threads per
-// query row do the softmax.  What differs is how the operands arrive: each 64-channel slab is its own TMA box, and a slab
+// query/key and value sizes that are multiples of 8.  Each 64-channel slab of an operand is a TMA box of its own, and a slab
 // that reaches past a head's channels is filled with zeros by the copy.
 //
 //   Latent attention: the unrotated part of K comes from the expanded keys of the head, the rotated part straight from the
 //   cache rows that all heads share.
 //   Windowed attention: the key tiles are those of the first `keep` tokens and then those of the window; groups of query
-//   heads share a key/value head; a sink enters the sum at the end.  With two maps (differential attention) the steps of a
-//   tile alternate between them: the two S buffers and two halves of O belong to one map each, the value tile to both.
-//   The softmax weights enter P V as the sum of two bf16 numbers (SPLIT), so they keep 32-bit accuracy: a tile's P takes
-//   the 128 columns that held its S.
+//   heads share a key/value head; a sink enters the sum at the end.  The softmax weights enter P V as the sum of two bf16
+//   numbers (SPLIT), so they keep 32-bit accuracy: a tile's P takes the 128 columns that held its S.
 //
-// Normalisation, the head's own norm of differential attention and the output gate are applied as the result leaves.
+// One CTA per SM walks the items (128 queries of one head), latest queries first.  The steps of an item, 128 queries against
+// 128 keys, alternate between two streams, each with a buffer for S / P and an accumulator O of its own in tensor memory and
+// eight softmax warps (two threads per query row), so that the exponentials of one stream run beside the products, the
+// loads and the row maxima of the other.  With two maps (differential attention) the streams are the maps, otherwise the
+// even and the odd key tiles, whose partial results meet at the end.  A TMA warp streams Q, K and V (two stages of K and V),
+// one thread issues S = Q K^T, another O += P V with P read back from tensor memory; all of them run ahead into the next item.
+// Sum of the streams, the head's own norm of differential attention and the output gate are applied as the result leaves.
 #include <algorithm>
 
 #include "decoder.cuh"
@@ -23,15 +24,19 @@ using namespace sm100;
 
 namespace {
 
-constexpr int BQ = 128, BKV = 128, NS = 2, CW = BKV / NS, THREADS = 128 + NS * 128;
+constexpr int BQ = 128, BKV = 128, NS = 2, CW = BKV / NS, THREADS = 128 + 2 * NS * 128;
 constexpr int SLAB = 128 * 64 * 2;                    // one box: 128 tokens x 64 channels
 constexpr int MAX_SLABS = 13;                         // 16 KB each: (maps + 2) per query/key slab (Q + two K stages), 2 per value slab
+constexpr int MAX_V = 128;                            // value columns of one launch
 constexpr float LOG2E = 1.4426950408889634f;
+// registers per thread: launched with 96 (640 threads); the first warpgroup's surplus goes to the softmax warps
+constexpr int REGS_ROLES = 32, REGS_SOFTMAX = 112;
 
 struct SlabAttn {
   bf16* o; const bf16* gate; unsigned int* status;
   long long ld_gate;
-  int T, first, N, heads, vdim;
+  int T, first, N, heads, vdim, items, qtiles;
+  int col0, cols;              // value columns of this launch
   int per;                     // query heads per key/value head
   int n_un, n_rot, n_v;        // slabs of the unrotated part, the rotated part, the values
   int k_un, k_rot;             // 16-channel steps of the two parts
@@ -40,6 +45,25 @@ struct SlabAttn {
   const float* sink;           // [heads] or null
   const float* lambda;         // two maps: o = a1 - lambda a2, then o / rms(o) * out_scale
   float out_scale, eps;
+};
+
+// One item: 128 queries of one head and the key tiles that they see: first those of the kept tokens before the window, then
+// those from `lo`, the first token that any of the queries sees through the window.
+struct Item {
+  int h, b, q0, lo, kept, nkeep, ntile;
+  __device__ __forceinline__ Item(const SlabAttn& p, int item) {
+    const int per = p.items / p.qtiles;               // heads x columns
+    const int rem = item % per;
+    h = rem % p.heads;
+    b = rem / p.heads;
+    q0 = (p.qtiles - 1 - item / per) * BQ;
+    const int last = min(p.first + q0 + BQ - 1, p.N - 1);
+    lo = max(0, p.first + q0 - p.window + 1);
+    kept = min(p.keep, lo);
+    nkeep = (kept + BKV - 1) / BKV;
+    ntile = nkeep + (last - lo) / BKV + 1;
+  }
+  __device__ __forceinline__ int key(int i) const { return i < nkeep ? i * BKV : lo + (i - nkeep) * BKV; }
 };
 
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
@@ -57,41 +81,34 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
   grid_launch_dependents();
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-  const int nqk = p.n_un + p.n_rot;
-  const int q_bytes = nqk * SLAB, v_bytes = p.n_v * SLAB;
+  const int q_bytes = (p.n_un + p.n_rot) * SLAB, v_bytes = p.n_v * SLAB;
   uint8_t* sQ = smem;
   uint8_t* sK = sQ + MAPS * q_bytes;     // 2 stages
   uint8_t* sV = sK + 2 * q_bytes;        // 2 stages
   uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * v_bytes);
   uint64_t* q_full = bars;
-  uint64_t* k_full = bars + 1;    // [2]
-  uint64_t* v_full = bars + 3;    // [2]
-  uint64_t* s_full = bars + 5;    // [2] S of a tile is in TMEM; also frees the tile's K stage
-  uint64_t* p_ready = bars + 7;   // [2]
-  uint64_t* pv_done = bars + 9;   // [2] P V of a step has been accumulated; also frees its S/P buffer
-  uint64_t* v_free = bars + 11;   // [2] every map's P V of a tile has been accumulated
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 13);
+  uint64_t* q_free = bars + 1;    // the item's last S has been executed
+  uint64_t* k_full = bars + 2;    // [2 stages]
+  uint64_t* k_free = bars + 4;    // [2 stages]
+  uint64_t* v_full = bars + 6;    // [2 stages]
+  uint64_t* v_free = bars + 8;    // [2 stages]
+  uint64_t* s_full = bars + 10;   // [2 streams]
+  uint64_t* p_ready = bars + 12;  // [2 streams]
+  uint64_t* pv_done = bars + 14;  // [2 streams] a step's P V has been accumulated; also frees the stream's S / P buffer
+  uint64_t* o_free = bars + 16;   // every softmax warp has read the item's O
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 17);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  float* xmax = reinterpret_cast<float*>(bars + 32);   // [2 parities][NS][128 rows]
-  float* xl = xmax + 2 * NS * 128;                     // [NS][128 rows]
+  float* xmax = reinterpret_cast<float*>(bars + 32);   // [2 parities][2 streams][NS][128 rows]
+  float* xl = xmax + 4 * NS * 128;                     // [2 streams][NS][128 rows]
+  float* xm = xl + 2 * NS * 128;                       // [2 streams][128 rows]
+  float* xs = xm + 2 * 128;                            // [2 streams][NS][128 rows]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int qt = gridDim.x - 1 - blockIdx.x;  // heavy (late) query tiles first
-  const int h = blockIdx.y, b = blockIdx.z, hk = h / p.per;
-  const int q0 = qt * BQ;
-  // Key tiles: first those of the kept tokens before the window, then those from `lo`, the first token that any query of
-  // this block sees through the window.  A step is one map of one tile.
-  const int last = min(p.first + q0 + BQ - 1, p.N - 1);
-  const int lo = max(0, p.first + q0 - p.window + 1), kept = min(p.keep, lo);
-  const int nkeep = (kept + BKV - 1) / BKV, ntile = nkeep + (last - lo) / BKV + 1;
-  const int nstep = ntile * MAPS;
-  auto tile_key = [&](int i) { return i < nkeep ? i * BKV : lo + (i - nkeep) * BKV; };
-
   if (threadIdx.x == 0) {
-    mbar_init(q_full, 1);
+    mbar_init(q_full, 1); mbar_init(q_free, 1); mbar_init(o_free, 4 * NS * 2);
     for (int i = 0; i < 2; i++) {
-      mbar_init(&k_full[i], 1); mbar_init(&v_full[i], 1);
-      mbar_init(&s_full[i], 1); mbar_init(&p_ready[i], NS * 4); mbar_init(&pv_done[i], 1); mbar_init(&v_free[i], 1);
+      mbar_init(&k_full[i], 1); mbar_init(&k_free[i], 1); mbar_init(&v_full[i], 1); mbar_init(&v_free[i], 1);
+      mbar_init(&s_full[i], 1); mbar_init(&p_ready[i], NS * 4); mbar_init(&pv_done[i], 1);
     }
     *abort_flag = 0;
     fence_barrier_init();
@@ -102,266 +119,328 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
-  const uint32_t tS[2] = {tmem_base, tmem_base + 128};
-  const uint32_t tO = tmem_base + 256;
+  grid_dependency_wait();
 
-  if (warp == 0) {
-    if (lane == 0) {
+  // Every role walks the same items in the same order and counts what it has seen: n items, kc key tiles, vc value tiles, cx[X]
+  // steps of stream X.  The phase of a barrier is that count (of its stage's turns), modulo two.
+  if (warp < 4) {
+    reg_dealloc<REGS_ROLES>();
+    if (warp == 0 && lane == 0) {
       // ---------------- TMA producer ----------------
-      mbar_expect_tx(q_full, MAPS * q_bytes);
-#pragma unroll
-      for (int m = 0; m < MAPS; m++) {
-        for (int j = 0; j < p.n_un; j++) tma_load_4d(sQ + m * q_bytes + j * SLAB, &tmQu, q_full, j * 64, h * MAPS + m, q0, b);
-        for (int j = 0; j < p.n_rot; j++) tma_load_4d(sQ + m * q_bytes + (p.n_un + j) * SLAB, &tmQr, q_full, j * 64, h * MAPS + m, q0, b);
-      }
+      int n = 0, kc = 0, vc = 0;
       bool ok = true;
-      uint32_t k_issued = 0, v_issued = 0;
-      for (int s = 0; s < nstep && ok; s++) {
-        const int st = s & 1, i = s / MAPS, m = s % MAPS, vt = i & 1;
-        const int key = tile_key(i);
-        // the stage's previous user is step s-2, or tile i-2 for the values
-        if (s >= 2 && !mbar_wait(&s_full[st], ((s - 2) >> 1) & 1, abort_flag, p.status)) { ok = false; break; }
-        uint8_t* k = sK + st * q_bytes;
-        mbar_expect_tx(&k_full[st], q_bytes);
-        for (int j = 0; j < p.n_un; j++) tma_load_4d(k + j * SLAB, &tmKu, &k_full[st], j * 64, hk * MAPS + m, key, b);
-        for (int j = 0; j < p.n_rot; j++) tma_load_3d(k + (p.n_un + j) * SLAB, &tmKr, &k_full[st], j * 64, key, b);
-        k_issued = s + 1;
-        if (m) continue;
-        if (i >= 2 && !mbar_wait(&v_free[vt], ((i - 2) >> 1) & 1, abort_flag, p.status)) { ok = false; break; }
-        uint8_t* v = sV + vt * v_bytes;
-        mbar_expect_tx(&v_full[vt], v_bytes);
-        for (int j = 0; j < p.n_v; j++) tma_load_4d(v + j * SLAB, &tmV, &v_full[vt], j * 64, hk, key, b);
-        v_issued = i + 1;
+      for (int item = blockIdx.x; item < p.items && ok; item += gridDim.x) {
+        const Item it(p, item);
+        const int hk = it.h / p.per;
+        if (n >= 1 && !mbar_wait(q_free, (n - 1) & 1, abort_flag, p.status)) break;
+        mbar_expect_tx(q_full, MAPS * q_bytes);
+#pragma unroll
+        for (int m = 0; m < MAPS; m++) {
+          for (int j = 0; j < p.n_un; j++) tma_load_4d(sQ + m * q_bytes + j * SLAB, &tmQu, q_full, j * 64, it.h * MAPS + m, it.q0, it.b);
+          for (int j = 0; j < p.n_rot; j++) tma_load_4d(sQ + m * q_bytes + (p.n_un + j) * SLAB, &tmQr, q_full, j * 64, it.h * MAPS + m, it.q0, it.b);
+        }
+        n++;
+        for (int i = 0; i < it.ntile && ok; i++) {
+          const int key = it.key(i);
+#pragma unroll
+          for (int m = 0; m < MAPS; m++) {
+            const int st = kc & 1;
+            if (kc >= 2 && !mbar_wait(&k_free[st], ((kc - 2) >> 1) & 1, abort_flag, p.status)) { ok = false; break; }
+            uint8_t* k = sK + st * q_bytes;
+            mbar_expect_tx(&k_full[st], q_bytes);
+            for (int j = 0; j < p.n_un; j++) tma_load_4d(k + j * SLAB, &tmKu, &k_full[st], j * 64, hk * MAPS + m, key, it.b);
+            for (int j = 0; j < p.n_rot; j++) tma_load_3d(k + (p.n_un + j) * SLAB, &tmKr, &k_full[st], j * 64, key, it.b);
+            kc++;
+          }
+          const int vt = vc & 1;
+          if (!ok || (vc >= 2 && !mbar_wait(&v_free[vt], ((vc - 2) >> 1) & 1, abort_flag, p.status))) { ok = false; break; }
+          uint8_t* v = sV + vt * v_bytes;
+          mbar_expect_tx(&v_full[vt], v_bytes);
+          for (int j = 0; j < p.n_v; j++) tma_load_4d(v + j * SLAB, &tmV, &v_full[vt], p.col0 + j * 64, hk, key, it.b);
+          vc++;
+        }
       }
       if (*abort_flag) {
         // let loads already in flight land before the CTA exits
-        auto drain = [&](uint64_t* bar, uint32_t ph) { for (uint32_t it = 0; it < WAIT_LIMIT && !mbar_try_wait(bar, ph); ++it) {} };
-        drain(q_full, 0);
-        for (int st = 0; st < 2; st++) {
-          for (int i = (int)k_issued - 1; i >= 0 && i >= (int)k_issued - 2; i--) if ((i & 1) == st) drain(&k_full[st], (i >> 1) & 1);
-          for (int i = (int)v_issued - 1; i >= 0 && i >= (int)v_issued - 2; i--) if ((i & 1) == st) drain(&v_full[st], (i >> 1) & 1);
-        }
+        auto drain = [&](uint64_t* bar, int turn) { for (uint32_t t = 0; t < WAIT_LIMIT && !mbar_try_wait(bar, turn & 1); ++t) {} };
+        if (n >= 1) drain(q_full, n - 1);
+        for (int i = max(0, kc - 2); i < kc; i++) drain(&k_full[i & 1], i >> 1);
+        for (int i = max(0, vc - 2); i < vc; i++) drain(&v_full[i & 1], i >> 1);
       }
-    }
-  } else if (warp == 1) {
-    if (lane == 0) {
+    } else if (warp == 1 && lane == 0) {
       // ---------------- S = Q K^T issuer ----------------
       constexpr uint32_t idesc_s = idesc_bf16(BQ, BKV, false, false);  // both operands K-major
-      const uint32_t q_addr = smem_u32(sQ);
-      bool ok = mbar_wait(q_full, 0, abort_flag, p.status);
-      for (int s = 0; s < nstep && ok; s++) {
-        const int st = s & 1;
-        if (!mbar_wait(&k_full[st], (s >> 1) & 1, abort_flag, p.status)) break;
-        // S(s) overwrites the buffer that held P(s-2): its P V must have been executed
-        if (s >= 2 && !mbar_wait(&pv_done[st], ((s - 2) >> 1) & 1, abort_flag, p.status)) break;
-        tc_fence_after();
-        const uint32_t k_addr = smem_u32(sK + st * q_bytes), qm_addr = q_addr + (s % MAPS) * q_bytes;
-        for (int k = 0; k < p.k_un; k++) {
-          const uint32_t off = (k >> 2) * SLAB + (k & 3) * 32;
-          mma_ss(tS[st], smem_desc_sw128(qm_addr + off, 16, 1024), smem_desc_sw128(k_addr + off, 16, 1024), idesc_s, k > 0);
+      int n = 0, kc = 0, cx[2] = {0, 0};
+      bool ok = true;
+      for (int item = blockIdx.x; item < p.items && ok; item += gridDim.x, n++) {
+        const Item it(p, item);
+        if (!mbar_wait(q_full, n & 1, abort_flag, p.status)) break;
+        for (int i = 0; i < it.ntile && ok; i++) {
+#pragma unroll
+          for (int m = 0; m < MAPS; m++, kc++) {
+            const int X = MAPS == 2 ? m : i & 1, st = kc & 1;
+            const int turns = X ? cx[1] : cx[0];
+            // S overwrites the buffer that held the stream's previous P: its P V must have been executed
+            if (!mbar_wait(&k_full[st], (kc >> 1) & 1, abort_flag, p.status) ||
+                (turns >= 1 && !mbar_wait(&pv_done[X], (turns - 1) & 1, abort_flag, p.status))) { ok = false; break; }
+            tc_fence_after();
+            const uint32_t k_addr = smem_u32(sK + st * q_bytes), q_addr = smem_u32(sQ) + m * q_bytes, tS = tmem_base + X * 128;
+            for (int k = 0; k < p.k_un; k++) {
+              const uint32_t off = (k >> 2) * SLAB + (k & 3) * 32;
+              mma_ss(tS, smem_desc_sw128(q_addr + off, 16, 1024), smem_desc_sw128(k_addr + off, 16, 1024), idesc_s, k > 0);
+            }
+            for (int k = 0; k < p.k_rot; k++) {
+              const uint32_t off = (p.n_un + (k >> 2)) * SLAB + (k & 3) * 32;
+              mma_ss(tS, smem_desc_sw128(q_addr + off, 16, 1024), smem_desc_sw128(k_addr + off, 16, 1024), idesc_s, 1);
+            }
+            tc_commit(&s_full[X]);
+            tc_commit(&k_free[st]);
+            if (X) cx[1]++; else cx[0]++;
+          }
         }
-        for (int k = 0; k < p.k_rot; k++) {
-          const uint32_t off = (p.n_un + (k >> 2)) * SLAB + (k & 3) * 32;
-          mma_ss(tS[st], smem_desc_sw128(qm_addr + off, 16, 1024), smem_desc_sw128(k_addr + off, 16, 1024), idesc_s, 1);
-        }
-        tc_commit(&s_full[st]);
+        if (ok) tc_commit(q_free);
       }
-    }
-  } else if (warp == 2) {
-    if (lane == 0) {
+    } else if (warp == 2 && lane == 0) {
       // ---------------- O += P V issuer ----------------
-      const uint32_t idesc_o = idesc_bf16(BQ, (p.vdim + 15) / 16 * 16, false, true);    // V is N-contiguous
-      for (int s = 0; s < nstep; s++) {
-        const int st = s & 1, i = s / MAPS, m = s % MAPS, vt = i & 1;
-        if (!mbar_wait(&p_ready[st], (s >> 1) & 1, abort_flag, p.status)) break;
-        if (m == 0 && !mbar_wait(&v_full[vt], (i >> 1) & 1, abort_flag, p.status)) break;
-        tc_fence_after();
-        const uint32_t v_addr = smem_u32(sV + vt * v_bytes), tOm = tO + m * 128;
+      const uint32_t idesc_o = idesc_bf16(BQ, (p.cols + 15) / 16 * 16, false, true);    // V is N-contiguous
+      int n = 0, vc = 0, cx[2] = {0, 0};
+      bool ok = true;
+      for (int item = blockIdx.x; item < p.items && ok; item += gridDim.x, n++) {
+        const Item it(p, item);
+        for (int i = 0; i < it.ntile && ok; i++, vc++) {
+          const int vt = vc & 1;
+          const uint32_t v_addr = smem_u32(sV + vt * v_bytes);
 #pragma unroll
-        for (int k = 0; k < BKV / 16; k++) {
-          const uint64_t vd = smem_desc_sw128(v_addr + k * 2048, SLAB, 1024);
-          mma_ts(tOm, tS[st] + k * 8, vd, idesc_o, (i > 0 || k > 0) ? 1u : 0u);
-          if (SPLIT) mma_ts(tOm, tS[st] + BKV / 2 + k * 8, vd, idesc_o, 1u);
+          for (int m = 0; m < MAPS; m++) {
+            const int X = MAPS == 2 ? m : i & 1;
+            const bool fresh = MAPS == 2 ? i == 0 : i < 2;      // the stream's first step of the item overwrites O
+            if (!mbar_wait(&p_ready[X], (X ? cx[1] : cx[0]) & 1, abort_flag, p.status) ||
+                (m == 0 && !mbar_wait(&v_full[vt], (vc >> 1) & 1, abort_flag, p.status)) ||
+                (i == 0 && m == 0 && n >= 1 && !mbar_wait(o_free, (n - 1) & 1, abort_flag, p.status))) { ok = false; break; }
+            tc_fence_after();
+            const uint32_t tP = tmem_base + X * 128, tO = tmem_base + 256 + X * 128;
+#pragma unroll
+            for (int k = 0; k < BKV / 16; k++) {
+              const uint64_t vd = smem_desc_sw128(v_addr + k * 2048, SLAB, 1024);
+              // 32 keys: 16 columns of P and, with SPLIT, 16 columns of what rounding took from it
+              mma_ts(tO, tP + (k >> 1) * 32 + (k & 1) * 8, vd, idesc_o, (!fresh || k > 0) ? 1u : 0u);
+              if (SPLIT) mma_ts(tO, tP + (k >> 1) * 32 + 16 + (k & 1) * 8, vd, idesc_o, 1u);
+            }
+            tc_commit(&pv_done[X]);
+            if (X) cx[1]++; else cx[0]++;
+          }
+          if (ok) tc_commit(&v_free[vt]);
         }
-        tc_commit(&pv_done[st]);
-        if (m == MAPS - 1) tc_commit(&v_free[vt]);
       }
     }
-  } else if (warp >= 4) {
-    // ---------------- softmax: NS threads per query row, each owns CW = 128 / NS of the keys of a tile ----------------
-    const int quad = warp & 3;
-    const int hs = (warp - 4) >> 2;        // which CW keys of each tile; which 32-column chunks of O
+  } else {
+    // ---------------- softmax: stream X, two threads per query row, each owns CW of the keys of a tile ----------------
+    reg_alloc<REGS_SOFTMAX>();
+    const int quad = warp & 3, X = (warp - 4) >> 3, hs = ((warp - 4) >> 2) & 1;
     const int r = quad * 32 + lane;
-    const int q = p.first + q0 + r;        // position of this row's query
-    const bool row_ok = q0 + r < p.T;
     const uint32_t lane_off = (uint32_t)(quad * 32) << 16;
-    const int ochunks = (p.vdim + 31) / 32;
+    const uint32_t tS = tmem_base + X * 128 + hs * CW + lane_off, tO = tmem_base + 256 + lane_off;
+    const int ochunks = (p.cols + 31) / 32;
     const float c = p.c;
-    float m_row[MAPS], l_row[MAPS];      // l_row: this thread's share of the row sum (same m_row in all threads of a row)
-#pragma unroll
-    for (int m = 0; m < MAPS; m++) { m_row[m] = -INFINITY; l_row[m] = 0.f; }
+    const uint64_t c2 = pack2(c, c);
+    int cx[2] = {0, 0};
     bool ok = true;
-    for (int i = 0; i < ntile; i++) {
-      const int k0 = tile_key(i) + hs * CW;
-      // keys from k0 on that this row sees: [k0 + a0, k0 + a1)
-      const int a1 = i < nkeep ? kept - k0 : q + 1 - k0;
-      const int a0 = i < nkeep || k0 >= q + 1 - p.window ? 0 : q + 1 - p.window - k0;      // below a0 only kept tokens
-#pragma unroll
-      for (int m = 0; m < MAPS; m++) {
-        const int s = i * MAPS + m, st = s & 1;
-        float &m_used = m_row[m], &l = l_row[m];
-        // After a timed-out wait the warp keeps walking the loop (skipping the work) so that it still
-        // meets its partner warps at every row barrier.
-        if (ok && !mbar_wait(&s_full[st], (s >> 1) & 1, abort_flag, p.status)) ok = false;
+    for (int item = blockIdx.x; item < p.items; item += gridDim.x) {
+      const Item it(p, item);
+      const int q = p.first + it.q0 + r;       // position of this row's query
+      float m_used = -INFINITY, l = 0.f;       // l: this thread's share of the row sum (same m_used in both threads of a row)
+      const int steps = MAPS == 2 ? it.ntile : (it.ntile + 1 - X) / 2;
+      const int before = X ? cx[1] : cx[0];
+      for (int s = 0; s < steps; s++) {
+        const int turn = before + s, i = MAPS == 2 ? s : 2 * s + X;
+        const int k0 = it.key(i) + hs * CW;
+        // keys from k0 on that this row sees: [k0 + a0, k0 + a1), and below a0 the kept tokens
+        const int a1 = i < it.nkeep ? it.kept - k0 : q + 1 - k0;
+        const int a0 = i < it.nkeep ? 0 : q + 1 - p.window - k0;
+        const int ak = p.keep - k0;
+        // After a timed-out wait the warp keeps walking the loop (skipping the work) so that it still meets its partner
+        // warps at every barrier.
+        if (ok && !mbar_wait(&s_full[X], turn & 1, abort_flag, p.status)) ok = false;
         ok = __all_sync(0xffffffffu, ok);
-        if (!ok) { asm volatile("bar.sync %0, %1;" ::"r"(2 + quad), "n"(NS * 32) : "memory"); continue; }
         tc_fence_after();
-        float x[CW];
+        // Per group of 32 keys the warp decides together: every lane sees all of it, no lane sees any of it, or mixed.
+        bool mixed[CW / 32], empty[CW / 32];
 #pragma unroll
-        for (int u = 0; u < CW / 32; u++)
-          tmem_ld32(tS[st] + lane_off + hs * CW + u * 32, *reinterpret_cast<uint32_t(*)[32]>(&x[u * 32]));
-        tmem_ld_wait();
-        if (a1 < CW || a0 > 0) {
-#pragma unroll
-          for (int j = 0; j < CW; j++) x[j] = j < a1 && (j >= a0 || k0 + j < p.keep) ? x[j] : -INFINITY;
+        for (int u = 0; u < CW / 32; u++) {
+          mixed[u] = !__all_sync(0xffffffffu, a1 >= 32 * u + 32 && (a0 <= 32 * u || ak >= 32 * u + 32));
+          empty[u] = mixed[u] && __all_sync(0xffffffffu, a1 <= 32 * u || (a0 >= 32 * u + 32 && ak <= 32 * u));
         }
-        float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+        auto load = [&](int u, float (&x)[32]) {
+          tmem_ld32(tS + u * 32, reinterpret_cast<uint32_t(&)[32]>(x));
+          tmem_ld_wait();
+          if (mixed[u]) {
 #pragma unroll
-        for (int j = 0; j < CW; j += 4) {
-          mx[0] = fmaxf(mx[0], x[j]); mx[1] = fmaxf(mx[1], x[j + 1]);
-          mx[2] = fmaxf(mx[2], x[j + 2]); mx[3] = fmaxf(mx[3], x[j + 3]);
+            for (int j = 0; j < 32; j++) x[j] = 32 * u + j < a1 && (32 * u + j >= a0 || 32 * u + j < ak) ? x[j] : -INFINITY;
+          }
+        };
+        float mt = -INFINITY;
+        if (ok) {
+          float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+          for (int u = 0; u < CW / 32; u++) {
+            if (empty[u]) continue;
+            float x[32];
+            load(u, x);
+#pragma unroll
+            for (int j = 0; j < 32; j += 8) {
+              mx[0] = max3(mx[0], x[j], x[j + 1]); mx[1] = max3(mx[1], x[j + 2], x[j + 3]);
+              mx[2] = max3(mx[2], x[j + 4], x[j + 5]); mx[3] = max3(mx[3], x[j + 6], x[j + 7]);
+            }
+          }
+          mt = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * c;   // scaled units (c > 0 keeps the argmax)
         }
-        float mt = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * c;   // scaled units (c > 0 keeps the argmax)
-        // combine the partial row maxima; after this barrier every thread of the row holds its part of S in
-        // registers, so P may overwrite S in TMEM
-        xmax[st * (NS * 128) + hs * 128 + r] = mt;
-        asm volatile("bar.sync %0, %1;" ::"r"(2 + quad), "n"(NS * 32) : "memory");
-#pragma unroll
-        for (int o = 1; o < NS; o++) mt = fmaxf(mt, xmax[st * (NS * 128) + ((hs + o) % NS) * 128 + r]);
+        float* xe = xmax + ((turn & 1) * 2 + X) * (NS * 128);
+        xe[hs * 128 + r] = mt;
+        asm volatile("bar.sync %0, %1;" ::"r"(2 + 4 * X + quad), "n"(NS * 32) : "memory");
+        mt = fmaxf(mt, xe[(hs ^ 1) * 128 + r]);
+        if (!ok) continue;
         const bool grow = mt > m_used + 8.f || (m_used == -INFINITY && mt > -INFINITY);
         if (__any_sync(0xffffffffu, grow)) {
           const float m_new = fmaxf(m_used, mt);
           const float alpha = (m_used == -INFINITY) ? 0.f : fast_exp2(m_used - m_new);
           l *= alpha;
           m_used = m_new;
-          if (i > 0) {
-            // O lives in TMEM and is being accumulated by the tensor core: wait for this map's previous P V
-            bool w = mbar_wait(&pv_done[(s - MAPS) & 1], ((s - MAPS) >> 1) & 1, abort_flag, p.status);
+          if (s > 0) {
+            // O is being accumulated by the tensor core: wait for the stream's previous P V
+            bool w = mbar_wait(&pv_done[X], (turn - 1) & 1, abort_flag, p.status);
             w = __all_sync(0xffffffffu, w);
             if (!w) { ok = false; continue; }
             tc_fence_after();
             for (int u = hs; u < ochunks; u += NS) {
               uint32_t rr[32];
-              tmem_ld32(tO + m * 128 + lane_off + u * 32, rr);
+              tmem_ld32(tO + X * 128 + u * 32, rr);
               tmem_ld_wait();
 #pragma unroll
               for (int j = 0; j < 32; j++) rr[j] = __float_as_uint(__uint_as_float(rr[j]) * alpha);
-              tmem_st32(tO + m * 128 + lane_off + u * 32, rr);
+              tmem_st32(tO + X * 128 + u * 32, rr);
             }
             tmem_st_wait();
           }
         }
         const float mm = (m_used == -INFINITY) ? 0.f : m_used;
-        float sm[4] = {0.f, 0.f, 0.f, 0.f};
+        const uint64_t nm2 = pack2(-mm, -mm);
+        uint64_t sm2[2] = {0ull, 0ull};   // (+0, +0)
 #pragma unroll
         for (int u = 0; u < CW / 32; u++) {
           uint32_t pk[16], pl[16];
+          if (empty[u]) {
 #pragma unroll
-          for (int j = 0; j < 16; j += 2) {
-            const float p0 = fast_exp2(fmaf(x[u * 32 + 2 * j], c, -mm)), p1 = fast_exp2(fmaf(x[u * 32 + 2 * j + 1], c, -mm));
-            const float p2 = fast_exp2(fmaf(x[u * 32 + 2 * j + 2], c, -mm)), p3 = fast_exp2(fmaf(x[u * 32 + 2 * j + 3], c, -mm));
-            sm[0] += p0; sm[1] += p1; sm[2] += p2; sm[3] += p3;
-            pk[j] = pack_bf16(p0, p1);
-            pk[j + 1] = pack_bf16(p2, p3);
-            if (SPLIT) {
-              pl[j] = pack_bf16(p0 - bf16_low(pk[j]), p1 - bf16_high(pk[j]));
-              pl[j + 1] = pack_bf16(p2 - bf16_low(pk[j + 1]), p3 - bf16_high(pk[j + 1]));
+            for (int j = 0; j < 16; j++) pk[j] = pl[j] = 0u;
+          } else {
+            float x[32];
+            load(u, x);
+#pragma unroll
+            for (int j = 0; j < 16; j += 2) {
+              float t0, t1, t2, t3;
+              unpack2(fma2(pack2(x[2 * j], x[2 * j + 1]), c2, nm2), t0, t1);
+              unpack2(fma2(pack2(x[2 * j + 2], x[2 * j + 3]), c2, nm2), t2, t3);
+              const float p0 = fast_exp2(t0), p1 = fast_exp2(t1), p2 = fast_exp2(t2), p3 = fast_exp2(t3);
+              sm2[0] = add2(sm2[0], pack2(p0, p1));
+              sm2[1] = add2(sm2[1], pack2(p2, p3));
+              pk[j] = pack_bf16(p0, p1);
+              pk[j + 1] = pack_bf16(p2, p3);
+              if (SPLIT) {
+                pl[j] = pack_bf16(p0 - bf16_low(pk[j]), p1 - bf16_high(pk[j]));
+                pl[j + 1] = pack_bf16(p2 - bf16_low(pk[j + 1]), p3 - bf16_high(pk[j + 1]));
+              }
             }
           }
-          tmem_st16(tS[st] + lane_off + hs * (CW / 2) + u * 16, pk);
-          if (SPLIT) tmem_st16(tS[st] + BKV / 2 + lane_off + hs * (CW / 2) + u * 16, pl);
+          // over S columns that this thread has loaded for the last time
+          tmem_st16(tS + u * 32, pk);
+          if (SPLIT) tmem_st16(tS + u * 32 + 16, pl);
         }
-        l += (sm[0] + sm[1]) + (sm[2] + sm[3]);
+        {
+          float s0, s1, s2, s3;
+          unpack2(sm2[0], s0, s1);
+          unpack2(sm2[1], s2, s3);
+          l += (s0 + s1) + (s2 + s3);
+        }
         tmem_st_wait();
         tc_fence_before();
         __syncwarp();
-        if (lane == 0) mbar_arrive(&p_ready[st]);
+        if (lane == 0) mbar_arrive(&p_ready[X]);
       }
-    }
-    // 1 / (row sum), the sink's term included
-    float inv[MAPS];
-#pragma unroll
-    for (int m = 0; m < MAPS; m++) {
-      float l = l_row[m];
-      xl[hs * 128 + r] = l;
-      asm volatile("bar.sync %0, %1;" ::"r"(2 + quad), "n"(NS * 32) : "memory");
-#pragma unroll
-      for (int o = 1; o < NS; o++) l += xl[((hs + o) % NS) * 128 + r];
-      asm volatile("bar.sync %0, %1;" ::"r"(2 + quad), "n"(NS * 32) : "memory");
-      if (p.sink) {
-        const float z = __ldg(p.sink + h) * LOG2E, top = fmaxf(z, m_row[m]), f = fast_exp2(m_row[m] - top);
-        inv[m] = f / (l * f + fast_exp2(z - top));
-      } else {
-        inv[m] = 1.f / l;
-      }
-      const int s = (ntile - 1) * MAPS + m;
-      ok = ok && mbar_wait(&pv_done[s & 1], (s >> 1) & 1, abort_flag, p.status);
-    }
-    ok = __all_sync(0xffffffffu, ok);
-    if (ok) tc_fence_after();
-    const long long row = (long long)b * p.T + q0 + r;
-    float lam = 0.f, rms = 1.f;
-    if constexpr (MAPS == 2) {
-      // the head's own norm: mean square of a1 - lambda a2 over both threads of the row
-      lam = __ldg(p.lambda) * inv[1];
-      float ss = 0.f;
-      if (ok) {
-        for (int u = hs; u < ochunks; u += NS) {
-          uint32_t r1[32], r2[32];
-          tmem_ld32(tO + lane_off + u * 32, r1);
-          tmem_ld32(tO + 128 + lane_off + u * 32, r2);
-          tmem_ld_wait();
-#pragma unroll
-          for (int j = 0; j < 32; j++) {
-            const float v = __uint_as_float(r1[j]) * inv[0] - __uint_as_float(r2[j]) * lam;
-            ss += u * 32 + j < p.vdim ? v * v : 0.f;
-          }
+      cx[0] += MAPS == 2 ? it.ntile : (it.ntile + 1) / 2;
+      cx[1] += MAPS == 2 ? it.ntile : it.ntile / 2;
+      // ---- the item's result = f[0] O_0 + f[1] O_1; the four warps of a quad take 32 columns each ----
+      xl[(X * NS + hs) * 128 + r] = l;
+      if (hs == 0) xm[X * 128 + r] = m_used;
+      asm volatile("bar.sync %0, %1;" ::"r"(10 + quad), "n"(2 * NS * 32) : "memory");
+      const bool second = MAPS == 2 || it.ntile > 1;      // O_1 holds something
+      float f[2];
+      {
+        const float m0 = xm[r], m1 = xm[128 + r], l0 = xl[r] + xl[128 + r], l1 = xl[256 + r] + xl[384 + r];
+        const float z = p.sink ? __ldg(p.sink + it.h) * LOG2E : -INFINITY;
+        if constexpr (MAPS == 2) {
+          const float t0 = fmaxf(m0, z), t1 = fmaxf(m1, z), e0 = fast_exp2(m0 - t0), e1 = fast_exp2(m1 - t1);
+          f[0] = e0 / (l0 * e0 + fast_exp2(z - t0));
+          f[1] = -__ldg(p.lambda) * e1 / (l1 * e1 + fast_exp2(z - t1));
+        } else {
+          const float top = fmaxf(fmaxf(m0, m1), z), e0 = fast_exp2(m0 - top), e1 = fast_exp2(m1 - top);
+          const float inv = 1.f / (l0 * e0 + l1 * e1 + fast_exp2(z - top));
+          f[0] = e0 * inv; f[1] = e1 * inv;
         }
       }
-      xl[hs * 128 + r] = ss;
-      asm volatile("bar.sync %0, %1;" ::"r"(2 + quad), "n"(NS * 32) : "memory");
+      ok = ok && mbar_wait(&pv_done[0], (cx[0] - 1) & 1, abort_flag, p.status);
+      if (second) ok = ok && mbar_wait(&pv_done[1], (cx[1] - 1) & 1, abort_flag, p.status);
+      ok = __all_sync(0xffffffffu, ok);
+      const int u = X * NS + hs;
+      const bool mine = ok && u < ochunks;
+      float v[32];
+      if (mine) {
+        tc_fence_after();
+        tmem_ld32(tO + u * 32, reinterpret_cast<uint32_t(&)[32]>(v));
+        if (second) {
+          uint32_t v1[32];
+          tmem_ld32(tO + 128 + u * 32, v1);
+          tmem_ld_wait();
 #pragma unroll
-      for (int o = 1; o < NS; o++) ss += xl[((hs + o) % NS) * 128 + r];
-      rms = p.out_scale / sqrtf(ss / p.vdim + p.eps);
-    }
-    if (ok) {
-      if (p.gate_mode == FEMTO_GATE_HEAD && row_ok) rms *= 1.f / (1.f + expf(-__bfloat162float(p.gate[row * p.ld_gate + h])));
-      const bf16* gate = p.gate_mode == FEMTO_GATE_ELEMENT ? p.gate + row * p.ld_gate + (long long)h * p.vdim : nullptr;
-      bf16* o = p.o + (row * p.heads + h) * p.vdim;
-      for (int u = hs; u < ochunks; u += NS) {
-        uint32_t r1[32], r2[32];
-        tmem_ld32(tO + lane_off + u * 32, r1);
-        if constexpr (MAPS == 2) tmem_ld32(tO + 128 + lane_off + u * 32, r2);
-        tmem_ld_wait();
-        if (row_ok) {
+          for (int j = 0; j < 32; j++) v[j] = v[j] * f[0] + __uint_as_float(v1[j]) * f[1];
+        } else {
+          tmem_ld_wait();
 #pragma unroll
-          for (int j = 0; j < 32; j += 8) {
-            if (u * 32 + j < p.vdim) {
-              float v[8];
+          for (int j = 0; j < 32; j++) v[j] *= f[0];
+        }
+        tc_fence_before();
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(o_free);
+      const bool row_ok = it.q0 + r < p.T;
+      const long long row = (long long)it.b * p.T + it.q0 + r;
+      float mul = 1.f;
+      if constexpr (MAPS == 2) {      // the head's own norm
+        float ss = 0.f;
+        if (mine) {
 #pragma unroll
-              for (int e = 0; e < 8; e++) {
-                v[e] = __uint_as_float(r1[j + e]) * inv[0];
-                if constexpr (MAPS == 2) v[e] -= __uint_as_float(r2[j + e]) * lam;
-                v[e] *= rms;
-              }
-              if (gate) {
-                float z[8];
-                load_vec<bf16, 8>(gate + u * 32 + j, z);
+          for (int j = 0; j < 32; j++) ss += u * 32 + j < p.cols ? v[j] * v[j] : 0.f;
+        }
+        xs[u * 128 + r] = ss;
+        asm volatile("bar.sync %0, %1;" ::"r"(10 + quad), "n"(2 * NS * 32) : "memory");
+        ss = (xs[r] + xs[128 + r]) + (xs[256 + r] + xs[384 + r]);
+        mul = p.out_scale / sqrtf(ss / p.cols + p.eps);
+      }
+      if (mine && row_ok) {
+        if (p.gate_mode == FEMTO_GATE_HEAD) mul *= 1.f / (1.f + expf(-__bfloat162float(p.gate[row * p.ld_gate + it.h])));
+        const bf16* gate = p.gate_mode == FEMTO_GATE_ELEMENT ? p.gate + row * p.ld_gate + (long long)it.h * p.vdim + p.col0 + u * 32 : nullptr;
+        bf16* o = p.o + (row * p.heads + it.h) * p.vdim + p.col0 + u * 32;
 #pragma unroll
-                for (int e = 0; e < 8; e++) v[e] *= __fdividef(1.f, 1.f + __expf(-z[e]));
-              }
-              store_vec<bf16, 8>(o + u * 32 + j, v);
+        for (int j = 0; j < 32; j += 8) {
+          if (u * 32 + j < p.cols) {
+            float w[8];
+#pragma unroll
+            for (int e = 0; e < 8; e++) w[e] = v[j + e] * mul;
+            if (gate) {
+              float z[8];
+              load_vec<bf16, 8>(gate + j, z);
+#pragma unroll
+              for (int e = 0; e < 8; e++) w[e] *= __fdividef(1.f, 1.f + __expf(-z[e]));
             }
+            store_vec<bf16, 8>(o + j, w);
           }
         }
       }
@@ -377,19 +456,26 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
 }
 
 int slabs(int n) { return (n + 63) / 64; }
-size_t smem_bytes(int maps, int nqk, int nv) { return (size_t)SLAB * ((maps + 2) * nqk + 2 * nv) + 1024 + 256 + 3 * NS * 128 * 4; }
+size_t smem_bytes(int maps, int nqk, int nv) { return (size_t)SLAB * ((maps + 2) * nqk + 2 * nv) + 1024 + 256 + 14 * 128 * 4 + 4 * 128 * 4; }
 
 template <int MAPS, bool SPLIT>
 int launch(const CUtensorMap& tmQu, const CUtensorMap& tmQr, const CUtensorMap& tmKu, const CUtensorMap& tmKr, const CUtensorMap& tmV,
-           const SlabAttn& p, int B, cudaStream_t s) {
+           SlabAttn p, int B, cudaStream_t s) {
   static PerDevice attr;
   const int dev = PerDevice::current();
   if (dev < 0 || !attr.done[dev]) {
     CUDA_TRY(cudaFuncSetAttribute(slab_attn_kernel<MAPS, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     if (dev >= 0) attr.done[dev] = true;
   }
-  slab_attn_kernel<MAPS, SPLIT><<<dim3(cdiv(p.T, BQ), p.heads, B), THREADS, smem_bytes(MAPS, p.n_un + p.n_rot, p.n_v), s>>>(tmQu, tmQr, tmKu, tmKr, tmV, p);
-  KERNEL_CHECK();
+  p.qtiles = cdiv(p.T, BQ);
+  p.items = p.qtiles * p.heads * B;
+  const int grid = std::min(p.items, device_sm_count());
+  for (p.col0 = 0; p.col0 < p.vdim; p.col0 += MAX_V) {      // wide values: the attention once per 128 columns
+    p.cols = std::min(MAX_V, p.vdim - p.col0);
+    p.n_v = slabs(p.cols);
+    CUDA_TRY(launch_dependent(slab_attn_kernel<MAPS, SPLIT>, grid, THREADS, smem_bytes(MAPS, p.n_un + p.n_rot, p.n_v), s, tmQu, tmQr, tmKu, tmKr, tmV, p));
+    KERNEL_CHECK();
+  }
   return 0;
 }
 
@@ -397,7 +483,7 @@ int launch(const CUtensorMap& tmQu, const CUtensorMap& tmQr, const CUtensorMap& 
 
 bool latent_attention_tc_supported(const LatentArgs& a) {
   if ((a.dim | a.rot_dim | a.vdim) & 7 || a.vdim > 256 || !(a.scale > 0.f)) return false;
-  if (3 * (slabs(a.dim) + slabs(a.rot_dim)) + 2 * slabs(a.vdim) > MAX_SLABS) return false;
+  if (3 * (slabs(a.dim) + slabs(a.rot_dim)) + 2 * slabs(std::min(a.vdim, MAX_V)) > MAX_SLABS) return false;
   return aligned16(a.q) && aligned16(a.kv) && aligned16(a.latent) && aligned16(a.o);
 }
 
@@ -429,14 +515,14 @@ int latent_attention_tc(const LatentArgs& a, cudaStream_t s) {
   SlabAttn p = {};
   p.o = (bf16*)a.o; p.gate = (const bf16*)a.gate; p.status = a.d->status; p.ld_gate = a.ld_gate; p.gate_mode = FEMTO_GATE_HEAD;
   p.T = a.T; p.first = a.first; p.N = (int)N; p.heads = a.heads; p.per = 1; p.vdim = a.vdim; p.window = 1 << 30;
-  p.n_un = slabs(a.dim); p.n_rot = slabs(a.rot_dim); p.n_v = slabs(a.vdim);
+  p.n_un = slabs(a.dim); p.n_rot = slabs(a.rot_dim);
   p.k_un = cdiv(a.dim, 16); p.k_rot = cdiv(a.rot_dim, 16); p.c = a.scale * LOG2E;
   return launch<1, false>(tmQu, tmQr, tmKu, tmKr, tmV, p, a.B, s);
 }
 
 bool window_attention_tc_supported(const WindowAttnArgs& a) {
-  if ((a.dim | a.vdim) & 7 || a.vdim > (a.maps == 2 ? 128 : 256) || !(a.scale > 0.f)) return false;
-  if ((a.maps + 2) * slabs(a.dim) + 2 * slabs(a.vdim) > MAX_SLABS) return false;
+  if ((a.dim | a.vdim) & 7 || a.vdim > (a.maps == 2 ? MAX_V : 256) || !(a.scale > 0.f)) return false;
+  if ((a.maps + 2) * slabs(a.dim) + 2 * slabs(std::min(a.vdim, MAX_V)) > MAX_SLABS) return false;
   if ((a.ldq | a.ld | a.vo | a.ld_gate) & 7) return false;
   return aligned16(a.q) && aligned16(a.kv) && aligned16(a.o) && (a.gate_mode != FEMTO_GATE_ELEMENT || aligned16(a.gate));
 }
@@ -463,6 +549,6 @@ int window_attention_tc(const WindowAttnArgs& a, cudaStream_t s) {
   p.o = (bf16*)a.o; p.gate = (const bf16*)a.gate; p.status = a.status; p.ld_gate = a.ld_gate; p.gate_mode = a.gate_mode;
   p.T = a.T; p.first = a.first; p.N = (int)N; p.heads = a.heads; p.per = a.heads / a.kv_heads; p.vdim = a.vdim;
   p.window = a.window; p.keep = a.keep; p.sink = a.sink; p.lambda = a.lambda; p.out_scale = a.out_scale; p.eps = a.eps;
-  p.n_un = slabs(a.dim); p.n_v = slabs(a.vdim); p.k_un = cdiv(a.dim, 16); p.c = a.scale * LOG2E;
+  p.n_un = slabs(a.dim); p.k_un = cdiv(a.dim, 16); p.c = a.scale * LOG2E;
   return a.maps == 2 ? launch<2, true>(tmQ, tmQ, tmK, tmK, tmV, p, a.B, s) : launch<1, true>(tmQ, tmQ, tmK, tmK, tmV, p, a.B, s);
 }
