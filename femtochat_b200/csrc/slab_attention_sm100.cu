@@ -6,14 +6,14 @@
 //   cache rows that all heads share.
 //   Windowed attention: the key tiles are those of the first `keep` tokens and then those of the window; groups of query
 //   heads share a key/value head; a sink enters the sum at the end.  The softmax weights enter P V as the sum of two bf16
-//   numbers (SPLIT), so they keep 32-bit accuracy: a tile's P takes the 128 columns that held its S.
+//   numbers (SPLIT), so they keep 32-bit accuracy: a tile's P takes the columns that held its S.
 //
 // One CTA per SM walks the items (128 queries of one head), latest queries first.  The steps of an item, 128 queries against
-// 128 keys, alternate between two streams, each with a buffer for S / P and an accumulator O of its own in tensor memory and
-// eight softmax warps (two threads per query row), so that the exponentials of one stream run beside the products, the
-// loads and the row maxima of the other.  With two maps (differential attention) the streams are the maps, otherwise the
-// even and the odd key tiles, whose partial results meet at the end.  A TMA warp streams Q, K and V (two stages of K and V),
-// one thread issues S = Q K^T, another O += P V with P read back from tensor memory; all of them run ahead into the next item.
+// 64 keys, alternate between two streams, each with two buffers for S / P and an accumulator O of its own in tensor memory and
+// four softmax warps (one thread per query row): S of a stream's next step is there before the softmax of this one is
+// done, and the exponentials of one stream run beside the loads and the row maxima of the other.  With two maps (differential attention) the streams are the maps, otherwise the
+// even and the odd key tiles, whose partial results meet at the end.  A TMA warp streams Q, K and V (four stages of K and V),
+// one warp issues S = Q K^T, another O += P V with P read back from tensor memory; all of them run ahead into the next item.
 // Sum of the streams, the head's own norm of differential attention and the output gate are applied as the result leaves.
 #include <algorithm>
 
@@ -24,14 +24,12 @@ using namespace sm100;
 
 namespace {
 
-constexpr int BQ = 128, BKV = 128, NS = 2, CW = BKV / NS, THREADS = 128 + 2 * NS * 128;
-constexpr int SLAB = 128 * 64 * 2;                    // one box: 128 tokens x 64 channels
-constexpr int MAX_SLABS = 13;                         // 16 KB each: (maps + 2) per query/key slab (Q + two K stages), 2 per value slab
+constexpr int BQ = 128, BKV = 64, THREADS = 128 + 2 * 128;
+constexpr int STAGES = 4;                             // of K and of V
+constexpr int SLAB_Q = BQ * 64 * 2, SLAB = BKV * 64 * 2;   // one box: 128 queries or 64 keys x 64 channels
+constexpr int MAX_SLABS = 26;                         // 8 KB each: 2 maps + STAGES per query/key slab, STAGES per value slab
 constexpr int MAX_V = 128;                            // value columns of one launch
 constexpr float LOG2E = 1.4426950408889634f;
-// registers per thread: launched with 96 (640 threads); the first warpgroup's surplus goes to the softmax warps
-constexpr int REGS_ROLES = 32, REGS_SOFTMAX = 112;
-
 struct SlabAttn {
   bf16* o; const bf16* gate; unsigned int* status;
   long long ld_gate;
@@ -73,6 +71,16 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 __device__ __forceinline__ float bf16_low(uint32_t v) { return __uint_as_float(v << 16); }
 __device__ __forceinline__ float bf16_high(uint32_t v) { return __uint_as_float(v & 0xffff0000u); }
 
+// S (+)= Q K^T over `steps` groups of 16 channels.  A descriptor counts in units of 16 bytes: 16 channels further are 2 of them.
+__device__ __forceinline__ void issue_slabs(uint32_t tS, uint64_t qd, uint64_t kd, int steps, bool accumulate, uint32_t idesc) {
+  for (; steps > 0; steps -= 4, qd += SLAB_Q >> 4, kd += SLAB >> 4) {
+#pragma unroll
+    for (int k = 0; k < 4; k++)
+      if (k < steps) mma_ss(tS, qd + 2 * k, kd + 2 * k, idesc, k > 0 || accumulate);
+    accumulate = true;
+  }
+}
+
 template <int MAPS, bool SPLIT>
 __global__ void __launch_bounds__(THREADS, 1)
 slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant__ CUtensorMap tmQr,
@@ -81,34 +89,33 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
   grid_launch_dependents();
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-  const int q_bytes = (p.n_un + p.n_rot) * SLAB, v_bytes = p.n_v * SLAB;
+  const int q_bytes = (p.n_un + p.n_rot) * SLAB_Q, k_bytes = (p.n_un + p.n_rot) * SLAB, v_bytes = p.n_v * SLAB;
   uint8_t* sQ = smem;
-  uint8_t* sK = sQ + MAPS * q_bytes;     // 2 stages
-  uint8_t* sV = sK + 2 * q_bytes;        // 2 stages
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * v_bytes);
+  uint8_t* sK = sQ + MAPS * q_bytes;
+  uint8_t* sV = sK + STAGES * k_bytes;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + STAGES * v_bytes);
   uint64_t* q_full = bars;
   uint64_t* q_free = bars + 1;    // the item's last S has been executed
-  uint64_t* k_full = bars + 2;    // [2 stages]
-  uint64_t* k_free = bars + 4;    // [2 stages]
-  uint64_t* v_full = bars + 6;    // [2 stages]
-  uint64_t* v_free = bars + 8;    // [2 stages]
-  uint64_t* s_full = bars + 10;   // [2 streams]
-  uint64_t* p_ready = bars + 12;  // [2 streams]
-  uint64_t* pv_done = bars + 14;  // [2 streams] a step's P V has been accumulated; also frees the stream's S / P buffer
-  uint64_t* o_free = bars + 16;   // every softmax warp has read the item's O
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 17);
+  uint64_t* o_free = bars + 2;    // every softmax warp has read the item's O
+  uint64_t* k_full = bars + 3;    // [STAGES]
+  uint64_t* k_free = bars + 7;    // [STAGES]
+  uint64_t* v_full = bars + 11;   // [STAGES]
+  uint64_t* v_free = bars + 15;   // [STAGES]
+  uint64_t* s_full = bars + 19;   // [2 streams][2 buffers]
+  uint64_t* p_ready = bars + 23;  // [2 streams][2 buffers]
+  uint64_t* pv_done = bars + 27;  // [2 streams][2 buffers] a step's P V has been accumulated; also frees its S / P buffer
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 31);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  float* xmax = reinterpret_cast<float*>(bars + 32);   // [2 parities][2 streams][NS][128 rows]
-  float* xl = xmax + 4 * NS * 128;                     // [2 streams][NS][128 rows]
-  float* xm = xl + 2 * NS * 128;                       // [2 streams][128 rows]
-  float* xs = xm + 2 * 128;                            // [2 streams][NS][128 rows]
+  float* xl = reinterpret_cast<float*>(bars + 32);     // [2 streams][128 rows] row sums, maxima, squares of the results
+  float* xm = xl + 2 * 128;
+  float* xs = xm + 2 * 128;
 
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    mbar_init(q_full, 1); mbar_init(q_free, 1); mbar_init(o_free, 4 * NS * 2);
-    for (int i = 0; i < 2; i++) {
+    mbar_init(q_full, 1); mbar_init(q_free, 1); mbar_init(o_free, 8);
+    for (int i = 0; i < 4; i++) {
       mbar_init(&k_full[i], 1); mbar_init(&k_free[i], 1); mbar_init(&v_full[i], 1); mbar_init(&v_free[i], 1);
-      mbar_init(&s_full[i], 1); mbar_init(&p_ready[i], NS * 4); mbar_init(&pv_done[i], 1);
+      mbar_init(&s_full[i], 1); mbar_init(&p_ready[i], 4); mbar_init(&pv_done[i], 1);
     }
     *abort_flag = 0;
     fence_barrier_init();
@@ -122,41 +129,46 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
   grid_dependency_wait();
 
   // Every role walks the same items in the same order and counts what it has seen: n items, kc key tiles, vc value tiles, cx[X]
-  // steps of stream X.  The phase of a barrier is that count (of its stage's turns), modulo two.
+  // steps of stream X (its turn t uses buffer t & 1).  The phase of a barrier is the count of its own turns, modulo two.
   if (warp < 4) {
-    reg_dealloc<REGS_ROLES>();
-    if (warp == 0 && lane == 0) {
+    if (warp == 0) {
       // ---------------- TMA producer ----------------
       int n = 0, kc = 0, vc = 0;
       bool ok = true;
       for (int item = blockIdx.x; item < p.items && ok; item += gridDim.x) {
         const Item it(p, item);
         const int hk = it.h / p.per;
-        if (n >= 1 && !mbar_wait(q_free, (n - 1) & 1, abort_flag, p.status)) break;
-        mbar_expect_tx(q_full, MAPS * q_bytes);
+        if (n >= 1 && !mbar_wait_warp(q_free, (n - 1) & 1, abort_flag, p.status)) break;
+        if (elect_one()) {
+          mbar_expect_tx(q_full, MAPS * q_bytes);
 #pragma unroll
-        for (int m = 0; m < MAPS; m++) {
-          for (int j = 0; j < p.n_un; j++) tma_load_4d(sQ + m * q_bytes + j * SLAB, &tmQu, q_full, j * 64, it.h * MAPS + m, it.q0, it.b);
-          for (int j = 0; j < p.n_rot; j++) tma_load_4d(sQ + m * q_bytes + (p.n_un + j) * SLAB, &tmQr, q_full, j * 64, it.h * MAPS + m, it.q0, it.b);
+          for (int m = 0; m < MAPS; m++) {
+            for (int j = 0; j < p.n_un; j++) tma_load_4d(sQ + m * q_bytes + j * SLAB_Q, &tmQu, q_full, j * 64, it.h * MAPS + m, it.q0, it.b);
+            for (int j = 0; j < p.n_rot; j++) tma_load_4d(sQ + m * q_bytes + (p.n_un + j) * SLAB_Q, &tmQr, q_full, j * 64, it.h * MAPS + m, it.q0, it.b);
+          }
         }
         n++;
         for (int i = 0; i < it.ntile && ok; i++) {
           const int key = it.key(i);
 #pragma unroll
           for (int m = 0; m < MAPS; m++) {
-            const int st = kc & 1;
-            if (kc >= 2 && !mbar_wait(&k_free[st], ((kc - 2) >> 1) & 1, abort_flag, p.status)) { ok = false; break; }
-            uint8_t* k = sK + st * q_bytes;
-            mbar_expect_tx(&k_full[st], q_bytes);
-            for (int j = 0; j < p.n_un; j++) tma_load_4d(k + j * SLAB, &tmKu, &k_full[st], j * 64, hk * MAPS + m, key, it.b);
-            for (int j = 0; j < p.n_rot; j++) tma_load_3d(k + (p.n_un + j) * SLAB, &tmKr, &k_full[st], j * 64, key, it.b);
+            const int st = kc % STAGES;
+            if (kc >= STAGES && !mbar_wait_warp(&k_free[st], (kc / STAGES - 1) & 1, abort_flag, p.status)) { ok = false; break; }
+            if (elect_one()) {
+              uint8_t* k = sK + st * k_bytes;
+              mbar_expect_tx(&k_full[st], k_bytes);
+              for (int j = 0; j < p.n_un; j++) tma_load_4d(k + j * SLAB, &tmKu, &k_full[st], j * 64, hk * MAPS + m, key, it.b);
+              for (int j = 0; j < p.n_rot; j++) tma_load_3d(k + (p.n_un + j) * SLAB, &tmKr, &k_full[st], j * 64, key, it.b);
+            }
             kc++;
           }
-          const int vt = vc & 1;
-          if (!ok || (vc >= 2 && !mbar_wait(&v_free[vt], ((vc - 2) >> 1) & 1, abort_flag, p.status))) { ok = false; break; }
-          uint8_t* v = sV + vt * v_bytes;
-          mbar_expect_tx(&v_full[vt], v_bytes);
-          for (int j = 0; j < p.n_v; j++) tma_load_4d(v + j * SLAB, &tmV, &v_full[vt], p.col0 + j * 64, hk, key, it.b);
+          const int vt = vc % STAGES;
+          if (!ok || (vc >= STAGES && !mbar_wait_warp(&v_free[vt], (vc / STAGES - 1) & 1, abort_flag, p.status))) { ok = false; break; }
+          if (elect_one()) {
+            uint8_t* v = sV + vt * v_bytes;
+            mbar_expect_tx(&v_full[vt], v_bytes);
+            for (int j = 0; j < p.n_v; j++) tma_load_4d(v + j * SLAB, &tmV, &v_full[vt], p.col0 + j * 64, hk, key, it.b);
+          }
           vc++;
         }
       }
@@ -164,82 +176,82 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
         // let loads already in flight land before the CTA exits
         auto drain = [&](uint64_t* bar, int turn) { for (uint32_t t = 0; t < WAIT_LIMIT && !mbar_try_wait(bar, turn & 1); ++t) {} };
         if (n >= 1) drain(q_full, n - 1);
-        for (int i = max(0, kc - 2); i < kc; i++) drain(&k_full[i & 1], i >> 1);
-        for (int i = max(0, vc - 2); i < vc; i++) drain(&v_full[i & 1], i >> 1);
+        for (int i = max(0, kc - STAGES); i < kc; i++) drain(&k_full[i % STAGES], i / STAGES);
+        for (int i = max(0, vc - STAGES); i < vc; i++) drain(&v_full[i % STAGES], i / STAGES);
       }
-    } else if (warp == 1 && lane == 0) {
+    } else if (warp == 1) {
       // ---------------- S = Q K^T issuer ----------------
       constexpr uint32_t idesc_s = idesc_bf16(BQ, BKV, false, false);  // both operands K-major
+      const uint64_t q_desc = smem_desc_sw128(smem_u32(sQ), 16, 1024), k_desc = smem_desc_sw128(smem_u32(sK), 16, 1024);
       int n = 0, kc = 0, cx[2] = {0, 0};
       bool ok = true;
       for (int item = blockIdx.x; item < p.items && ok; item += gridDim.x, n++) {
         const Item it(p, item);
-        if (!mbar_wait(q_full, n & 1, abort_flag, p.status)) break;
+        if (!mbar_wait_warp(q_full, n & 1, abort_flag, p.status)) break;
         for (int i = 0; i < it.ntile && ok; i++) {
 #pragma unroll
           for (int m = 0; m < MAPS; m++, kc++) {
-            const int X = MAPS == 2 ? m : i & 1, st = kc & 1;
-            const int turns = X ? cx[1] : cx[0];
-            // S overwrites the buffer that held the stream's previous P: its P V must have been executed
-            if (!mbar_wait(&k_full[st], (kc >> 1) & 1, abort_flag, p.status) ||
-                (turns >= 1 && !mbar_wait(&pv_done[X], (turns - 1) & 1, abort_flag, p.status))) { ok = false; break; }
+            const int X = MAPS == 2 ? m : i & 1, st = kc % STAGES;
+            const int turn = X ? cx[1] : cx[0], xb = 2 * X + (turn & 1);
+            // S overwrites the buffer that held P of the stream's last step but one: its P V must have been executed
+            if (!mbar_wait_warp(&k_full[st], (kc / STAGES) & 1, abort_flag, p.status) ||
+                (turn >= 2 && !mbar_wait_warp(&pv_done[xb], ((turn - 2) >> 1) & 1, abort_flag, p.status))) { ok = false; break; }
             tc_fence_after();
-            const uint32_t k_addr = smem_u32(sK + st * q_bytes), q_addr = smem_u32(sQ) + m * q_bytes, tS = tmem_base + X * 128;
-            for (int k = 0; k < p.k_un; k++) {
-              const uint32_t off = (k >> 2) * SLAB + (k & 3) * 32;
-              mma_ss(tS, smem_desc_sw128(q_addr + off, 16, 1024), smem_desc_sw128(k_addr + off, 16, 1024), idesc_s, k > 0);
+            const uint32_t tS = tmem_base + xb * BKV;
+            const uint64_t qd = q_desc + (uint32_t)(m * q_bytes >> 4), kd = k_desc + (uint32_t)(st * k_bytes >> 4);
+            if (elect_one()) {
+              issue_slabs(tS, qd, kd, p.k_un, false, idesc_s);
+              if (p.k_rot) issue_slabs(tS, qd + (uint32_t)(p.n_un * SLAB_Q >> 4), kd + (uint32_t)(p.n_un * SLAB >> 4), p.k_rot, true, idesc_s);
+              tc_commit(&s_full[xb]);
+              tc_commit(&k_free[st]);
+              if (i == it.ntile - 1 && m == MAPS - 1) tc_commit(q_free);
             }
-            for (int k = 0; k < p.k_rot; k++) {
-              const uint32_t off = (p.n_un + (k >> 2)) * SLAB + (k & 3) * 32;
-              mma_ss(tS, smem_desc_sw128(q_addr + off, 16, 1024), smem_desc_sw128(k_addr + off, 16, 1024), idesc_s, 1);
-            }
-            tc_commit(&s_full[X]);
-            tc_commit(&k_free[st]);
             if (X) cx[1]++; else cx[0]++;
           }
         }
-        if (ok) tc_commit(q_free);
       }
-    } else if (warp == 2 && lane == 0) {
+    } else if (warp == 2) {
       // ---------------- O += P V issuer ----------------
+      const uint64_t v_desc = smem_desc_sw128(smem_u32(sV), SLAB, 1024);
       const uint32_t idesc_o = idesc_bf16(BQ, (p.cols + 15) / 16 * 16, false, true);    // V is N-contiguous
       int n = 0, vc = 0, cx[2] = {0, 0};
       bool ok = true;
       for (int item = blockIdx.x; item < p.items && ok; item += gridDim.x, n++) {
         const Item it(p, item);
         for (int i = 0; i < it.ntile && ok; i++, vc++) {
-          const int vt = vc & 1;
-          const uint32_t v_addr = smem_u32(sV + vt * v_bytes);
+          const int vt = vc % STAGES;
+          const uint64_t vd = v_desc + (uint32_t)(vt * v_bytes >> 4);
 #pragma unroll
           for (int m = 0; m < MAPS; m++) {
             const int X = MAPS == 2 ? m : i & 1;
+            const int turn = X ? cx[1] : cx[0], xb = 2 * X + (turn & 1);
             const bool fresh = MAPS == 2 ? i == 0 : i < 2;      // the stream's first step of the item overwrites O
-            if (!mbar_wait(&p_ready[X], (X ? cx[1] : cx[0]) & 1, abort_flag, p.status) ||
-                (m == 0 && !mbar_wait(&v_full[vt], (vc >> 1) & 1, abort_flag, p.status)) ||
-                (i == 0 && m == 0 && n >= 1 && !mbar_wait(o_free, (n - 1) & 1, abort_flag, p.status))) { ok = false; break; }
+            if (!mbar_wait_warp(&p_ready[xb], (turn >> 1) & 1, abort_flag, p.status) ||
+                (m == 0 && !mbar_wait_warp(&v_full[vt], (vc / STAGES) & 1, abort_flag, p.status)) ||
+                (i == 0 && m == 0 && n >= 1 && !mbar_wait_warp(o_free, (n - 1) & 1, abort_flag, p.status))) { ok = false; break; }
             tc_fence_after();
-            const uint32_t tP = tmem_base + X * 128, tO = tmem_base + 256 + X * 128;
+            const uint32_t tP = tmem_base + xb * BKV, tO = tmem_base + 256 + X * 128;
+            if (elect_one()) {
 #pragma unroll
-            for (int k = 0; k < BKV / 16; k++) {
-              const uint64_t vd = smem_desc_sw128(v_addr + k * 2048, SLAB, 1024);
-              // 32 keys: 16 columns of P and, with SPLIT, 16 columns of what rounding took from it
-              mma_ts(tO, tP + (k >> 1) * 32 + (k & 1) * 8, vd, idesc_o, (!fresh || k > 0) ? 1u : 0u);
-              if (SPLIT) mma_ts(tO, tP + (k >> 1) * 32 + 16 + (k & 1) * 8, vd, idesc_o, 1u);
+              for (int k = 0; k < BKV / 16; k++) {
+                // 32 keys: 16 columns of P and, with SPLIT, 16 columns of what rounding took from it; 16 keys of V are 2048 bytes
+                mma_ts(tO, tP + (k >> 1) * 32 + (k & 1) * 8, vd + k * 128, idesc_o, (!fresh || k > 0) ? 1u : 0u);
+                if (SPLIT) mma_ts(tO, tP + (k >> 1) * 32 + 16 + (k & 1) * 8, vd + k * 128, idesc_o, 1u);
+              }
+              tc_commit(&pv_done[xb]);
+              if (m == MAPS - 1) tc_commit(&v_free[vt]);
             }
-            tc_commit(&pv_done[X]);
             if (X) cx[1]++; else cx[0]++;
           }
-          if (ok) tc_commit(&v_free[vt]);
         }
       }
     }
   } else {
-    // ---------------- softmax: stream X, two threads per query row, each owns CW of the keys of a tile ----------------
-    reg_alloc<REGS_SOFTMAX>();
-    const int quad = warp & 3, X = (warp - 4) >> 3, hs = ((warp - 4) >> 2) & 1;
+    // ---------------- softmax: stream X (four warps each), one thread per query row ----------------
+    const int quad = warp & 3, X = (warp - 4) >> 2;
     const int r = quad * 32 + lane;
     const uint32_t lane_off = (uint32_t)(quad * 32) << 16;
-    const uint32_t tS = tmem_base + X * 128 + hs * CW + lane_off, tO = tmem_base + 256 + lane_off;
+    const uint32_t tO = tmem_base + 256 + lane_off;
     const int ochunks = (p.cols + 31) / 32;
     const float c = p.c;
     const uint64_t c2 = pack2(c, c);
@@ -248,57 +260,48 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
     for (int item = blockIdx.x; item < p.items; item += gridDim.x) {
       const Item it(p, item);
       const int q = p.first + it.q0 + r;       // position of this row's query
-      float m_used = -INFINITY, l = 0.f;       // l: this thread's share of the row sum (same m_used in both threads of a row)
+      float m_used = -INFINITY, l = 0.f;
       const int steps = MAPS == 2 ? it.ntile : (it.ntile + 1 - X) / 2;
       const int before = X ? cx[1] : cx[0];
-      for (int s = 0; s < steps; s++) {
-        const int turn = before + s, i = MAPS == 2 ? s : 2 * s + X;
-        const int k0 = it.key(i) + hs * CW;
+      for (int s = 0; s < steps && ok; s++) {
+        const int turn = before + s, i = MAPS == 2 ? s : 2 * s + X, xb = 2 * X + (turn & 1);
+        const uint32_t tS = tmem_base + xb * BKV + lane_off;
+        const int k0 = it.key(i);
         // keys from k0 on that this row sees: [k0 + a0, k0 + a1), and below a0 the kept tokens
         const int a1 = i < it.nkeep ? it.kept - k0 : q + 1 - k0;
         const int a0 = i < it.nkeep ? 0 : q + 1 - p.window - k0;
         const int ak = p.keep - k0;
-        // After a timed-out wait the warp keeps walking the loop (skipping the work) so that it still meets its partner
-        // warps at every barrier.
-        if (ok && !mbar_wait(&s_full[X], turn & 1, abort_flag, p.status)) ok = false;
+        ok = mbar_wait(&s_full[xb], (turn >> 1) & 1, abort_flag, p.status);
         ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
         tc_fence_after();
         // Per group of 32 keys the warp decides together: every lane sees all of it, no lane sees any of it, or mixed.
-        bool mixed[CW / 32], empty[CW / 32];
+        bool mixed[2], empty[2];
 #pragma unroll
-        for (int u = 0; u < CW / 32; u++) {
+        for (int u = 0; u < 2; u++) {
           mixed[u] = !__all_sync(0xffffffffu, a1 >= 32 * u + 32 && (a0 <= 32 * u || ak >= 32 * u + 32));
           empty[u] = mixed[u] && __all_sync(0xffffffffu, a1 <= 32 * u || (a0 >= 32 * u + 32 && ak <= 32 * u));
         }
-        auto load = [&](int u, float (&x)[32]) {
-          tmem_ld32(tS + u * 32, reinterpret_cast<uint32_t(&)[32]>(x));
-          tmem_ld_wait();
+        float x[2][32];
+#pragma unroll
+        for (int u = 0; u < 2; u++)
+          if (!empty[u]) tmem_ld32(tS + u * 32, reinterpret_cast<uint32_t(&)[32]>(x[u]));
+        tmem_ld_wait();
+        float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+        for (int u = 0; u < 2; u++) {
+          if (empty[u]) continue;
           if (mixed[u]) {
 #pragma unroll
-            for (int j = 0; j < 32; j++) x[j] = 32 * u + j < a1 && (32 * u + j >= a0 || 32 * u + j < ak) ? x[j] : -INFINITY;
+            for (int j = 0; j < 32; j++) x[u][j] = 32 * u + j < a1 && (32 * u + j >= a0 || 32 * u + j < ak) ? x[u][j] : -INFINITY;
           }
-        };
-        float mt = -INFINITY;
-        if (ok) {
-          float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-          for (int u = 0; u < CW / 32; u++) {
-            if (empty[u]) continue;
-            float x[32];
-            load(u, x);
-#pragma unroll
-            for (int j = 0; j < 32; j += 8) {
-              mx[0] = max3(mx[0], x[j], x[j + 1]); mx[1] = max3(mx[1], x[j + 2], x[j + 3]);
-              mx[2] = max3(mx[2], x[j + 4], x[j + 5]); mx[3] = max3(mx[3], x[j + 6], x[j + 7]);
-            }
+          for (int j = 0; j < 32; j += 8) {
+            mx[0] = max3(mx[0], x[u][j], x[u][j + 1]); mx[1] = max3(mx[1], x[u][j + 2], x[u][j + 3]);
+            mx[2] = max3(mx[2], x[u][j + 4], x[u][j + 5]); mx[3] = max3(mx[3], x[u][j + 6], x[u][j + 7]);
           }
-          mt = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * c;   // scaled units (c > 0 keeps the argmax)
         }
-        float* xe = xmax + ((turn & 1) * 2 + X) * (NS * 128);
-        xe[hs * 128 + r] = mt;
-        asm volatile("bar.sync %0, %1;" ::"r"(2 + 4 * X + quad), "n"(NS * 32) : "memory");
-        mt = fmaxf(mt, xe[(hs ^ 1) * 128 + r]);
-        if (!ok) continue;
+        const float mt = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * c;   // scaled units (c > 0 keeps the argmax)
         const bool grow = mt > m_used + 8.f || (m_used == -INFINITY && mt > -INFINITY);
         if (__any_sync(0xffffffffu, grow)) {
           const float m_new = fmaxf(m_used, mt);
@@ -307,11 +310,12 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
           m_used = m_new;
           if (s > 0) {
             // O is being accumulated by the tensor core: wait for the stream's previous P V
-            bool w = mbar_wait(&pv_done[X], (turn - 1) & 1, abort_flag, p.status);
-            w = __all_sync(0xffffffffu, w);
-            if (!w) { ok = false; continue; }
+            ok = mbar_wait(&pv_done[xb ^ 1], ((turn - 1) >> 1) & 1, abort_flag, p.status);
+            ok = __all_sync(0xffffffffu, ok);
+            if (!ok) break;
             tc_fence_after();
-            for (int u = hs; u < ochunks; u += NS) {
+#pragma unroll 1
+            for (int u = 0; u < ochunks; u++) {
               uint32_t rr[32];
               tmem_ld32(tO + X * 128 + u * 32, rr);
               tmem_ld_wait();
@@ -326,19 +330,17 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
         const uint64_t nm2 = pack2(-mm, -mm);
         uint64_t sm2[2] = {0ull, 0ull};   // (+0, +0)
 #pragma unroll
-        for (int u = 0; u < CW / 32; u++) {
+        for (int u = 0; u < 2; u++) {
           uint32_t pk[16], pl[16];
           if (empty[u]) {
 #pragma unroll
             for (int j = 0; j < 16; j++) pk[j] = pl[j] = 0u;
           } else {
-            float x[32];
-            load(u, x);
 #pragma unroll
             for (int j = 0; j < 16; j += 2) {
               float t0, t1, t2, t3;
-              unpack2(fma2(pack2(x[2 * j], x[2 * j + 1]), c2, nm2), t0, t1);
-              unpack2(fma2(pack2(x[2 * j + 2], x[2 * j + 3]), c2, nm2), t2, t3);
+              unpack2(fma2(pack2(x[u][2 * j], x[u][2 * j + 1]), c2, nm2), t0, t1);
+              unpack2(fma2(pack2(x[u][2 * j + 2], x[u][2 * j + 3]), c2, nm2), t2, t3);
               const float p0 = fast_exp2(t0), p1 = fast_exp2(t1), p2 = fast_exp2(t2), p3 = fast_exp2(t3);
               sm2[0] = add2(sm2[0], pack2(p0, p1));
               sm2[1] = add2(sm2[1], pack2(p2, p3));
@@ -350,8 +352,7 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
               }
             }
           }
-          // over S columns that this thread has loaded for the last time
-          tmem_st16(tS + u * 32, pk);
+          tmem_st16(tS + u * 32, pk);      // over the S columns that this thread has loaded
           if (SPLIT) tmem_st16(tS + u * 32 + 16, pl);
         }
         {
@@ -363,18 +364,33 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
         tmem_st_wait();
         tc_fence_before();
         __syncwarp();
-        if (lane == 0) mbar_arrive(&p_ready[X]);
+        if (lane == 0) mbar_arrive(&p_ready[xb]);
       }
       cx[0] += MAPS == 2 ? it.ntile : (it.ntile + 1) / 2;
       cx[1] += MAPS == 2 ? it.ntile : it.ntile / 2;
-      // ---- the item's result = f[0] O_0 + f[1] O_1; the four warps of a quad take 32 columns each ----
-      xl[(X * NS + hs) * 128 + r] = l;
-      if (hs == 0) xm[X * 128 + r] = m_used;
-      asm volatile("bar.sync %0, %1;" ::"r"(10 + quad), "n"(2 * NS * 32) : "memory");
+      // ---- the item's result = f[0] O_0 + f[1] O_1; the two warps of a quad take 64 columns each ----
+      const bool row_ok = it.q0 + r < p.T;
+      const long long row = (long long)it.b * p.T + it.q0 + r;
+      const int col = X * 64;              // first column of this thread
+      // what the result is multiplied by is on its way while the last products run
+      float head_gate = 0.f;
+      uint4 gate[8];
+      if (row_ok) {
+        if (p.gate_mode == FEMTO_GATE_HEAD) head_gate = __bfloat162float(p.gate[row * p.ld_gate + it.h]);
+        if (p.gate_mode == FEMTO_GATE_ELEMENT) {
+          const uint4* g = reinterpret_cast<const uint4*>(p.gate + row * p.ld_gate + (long long)it.h * p.vdim + p.col0 + col);
+#pragma unroll
+          for (int j = 0; j < 8; j++)
+            if (col + j * 8 < p.cols) gate[j] = __ldg(g + j);
+        }
+      }
+      xl[X * 128 + r] = l;
+      xm[X * 128 + r] = m_used;
+      asm volatile("bar.sync %0, %1;" ::"r"(2 + quad), "n"(64) : "memory");
       const bool second = MAPS == 2 || it.ntile > 1;      // O_1 holds something
       float f[2];
       {
-        const float m0 = xm[r], m1 = xm[128 + r], l0 = xl[r] + xl[128 + r], l1 = xl[256 + r] + xl[384 + r];
+        const float m0 = xm[r], m1 = xm[128 + r], l0 = xl[r], l1 = xl[128 + r];
         const float z = p.sink ? __ldg(p.sink + it.h) * LOG2E : -INFINITY;
         if constexpr (MAPS == 2) {
           const float t0 = fmaxf(m0, z), t1 = fmaxf(m1, z), e0 = fast_exp2(m0 - t0), e1 = fast_exp2(m1 - t1);
@@ -386,18 +402,15 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
           f[0] = e0 * inv; f[1] = e1 * inv;
         }
       }
-      ok = ok && mbar_wait(&pv_done[0], (cx[0] - 1) & 1, abort_flag, p.status);
-      if (second) ok = ok && mbar_wait(&pv_done[1], (cx[1] - 1) & 1, abort_flag, p.status);
+      ok = ok && mbar_wait(&pv_done[(cx[0] - 1) & 1], ((cx[0] - 1) >> 1) & 1, abort_flag, p.status);
+      if (second) ok = ok && mbar_wait(&pv_done[2 + ((cx[1] - 1) & 1)], ((cx[1] - 1) >> 1) & 1, abort_flag, p.status);
       ok = __all_sync(0xffffffffu, ok);
-      const int u = X * NS + hs;
-      const bool mine = ok && u < ochunks;
-      float v[32];
-      if (mine) {
-        tc_fence_after();
-        tmem_ld32(tO + u * 32, reinterpret_cast<uint32_t(&)[32]>(v));
+      tc_fence_after();
+      auto result = [&](int u, float (&v)[32]) {
+        tmem_ld32(tO + col + u * 32, reinterpret_cast<uint32_t(&)[32]>(v));
         if (second) {
           uint32_t v1[32];
-          tmem_ld32(tO + 128 + u * 32, v1);
+          tmem_ld32(tO + 128 + col + u * 32, v1);
           tmem_ld_wait();
 #pragma unroll
           for (int j = 0; j < 32; j++) v[j] = v[j] * f[0] + __uint_as_float(v1[j]) * f[1];
@@ -406,44 +419,52 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
 #pragma unroll
           for (int j = 0; j < 32; j++) v[j] *= f[0];
         }
-        tc_fence_before();
-      }
-      __syncwarp();
-      if (lane == 0) mbar_arrive(o_free);
-      const bool row_ok = it.q0 + r < p.T;
-      const long long row = (long long)it.b * p.T + it.q0 + r;
+      };
       float mul = 1.f;
       if constexpr (MAPS == 2) {      // the head's own norm
         float ss = 0.f;
-        if (mine) {
+#pragma unroll 1
+        for (int u = 0; u < 2; u++) {
+          if (!ok || col + u * 32 >= p.cols) break;
+          float v[32];
+          result(u, v);
 #pragma unroll
-          for (int j = 0; j < 32; j++) ss += u * 32 + j < p.cols ? v[j] * v[j] : 0.f;
+          for (int j = 0; j < 32; j++) ss += col + u * 32 + j < p.cols ? v[j] * v[j] : 0.f;
         }
-        xs[u * 128 + r] = ss;
-        asm volatile("bar.sync %0, %1;" ::"r"(10 + quad), "n"(2 * NS * 32) : "memory");
-        ss = (xs[r] + xs[128 + r]) + (xs[256 + r] + xs[384 + r]);
-        mul = p.out_scale / sqrtf(ss / p.cols + p.eps);
+        xs[X * 128 + r] = ss;
+        asm volatile("bar.sync %0, %1;" ::"r"(2 + quad), "n"(64) : "memory");
+        mul = p.out_scale / sqrtf((xs[r] + xs[128 + r]) / p.cols + p.eps);
       }
-      if (mine && row_ok) {
-        if (p.gate_mode == FEMTO_GATE_HEAD) mul *= 1.f / (1.f + expf(-__bfloat162float(p.gate[row * p.ld_gate + it.h])));
-        const bf16* gate = p.gate_mode == FEMTO_GATE_ELEMENT ? p.gate + row * p.ld_gate + (long long)it.h * p.vdim + p.col0 + u * 32 : nullptr;
-        bf16* o = p.o + (row * p.heads + it.h) * p.vdim + p.col0 + u * 32;
+      if (p.gate_mode == FEMTO_GATE_HEAD) mul *= __fdividef(1.f, 1.f + __expf(-head_gate));
+      bf16* o = p.o + (row * p.heads + it.h) * p.vdim + p.col0 + col;
 #pragma unroll
-        for (int j = 0; j < 32; j += 8) {
-          if (u * 32 + j < p.cols) {
+      for (int u = 0; u < 2; u++) {
+        if (!ok || col + u * 32 >= p.cols) continue;
+        float v[32];
+        result(u, v);
+        __syncwarp();
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+          if (row_ok && col + u * 32 + j * 8 < p.cols) {
             float w[8];
 #pragma unroll
-            for (int e = 0; e < 8; e++) w[e] = v[j + e] * mul;
-            if (gate) {
-              float z[8];
-              load_vec<bf16, 8>(gate + j, z);
+            for (int e = 0; e < 8; e++) w[e] = v[8 * j + e] * mul;
+            if (p.gate_mode == FEMTO_GATE_ELEMENT) {
+              const uint32_t* g = reinterpret_cast<const uint32_t*>(&gate[u * 4 + j]);
 #pragma unroll
-              for (int e = 0; e < 8; e++) w[e] *= __fdividef(1.f, 1.f + __expf(-z[e]));
+              for (int e = 0; e < 8; e += 2) {
+                w[e] *= __fdividef(1.f, 1.f + __expf(-bf16_low(g[e / 2])));
+                w[e + 1] *= __fdividef(1.f, 1.f + __expf(-bf16_high(g[e / 2])));
+              }
             }
-            store_vec<bf16, 8>(o + j, w);
+            store_vec<bf16, 8>(o + u * 32 + 8 * j, w);
           }
         }
+        __syncwarp();
       }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(o_free);
     }
   }
 
@@ -456,7 +477,7 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
 }
 
 int slabs(int n) { return (n + 63) / 64; }
-size_t smem_bytes(int maps, int nqk, int nv) { return (size_t)SLAB * ((maps + 2) * nqk + 2 * nv) + 1024 + 256 + 14 * 128 * 4 + 4 * 128 * 4; }
+size_t smem_bytes(int maps, int nqk, int nv) { return (size_t)SLAB * ((2 * maps + STAGES) * nqk + STAGES * nv) + 1024 + 256 + 6 * 128 * 4; }
 
 template <int MAPS, bool SPLIT>
 int launch(const CUtensorMap& tmQu, const CUtensorMap& tmQr, const CUtensorMap& tmKu, const CUtensorMap& tmKr, const CUtensorMap& tmV,
@@ -483,7 +504,7 @@ int launch(const CUtensorMap& tmQu, const CUtensorMap& tmQr, const CUtensorMap& 
 
 bool latent_attention_tc_supported(const LatentArgs& a) {
   if ((a.dim | a.rot_dim | a.vdim) & 7 || a.vdim > 256 || !(a.scale > 0.f)) return false;
-  if (3 * (slabs(a.dim) + slabs(a.rot_dim)) + 2 * slabs(std::min(a.vdim, MAX_V)) > MAX_SLABS) return false;
+  if ((2 + STAGES) * (slabs(a.dim) + slabs(a.rot_dim)) + STAGES * slabs(std::min(a.vdim, MAX_V)) > MAX_SLABS) return false;
   return aligned16(a.q) && aligned16(a.kv) && aligned16(a.latent) && aligned16(a.o);
 }
 
@@ -491,26 +512,26 @@ int latent_attention_tc(const LatentArgs& a, cudaStream_t s) {
   const uint64_t N = a.first + a.T, H = a.heads, hd = a.dim + a.rot_dim, wide = H * (a.dim + a.vdim);
   CUtensorMap tmQu, tmQr, tmKu, tmKr, tmV;
   const bf16 *q = (const bf16*)a.q, *kv = (const bf16*)a.kv;
-  const uint32_t box4[4] = {64, 1, 128, 1}, box3[3] = {64, 128, 1};
+  const uint32_t boxQ[4] = {64, 1, BQ, 1}, boxK[4] = {64, 1, BKV, 1}, box3[3] = {64, BKV, 1};
   {
     const uint64_t d[4] = {(uint64_t)a.dim, H, (uint64_t)a.T, (uint64_t)a.B}, st[3] = {hd, H * hd, H * hd * a.T};
-    FEMTO_TRY(make_tmap_nd_bf16(&tmQu, q, 4, d, st, box4));
+    FEMTO_TRY(make_tmap_nd_bf16(&tmQu, q, 4, d, st, boxQ));
   }
   tmQr = tmQu;
   {
     const uint64_t d[4] = {(uint64_t)a.dim, H, N, (uint64_t)a.B}, st[3] = {(uint64_t)a.dim, wide, wide * a.maxT};
-    FEMTO_TRY(make_tmap_nd_bf16(&tmKu, kv, 4, d, st, box4));
+    FEMTO_TRY(make_tmap_nd_bf16(&tmKu, kv, 4, d, st, boxK));
   }
   tmKr = tmKu;
   if (a.rot_dim > 0) {
     const uint64_t d[4] = {(uint64_t)a.rot_dim, H, (uint64_t)a.T, (uint64_t)a.B}, st[3] = {hd, H * hd, H * hd * a.T};
-    FEMTO_TRY(make_tmap_nd_bf16(&tmQr, q + a.dim, 4, d, st, box4));
+    FEMTO_TRY(make_tmap_nd_bf16(&tmQr, q + a.dim, 4, d, st, boxQ));
     const uint64_t dk[3] = {(uint64_t)a.rot_dim, N, (uint64_t)a.B}, sk[2] = {(uint64_t)a.ld, (uint64_t)a.ld * a.maxT};
     FEMTO_TRY(make_tmap_nd_bf16(&tmKr, (const bf16*)a.latent + a.lp, 3, dk, sk, box3));
   }
   {
     const uint64_t d[4] = {(uint64_t)a.vdim, H, N, (uint64_t)a.B}, st[3] = {(uint64_t)a.vdim, wide, wide * a.maxT};
-    FEMTO_TRY(make_tmap_nd_bf16(&tmV, kv + H * a.dim, 4, d, st, box4));
+    FEMTO_TRY(make_tmap_nd_bf16(&tmV, kv + H * a.dim, 4, d, st, boxK));
   }
   SlabAttn p = {};
   p.o = (bf16*)a.o; p.gate = (const bf16*)a.gate; p.status = a.d->status; p.ld_gate = a.ld_gate; p.gate_mode = FEMTO_GATE_HEAD;
@@ -522,7 +543,7 @@ int latent_attention_tc(const LatentArgs& a, cudaStream_t s) {
 
 bool window_attention_tc_supported(const WindowAttnArgs& a) {
   if ((a.dim | a.vdim) & 7 || a.vdim > (a.maps == 2 ? MAX_V : 256) || !(a.scale > 0.f)) return false;
-  if ((a.maps + 2) * slabs(a.dim) + 2 * slabs(std::min(a.vdim, MAX_V)) > MAX_SLABS) return false;
+  if ((2 * a.maps + STAGES) * slabs(a.dim) + STAGES * slabs(std::min(a.vdim, MAX_V)) > MAX_SLABS) return false;
   if ((a.ldq | a.ld | a.vo | a.ld_gate) & 7) return false;
   return aligned16(a.q) && aligned16(a.kv) && aligned16(a.o) && (a.gate_mode != FEMTO_GATE_ELEMENT || aligned16(a.gate));
 }
@@ -531,19 +552,19 @@ int window_attention_tc(const WindowAttnArgs& a, cudaStream_t s) {
   const uint64_t N = a.first + a.T, H = a.heads, G = a.kv_heads, M = a.maps, D = a.dim, E = a.vdim;
   CUtensorMap tmQ, tmK, tmV;
   const bf16* kv = (const bf16*)a.kv;
-  const uint32_t box[4] = {64, 1, 128, 1};
+  const uint32_t boxQ[4] = {64, 1, BQ, 1}, boxK[4] = {64, 1, BKV, 1};
   {
     const uint64_t d[4] = {D, H * M, (uint64_t)a.T, (uint64_t)a.B}, st[3] = {D, (uint64_t)a.ldq, (uint64_t)a.ldq * a.T};
-    FEMTO_TRY(make_tmap_nd_bf16(&tmQ, a.q, 4, d, st, box));
+    FEMTO_TRY(make_tmap_nd_bf16(&tmQ, a.q, 4, d, st, boxQ));
   }
   const uint64_t ld = a.ld, col = ld * a.maxT;
   {
     const uint64_t d[4] = {D, G * M, N, (uint64_t)a.B}, st[3] = {D, ld, col};
-    FEMTO_TRY(make_tmap_nd_bf16(&tmK, kv, 4, d, st, box));
+    FEMTO_TRY(make_tmap_nd_bf16(&tmK, kv, 4, d, st, boxK));
   }
   {
     const uint64_t d[4] = {E, G, N, (uint64_t)a.B}, st[3] = {E, ld, col};
-    FEMTO_TRY(make_tmap_nd_bf16(&tmV, kv + a.vo, 4, d, st, box));
+    FEMTO_TRY(make_tmap_nd_bf16(&tmV, kv + a.vo, 4, d, st, boxK));
   }
   SlabAttn p = {};
   p.o = (bf16*)a.o; p.gate = (const bf16*)a.gate; p.status = a.status; p.ld_gate = a.ld_gate; p.gate_mode = a.gate_mode;

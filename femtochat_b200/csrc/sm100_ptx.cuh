@@ -51,6 +51,16 @@ __device__ __forceinline__ bool mbar_wait_limit(uint64_t* bar, uint32_t parity, 
 __device__ __forceinline__ bool mbar_wait(uint64_t* bar, uint32_t parity, volatile int* abort_flag, unsigned int* status) {
   return mbar_wait_limit(bar, parity, abort_flag, status, WAIT_LIMIT);
 }
+// The roles that issue copies and products run with the whole warp converged, so that the compiler keeps addresses and
+// descriptors in uniform registers, and one elected lane executes the instruction itself.
+__device__ __forceinline__ bool elect_one() {
+  uint32_t p;
+  asm volatile("{\n\t.reg .pred p;\n\telect.sync _|p, 0xffffffff;\n\tselp.u32 %0, 1, 0, p;\n\t}" : "=r"(p));
+  return p != 0;
+}
+__device__ __forceinline__ bool mbar_wait_warp(uint64_t* bar, uint32_t parity, volatile int* abort_flag, unsigned int* status) {
+  return __all_sync(0xffffffffu, mbar_wait(bar, parity, abort_flag, status));
+}
 
 // 2^x on the special-function unit (ex2.approx.ftz: relative error about 2^-22, flushes denormals).
 __device__ __forceinline__ float fast_exp2(float x) {
