@@ -11,10 +11,11 @@
 // One CTA per SM walks the items (128 queries of one head), latest queries first.  The steps of an item, 128 queries against
 // 64 keys, alternate between two streams, each with two buffers for S / P and an accumulator O of its own in tensor memory and
 // four softmax warps (one thread per query row): S of a stream's next step is there before the softmax of this one is
-// done, and the exponentials of one stream run beside the loads and the row maxima of the other.  With two maps (differential attention) the streams are the maps, otherwise the
-// even and the odd key tiles, whose partial results meet at the end.  A TMA warp streams Q, K and V (four stages of K and V),
-// one warp issues S = Q K^T, another O += P V with P read back from tensor memory; all of them run ahead into the next item.
-// Sum of the streams, the head's own norm of differential attention and the output gate are applied as the result leaves.
+// done, and the exponentials of one stream run beside the loads and the row maxima of the other.  With two maps (differential
+// attention) the streams are the maps, otherwise the even and the odd key tiles, whose partial results meet at the end.  One
+// warp loads Q and K, one V (four stages of each), one issues S = Q K^T, another O += P V with P read back from tensor
+// memory; all of them run ahead into the next item.  Sum of the streams, the head's own norm of differential attention and
+// the output gate are applied as the result leaves.
 #include <algorithm>
 
 #include "decoder.cuh"
@@ -30,6 +31,8 @@ constexpr int SLAB_Q = BQ * 64 * 2, SLAB = BKV * 64 * 2;   // one box: 128 queri
 constexpr int MAX_SLABS = 26;                         // 8 KB each: 2 maps + STAGES per query/key slab, STAGES per value slab
 constexpr int MAX_V = 128;                            // value columns of one launch
 constexpr float LOG2E = 1.4426950408889634f;
+// registers per thread: 384 threads launch with 168 = (128 * 104 + 256 * 200) / 384
+constexpr int REGS_ROLES = 104, REGS_SOFTMAX = 200;
 struct SlabAttn {
   bf16* o; const bf16* gate; unsigned int* status;
   long long ld_gate;
@@ -131,9 +134,12 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
   // Every role walks the same items in the same order and counts what it has seen: n items, kc key tiles, vc value tiles, cx[X]
   // steps of stream X (its turn t uses buffer t & 1).  The phase of a barrier is the count of its own turns, modulo two.
   if (warp < 4) {
+    reg_dealloc<REGS_ROLES>();
+    // let loads already in flight land before the CTA exits
+    auto drain = [&](uint64_t* bar, int turn) { for (uint32_t t = 0; t < WAIT_LIMIT && !mbar_try_wait(bar, turn & 1); ++t) {} };
     if (warp == 0) {
-      // ---------------- TMA producer ----------------
-      int n = 0, kc = 0, vc = 0;
+      // ---------------- loads of Q and K ----------------
+      int n = 0, kc = 0;
       bool ok = true;
       for (int item = blockIdx.x; item < p.items && ok; item += gridDim.x) {
         const Item it(p, item);
@@ -162,23 +168,31 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
             }
             kc++;
           }
-          const int vt = vc % STAGES;
-          if (!ok || (vc >= STAGES && !mbar_wait_warp(&v_free[vt], (vc / STAGES - 1) & 1, abort_flag, p.status))) { ok = false; break; }
-          if (elect_one()) {
-            uint8_t* v = sV + vt * v_bytes;
-            mbar_expect_tx(&v_full[vt], v_bytes);
-            for (int j = 0; j < p.n_v; j++) tma_load_4d(v + j * SLAB, &tmV, &v_full[vt], p.col0 + j * 64, hk, key, it.b);
-          }
-          vc++;
         }
       }
       if (*abort_flag) {
-        // let loads already in flight land before the CTA exits
-        auto drain = [&](uint64_t* bar, int turn) { for (uint32_t t = 0; t < WAIT_LIMIT && !mbar_try_wait(bar, turn & 1); ++t) {} };
         if (n >= 1) drain(q_full, n - 1);
         for (int i = max(0, kc - STAGES); i < kc; i++) drain(&k_full[i % STAGES], i / STAGES);
-        for (int i = max(0, vc - STAGES); i < vc; i++) drain(&v_full[i % STAGES], i / STAGES);
       }
+    } else if (warp == 3) {
+      // ---------------- loads of V ----------------
+      int vc = 0;
+      bool ok = true;
+      for (int item = blockIdx.x; item < p.items && ok; item += gridDim.x) {
+        const Item it(p, item);
+        const int hk = it.h / p.per;
+        for (int i = 0; i < it.ntile; i++, vc++) {
+          const int vt = vc % STAGES;
+          if (vc >= STAGES && !mbar_wait_warp(&v_free[vt], (vc / STAGES - 1) & 1, abort_flag, p.status)) { ok = false; break; }
+          if (elect_one()) {
+            uint8_t* v = sV + vt * v_bytes;
+            mbar_expect_tx(&v_full[vt], v_bytes);
+            for (int j = 0; j < p.n_v; j++) tma_load_4d(v + j * SLAB, &tmV, &v_full[vt], p.col0 + j * 64, hk, it.key(i), it.b);
+          }
+        }
+      }
+      if (*abort_flag)
+        for (int i = max(0, vc - STAGES); i < vc; i++) drain(&v_full[i % STAGES], i / STAGES);
     } else if (warp == 1) {
       // ---------------- S = Q K^T issuer ----------------
       constexpr uint32_t idesc_s = idesc_bf16(BQ, BKV, false, false);  // both operands K-major
@@ -248,6 +262,7 @@ slab_attn_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant
     }
   } else {
     // ---------------- softmax: stream X (four warps each), one thread per query row ----------------
+    reg_alloc<REGS_SOFTMAX>();
     const int quad = warp & 3, X = (warp - 4) >> 2;
     const int r = quad * 32 + lane;
     const uint32_t lane_off = (uint32_t)(quad * 32) << 16;
