@@ -5,6 +5,7 @@
 #include <algorithm>
 
 #include "decoder.cuh"
+#include "warp_mma.cuh"
 
 namespace {
 
@@ -243,19 +244,6 @@ __global__ void __launch_bounds__(1024) k_absorb_q(const LatentArgs a) {
 // keys (read as they lie) and as values (read transposed).  Queries and softmax weights are sums of two bf16 numbers, so
 // scores and weights keep fp32 accuracy.  For the scores the warps share the channels, so a warp's part of the queries
 // stays in registers for the whole kernel and shared memory is read once; their partial sums meet in shared memory.
-__device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)) : "memory");
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)) : "memory");
-}
-__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ int swz(int row, int col, int width) { return row * width + ((((col >> 3) ^ (row & 7)) << 3) | (col & 7)); }
-
 // NK: 16-channel steps per warp (width <= 128 NK); NP: pairs of 8-channel tiles of the result per warp (lp <= 128 NP)
 template <int NK, int NP>
 __global__ void __launch_bounds__(256) k_latent_decode_mma(const LatentArgs a, int splits, int tiles_per, int KT, int width) {

@@ -7,6 +7,7 @@
 #include <algorithm>
 
 #include "decoder.cuh"
+#include "warp_mma.cuh"
 
 namespace {
 
@@ -325,21 +326,188 @@ __global__ void __launch_bounds__(256) k_window_decode(const WindowAttnArgs a, c
   }
 }
 
-// grid (heads, rows): the splits of a head in order, the sink, the difference of the maps and its norm, the gate.
+// The tensor-core form for bf16: the pairs are the 16 rows of an mma tile, and each of the four warps of a block takes tiles of
+// 32 visible keys of its own, which arrive in its part of shared memory by cp.async; the warps' results meet at the end.
+// A query's row has zeros in the other map's channels, so that both maps run as one product with whole cached rows; the
+// softmax weights are sums of two bf16 numbers and keep 32-bit accuracy.
+// KS: steps of 16 key channels (maps dim <= 16 KS), NE: pairs of 8-channel tiles of the result (vdim <= 16 NE)
+constexpr int DW = 4, DT = 32;      // warps of a block, keys of a tile
+template <int KS, int NE>
+__global__ void __launch_bounds__(32 * DW, KS <= 8 ? 3 : 1) k_window_decode_mma(const WindowAttnArgs a, const DecodeShape sh) {
+  pdl_trigger();
+  extern __shared__ __align__(16) uint8_t raw[];
+  const int D = a.dim, E = a.vdim, MD = a.maps * D;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c2 = 2 * (lane & 3);
+  bf16* ks = reinterpret_cast<bf16*>(raw) + warp * DT * (sh.pk + sh.pv);      // [DT][pk], swizzled
+  bf16* vs = ks + DT * sh.pk;                                                // [DT][pv]
+  const int hk = blockIdx.x / sh.groups, h0 = hk * sh.per + blockIdx.x % sh.groups * sh.hq;
+  const int nv = min(sh.hq, (hk + 1) * sh.per - h0) * a.maps;
+  const long long row = blockIdx.z;
+  const int b = (int)(row / a.T), pos = a.first + (int)(row % a.T);
+  const Visible vis(pos, a.window, a.keep);
+  const bf16* kv = reinterpret_cast<const bf16*>(a.kv) + (long long)b * a.maxT * a.ld;
+  const bf16* ksrc = kv + (long long)hk * MD;
+  const bf16* vsrc = kv + a.vo + (long long)hk * E;
+  const bf16* q = reinterpret_cast<const bf16*>(a.q) + row * a.ldq + (long long)h0 * MD;
+  // the padding of the staged rows stays zero
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  for (int i = lane; i < DT * (sh.pk - MD) / 8; i += 32) { const int w = (sh.pk - MD) / 8; *reinterpret_cast<uint4*>(ks + swz(i / w, MD + i % w * 8, sh.pk)) = zero; }
+  for (int i = lane; i < DT * (sh.pv - E) / 8; i += 32) { const int w = (sh.pv - E) / 8; *reinterpret_cast<uint4*>(vs + swz(i / w, E + i % w * 8, sh.pv)) = zero; }
+  auto stage = [&](bf16* dst, int pitch, const bf16* src, int i0, int n, int units) {
+    int r = lane / units, u = lane % units;
+    const int dr = 32 / units, du = 32 % units;      // a step of 32 units
+#pragma unroll 4
+    while (r < DT) {
+      if (r < n) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(dst + swz(r, u * 8, pitch))), "l"(src + (long long)vis.key(i0 + r) * a.ld + u * 8) : "memory");
+      else *reinterpret_cast<uint4*>(dst + swz(r, u * 8, pitch)) = zero;
+      r += dr; u += du;
+      if (u >= units) { u -= units; r++; }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  const int first = blockIdx.y * sh.tiles_per, last = min(first + sh.tiles_per, (vis.n + DT - 1) / DT);
+  pdl_wait();
+  uint32_t qa[KS][4];
+  float o[NE][2][4] = {}, m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  for (int t = first + warp; t < last; t += DW) {
+    const int n = min(DT, vis.n - t * DT);
+    __syncwarp();
+    stage(ks, sh.pk, ksrc, t * DT, n, MD / 8);
+    stage(vs, sh.pv, vsrc, t * DT, n, E / 8);
+    if (t == first + warp) {
+#pragma unroll
+      for (int k = 0; k < KS; k++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+          const int v = g + 8 * (e & 1), c = k * 16 + 8 * (e >> 1) + c2 - (a.maps == 2 ? v % 2 * D : 0);
+          qa[k][e] = v < nv && c >= 0 && c < D ? *reinterpret_cast<const uint32_t*>(q + v * D + c) : 0u;
+        }
+    }
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncwarp();
+    float s[4][4] = {};
+#pragma unroll
+    for (int k = 0; k < KS; k++) {
+      if (k * 16 >= MD) break;
+#pragma unroll
+      for (int j = 0; j < 2; j++) {
+        uint32_t kb[4];
+        ldsm4(kb, ks + swz(16 * j + (lane & 7) + 8 * (lane >> 4), k * 16 + 8 * ((lane >> 3) & 1), sh.pk));
+        mma16816(s[2 * j], qa[k], kb[0], kb[1]);
+        mma16816(s[2 * j + 1], qa[k], kb[2], kb[3]);
+      }
+    }
+    // softmax of rows g and g + 8, each shared by four lanes
+    float f[2];
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+      float mn = m[e];
+#pragma unroll
+      for (int j = 0; j < 4; j++)
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+          float& x = s[j][2 * e + i];
+          x = 8 * j + c2 + i < n ? x * a.scale : -INFINITY;
+          mn = fmaxf(mn, x);
+        }
+      mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 1));
+      mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 2));      // finite: a tile holds at least one visible key
+      f[e] = __expf(m[e] - mn);
+      m[e] = mn;
+      l[e] *= f[e];
+#pragma unroll
+      for (int j = 0; j < 4; j++)
+#pragma unroll
+        for (int i = 0; i < 2; i++) { float& x = s[j][2 * e + i]; x = __expf(x - mn); l[e] += x; }
+    }
+#pragma unroll
+    for (int j = 0; j < NE; j++)
+#pragma unroll
+      for (int i = 0; i < 2; i++) { o[j][i][0] *= f[0]; o[j][i][1] *= f[0]; o[j][i][2] *= f[1]; o[j][i][3] *= f[1]; }
+    uint32_t ph[2][4], pl[2][4];
+#pragma unroll
+    for (int k = 0; k < 2; k++)
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const float x = s[2 * k + (e >> 1)][2 * (e & 1)], y = s[2 * k + (e >> 1)][2 * (e & 1) + 1];
+        const __nv_bfloat162 hi = __floats2bfloat162_rn(x, y);
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(x - __bfloat162float(hi.x), y - __bfloat162float(hi.y));
+        ph[k][e] = *reinterpret_cast<const uint32_t*>(&hi);
+        pl[k][e] = *reinterpret_cast<const uint32_t*>(&lo);
+      }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncwarp();
+#pragma unroll
+    for (int j = 0; j < NE; j++) {
+      if (j * 16 >= E) break;
+#pragma unroll
+      for (int k = 0; k < 2; k++) {
+        uint32_t vb[4];
+        ldsm4t(vb, vs + swz(16 * k + (lane & 15), j * 16 + 8 * (lane >> 4), sh.pv));
+#pragma unroll
+        for (int i = 0; i < 2; i++) { mma16816(o[j][i], ph[k], vb[2 * i], vb[2 * i + 1]); mma16816(o[j][i], pl[k], vb[2 * i], vb[2 * i + 1]); }
+      }
+    }
+  }
+#pragma unroll
+  for (int e = 0; e < 2; e++) {
+    l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
+    l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
+  }
+  // the warps' results through shared memory: [DW][16][E], and their maxima and sums
+  __shared__ float sm[DW][16], sl[DW][16];
+  float* os = reinterpret_cast<float*>(raw);
+  __syncthreads();
+#pragma unroll
+  for (int e = 0; e < 2; e++) {
+    const int v = g + 8 * e;
+    if ((lane & 3) == 0) { sm[warp][v] = m[e]; sl[warp][v] = l[e]; }
+#pragma unroll
+    for (int j = 0; j < NE; j++)
+#pragma unroll
+      for (int i = 0; i < 2; i++) {
+        const int c = j * 16 + 8 * i + c2;
+        if (v < nv && c < E) *reinterpret_cast<float2*>(os + (warp * 16 + v) * E + c) = make_float2(o[j][i][2 * e], o[j][i][2 * e + 1]);
+      }
+  }
+  __syncthreads();
+  for (int i = tid; i < nv * E; i += 32 * DW) {
+    const int v = i / E, c = i % E;
+    float M = -INFINITY, L = 0.f, x = 0.f;
+#pragma unroll
+    for (int w = 0; w < DW; w++) M = fmaxf(M, sm[w][v]);
+#pragma unroll
+    for (int w = 0; w < DW; w++) {
+      const float r = sm[w][v] == -INFINITY ? 0.f : __expf(sm[w][v] - M);
+      L += r * sl[w][v];
+      x = fmaf(r, os[(w * 16 + v) * E + c], x);
+    }
+    float* dst = a.part + (((row * a.heads + h0) * a.maps + v) * sh.splits + blockIdx.y) * (E + 2);
+    if (c == 0) { dst[0] = M; dst[1] = L; }
+    dst[2 + c] = x;
+  }
+}
+
+// grid (heads, rows): the splits of a head, the sink, the difference of the maps and its norm, the gate.  Four groups of 128
+// threads take every fourth split.
 template <typename T, int MAPS>
-__global__ void __launch_bounds__(128) k_window_combine(const WindowAttnArgs a, int splits) {
+__global__ void __launch_bounds__(512) k_window_combine(const WindowAttnArgs a, int splits) {
   pdl_trigger();
   extern __shared__ float sm[];
   float* ws = sm;                 // [MAPS][splits]
-  __shared__ float red[4];
-  const int h = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, E = a.vdim;
+  __shared__ float os[3][MAPS][256], red[4];
+  const int h = blockIdx.x, tid = threadIdx.x & 127, part = threadIdx.x >> 7, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, E = a.vdim;
   const long long row = blockIdx.y;
   const T* gp = reinterpret_cast<const T*>(a.gate) + (a.gate_mode == FEMTO_GATE_NONE ? 0 : row * a.ld_gate + (a.gate_mode == FEMTO_GATE_HEAD ? h : h * E));
   const float* p = a.part + (row * a.heads + h) * MAPS * (long long)splits * (E + 2);
+  const float z = a.sink ? a.sink[h] : -INFINITY, lam = MAPS == 2 ? *a.lambda : 0.f;
   pdl_wait();
+  float gate[2] = {0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < 2; i++)
+    if (!part && tid + 128 * i < E && a.gate_mode != FEMTO_GATE_NONE) gate[i] = to_f<T>(gp[a.gate_mode == FEMTO_GATE_HEAD ? 0 : tid + 128 * i]);
   if (warp < MAPS) {
     const float* pm = p + (long long)warp * splits * (E + 2);
-    const float z = a.sink ? a.sink[h] : -INFINITY;
     float M = z, L = 0.f;
     for (int s = lane; s < splits; s += 32) { const float m = pm[(long long)s * (E + 2)]; ws[warp * splits + s] = m; M = fmaxf(M, m); }
     M = warp_max(M);
@@ -355,34 +523,43 @@ __global__ void __launch_bounds__(128) k_window_combine(const WindowAttnArgs a, 
     for (int s = lane; s < splits; s += 32) ws[warp * splits + s] *= L;
   }
   __syncthreads();
-  float v[2] = {0.f, 0.f};
+  float o[MAPS][2];
 #pragma unroll
-  for (int mp = MAPS - 1; mp >= 0; mp--) {
-    float o[2] = {0.f, 0.f};
+  for (int mp = 0; mp < MAPS; mp++) {
     const float* pm = p + (long long)mp * splits * (E + 2) + 2;
-#pragma unroll 8
-    for (int s = 0; s < splits; s++) {
-      const float w = ws[mp * splits + s];
-      if (tid < E) o[0] = fmaf(w, pm[(long long)s * (E + 2) + tid], o[0]);
-      if (tid + 128 < E) o[1] = fmaf(w, pm[(long long)s * (E + 2) + tid + 128], o[1]);
+#pragma unroll
+    for (int i = 0; i < 2; i++) {
+      o[mp][i] = 0.f;
+      const int c = tid + 128 * i;
+      if (c < E)
+#pragma unroll 4
+        for (int s = part; s < splits; s += 4) o[mp][i] = fmaf(ws[mp * splits + s], pm[(long long)s * (E + 2) + c], o[mp][i]);
+      if (part) os[part - 1][mp][c] = o[mp][i];
     }
-    if (mp == 1) { const float lam = *a.lambda; v[0] = -lam * o[0]; v[1] = -lam * o[1]; }
-    else { v[0] += o[0]; v[1] += o[1]; }
+  }
+  __syncthreads();
+  if (part) return;
+  float v[2];
+#pragma unroll
+  for (int i = 0; i < 2; i++) {
+#pragma unroll
+    for (int mp = 0; mp < MAPS; mp++) o[mp][i] += (os[0][mp][tid + 128 * i] + os[1][mp][tid + 128 * i]) + os[2][mp][tid + 128 * i];
+    v[i] = MAPS == 2 ? o[0][i] - lam * o[MAPS - 1][i] : o[0][i];
   }
   if (MAPS == 2) {
-    const float ss = warp_sum(v[0] * v[0] + v[1] * v[1]);
+    const float ss = warp_sum(v[0] * v[0] + v[1] * v[1]);      // channels past vdim hold zeros
     if (lane == 0) red[warp] = ss;
-    __syncthreads();
+    asm volatile("bar.sync 1, 128;" ::: "memory");
     const float f = a.out_scale / sqrtf((red[0] + red[1] + red[2] + red[3]) / E + a.eps);
     v[0] *= f; v[1] *= f;
   }
-  T* o = reinterpret_cast<T*>(a.o) + row * (long long)a.heads * E + (long long)h * E;
+  T* o_row = reinterpret_cast<T*>(a.o) + row * (long long)a.heads * E + (long long)h * E;
 #pragma unroll
   for (int i = 0; i < 2; i++) {
     const int c = tid + 128 * i;
     if (c >= E) continue;
-    if (a.gate_mode != FEMTO_GATE_NONE) v[i] /= 1.f + expf(-to_f<T>(gp[a.gate_mode == FEMTO_GATE_HEAD ? 0 : c]));
-    o[c] = from_f<T>(v[i]);
+    if (a.gate_mode != FEMTO_GATE_NONE) v[i] /= 1.f + expf(-gate[i]);
+    o_row[c] = from_f<T>(v[i]);
   }
 }
 
@@ -399,35 +576,46 @@ template <typename T> int window_decode(const WindowAttnArgs& a, cudaStream_t s)
   sh.per = a.heads / a.kv_heads;
   sh.hq = std::min(sh.per, VH / a.maps);
   sh.groups = cdiv(sh.per, sh.hq);
-  // odd numbers of 16-byte units between staged rows keep the vector loads of neighbouring keys on different banks
-  sh.pk = (cdiv(a.maps * a.dim * es, 16) | 1) * V;
-  sh.pv = (cdiv(a.vdim * es, 16) | 1) * V;
-  auto bytes = [&](int kt) {
-    return std::max((size_t)es * kt * (sh.pk + sh.pv) + 4 * (size_t)(VH * ((a.dim + 3) & ~3) + VH * kt + 3 * VH), (size_t)4 * (VH / 2) * a.vdim);
-  };
-  sh.KT = bytes(64) <= 200 * 1024 ? 64 : 32;
-  const int seen = (int)std::min<long long>(a.first + a.T, (long long)a.window + a.keep);
-  const int tiles = cdiv(seen, sh.KT), blocks = a.kv_heads * sh.groups * rows;
-  int splits = std::max(1, std::min(tiles, cdiv(2 * device_sm_count(), blocks)));
-  sh.tiles_per = cdiv(tiles, splits);
+  const bool vec = a.dim % V == 0 && a.vdim % V == 0 && a.ld % V == 0 && a.vo % V == 0 && aligned16(a.kv);
+  const bool tc = es == 2 && vec && a.maps * a.dim <= 256 && a.vdim <= 256 && (a.ldq & 1) == 0;
+  const int seen = (int)std::min<long long>(a.first + a.T, (long long)a.window + a.keep), blocks = a.kv_heads * sh.groups * rows;
+  size_t smem;
+  int tiles;
+  if (tc) {
+    sh.pk = round_up(a.maps * a.dim, 64); sh.pv = round_up(a.vdim, 64); sh.KT = DT;
+    smem = (size_t)2 * DW * DT * (sh.pk + sh.pv);
+    tiles = cdiv(seen, DT);
+    // a block's four warps have a tile each, more when that makes more blocks than run at once
+    sh.tiles_per = std::max(DW, cdiv(tiles, std::max(1, 3 * device_sm_count() / blocks)));
+  } else {
+    // odd numbers of 16-byte units between staged rows keep the vector loads of neighbouring keys on different banks
+    sh.pk = (cdiv(a.maps * a.dim * es, 16) | 1) * V;
+    sh.pv = (cdiv(a.vdim * es, 16) | 1) * V;
+    auto bytes = [&](int kt) {
+      return std::max((size_t)es * kt * (sh.pk + sh.pv) + 4 * (size_t)(VH * ((a.dim + 3) & ~3) + VH * kt + 3 * VH), (size_t)4 * (VH / 2) * a.vdim);
+    };
+    sh.KT = bytes(64) <= 200 * 1024 ? 64 : 32;
+    smem = bytes(sh.KT);
+    tiles = cdiv(seen, sh.KT);
+    sh.tiles_per = cdiv(tiles, std::max(1, std::min(tiles, cdiv(2 * device_sm_count(), blocks))));
+  }
   auto floats = [&] { return (size_t)rows * a.heads * a.maps * cdiv(tiles, sh.tiles_per) * (a.vdim + 2); };
   while (floats() > a.part_floats && sh.tiles_per < tiles) sh.tiles_per++;
   if (floats() > a.part_floats) return femto_fail(FEMTO_ERR_STATE, "attention: no room for the partial results of %d rows", rows);
   sh.splits = cdiv(tiles, sh.tiles_per);
   const dim3 grid(a.kv_heads * sh.groups, sh.splits, rows);
-  const size_t smem = bytes(sh.KT);
-  const bool vec = a.dim % V == 0 && a.vdim % V == 0 && a.ld % V == 0 && a.vo % V == 0 && aligned16(a.kv);
-  if (vec) {
-    FEMTO_TRY(allow_smem(k_window_decode<T, true>, smem));
-    CUDA_TRY(launch_dependent(k_window_decode<T, true>, grid, 256, smem, s, a, sh));
-  } else {
-    FEMTO_TRY(allow_smem(k_window_decode<T, false>, smem));
-    CUDA_TRY(launch_dependent(k_window_decode<T, false>, grid, 256, smem, s, a, sh));
-  }
+#define LAUNCH(KERNEL, THREADS) do { FEMTO_TRY(allow_smem(KERNEL, smem)); CUDA_TRY(launch_dependent(KERNEL, grid, THREADS, smem, s, a, sh)); } while (0)
+  if (tc) {
+    if (sh.pk <= 64 && sh.pv <= 64) LAUNCH((k_window_decode_mma<4, 4>), 32 * DW);
+    else if (sh.pk <= 128 && sh.pv <= 128) LAUNCH((k_window_decode_mma<8, 8>), 32 * DW);
+    else LAUNCH((k_window_decode_mma<16, 16>), 32 * DW);
+  } else if (vec) LAUNCH((k_window_decode<T, true>), 256);
+  else LAUNCH((k_window_decode<T, false>), 256);
+#undef LAUNCH
   KERNEL_CHECK();
   const size_t ws = 4 * (size_t)a.maps * sh.splits;
-  if (a.maps == 2) CUDA_TRY(launch_dependent(k_window_combine<T, 2>, dim3(a.heads, rows), 128, ws, s, a, sh.splits));
-  else CUDA_TRY(launch_dependent(k_window_combine<T, 1>, dim3(a.heads, rows), 128, ws, s, a, sh.splits));
+  if (a.maps == 2) CUDA_TRY(launch_dependent(k_window_combine<T, 2>, dim3(a.heads, rows), 512, ws, s, a, sh.splits));
+  else CUDA_TRY(launch_dependent(k_window_combine<T, 1>, dim3(a.heads, rows), 512, ws, s, a, sh.splits));
   KERNEL_CHECK();
   return 0;
 }
@@ -435,7 +623,7 @@ template <typename T> int window_decode(const WindowAttnArgs& a, cudaStream_t s)
 }  // namespace
 
 size_t window_attention_part_floats(int max_batch, int heads, int maps, int vdim) {
-  return (size_t)heads * maps * (vdim + 2) * ((size_t)max_batch * ATTN_FEW + 2 * 160);
+  return (size_t)heads * maps * (vdim + 2) * ((size_t)max_batch * ATTN_FEW + 3 * 160);
 }
 
 int diff_lambda(const float* lq1, const float* lk1, const float* lq2, const float* lk2, int dim, float diff, float* out, cudaStream_t s) {
