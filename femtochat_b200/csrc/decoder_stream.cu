@@ -576,17 +576,13 @@ int rows_linear(DecoderStack* d, const void* X, long long ldx, const void* W, lo
   g.ws = d->gemm_ws; g.ws_bytes = d->gemm_ws_bytes; g.status = d->status;
   g.A = X; g.lda = ldx; g.a_kmajor = true; g.B = W; g.ldb = ldw; g.b_kmajor = true;
   g.C = C; g.ldc = ldc; g.M = M; g.N = N; g.K = K; g.epi = epi; g.beta = 0.f; g.any_size = true; g.bias = out.bias;
-  if (out.n2) {      // two products: this part, and for every column of tokens the rest
+  if (out.n2) {      // two products: this part, and the rest as a batch over the columns of tokens
     g.N = out.n2;
     FEMTO_TRY(gemm<T>(g, s));
-    g.B = (const T*)W + out.n2 * ldw; g.N = N - out.n2; g.M = out.T2; g.ldc = out.ld2;
+    g.B = (const T*)W + out.n2 * ldw; g.N = N - out.n2; g.M = out.T2; g.batch = M / out.T2; g.strideA = out.T2 * ldx;
+    g.C = out.C2; g.ldc = out.ld2; g.strideC = out.stride2;
     if (g.bias) g.bias += out.n2;
-    for (int b = 0; b < M / out.T2; b++) {
-      g.A = (const T*)X + (long long)b * out.T2 * ldx;
-      g.C = (T*)out.C2 + b * out.stride2;
-      FEMTO_TRY(gemm<T>(g, s));
-    }
-    return 0;
+    return gemm<T>(g, s);
   }
   if (epi != EPI_SWIGLU) {
     FEMTO_TRY(gemm<T>(g, s));

@@ -273,7 +273,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
         if (below_diagonal(g, mt, nt, TILE_M)) continue;
         const int m0 = mt * TILE_M + rank * BM;           // first row of A this CTA loads
         const int n0 = nt * BN + rank * G::BN_LOCAL;      // first column of B this CTA loads (its half, in a pair)
-        const int bb = g.groups ? __ldg(g.groups + 1 + mt * TILE_M / g.group_rows) : bz;   // which matrix of B
+        const int bb = g.groups ? __ldg(g.groups + 1 + mt * TILE_M / g.group_rows) : g.strideB ? bz : 0;   // which matrix of B
         for (int kb = kb0; kb < kb1; kb++) {
           if (!mbar_wait(&empty[stage], phase ^ 1, abort_flag, g.status)) { ok = false; break; }
           uint8_t* sa = smem + stage * STAGE_BYTES;
@@ -852,7 +852,7 @@ int gemm_tc_bf16(const GemmArgs& g, cudaStream_t s) {
     g_pair_mode = (e && e[0] == '0') ? 0 : 1;
   }
   bool pair = (g_pair_mode != 0) && g.M >= 2 * BM && sms >= 2 && (!g.groups || g.group_rows % (2 * BM) == 0);
-  const int nbB = g.groups ? g.n_groups : nb;      // matrices of B
+  const int nbB = g.groups ? g.n_groups : g.strideB ? nb : 1;      // matrices of B: one for the whole batch when they are no distance apart
   if (pair) {
     if (g.a_kmajor) pair = make_tmap_3d_bf16(&tmA, g.A, g.K, g.M, nb, g.lda, g.strideA, 64, BM) == 0;
     else pair = make_tmap_4d_slabs_bf16(&tmA, g.A, g.M, g.K, nb, g.lda, g.strideA, BK, BM / 64) == 0;

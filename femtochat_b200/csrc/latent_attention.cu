@@ -653,11 +653,8 @@ template <typename T> int latent_attention(const LatentArgs& a, cudaStream_t s) 
   g.ws = a.d->gemm_ws; g.ws_bytes = a.d->gemm_ws_bytes; g.status = a.d->status;
   g.A = a.latent; g.lda = a.ld; g.strideA = (long long)a.maxT * a.ld; g.B = a.w_kv; g.ldb = a.lp; g.strideB = 0;
   g.C = a.kv; g.ldc = wide; g.strideC = (long long)a.maxT * wide; g.M = N; g.N = wide; g.K = a.lp; g.epi = EPI_STORE; g.any_size = true;
-  for (int b = 0; b < a.B; b++) {
-    FEMTO_TRY(gemm<T>(g, s));
-    g.A = reinterpret_cast<const T*>(g.A) + g.strideA;
-    g.C = reinterpret_cast<T*>(g.C) + g.strideC;
-  }
+  g.batch = a.B;
+  FEMTO_TRY(gemm<T>(g, s));
   if (sizeof(T) == 2 && latent_attention_tc_supported(a)) return latent_attention_tc(a, s);
   const size_t smem = 4 * (size_t)((SQ + SK) * (a.dim + a.rot_dim + 1) + SK * a.vdim + SQ * (SK + 1) + 2 * SQ);
   FEMTO_TRY(allow_smem(k_latent_attn_simt<T>, smem));
