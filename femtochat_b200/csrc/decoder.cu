@@ -530,7 +530,8 @@ static int feed_forward(DecoderStack* d, const DecLayer& l, const float* theta, 
   }
   MoeArgs a;
   a.ldz = round_up(q.experts, 4);
-  FEMTO_TRY(rows_linear<T>(d, h, w, l.w_router, w, d->moe_z, a.ldz, R, q.experts, w, EPI_F32, s));
+  if (sizeof(T) == 2 && R > ROWS_STREAM && (w & 7) == 0 && q.experts <= MOE_ROUTE) a.router = l.w_router;
+  else FEMTO_TRY(rows_linear<T>(d, h, w, l.w_router, w, d->moe_z, a.ldz, R, q.experts, w, EPI_F32, s));
   a.z = d->moe_z; a.bias = theta + l.router_bias; a.rows = R; a.experts = q.experts; a.top = q.top; a.width = w;
   a.h = h; a.weight = d->moe_weight; a.expert = d->moe_expert; a.slot = d->moe_slot; a.counts = d->moe_counts; a.groups = d->moe_groups;
   a.lists = d->moe_lists; a.xs = d->moe_x;

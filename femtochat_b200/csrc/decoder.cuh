@@ -247,6 +247,7 @@ constexpr int ATTN_FEW = 8;            // columns with at most this many new tok
 struct MoeArgs {
   const float* z = nullptr; long long ldz = 0;         // router logits [rows][ldz], without the bias
   const float* bias = nullptr;
+  const void* router = nullptr;  // instead of z: router weights [experts][width], at most MOE_ROUTE of them in bf16
   int rows = 0, experts = 0, top = 0, width = 0, group_rows = 0, max_lists = 0;
   const void* h = nullptr;       // [rows][width]
   float* weight = nullptr; int *expert = nullptr, *slot = nullptr;   // [rows * top]
@@ -255,6 +256,7 @@ struct MoeArgs {
   int* lists = nullptr;          // few rows: number of lists, (expert, start, length) of each, from 1 + 3 max_lists on the pairs
   void* xs = nullptr;            // sorted inputs
 };
+constexpr int MOE_ROUTE = 64;          // experts up to which moe_sort can multiply by the router itself
 bool moe_supported(int experts, int top);
 int moe_group_rows(long long rows, int experts, int top);
 long long moe_max_slots(long long rows, int experts, int top, int group_rows);

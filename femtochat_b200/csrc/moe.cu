@@ -8,6 +8,7 @@
 
 #include "decoder.cuh"
 #include "streaming.cuh"
+#include "warp_mma.cuh"
 
 namespace {
 
@@ -47,12 +48,12 @@ __device__ __forceinline__ void choose(const float* __restrict__ z, const float*
   weight = p / warp_sum(p);
 }
 
+// The choices of a block's TOPK_ROWS rows (logits z with pitch ldz, of these rows): weights, experts, and every choice's place
+// among the rows of its expert.  By 256 threads.
 constexpr int TOPK_ROWS = 32;
 template <int PER>
-__global__ void __launch_bounds__(256) k_moe_choose(const MoeArgs a) {
-  pdl_trigger();
-  pdl_wait();
-  __shared__ int count[MAX_EXPERTS];
+__device__ __forceinline__ void choose_rows(const MoeArgs& a, const float* z, long long ldz) {
+  __shared__ int count[32 * PER];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int e = threadIdx.x; e < a.experts; e += 256) count[e] = 0;
   __syncthreads();
@@ -64,7 +65,7 @@ __global__ void __launch_bounds__(256) k_moe_choose(const MoeArgs a) {
     if (row >= a.rows) continue;
     float w;
     int e;
-    choose<PER>(a.z + row * a.ldz, a.bias, a.experts, a.top, lane, e, w);
+    choose<PER>(z + (i * 8 + warp) * ldz, a.bias, a.experts, a.top, lane, e, w);
     if (lane < a.top) {
       a.weight[row * a.top + lane] = w;
       id[i] = e;
@@ -81,6 +82,55 @@ __global__ void __launch_bounds__(256) k_moe_choose(const MoeArgs a) {
     a.expert[pair] = id[i];
     a.slot[pair] = count[id[i]] + at[i];      // place among the expert's rows
   }
+}
+
+template <int PER>
+__global__ void __launch_bounds__(256) k_moe_choose(const MoeArgs a) {
+  pdl_trigger();
+  pdl_wait();
+  choose_rows<PER>(a, a.z + (long long)blockIdx.x * TOPK_ROWS * a.ldz, a.ldz);
+}
+
+// Router and choice in one launch, bf16 rows and at most 8 NT experts: 32 rows per block, two tiles of 16 rows by four parts of
+// the channels.  Rows and weights go straight from global memory into the fragments: a lane takes 16 consecutive bytes of
+// each, and since both are read in the same order the permutation of the channels inside a step does not matter.
+template <int NT>
+__global__ void __launch_bounds__(256) k_moe_route(const MoeArgs a) {
+  pdl_trigger();
+  constexpr int ZP = 8 * NT + 1;
+  __shared__ float z[4][TOPK_ROWS][ZP];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c2 = 2 * (lane & 3);
+  const int rt = warp & 1, part = warp >> 1, K = a.width;
+  const long long row = (long long)blockIdx.x * TOPK_ROWS + rt * 16 + g;
+  const bf16* h = reinterpret_cast<const bf16*>(a.h);
+  const bf16 *x0 = h + min(row, (long long)a.rows - 1) * K, *x1 = h + min(row + 8, (long long)a.rows - 1) * K;
+  const bf16* w = reinterpret_cast<const bf16*>(a.router);
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  pdl_wait();
+  float acc[NT][4] = {};
+#pragma unroll 4
+  for (int k0 = part * 32; k0 < K; k0 += 128) {
+    const int k = k0 + (lane & 3) * 8;
+    const uint4 p = k < K ? *reinterpret_cast<const uint4*>(x0 + k) : zero, q = k < K ? *reinterpret_cast<const uint4*>(x1 + k) : zero;
+    const uint32_t lo[4] = {p.x, q.x, p.y, q.y}, hi[4] = {p.z, q.z, p.w, q.w};
+#pragma unroll
+    for (int t = 0; t < NT; t++) {
+      const uint4 b = k < K && 8 * t + g < a.experts ? __ldg(reinterpret_cast<const uint4*>(w + (long long)(8 * t + g) * K + k)) : zero;
+      mma16816(acc[t], lo, b.x, b.y);
+      mma16816(acc[t], hi, b.z, b.w);
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < NT; t++)
+#pragma unroll
+    for (int e = 0; e < 4; e++) z[part][rt * 16 + g + 8 * (e >> 1)][8 * t + c2 + (e & 1)] = acc[t][e];
+  __syncthreads();
+  for (int i = threadIdx.x; i < TOPK_ROWS * 8 * NT; i += 256) {
+    const int r = i / (8 * NT), c = i % (8 * NT);
+    z[0][r][c] = (z[0][r][c] + z[1][r][c]) + (z[2][r][c] + z[3][r][c]);
+  }
+  __syncthreads();
+  choose_rows<(NT + 3) / 4>(a, &z[0][0][0], ZP);
 }
 
 // Places every (row, choice) pair: slot = start of its expert's run + place, and the row's input is copied there.  Every block
@@ -202,9 +252,19 @@ long long moe_max_slots(long long rows, int experts, int top, int group_rows) {
 template <typename T> int moe_sort(const MoeArgs& a, cudaStream_t s) {
   constexpr int V = VecN<T>::n;
   FEMTO_TRY(fill_zero(a.counts, 4 * (size_t)a.experts, s));
-#define LAUNCH(PER) CUDA_TRY(launch_dependent(k_moe_choose<PER>, cdiv(a.rows, TOPK_ROWS), 256, 0, s, a))
-  DISPATCH_PER(a.experts, LAUNCH);
+  const int choosers = cdiv(a.rows, TOPK_ROWS);
+  if (a.router) {
+#define LAUNCH(NT) CUDA_TRY(launch_dependent(k_moe_route<NT>, choosers, 256, 0, s, a))
+    if (a.experts <= 8) LAUNCH(1);
+    else if (a.experts <= 16) LAUNCH(2);
+    else if (a.experts <= 32) LAUNCH(4);
+    else LAUNCH(8);
 #undef LAUNCH
+  } else {
+#define LAUNCH(PER) CUDA_TRY(launch_dependent(k_moe_choose<PER>, choosers, 256, 0, s, a))
+    DISPATCH_PER(a.experts, LAUNCH);
+#undef LAUNCH
+  }
   KERNEL_CHECK();
   const int blocks = cdiv((long long)a.rows * a.top, PLACE_PAIRS);
   if (a.width % V == 0 && aligned16(a.h) && aligned16(a.xs)) CUDA_TRY(launch_dependent(k_moe_place<T, V>, blocks, 256, 0, s, a));
