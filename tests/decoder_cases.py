@@ -66,6 +66,7 @@ SINGLE = {
     "latent, aligned sizes": (config(latent(heads=4, dim=128, rot_dim=64, vdim=128, q_rank=192, kv_rank=128, ff=512, scale=0.07), width=256, vocab=320), (8, 8)),
     "latent, dim 64": (config(latent(heads=2, dim=64, rot_dim=64, vdim=64, q_rank=64, kv_rank=256, ff=256), width=128), (8, 8)),
     "latent, vdim 96": (config(latent(heads=5, dim=48, rot_dim=16, vdim=96, q_rank=40, kv_rank=72, ff=256), width=128), (8, 8)),
+    "latent, wide values": (config(latent(heads=2, dim=64, rot_dim=16, vdim=160, q_rank=40, kv_rank=72)), (8, 8)),
     "latent, one head, odd sizes": (config(latent(heads=1, dim=5, rot_dim=2, vdim=3, q_rank=7, kv_rank=9, ff=20), width=34), (8, 8)),
     "differential": (zurevik(differential()), (8, 8)),
     "differential, one key head": (zurevik(differential(heads=6, kv_heads=1, dim=8, vdim=40, size=5, keep=1, scale=0.5, diff=0.2)), (8, 8)),
@@ -84,6 +85,7 @@ SINGLE = {
     "sinks, no softcap": (zurevik(sinks(size=400), softcap=None, embed_scale=0.3), (8, 8)),
     "sinks, aligned sizes": (zurevik(sinks(heads=4, kv_heads=2, dim=128, vdim=128, size=70, scale=0.09), width=256, vocab=320), (8, 8)),
     "sinks, wide": (zurevik(sinks(heads=2, kv_heads=1, dim=256, vdim=200, scale=0.05)), (8, 8)),
+    "sinks, wide values": (zurevik(sinks(heads=4, kv_heads=2, dim=64, vdim=200, scale=0.12), width=64), (8, 8)),
     "sinks, one head, odd sizes": (zurevik(sinks(heads=1, kv_heads=1, dim=7, vdim=5, scale=0.6), width=34, vocab=61), (8, 8)),
     "sinks, shared keys": (zurevik(sinks(size=9), sinks(size=30, kv_from=0, scale=0.35), sinks(size=4, kv_from=0, heads=2)), (8, 8)),
 }
@@ -94,7 +96,10 @@ EXPERTS = {
     "one of three": zurevik(differential(mlp=moe(experts=3, top=1))),
     "all of four": zurevik(sinks(mlp=moe(experts=4, top=4, ff=9))),
     "one expert": zurevik(sinks(mlp=moe(experts=1, top=1))),
+    "three of twenty": zurevik(sinks(mlp=moe(experts=20, top=3, ff=16))),
     "five of forty": zurevik(sinks(mlp=moe(experts=40, top=5, ff=16))),
+    "one of seventy": zurevik(sinks(mlp=moe(experts=70, top=1, ff=8))),
+    "two of three hundred": zurevik(sinks(mlp=moe(experts=300, top=2, ff=8))),
     "odd sizes": zurevik(sinks(heads=1, kv_heads=1, dim=7, vdim=5, mlp=moe(ff=13, experts=6, top=3)), width=34, vocab=61),
     "aligned sizes": zurevik(sinks(heads=2, kv_heads=2, dim=64, vdim=64, mlp=moe(ff=256, experts=4, top=2)), width=256, vocab=320),
     "between norms": config(latent(ff=0), latent(ff=0)),

@@ -105,6 +105,20 @@ def test_columns_equal_each_alone(dtype):
     ok(model)
 
 
+@BOTH
+def test_more_query_tiles_than_multiprocessors(dtype):
+    """Every block of the prompt's attention works through several items; columns with the same tokens agree."""
+    cfg = dc.zurevik(dc.sinks(heads=12, kv_heads=3, dim=32, vdim=40, size=100), dc.differential(heads=12, kv_heads=4, dim=16, vdim=24, size=70, keep=3), width=48)
+    model, w = dc.model_and_weights(cfg, (8, 8), dtype, seed=37)
+    B, n = 9, 300
+    t = dc.tokens(n, cfg["vocab"], 8)
+    want = lo.Sequence(cfg, w).feed(t)
+    z = fb.extend(model, cache_for(model, n, B), t[None].repeat(B, 1), want=list(range(B * n))).cpu().view(B, n, -1)
+    for b in range(B):
+        assert dc.rel_error(z[b], want) < TOL[dtype], b
+    ok(model)
+
+
 def test_internal_portions():
     """A prompt longer than one internal pass, several columns, a ragged choice of positions."""
     cfg = dc.ZMIXED
